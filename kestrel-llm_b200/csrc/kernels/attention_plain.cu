@@ -30,12 +30,12 @@
 #define PA_MAX_PER_LANE 18    // head size up to 576 (a cached latent of 512 numbers beside a shared key part of 64)
 #define PA_KEYS 4
 
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(PA_WARPS * 32)
 attention_plain_kernel(const T *__restrict__ q, const T *__restrict__ k_cache, const T *__restrict__ v_cache,
                        const int *__restrict__ positions, const int *__restrict__ seq_of_token,
                        const int *__restrict__ block_table, int table_stride, int page_size,
-                       T *__restrict__ out, int nq, int nkv, int hd, int vd, int v_ld, int window, int keep_first,
+                       TO *__restrict__ out, int nq, int nkv, int hd, int vd, int v_ld, int window, int keep_first,
                        const float *__restrict__ gate, float scale, const ScoreOpts opts) {
     pdl_launch_dependents();
     pdl_wait();
@@ -151,11 +151,11 @@ attention_plain_kernel(const T *__restrict__ q, const T *__restrict__ k_cache, c
         }
         float inv = sigmoid ? 1.0f : 1.0f / L;
         if (gate) inv *= gate[(size_t)t * nq + h];
-        T *orow = out + ((size_t)t * nq + h) * vd;
+        TO *orow = out + ((size_t)t * nq + h) * vd;
 #pragma unroll
         for (int c = 0; c < PA_MAX_PER_LANE; ++c) {
             int i = lane + 32 * c;
-            if (c < per_lane_v && i < vd) orow[i] = from_f32<T>(o[c] * inv);
+            if (c < per_lane_v && i < vd) orow[i] = from_f32<TO>(o[c] * inv);
         }
     }
 }
@@ -172,13 +172,26 @@ KESTREL_API int kestrel_attention_plain_scored(const void *q, const void *k_cach
                                           stream);
 }
 
-// the same with a learned number per head and bucket of distances added to the scores: rel [buckets, nq], the bucket of
-// a distance from rel_bucket [rel_far + 1] (distances beyond rel_far share its bucket); `v_ld` > 0: the V plane's rows hold v_ld
-// numbers of which the first vd are the value (a V plane that is the K plane of longer rows)
 KESTREL_API int kestrel_attention_plain_biased(const void *q, const void *k_cache, const void *v_cache,
                                                const int *positions, const int *seq_of_token,
                                                const int *block_table, int table_stride, int page_size,
                                                void *out, int dtype, int T, int nq, int nkv, int hd, int vd, int window,
+                                               int keep_first, const float *gate, float scale, float softcap, const float *r1,
+                                               const float *r2, const float *head_bias, int weighting, const float *sink,
+                                               const float *rel, const int *rel_bucket, int rel_far, int v_ld, cudaStream_t stream) {
+    return kestrel_attention_plain_to(q, k_cache, v_cache, positions, seq_of_token, block_table, table_stride, page_size, out, dtype, 0, T, nq, nkv,
+                                      hd, vd, window, keep_first, gate, scale, softcap, r1, r2, head_bias, weighting, sink, rel, rel_bucket, rel_far,
+                                      v_ld, stream);
+}
+
+// the same with a learned number per head and bucket of distances added to the scores: rel [buckets, nq], the bucket of
+// a distance from rel_bucket [rel_far + 1] (distances beyond rel_far share its bucket); `v_ld` > 0: the V plane's rows hold v_ld
+// numbers of which the first vd are the value (a V plane that is the K plane of longer rows); `out_f32`: the output is float32 whatever the storage type (heads
+// that are combined further before they are rounded)
+KESTREL_API int kestrel_attention_plain_to(const void *q, const void *k_cache, const void *v_cache,
+                                               const int *positions, const int *seq_of_token,
+                                               const int *block_table, int table_stride, int page_size,
+                                               void *out, int dtype, int out_f32, int T, int nq, int nkv, int hd, int vd, int window,
                                                int keep_first, const float *gate, float scale, float softcap, const float *r1,
                                                const float *r2, const float *head_bias, int weighting, const float *sink,
                                                const float *rel, const int *rel_bucket, int rel_far, int v_ld, cudaStream_t stream) {
@@ -192,10 +205,13 @@ KESTREL_API int kestrel_attention_plain_biased(const void *q, const void *k_cach
     KESTREL_REQUIRE(nq <= 65535, "attention_plain: %d query heads exceed the grid", nq);
     dim3 grid(T, nq);
     if (dtype == KESTREL_F32)
-        kestrel_launch(attention_plain_kernel<float>, dim3(grid), dim3(PA_WARPS * 32), 0, stream, (const float *)q, (const float *)k_cache, (const float *)v_cache, positions, seq_of_token,
+        kestrel_launch(attention_plain_kernel<float, float>, dim3(grid), dim3(PA_WARPS * 32), 0, stream, (const float *)q, (const float *)k_cache, (const float *)v_cache, positions, seq_of_token,
             block_table, table_stride, page_size, (float *)out, nq, nkv, hd, vd, v_ld > 0 ? v_ld : vd, window, keep_first, gate, scale, opts);
+    else if (dtype == KESTREL_BF16 && out_f32)
+        kestrel_launch(attention_plain_kernel<__nv_bfloat16, float>, dim3(grid), dim3(PA_WARPS * 32), 0, stream, (const __nv_bfloat16 *)q, (const __nv_bfloat16 *)k_cache, (const __nv_bfloat16 *)v_cache, positions,
+            seq_of_token, block_table, table_stride, page_size, (float *)out, nq, nkv, hd, vd, v_ld > 0 ? v_ld : vd, window, keep_first, gate, scale, opts);
     else if (dtype == KESTREL_BF16)
-        kestrel_launch(attention_plain_kernel<__nv_bfloat16>, dim3(grid), dim3(PA_WARPS * 32), 0, stream, (const __nv_bfloat16 *)q, (const __nv_bfloat16 *)k_cache, (const __nv_bfloat16 *)v_cache, positions,
+        kestrel_launch(attention_plain_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(grid), dim3(PA_WARPS * 32), 0, stream, (const __nv_bfloat16 *)q, (const __nv_bfloat16 *)k_cache, (const __nv_bfloat16 *)v_cache, positions,
             seq_of_token, block_table, table_stride, page_size, (__nv_bfloat16 *)out, nq, nkv, hd, vd, v_ld > 0 ? v_ld : vd, window, keep_first, gate, scale, opts);
     else
         return kestrel_fail(-2, "attention_plain: unknown dtype %d", dtype);

@@ -61,14 +61,16 @@ attn_prepare_ex_kernel(const float *__restrict__ partial, int S, size_t slice_st
                        const int *__restrict__ block_table, int table_stride, int page_size,
                        T *__restrict__ k_cache, T *__restrict__ v_cache, T *__restrict__ q_out, float *__restrict__ gate_out,
                        int nq, int nkv, int hd, int vd, int has_kv, const float *__restrict__ bias, int v_norm, int keep_x,
-                       const float *__restrict__ inv_freq, int rot, int rot_mode, float rot_scale, float q_temp_coef, int q_temp_every) {
+                       const float *__restrict__ inv_freq, int rot, int rot_mode, float rot_scale, float q_temp_coef, int q_temp_every,
+                       int maps, int q_pad) {
     extern __shared__ float apx_ss[];              // qk_norm = 2: sum of squares of every q and k head, then (keep_x) their columns
     __shared__ float apx_rot[APX_WARPS][32 * APX_PER_LANE];   // rotate-half pairing: a warp's head, so that a lane reaches its partner
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const float *row = partial + (size_t)t * ld;
-    const int n_heads = nq + (has_kv ? 2 * nkv : 0);
+    const int nqm = nq * maps, nkm = nkv * maps;       // rows of q and k: every map of a head is normed and turned by itself
+    const int n_heads = nqm + (has_kv ? nkm + nkv : 0);
     float mul_q = 1.f, mul_k = 1.f;
     if (qk_norm == 2) {
         const int n_qk = nq + (has_kv ? nkv : 0);
@@ -103,10 +105,10 @@ attn_prepare_ex_kernel(const float *__restrict__ partial, int S, size_t slice_st
     }
     for (int r = blockIdx.y * APX_WARPS + warp; r < n_heads; r += gridDim.y * APX_WARPS) {
         // which part: 0 = q head r, 1 = k head, 2 = v head
-        const int kind = r < nq ? 0 : (r < nq + nkv ? 1 : 2);
-        const int head = kind == 0 ? r : (kind == 1 ? r - nq : r - nq - nkv);
+        const int kind = r < nqm ? 0 : (r < nqm + nkm ? 1 : 2);
+        const int head = kind == 0 ? r : (kind == 1 ? r - nqm : r - nqm - nkm);
         const int n = kind == 2 ? vd : hd;
-        const int col0 = kind == 0 ? head * hd : (kind == 1 ? nq * hd + head * hd : nq * hd + nkv * hd + head * vd);
+        const int col0 = kind == 0 ? head * hd : (kind == 1 ? nqm * hd + head * hd : nqm * hd + nkm * hd + head * vd);
         float x[APX_PER_LANE];
         float ss = 0.f;
         if (keep_x && qk_norm == 2 && kind != 2) {                 // summed in the first pass
@@ -134,9 +136,16 @@ attn_prepare_ex_kernel(const float *__restrict__ partial, int S, size_t slice_st
             ss = warp_sum(ss);
             mul = 1.0f / sqrtf(ss / (float)n + eps);
         }
-        T *dst = kind == 0 ? q_out + ((size_t)t * nq + head) * hd
-                           : (kind == 1 ? k_cache + (slot_row + (size_t)head * page_size) * hd
+        // several maps a head: a cache row holds the maps' keys one after the other; a padded query row has the cache row's
+        // length and is zero outside its own map's place
+        const int own = head % maps * hd;
+        T *dst = kind == 0 ? q_out + ((size_t)t * nqm + head) * (q_pad ? maps * hd : hd) + (q_pad ? own : 0)
+                           : (kind == 1 ? k_cache + (slot_row + (size_t)(head / maps) * page_size) * (maps * hd) + own
                                         : v_cache + (slot_row + (size_t)head * page_size) * vd);
+        if (kind == 0 && q_pad && maps > 1) {
+            T *zero = q_out + ((size_t)t * nqm + head) * (maps * hd);
+            for (int i = lane; i < (maps - 1) * hd; i += 32) zero[i < own ? i : i + hd] = from_f32<T>(0.f);
+        }
 #pragma unroll
         for (int c = 0; c < APX_PER_LANE; ++c) {
             const int i = lane + 32 * c;
@@ -174,7 +183,7 @@ attn_prepare_ex_kernel(const float *__restrict__ partial, int S, size_t slice_st
         }
     }
     if (gate_out && blockIdx.y == 0) {
-        const int col0 = nq * hd + (has_kv ? nkv * (hd + vd) : 0);
+        const int col0 = nqm * hd + (has_kv ? nkm * hd + nkv * vd : 0);
         for (int h = threadIdx.x; h < nq; h += APX_WARPS * 32) {
             float z = sum_slices(row, S, slice_stride, col0 + h);
             if (bias) z += bias[col0 + h];
@@ -204,14 +213,30 @@ KESTREL_API int kestrel_attn_prepare_rotated(const float *partial, int S, long l
                                          gate_out, dtype, T, nq, nkv, hd, vd, has_kv, stream);
 }
 
-// the same with a query temperature: q times 1 + q_temp_coef * ln(floor((position + 1) / q_temp_every) + 1); q_temp_every = 0: none
 KESTREL_API int kestrel_attn_prepare_tempered(const float *partial, int S, long long slice_stride, int ld, const float *bias, const float *q_norm_w,
                                               const float *k_norm_w, int qk_norm, int v_norm, float norm_eps, const float *inv_freq, int rot,
                                               int rot_mode, float rot_scale, float q_temp_coef, int q_temp_every, const int *positions,
                                               const int *seq_of_token, const int *block_table, int table_stride, int page_size, void *k_cache,
                                               void *v_cache, void *q_out, float *gate_out, int dtype, int T, int nq, int nkv, int hd, int vd,
                                               int has_kv, cudaStream_t stream) {
+    return kestrel_attn_prepare_maps(partial, S, slice_stride, ld, bias, q_norm_w, k_norm_w, qk_norm, v_norm, norm_eps, inv_freq, rot, rot_mode,
+                                     rot_scale, q_temp_coef, q_temp_every, positions, seq_of_token, block_table, table_stride, page_size, k_cache,
+                                     v_cache, q_out, gate_out, dtype, T, nq, nkv, hd, vd, has_kv, 1, 0, stream);
+}
+
+// with a query temperature: q times 1 + q_temp_coef * ln(floor((position + 1) / q_temp_every) + 1); q_temp_every = 0: none.  With
+// `maps` > 1 a head has that many queries and keys of size hd, laid out [head][map], over one value: product columns
+// [q: nq*maps*hd | k: nkv*maps*hd | v: nkv*vd | gate: nq], K pages [page][kv head][slot][maps*hd], and q_out [T, nq*maps, hd]
+// or, with `q_pad`, [T, nq*maps, maps*hd] whose rows are zero outside their own map's place, so that a plain dot product
+// of such a row with a cache row is its map's score
+KESTREL_API int kestrel_attn_prepare_maps(const float *partial, int S, long long slice_stride, int ld, const float *bias, const float *q_norm_w,
+                                              const float *k_norm_w, int qk_norm, int v_norm, float norm_eps, const float *inv_freq, int rot,
+                                              int rot_mode, float rot_scale, float q_temp_coef, int q_temp_every, const int *positions,
+                                              const int *seq_of_token, const int *block_table, int table_stride, int page_size, void *k_cache,
+                                              void *v_cache, void *q_out, float *gate_out, int dtype, int T, int nq, int nkv, int hd, int vd,
+                                              int has_kv, int maps, int q_pad, cudaStream_t stream) {
     if (T == 0) return 0;
+    KESTREL_REQUIRE(maps >= 1 && (maps == 1 || qk_norm != 2), "attn_prepare_ex: %d maps a head (the norm over a whole projection takes one)", maps);
     KESTREL_REQUIRE(q_temp_every >= 0, "attn_prepare_ex: a query temperature every %d positions", q_temp_every);
     KESTREL_REQUIRE(!inv_freq || (rot > 0 && rot % 2 == 0 && rot <= hd && (rot_mode == 0 || rot_mode == 1)),
                     "attn_prepare_ex: %d rotated dimensions of a head of %d (mode %d)", rot, hd, rot_mode);
@@ -223,18 +248,18 @@ KESTREL_API int kestrel_attn_prepare_tempered(const float *partial, int S, long 
     if (keep_x) smem += (size_t)(nq + nkv) * hd * sizeof(float);
     KESTREL_REQUIRE(T > 0 && nq >= 0 && nkv > 0 && hd > 0 && vd > 0 && S > 0 && (nq > 0 || has_kv), "attn_prepare_ex: bad sizes");
     KESTREL_REQUIRE(hd <= 32 * APX_PER_LANE && vd <= 32 * APX_PER_LANE, "attn_prepare_ex: head size %d / %d exceeds %d", hd, vd, 32 * APX_PER_LANE);
-    const int need = nq * hd + (has_kv ? nkv * (hd + vd) : 0) + (gate_out ? nq : 0);
+    const int need = nq * maps * hd + (has_kv ? nkv * (maps * hd + vd) : 0) + (gate_out ? nq : 0);
     KESTREL_REQUIRE(ld >= need, "attn_prepare_ex: the product has %d columns, the heads need %d", ld, need);
     // few tokens: a block per four head rows, so that the step's few tokens still fill the device
-    const int n_heads = nq + (has_kv ? 2 * nkv : 0);
+    const int n_heads = nq * maps + (has_kv ? nkv * (maps + 1) : 0);
     const int by = T >= 512 ? 1 : (n_heads + APX_WARPS - 1) / APX_WARPS;
     if (dtype == KESTREL_F32)
         kestrel_launch(attn_prepare_ex_kernel<float>, dim3(T, by), dim3(APX_WARPS * 32), smem, stream, partial, S, (size_t)slice_stride, ld, q_norm_w, k_norm_w, qk_norm, norm_eps,
-                       positions, seq_of_token, block_table, table_stride, page_size, (float *)k_cache, (float *)v_cache, (float *)q_out, gate_out, nq, nkv, hd, vd, has_kv, bias, v_norm, keep_x, inv_freq, rot, rot_mode, rot_scale, q_temp_coef, q_temp_every);
+                       positions, seq_of_token, block_table, table_stride, page_size, (float *)k_cache, (float *)v_cache, (float *)q_out, gate_out, nq, nkv, hd, vd, has_kv, bias, v_norm, keep_x, inv_freq, rot, rot_mode, rot_scale, q_temp_coef, q_temp_every, maps, q_pad);
     else if (dtype == KESTREL_BF16)
         kestrel_launch(attn_prepare_ex_kernel<__nv_bfloat16>, dim3(T, by), dim3(APX_WARPS * 32), smem, stream, partial, S, (size_t)slice_stride, ld, q_norm_w, k_norm_w, qk_norm, norm_eps,
                        positions, seq_of_token, block_table, table_stride, page_size, (__nv_bfloat16 *)k_cache, (__nv_bfloat16 *)v_cache, (__nv_bfloat16 *)q_out, gate_out, nq, nkv,
-                       hd, vd, has_kv, bias, v_norm, keep_x, inv_freq, rot, rot_mode, rot_scale, q_temp_coef, q_temp_every);
+                       hd, vd, has_kv, bias, v_norm, keep_x, inv_freq, rot, rot_mode, rot_scale, q_temp_coef, q_temp_every, maps, q_pad);
     else
         return kestrel_fail(-2, "attn_prepare_ex: unknown dtype %d", dtype);
     return kestrel_check_launch("attn_prepare_ex");

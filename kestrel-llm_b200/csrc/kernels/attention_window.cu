@@ -48,6 +48,7 @@ struct AwParams {
     const __nv_bfloat16 *v_cache;   // [pages, nkv, page_size, v_ld]: a value is the first vd numbers of its row (v_ld = vd unless the rows hold more)
     int v_ld;
     __nv_bfloat16 *out;             // [T, nq * vd]
+    float *out_f32;                 // if not null: the output goes here in float32 instead (heads that are combined further)
     const float *gate;              // [T, nq] or null
     const int *cu_seqlens, *kv_lens, *block_table;
     int table_stride, page_size, nq, nkv, hd, vd, window, keep_first;
@@ -287,6 +288,15 @@ attention_window_kernel(const AwParams p) {
                 inv = f / (fast_exp2(s2 - M) + l_r[h2] * f);
             }
             if (p.gate) inv *= p.gate[(size_t)tok * p.nq + head];
+            if (p.out_f32) {
+                float *dst = p.out_f32 + ((size_t)tok * p.nq + head) * vd;
+#pragma unroll
+                for (int j = 0; j < D / 8; ++j) {
+                    const int col = j * 8 + 2 * tq;
+                    if (col < vd) *reinterpret_cast<float2 *>(dst + col) = make_float2(o[j][2 * h2] * inv, o[j][2 * h2 + 1] * inv);
+                }
+                continue;
+            }
             __nv_bfloat16 *dst = p.out + ((size_t)tok * p.nq + head) * vd;
 #pragma unroll
             for (int j = 0; j < D / 8; ++j) {
@@ -352,7 +362,8 @@ attention_window_kernel(const AwParams p) {
             const int row = row0 + r, tok = tok_begin + row / G, head = kvh * G + row % G;
             float v = sigmoid ? acc : acc / L;
             if (p.gate) v *= p.gate[(size_t)tok * p.nq + head];
-            p.out[((size_t)tok * p.nq + head) * vd + col] = __float2bfloat16_rn(v);
+            if (p.out_f32) p.out_f32[((size_t)tok * p.nq + head) * vd + col] = v;
+            else p.out[((size_t)tok * p.nq + head) * vd + col] = __float2bfloat16_rn(v);
         }
     }
 }
@@ -392,7 +403,8 @@ attention_window_merge_kernel(const AwParams p, int ksplit, int D) {
         float acc = 0.f;
 #pragma unroll 8
         for (int s = 0; s < ksplit; ++s) acc = fmaf(p.part_o[(base + (size_t)s * 16) * D + col], f_s[s], acc);
-        p.out[((size_t)tok * p.nq + head) * vd + col] = __float2bfloat16_rn(acc * inv);
+        if (p.out_f32) p.out_f32[((size_t)tok * p.nq + head) * vd + col] = acc * inv;
+        else p.out[((size_t)tok * p.nq + head) * vd + col] = __float2bfloat16_rn(acc * inv);
     }
 }
 
@@ -471,6 +483,18 @@ KESTREL_API int kestrel_attention_window_biased(const void *q, const void *k_cac
                                                 float softcap, const float *r1, const float *r2, const float *head_bias, int weighting,
                                                 const float *sink, const float *rel, const int *rel_bucket, int rel_far, int v_ld,
                                                 int ksplit, float *scratch, cudaStream_t stream) {
+    return kestrel_attention_window_to(q, k_cache, v_cache, out, 0, gate, cu_seqlens, kv_lens, block_table, table_stride, page_size, nseq, max_count, nq,
+                                       nkv, hd, vd, window, keep_first, scale, softcap, r1, r2, head_bias, weighting, sink, rel, rel_bucket, rel_far, v_ld,
+                                       ksplit, scratch, stream);
+}
+
+// `out_f32`: the output is float32 (heads that are combined further before they are rounded)
+KESTREL_API int kestrel_attention_window_to(const void *q, const void *k_cache, const void *v_cache, void *out, int out_f32, const float *gate,
+                                                const int *cu_seqlens, const int *kv_lens, const int *block_table, int table_stride, int page_size,
+                                                int nseq, int max_count, int nq, int nkv, int hd, int vd, int window, int keep_first, float scale,
+                                                float softcap, const float *r1, const float *r2, const float *head_bias, int weighting,
+                                                const float *sink, const float *rel, const int *rel_bucket, int rel_far, int v_ld,
+                                                int ksplit, float *scratch, cudaStream_t stream) {
     if (nseq == 0 || max_count == 0) return 0;
     KESTREL_REQUIRE(ksplit >= 1 && ksplit <= 65535 && (ksplit == 1 || scratch), "attention_window: %d shares of the keys without scratch", ksplit);
     KESTREL_REQUIRE(weighting >= 0 && weighting <= 2 && softcap >= 0.f && (r1 == nullptr) == (r2 == nullptr), "attention_window: bad score options");
@@ -481,6 +505,7 @@ KESTREL_API int kestrel_attention_window_biased(const void *q, const void *k_cac
     p.k_cache = (const __nv_bfloat16 *)k_cache;
     p.v_cache = (const __nv_bfloat16 *)v_cache;
     p.out = (__nv_bfloat16 *)out;
+    p.out_f32 = out_f32 ? (float *)out : nullptr;
     p.gate = gate;
     p.cu_seqlens = cu_seqlens;
     p.kv_lens = kv_lens;

@@ -408,11 +408,12 @@ recurrence_scan_kernel(const float *__restrict__ r, const float *__restrict__ w,
 }
 
 // ---- per-head norm of the read-out, weight, optional sigmoid gate ---------------------------------
-// out = o / sqrt(mean(o^2) + eps) * w[h * w_stride + i] (* sigmoid(gate column g_col0 + h dv + i)) in the storage type
+// out = o / sqrt(mean(o^2) + eps) (* w[h * w_stride + i]) (* act(gate column g_col0 + h dv + i)) in the storage type; act: 0 the
+// sigmoid, 1 silu
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float *__restrict__ o, const float *__restrict__ w, int w_stride, float eps, const float *__restrict__ g_part,
-                      int Sg, size_t g_stride, int g_ld, int g_col0, T *__restrict__ out, int H, int dv) {
+                      int Sg, size_t g_stride, int g_ld, int g_col0, int g_act, T *__restrict__ out, int H, int dv) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -423,8 +424,12 @@ head_norm_gate_kernel(const float *__restrict__ o, const float *__restrict__ w, 
         ss = warp_sum(ss);
         const float rn = 1.0f / sqrtf(ss / (float)dv + eps);
         for (int i = lane; i < dv; i += 32) {
-            float y = o[base + i] * rn * w[(size_t)h * w_stride + i];
-            if (g_part) y *= lr_sigmoid(sum_slices(g_part, Sg, g_stride, (size_t)t * g_ld + g_col0 + (size_t)h * dv + i));
+            float y = o[base + i] * rn;
+            if (w) y *= w[(size_t)h * w_stride + i];
+            if (g_part) {
+                const float z = sum_slices(g_part, Sg, g_stride, (size_t)t * g_ld + g_col0 + (size_t)h * dv + i);
+                y *= g_act == 1 ? z * lr_sigmoid(z) : lr_sigmoid(z);
+            }
             out[base + i] = from_f32<T>(y);
         }
     }
@@ -502,16 +507,21 @@ KESTREL_API int kestrel_recurrence_scan(const float *r, const float *w, const fl
 
 KESTREL_API int kestrel_head_norm_gate(const float *o, const float *w, int w_stride, float eps, const float *g_part, int Sg, long long g_stride,
                                        int g_ld, int g_col0, void *out, int dtype, int T, int H, int dv, cudaStream_t stream) {
+    return kestrel_head_norm_act(o, w, w_stride, eps, g_part, Sg, g_stride, g_ld, g_col0, 0, out, dtype, T, H, dv, stream);
+}
+
+KESTREL_API int kestrel_head_norm_act(const float *o, const float *w, int w_stride, float eps, const float *g_part, int Sg, long long g_stride,
+                                      int g_ld, int g_col0, int g_act, void *out, int dtype, int T, int H, int dv, cudaStream_t stream) {
     if (T == 0) return 0;
-    KESTREL_REQUIRE(T > 0 && H > 0 && dv > 0 && (w_stride == 0 || w_stride == dv) && (!g_part || (Sg > 0 && g_col0 >= 0 && g_col0 + H * dv <= g_ld)),
+    KESTREL_REQUIRE(T > 0 && H > 0 && dv > 0 && (g_act == 0 || g_act == 1) && (w_stride == 0 || w_stride == dv) && (!g_part || (Sg > 0 && g_col0 >= 0 && g_col0 + H * dv <= g_ld)),
                     "head_norm_gate: bad sizes");
     const int by = T >= 512 ? 1 : (H + 3) / 4;
     if (dtype == KESTREL_F32)
         kestrel_launch(head_norm_gate_kernel<float>, dim3(T, by), dim3(128), 0, stream, o, w, w_stride, eps, g_part, Sg, (size_t)g_stride, g_ld, g_col0,
-                       (float *)out, H, dv);
+                       g_act, (float *)out, H, dv);
     else if (dtype == KESTREL_BF16)
         kestrel_launch(head_norm_gate_kernel<__nv_bfloat16>, dim3(T, by), dim3(128), 0, stream, o, w, w_stride, eps, g_part, Sg, (size_t)g_stride, g_ld,
-                       g_col0, (__nv_bfloat16 *)out, H, dv);
+                       g_col0, g_act, (__nv_bfloat16 *)out, H, dv);
     else
         return kestrel_fail(-2, "head_norm_gate: unknown dtype %d", dtype);
     return kestrel_check_launch("head_norm_gate");

@@ -72,6 +72,10 @@ KESTREL_API int kestrel_moe_route(const float *z_part, int S, long long slice_st
 // the sum of its two largest choice scores (its only one where a group is one expert), and only experts of the `keep`
 // best groups can be chosen.  Weights: the chosen experts' s divided by their sum (+ 1e-20), times `scale`.  Among equal
 // scores the lowest index wins.  A warp a token; all float32.
+//
+// Other routers of this form, by parameters: `softmax` - the scores are the softmax of z over all E outputs; `group_max` - a
+// group's score is its largest choice score; `renorm` 0 - the weights are the chosen scores as they are, times `scale`.  The
+// logits may be the first E of `ld` columns of a wider product.
 __device__ __forceinline__ void warp_argmax(float &best, int &arg) {
     for (int o = 16; o > 0; o >>= 1) {
         const float ob = __shfl_xor_sync(0xffffffffu, best, o);
@@ -81,18 +85,30 @@ __device__ __forceinline__ void warp_argmax(float &best, int &arg) {
 }
 
 __global__ void __launch_bounds__(32)
-moe_route_sigmoid_kernel(const float *__restrict__ z_part, int S, size_t slice_stride, const float *__restrict__ correction, int E, int top,
-                         int n_groups, int keep, float scale, int *__restrict__ ids, float *__restrict__ weights) {
+moe_route_scored_kernel(const float *__restrict__ z_part, int S, size_t slice_stride, int ld, const float *__restrict__ correction, int E, int top,
+                        int n_groups, int keep, float scale, int softmax, int group_max, int renorm, int *__restrict__ ids,
+                        float *__restrict__ weights) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float rs[];
     float *s = rs, *choice = rs + E, *gs = rs + 2 * E;          // s [E], choice [E], gs [n_groups]
     const int t = blockIdx.x, lane = threadIdx.x;
+    float zmax = -INFINITY, zsum = 0.f;
     for (int e = lane; e < E; e += 32) {
-        const float z = sum_slices(z_part, S, slice_stride, (size_t)t * E + e);
-        s[e] = 1.0f / (1.0f + expf(-z));
-        choice[e] = s[e] + (correction ? correction[e] : 0.f);
+        const float z = sum_slices(z_part, S, slice_stride, (size_t)t * ld + e);
+        s[e] = softmax ? z : 1.0f / (1.0f + expf(-z));
+        zmax = fmaxf(zmax, z);
     }
+    if (softmax) {
+        zmax = warp_max(zmax);
+        for (int e = lane; e < E; e += 32) {
+            s[e] = expf(s[e] - zmax);
+            zsum += s[e];
+        }
+        zsum = warp_sum(zsum);
+        for (int e = lane; e < E; e += 32) s[e] = s[e] / zsum;
+    }
+    for (int e = lane; e < E; e += 32) choice[e] = s[e] + (correction ? correction[e] : 0.f);
     __syncwarp();
     if (n_groups > 1 && keep < n_groups) {
         const int per = E / n_groups;
@@ -103,7 +119,7 @@ moe_route_sigmoid_kernel(const float *__restrict__ z_part, int S, size_t slice_s
                 if (v > a) { b = a; a = v; }
                 else if (v > b) b = v;
             }
-            gs[g] = per > 1 ? a + b : a;
+            gs[g] = per > 1 && !group_max ? a + b : a;
         }
         __syncwarp();
         // the groups that stay are marked by +inf; then every expert of another group is closed
@@ -136,29 +152,36 @@ moe_route_sigmoid_kernel(const float *__restrict__ z_part, int S, size_t slice_s
     }
     float denom = lane < top ? mine : 0.f;
     for (int o = 16; o > 0; o >>= 1) denom += __shfl_xor_sync(0xffffffffu, denom, o);
-    if (lane < top) weights[(size_t)t * top + lane] = mine / (denom + 1e-20f) * scale;
+    if (lane < top) weights[(size_t)t * top + lane] = (renorm ? mine / (denom + 1e-20f) : mine) * scale;
 }
 
 KESTREL_API int kestrel_moe_route_sigmoid(const float *z_part, int S, long long slice_stride, const float *correction, int n_groups, int keep,
                                           float scale, int *ids, float *weights, int T, int E, int top, cudaStream_t stream) {
+    return kestrel_moe_route_scored(z_part, S, slice_stride, E, correction, n_groups, keep, scale, 0, 0, 1, ids, weights, T, E, top, stream);
+}
+
+KESTREL_API int kestrel_moe_route_scored(const float *z_part, int S, long long slice_stride, int ld, const float *correction, int n_groups, int keep,
+                                         float scale, int softmax, int group_max, int renorm, int *ids, float *weights, int T, int E, int top,
+                                         cudaStream_t stream) {
     if (T == 0) return 0;
-    KESTREL_REQUIRE(T > 0 && E > 0 && top > 0 && top <= E && top <= 32 && S > 0, "moe_route_sigmoid: bad sizes E=%d top=%d", E, top);
-    KESTREL_REQUIRE(E <= 4096, "moe_route_sigmoid: %d experts exceed 4096", E);
+    KESTREL_REQUIRE(T > 0 && E > 0 && top > 0 && top <= E && top <= 32 && S > 0 && ld >= E, "moe_route_scored: bad sizes E=%d top=%d", E, top);
+    KESTREL_REQUIRE(E <= 4096, "moe_route_scored: %d experts exceed 4096", E);
     KESTREL_REQUIRE(n_groups >= 1 && E % n_groups == 0 && keep >= 1 && keep <= n_groups && (long long)keep * (E / n_groups) >= top,
-                    "moe_route_sigmoid: %d groups of %d experts, %d kept, %d chosen", n_groups, E, keep, top);
-    kestrel_launch(moe_route_sigmoid_kernel, dim3(T), dim3(32), (size_t)(2 * E + n_groups) * sizeof(float), stream, z_part, S, (size_t)slice_stride,
-                   correction, E, top, n_groups, keep, scale, ids, weights);
-    return kestrel_check_launch("moe_route_sigmoid");
+                    "moe_route_scored: %d groups of %d experts, %d kept, %d chosen", n_groups, E, keep, top);
+    kestrel_launch(moe_route_scored_kernel, dim3(T), dim3(32), (size_t)(2 * E + n_groups) * sizeof(float), stream, z_part, S, (size_t)slice_stride, ld,
+                   correction, E, top, n_groups, keep, scale, softmax, group_max, renorm, ids, weights);
+    return kestrel_check_launch("moe_route_scored");
 }
 
 // ------------------------------------------------------------------------------------------
 // One block groups the P = T * top pairs by expert.
 //   offsets [E + 1]; row_pair [P]: pair of sorted row r; pair_row [P]: sorted row of a pair;
 //   tile_expert / tile_row0 [ceil(P / rows) + E]; n_tiles [1]
+// Only the first `with_tiles` of the E router outputs get tiles: outputs behind them have no matrices (identity experts).
 // ------------------------------------------------------------------------------------------
 #define MG_THREADS 1024
 __global__ void __launch_bounds__(MG_THREADS)
-moe_group_kernel(const int *__restrict__ ids, int P, int E, int rows_per_tile, int *__restrict__ offsets, int *__restrict__ row_pair,
+moe_group_kernel(const int *__restrict__ ids, int P, int E, int with_tiles, int rows_per_tile, int *__restrict__ offsets, int *__restrict__ row_pair,
                  int *__restrict__ pair_row, int *__restrict__ tile_expert, int *__restrict__ tile_row0, int *__restrict__ n_tiles) {
     pdl_launch_dependents();
     pdl_wait();
@@ -172,7 +195,7 @@ moe_group_kernel(const int *__restrict__ ids, int P, int E, int rows_per_tile, i
         int acc = 0, nt = 0;
         for (int e = 0; e < E; ++e) {
             off[e] = acc;
-            for (int r = 0; r < cnt[e]; r += rows_per_tile) {
+            for (int r = 0; e < with_tiles && r < cnt[e]; r += rows_per_tile) {
                 tile_expert[nt] = e;
                 tile_row0[nt] = acc + r;
                 ++nt;
@@ -199,9 +222,14 @@ moe_group_kernel(const int *__restrict__ ids, int P, int E, int rows_per_tile, i
 
 KESTREL_API int kestrel_moe_group(const int *ids, int P, int E, int rows_per_tile, int *offsets, int *row_pair, int *pair_row, int *tile_expert,
                                   int *tile_row0, int *n_tiles, cudaStream_t stream) {
+    return kestrel_moe_group_some(ids, P, E, E, rows_per_tile, offsets, row_pair, pair_row, tile_expert, tile_row0, n_tiles, stream);
+}
+
+KESTREL_API int kestrel_moe_group_some(const int *ids, int P, int E, int with_tiles, int rows_per_tile, int *offsets, int *row_pair, int *pair_row,
+                                       int *tile_expert, int *tile_row0, int *n_tiles, cudaStream_t stream) {
     if (P == 0) return 0;
-    KESTREL_REQUIRE(P > 0 && E > 0 && E <= 8192 && rows_per_tile > 0, "moe_group: bad sizes");
-    kestrel_launch(moe_group_kernel, dim3(1), dim3(MG_THREADS), (size_t)(2 * E + 1) * sizeof(int), stream, ids, P, E, rows_per_tile, offsets, row_pair,
+    KESTREL_REQUIRE(P > 0 && E > 0 && E <= 8192 && with_tiles >= 0 && with_tiles <= E && rows_per_tile > 0, "moe_group: bad sizes");
+    kestrel_launch(moe_group_kernel, dim3(1), dim3(MG_THREADS), (size_t)(2 * E + 1) * sizeof(int), stream, ids, P, E, with_tiles, rows_per_tile, offsets, row_pair,
                    pair_row, tile_expert, tile_row0, n_tiles);
     return kestrel_check_launch("moe_group");
 }
@@ -227,7 +255,9 @@ __device__ __forceinline__ float expert_up_act(float z, int kind) {
     return r * r;
 }
 
+// a gated expert's activation: clamped as above, or with a negative `limit` the plain one, silu(g) u
 __device__ __forceinline__ float expert_act(float g, float u, float limit) {
+    if (limit < 0.f) return g / (1.0f + expf(-g)) * u;
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g * (1.0f / (1.0f + expf(-1.702f * g))) * (u + 1.0f);
@@ -593,4 +623,60 @@ KESTREL_API int kestrel_moe_combine(const float *y, const int *pair_row, int top
     KESTREL_REQUIRE(T > 0 && N > 0 && top > 0, "moe_combine: bad sizes");
     kestrel_launch(moe_combine_kernel, dim3(T), dim3(256), 0, stream, y, pair_row, top, out, N);
     return kestrel_check_launch("moe_combine");
+}
+
+// The same for a feed-forward with more to add.  Choices with ids >= `experts` are identity experts: they add their weight times
+// the token's input row x[t].  Where `shared` (float32 slices) is given - an expert that every token takes - it is added last, times
+// sigmoid(column sg_col of the product z) where `z_part` is given.
+template <typename T>
+__global__ void moe_combine_with_kernel(const float *__restrict__ y, const int *__restrict__ pair_row, const int *__restrict__ ids,
+                                        const float *__restrict__ weights, int top, int experts, const T *__restrict__ x, long long ldx,
+                                        const float *__restrict__ shared, int Ss, size_t shared_stride, const float *__restrict__ z_part, int Sz,
+                                        size_t z_stride, int z_ld, int sg_col, float *__restrict__ out, int N) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float direct_s;                        // the identity experts' weights, summed in the order of choice
+    __shared__ float gate_s;
+    __shared__ int row_s[32];                         // top <= 32; -1 for an identity expert
+    const int t = blockIdx.x;
+    if (threadIdx.x < 32) {
+        const int k = threadIdx.x;
+        const bool in = k < top;
+        const int id = in ? ids[(size_t)t * top + k] : 0;
+        row_s[k] = in && id < experts ? pair_row[(size_t)t * top + k] : -1;
+        const float w = in && id >= experts ? weights[(size_t)t * top + k] : 0.f;
+        const float sum = warp_sum(w);
+        if (k == 0) {
+            direct_s = sum;
+            gate_s = z_part ? 1.0f / (1.0f + expf(-sum_slices(z_part, Sz, z_stride, (size_t)t * z_ld + sg_col))) : 1.0f;
+        }
+    }
+    __syncthreads();
+    const float direct = direct_s, gate = gate_s;
+    for (int n = threadIdx.x; n < N; n += blockDim.x) {
+        float v = 0.f;
+        for (int k = 0; k < top; ++k)
+            if (row_s[k] >= 0) v += y[(size_t)row_s[k] * N + n];
+        if (direct != 0.f) v = fmaf(direct, to_f32<T>(x[(size_t)t * ldx + n]), v);
+        if (shared) v = fmaf(gate, sum_slices(shared, Ss, shared_stride, (size_t)t * N + n), v);
+        out[(size_t)t * N + n] = v;
+    }
+}
+
+KESTREL_API int kestrel_moe_combine_with(const float *y, const int *pair_row, const int *ids, const float *weights, int top, int experts,
+                                         const void *x, int dtype, long long ldx, const float *shared, int Ss, long long shared_stride,
+                                         const float *z_part, int Sz, long long z_stride, int z_ld, int sg_col, float *out, int T, int N,
+                                         cudaStream_t stream) {
+    if (T == 0) return 0;
+    KESTREL_REQUIRE(T > 0 && N > 0 && top > 0 && top <= 32 && experts >= 0 && (!shared || Ss > 0) && (!z_part || (Sz > 0 && sg_col >= 0 && sg_col < z_ld)),
+                    "moe_combine_with: bad sizes");
+    if (dtype == KESTREL_F32)
+        kestrel_launch(moe_combine_with_kernel<float>, dim3(T), dim3(256), 0, stream, y, pair_row, ids, weights, top, experts, (const float *)x, ldx,
+                       shared, Ss, (size_t)shared_stride, z_part, Sz, (size_t)z_stride, z_ld, sg_col, out, N);
+    else if (dtype == KESTREL_BF16)
+        kestrel_launch(moe_combine_with_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, y, pair_row, ids, weights, top, experts,
+                       (const __nv_bfloat16 *)x, ldx, shared, Ss, (size_t)shared_stride, z_part, Sz, (size_t)z_stride, z_ld, sg_col, out, N);
+    else
+        return kestrel_fail(-2, "moe_combine_with: unknown dtype %d", dtype);
+    return kestrel_check_launch("moe_combine_with");
 }

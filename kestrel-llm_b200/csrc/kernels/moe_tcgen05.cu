@@ -134,7 +134,9 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__
                         for (int j = 0; j < 16; ++j)
                             if (c + j < valid) {
                                 const float gg = fminf(g[j], limit), uu = fminf(fmaxf(u[j], -limit), limit);
-                                o[(size_t)(t0 + c + j) * ldo + n] = __float2bfloat16_rn(gg * (1.0f / (1.0f + expf(-1.702f * gg))) * (uu + 1.0f));
+                                // a negative limit: silu(g) u, without the clamp
+                                const float a = limit < 0.f ? g[j] / (1.0f + expf(-g[j])) * u[j] : gg * (1.0f / (1.0f + expf(-1.702f * gg))) * (uu + 1.0f);
+                                o[(size_t)(t0 + c + j) * ldo + n] = __float2bfloat16_rn(a);
                             }
                     }
                 } else if (!pair_weight) {          // an up product of experts without a gate: the activation `limit` names

@@ -6,6 +6,7 @@
 // A product reaches these kernels as float32 slices [S, T, N] that are summed in ascending s, as
 // everywhere in the library; all sums and norms are float32.
 #include "common.cuh"
+#include "xielu.cuh"
 #include <math.h>
 
 // ------------------------------------------------------------------------------------------
@@ -169,7 +170,8 @@ KESTREL_API int kestrel_partial_columns(const float *p, int S, long long slice_s
 }
 
 // ------------------------------------------------------------------------------------------
-// The same with an activation on the summed columns: 0 none, 1 the square of relu, 2 tanh, 3 silu, 4 gelu (erf), 5 gelu (tanh form).
+// The same with an activation on the summed columns: 0 none, 1 the square of relu, 2 tanh, 3 silu, 4 gelu (erf), 5 gelu (tanh
+// form), 6 xIELU with its two numbers in `act_p` (xielu.cuh).
 // ------------------------------------------------------------------------------------------
 __device__ __forceinline__ float column_act(float z, int act) {
     if (act == 4) return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));                                   // the exact gelu
@@ -182,7 +184,8 @@ __device__ __forceinline__ float column_act(float z, int act) {
 
 template <typename TOut>
 __global__ void partial_columns_act_kernel(const float *__restrict__ p, int S, size_t slice_stride, int ld, int col0,
-                                           const float *__restrict__ bias, int act, TOut *__restrict__ out, int n, size_t total) {
+                                           const float *__restrict__ bias, int act, const float *__restrict__ act_p,
+                                           TOut *__restrict__ out, int n, size_t total) {
     pdl_launch_dependents();
     pdl_wait();
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -191,19 +194,24 @@ __global__ void partial_columns_act_kernel(const float *__restrict__ p, int S, s
     int i = (int)(idx % n);
     float z = sum_slices(p, S, slice_stride, t * ld + col0 + i);
     if (bias) z += bias[col0 + i];
-    out[idx] = from_f32<TOut>(column_act(z, act));
+    out[idx] = from_f32<TOut>(act == 6 ? Xielu(act_p)(z) : column_act(z, act));
 }
 
 KESTREL_API int kestrel_partial_columns_act(const float *p, int S, long long slice_stride, int ld, int col0, const float *bias, int act, void *out,
                                             int dtype, int T, int n, cudaStream_t stream) {
+    return kestrel_partial_columns_act_with(p, S, slice_stride, ld, col0, bias, act, nullptr, out, dtype, T, n, stream);
+}
+
+KESTREL_API int kestrel_partial_columns_act_with(const float *p, int S, long long slice_stride, int ld, int col0, const float *bias, int act,
+                                                 const float *act_p, void *out, int dtype, int T, int n, cudaStream_t stream) {
     if (T == 0) return 0;
-    KESTREL_REQUIRE(T > 0 && n > 0 && S > 0 && col0 >= 0 && col0 + n <= ld && act >= 0 && act <= 5, "partial_columns_act: bad sizes or activation %d", act);
+    KESTREL_REQUIRE(T > 0 && n > 0 && S > 0 && col0 >= 0 && col0 + n <= ld && act >= 0 && act <= 6 && (act != 6 || act_p), "partial_columns_act: bad sizes or activation %d", act);
     size_t total = (size_t)T * n;
     unsigned blocks = (unsigned)((total + 255) / 256);
     if (dtype == KESTREL_F32)
-        kestrel_launch(partial_columns_act_kernel<float>, dim3(blocks), dim3(256), 0, stream, p, S, (size_t)slice_stride, ld, col0, bias, act, (float *)out, n, total);
+        kestrel_launch(partial_columns_act_kernel<float>, dim3(blocks), dim3(256), 0, stream, p, S, (size_t)slice_stride, ld, col0, bias, act, act_p, (float *)out, n, total);
     else if (dtype == KESTREL_BF16)
-        kestrel_launch(partial_columns_act_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, p, S, (size_t)slice_stride, ld, col0, bias, act, (__nv_bfloat16 *)out, n, total);
+        kestrel_launch(partial_columns_act_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, p, S, (size_t)slice_stride, ld, col0, bias, act, act_p, (__nv_bfloat16 *)out, n, total);
     else
         return kestrel_fail(-2, "partial_columns_act: unknown dtype %d", dtype);
     return kestrel_check_launch("partial_columns_act");
@@ -299,6 +307,7 @@ KESTREL_API int kestrel_combine_normed(const float *a, int Sa, long long stride_
 //     residual[t] += (y * sigmoid(g)) / sqrt(mean((y * sigmoid(g))^2) + eps) * w
 // and, where `next_w` is given, the next norm of the stream is made in the same pass:
 //     next_out[t] = residual[t] / sqrt(mean(residual[t]^2) + eps_next) * next_w       (storage type)
+// or, with `next_out` but no `next_w`, the stream itself in the storage type (sublayers that read it unnormed).
 // ------------------------------------------------------------------------------------------
 template <typename TOut, int Q>
 __global__ void __launch_bounds__(GN_VT_MAX / Q, 2 * Q)          // 2,048 threads an SM in every form
@@ -336,6 +345,10 @@ add_gated_normed_kernel(float *__restrict__ residual, const float *__restrict__ 
             {
                 const float x = residual[(size_t)t * d + i] + gn_row[i] * rn * w[i];
                 residual[(size_t)t * d + i] = x;
+                if (!next_w) {
+                    if (next_out) next_out[(size_t)t * d + i] = from_f32<TOut>(x);
+                    continue;
+                }
                 gn_row[i] = x;
                 s2[q] = fmaf(x, x, s2[q]);
             }
@@ -350,13 +363,13 @@ KESTREL_API int kestrel_add_gated_normed(float *residual, const float *y, int Sy
                                          long long stride_g, const float *g_bias, const float *w, float eps, const float *next_w, float eps_next,
                                          void *next_out, int next_dtype, int T, int d, cudaStream_t stream) {
     if (T == 0) return 0;
-    KESTREL_REQUIRE(T > 0 && d > 0 && Sy > 0 && (!g || Sg > 0) && d <= 12000 && ((next_w == nullptr) == (next_out == nullptr)),
+    KESTREL_REQUIRE(T > 0 && d > 0 && Sy > 0 && (!g || Sg > 0) && d <= 12000 && (!next_w || next_out),
                     "add_gated_normed: bad arguments T=%d d=%d", T, d);
     const int Q = gn_fold(T, d);
 #define GN_LAUNCH(TT, QQ) kestrel_launch(add_gated_normed_kernel<TT, QQ>, dim3(T), dim3(gn_threads(d) / QQ), (size_t)d * sizeof(float), stream, residual, y, Sy, \
                    (size_t)stride_y, y_bias, g, Sg, (size_t)stride_g, g_bias, w, eps, next_w, eps_next, (TT *)next_out, d)
 #define GN_LAUNCH_Q(TT) do { if (Q == 4) GN_LAUNCH(TT, 4); else if (Q == 2) GN_LAUNCH(TT, 2); else GN_LAUNCH(TT, 1); } while (0)
-    if (next_dtype == KESTREL_F32 || !next_w) GN_LAUNCH_Q(float);
+    if (next_dtype == KESTREL_F32 || !next_out) GN_LAUNCH_Q(float);
     else if (next_dtype == KESTREL_BF16) GN_LAUNCH_Q(__nv_bfloat16);
     else return kestrel_fail(-2, "add_gated_normed: unknown dtype %d", next_dtype);
 #undef GN_LAUNCH_Q

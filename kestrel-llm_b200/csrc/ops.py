@@ -151,6 +151,16 @@ class Partials:
         return out
 
 
+class StreamCopy:
+    """The residual stream in the storage type, handed from block to block in the place of a pending product by blocks whose
+    sublayers read the stream unnormed: nothing is left to add.  ``data`` [T, width]."""
+
+    __slots__ = ("data",)
+
+    def __init__(self, data: torch.Tensor):
+        self.data = data
+
+
 def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
     """out[t] = table[ids[t]] widened to float32, times ``scale``."""
     _need(table, "embed.table", dims=2)
@@ -496,19 +506,21 @@ def linear_add_into(x: torch.Tensor, w: torch.Tensor, residual: torch.Tensor) ->
     return True
 
 
-def linear_act(x: torch.Tensor, w: torch.Tensor, act: str, weights_static: bool = False) -> torch.Tensor:
-    """act(x w^T) in x's dtype, ``act`` one of `COLUMN_ACTS`.  bfloat16 with many tokens: the activation is the
+def linear_act(x: torch.Tensor, w: torch.Tensor, act: str, weights_static: bool = False, bias: Optional[torch.Tensor] = None,
+               act_params: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """act(x w^T + bias) in x's dtype, ``act`` one of `COLUMN_ACTS` (``act_params``: the numbers of one that has any).  bfloat16 with many tokens: the activation is the
     product's epilogue and the float32 product never reaches memory; otherwise the product comes as slices and
     `partial_columns_act` sums and activates them.  Both ways give the same bits where the product is one slice."""
     T, N = x.shape[0], w.shape[0]
-    if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.dim() == 2 and w.dim() == 2 and linear_act_fused:
+    if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.dim() == 2 and w.dim() == 2 and linear_act_fused and \
+            bias is None and act_params is None:
         out = torch.empty((T, N), dtype=torch.bfloat16, device=x.device)
         rc = library().kestrel_gemm_tc_act(x.data_ptr(), w.data_ptr(), out.data_ptr(), COLUMN_ACTS[act], T, N, x.shape[1], x.stride(0),
                                            w.stride(0), out.stride(0), _stream())
         if rc != 1:
             _check(rc)
             return out
-    return partial_columns_act(Partials(linear(x, w, weights_static=weights_static)), 0, N, x.dtype, act)
+    return partial_columns_act(Partials(linear(x, w, weights_static=weights_static), bias), 0, N, x.dtype, act, act_params)
 
 
 linear_act_fused = True          # tests switch the epilogue form off to hold both forms against each other
@@ -730,7 +742,7 @@ def attention(planner: Optional[AttentionPlanner], q: torch.Tensor, k_cache: tor
     the tiling of their rows and the cutting of key ranges into slices are decided natively
     (csrc/kernels/attention_dispatch.cu); float32 always takes the plain kernel."""
     _need(q, "attention.q", dims=2)
-    _need(out, "attention.out", q.dtype, 2)
+    _need(out, "attention.out", None if out.dtype == torch.float32 else q.dtype, 2)
     _need(k_cache, "attention.k_cache", q.dtype, 4)
     _need(v_cache, "attention.v_cache", q.dtype, 4)
     if q.shape[1] != nq * hd or out.shape != q.shape:
@@ -821,19 +833,26 @@ def partial_columns(p: Partials, col0: int, n: int, dtype: torch.dtype) -> torch
     return out
 
 
-COLUMN_ACTS = {None: 0, "none": 0, "relu2": 1, "tanh": 2, "silu": 3, "gelu": 4, "gelu_tanh": 5}
+COLUMN_ACTS = {None: 0, "none": 0, "relu2": 1, "tanh": 2, "silu": 3, "gelu": 4, "gelu_tanh": 5, "xielu": 6}
 
 
-def partial_columns_act(p: Partials, col0: int, n: int, dtype: torch.dtype, act: Optional[str]) -> torch.Tensor:
+def partial_columns_act(p: Partials, col0: int, n: int, dtype: torch.dtype, act: Optional[str],
+                        act_params: Optional[torch.Tensor] = None) -> torch.Tensor:
     """act(columns [col0, col0 + n) of a product, summed over its slices, plus its bias) in ``dtype``;
-    ``act`` None, "relu2" (the square of relu), "tanh", "silu", "gelu" (the exact one, with erf) or "gelu_tanh"."""
+    ``act`` None, "relu2" (the square of relu), "tanh", "silu", "gelu" (the exact one, with erf), "gelu_tanh" or "xielu" (with its two numbers in ``act_params``)."""
     if act not in COLUMN_ACTS:
         raise KernelError(f"partial_columns_act: activation {act!r} is none of {', '.join(str(k) for k in COLUMN_ACTS)}")
     out = torch.empty((p.tokens, n), dtype=dtype, device=p.data.device)
     if p.bias is not None and p.bias.shape[0] != p.width:
         raise KernelError("partial_columns_act: the bias does not fit the product's columns")
-    _check(library().kestrel_partial_columns_act(p.data.data_ptr(), p.slices, p.slice_stride, p.width, int(col0), _p(p.bias), COLUMN_ACTS[act],
-                                                 out.data_ptr(), _code(out, "partial_columns_act.out"), p.tokens, int(n), _stream()))
+    if (act == "xielu") != (act_params is not None):
+        raise KernelError(f"partial_columns_act: activation {act!r} {'needs its numbers' if act == 'xielu' else 'has no numbers of its own'}")
+    if act_params is not None:
+        _need(act_params, "partial_columns_act.act_params", torch.float32, 1)
+        if act_params.shape[0] != 2:
+            raise KernelError("partial_columns_act: xielu has two numbers")
+    _check(library().kestrel_partial_columns_act_with(p.data.data_ptr(), p.slices, p.slice_stride, p.width, int(col0), _p(p.bias), COLUMN_ACTS[act],
+                                                 _p(act_params), out.data_ptr(), _code(out, "partial_columns_act.out"), p.tokens, int(n), _stream()))
     return out
 
 
@@ -853,19 +872,21 @@ def combine_normed(a: Partials, wa: torch.Tensor, b: Partials, wb: torch.Tensor,
 def add_gated_normed(residual: torch.Tensor, y: Partials, gate: Optional[Partials], weight: torch.Tensor, eps: float,
                      next_weight: Optional[torch.Tensor] = None, next_eps: float = 0.0, next_out: Optional[torch.Tensor] = None) -> None:
     """residual += rmsnorm(y * sigmoid(gate)) * weight, y and gate the sums of their slices plus their
-    biases (no gate: y alone); with ``next_weight`` also next_out = rmsnorm(residual) * next_weight."""
+    biases (no gate: y alone); with ``next_weight`` also next_out = rmsnorm(residual) * next_weight, with ``next_out`` alone
+    next_out = residual in its own dtype."""
     _need(residual, "add_gated_normed.residual", torch.float32, 2)
     _need(weight, "add_gated_normed.weight", torch.float32, 1)
     T, d = residual.shape
     for p in (y, gate):
         if p is not None and (p.tokens != T or p.width != d or (p.bias is not None and p.bias.shape[0] != d)):
             raise KernelError("add_gated_normed: a product does not fit the residual stream")
-    if (next_weight is None) != (next_out is None):
-        raise KernelError("add_gated_normed: the next norm needs its weight and its output")
+    if next_weight is not None and next_out is None:
+        raise KernelError("add_gated_normed: the next norm needs its output")
     if next_out is not None:
         _need(next_out, "add_gated_normed.next_out", dims=2)
-        _need(next_weight, "add_gated_normed.next_weight", torch.float32, 1)
-        if next_out.shape != residual.shape or next_weight.shape[0] != d:
+        if next_weight is not None:
+            _need(next_weight, "add_gated_normed.next_weight", torch.float32, 1)
+        if next_out.shape != residual.shape or (next_weight is not None and next_weight.shape[0] != d):
             raise KernelError("add_gated_normed: the next norm's shapes differ")
     if weight.shape[0] != d:
         raise KernelError("add_gated_normed: the weight does not fit the row")
@@ -922,7 +943,7 @@ QK_NORM_MODES = {None: 0, False: 0, "none": 0, True: 1, "head": 1, "projection":
 def attn_prepare_ex(qkv: Partials, q_norm_w: Optional[torch.Tensor], k_norm_w: Optional[torch.Tensor], qk_norm, norm_eps: float,
                     positions: torch.Tensor, seq_of_token: torch.Tensor, block_table: torch.Tensor, page_size: int,
                     k_cache: torch.Tensor, v_cache: torch.Tensor, q_out: torch.Tensor, gate_out: Optional[torch.Tensor],
-                    nq: int, nkv: int, hd: int, vd: int, has_kv: bool, v_norm: bool = False, rotation=None, q_temp=None) -> None:
+                    nq: int, nkv: int, hd: int, vd: int, has_kv: bool, v_norm: bool = False, rotation=None, q_temp=None, maps: int = 1, q_pad: bool = False) -> None:
     """Columns [q | k | v | gate] of a fused product, plus the product's bias where it carries one:
     q and k divided by their root mean square - ``qk_norm`` "head" (or True): per head, times a
     weight [hd] where given; "projection": over all of q's columns at once and all of k's, times
@@ -930,13 +951,15 @@ def attn_prepare_ex(qkv: Partials, q_norm_w: Optional[torch.Tensor], k_norm_w: O
     ``q_out``, k and v into the cache pages (absent if ``has_kv`` is False), sigmoid of the gate
     columns to ``gate_out`` float32 [T, nq].  With ``rotation`` (a `Rotation` of parts/base.py: frequencies,
     rotated size, pairing, scale) q and k are turned by position after their norm.  ``q_temp`` = (coef, every): q
-    times 1 + coef ln(floor((position + 1) / every) + 1), a temperature that grows with the position."""
+    times 1 + coef ln(floor((position + 1) / every) + 1), a temperature that grows with the position.  ``maps`` > 1: a head
+    has that many queries and keys of size ``hd``, laid out [head][map], over one value; a cache row holds the maps' keys one
+    after the other, and with ``q_pad`` a query row has a cache row's length, zero outside its own map's place."""
     _need(q_out, "attn_prepare_ex.q_out", dims=2)
     _need(block_table, "attn_prepare_ex.block_table", torch.int32, 2)
     _need(k_cache, "attn_prepare_ex.k_cache", q_out.dtype, 4)
     _need(v_cache, "attn_prepare_ex.v_cache", q_out.dtype, 4)
     T = q_out.shape[0]
-    if qkv.tokens != T or q_out.shape[1] != nq * hd:
+    if qkv.tokens != T or q_out.shape[1] != nq * maps * hd * (maps if q_pad else 1):
         raise KernelError("attn_prepare_ex: shapes differ")
     if qk_norm not in QK_NORM_MODES:
         raise KernelError(f"attn_prepare_ex: qk_norm {qk_norm!r} is none of None, 'head', 'projection'")
@@ -949,7 +972,7 @@ def attn_prepare_ex(qkv: Partials, q_norm_w: Optional[torch.Tensor], k_norm_w: O
         for w, n, name in ((q_norm_w, nq * hd, "q"), (k_norm_w, nkv * hd, "k")):
             if (w is None and (name == "q" or has_kv)) or (w is not None and (w.dtype != torch.float32 or w.numel() != n)):
                 raise KernelError(f"attn_prepare_ex: the norm over the whole {name} projection needs a float32 weight of {n} entries")
-    if tuple(k_cache.shape[1:]) != (nkv, page_size, hd) or tuple(v_cache.shape[1:]) != (nkv, page_size, vd):
+    if tuple(k_cache.shape[1:]) != (nkv, page_size, maps * hd) or tuple(v_cache.shape[1:]) != (nkv, page_size, vd):
         raise KernelError("attn_prepare_ex: the cache planes do not fit the heads")
     if gate_out is not None:
         _need(gate_out, "attn_prepare_ex.gate_out", torch.float32, 2)
@@ -966,11 +989,11 @@ def attn_prepare_ex(qkv: Partials, q_norm_w: Optional[torch.Tensor], k_norm_w: O
     t_coef, t_every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 0)
     if q_temp and t_every <= 0:
         raise KernelError("attn_prepare_ex: a query temperature needs a positive number of positions a step")
-    _check(library().kestrel_attn_prepare_tempered(
+    _check(library().kestrel_attn_prepare_maps(
         qkv.data.data_ptr(), qkv.slices, qkv.slice_stride, qkv.width, _p(qkv.bias), _p(q_norm_w), _p(k_norm_w), mode, 1 if v_norm else 0,
         float(norm_eps), _p(inv_freq), rot or 0, rot_mode or 0, float(rotation.scale) if rotation is not None else 1.0, t_coef, t_every, positions.data_ptr(), seq_of_token.data_ptr(), block_table.data_ptr(), block_table.stride(0), int(page_size),
         k_cache.data_ptr(), v_cache.data_ptr(), q_out.data_ptr(), _p(gate_out), _code(q_out, "attn_prepare_ex.q_out"), T, nq, nkv, hd, vd,
-        1 if has_kv else 0, _stream()))
+        1 if has_kv else 0, int(maps), 1 if q_pad else 0, _stream()))
 
 
 WEIGHTINGS = {"softmax": 0, "softmax_sink": 1, "sigmoid": 2}
@@ -1032,9 +1055,9 @@ def attention_plain_ex(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Te
                        score: Optional[ScoreOptions] = None, v_ld: int = 0) -> None:
     """`attention_plain` with values of size ``vd`` (the first ``vd`` numbers of V rows of ``v_ld``, where that is given), the first ``keep_first`` keys of a request
     visible beyond the window, each head's output multiplied by ``gate`` [T, nq], and the layer's
-    `ScoreOptions`."""
+    `ScoreOptions`.  ``out`` may be float32 whatever the storage type."""
     _need(q, "attention.q", dims=2)
-    _need(out, "attention.out", q.dtype, 2)
+    _need(out, "attention.out", None if out.dtype == torch.float32 else q.dtype, 2)
     _need(k_cache, "attention.k_cache", q.dtype, 4)
     _need(v_cache, "attention.v_cache", q.dtype, 4)
     _need(block_table, "attention.block_table", torch.int32, 2)
@@ -1043,10 +1066,10 @@ def attention_plain_ex(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Te
         raise KernelError("attention: shapes differ")
     if gate is not None:
         _need(gate, "attention.gate", torch.float32, 2)
-    _check(library().kestrel_attention_plain_biased(
+    _check(library().kestrel_attention_plain_to(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), positions.data_ptr(), seq_of_token.data_ptr(), block_table.data_ptr(),
-        block_table.stride(0), int(page_size), out.data_ptr(), _code(q, "attention.q"), T, nq, nkv, hd, vd, int(window), int(keep_first),
-        _p(gate), float(scale), *(score or _NO_SCORE).args(nq), *(score or _NO_SCORE).rel_args(nq), int(v_ld), _stream()))
+        block_table.stride(0), int(page_size), out.data_ptr(), _code(q, "attention.q"), 1 if out.dtype == torch.float32 else 0, T, nq, nkv, hd, vd,
+        int(window), int(keep_first), _p(gate), float(scale), *(score or _NO_SCORE).args(nq), *(score or _NO_SCORE).rel_args(nq), int(v_ld), _stream()))
 
 
 def attention_window_supported(hd: int, vd: int, nq: int, nkv: int) -> bool:
@@ -1060,9 +1083,9 @@ def attention_window(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     """`attention_plain_ex` for bfloat16 on the tensor cores, over this step's requests as ``batch``
     describes them (cumulative lengths, lengths after the step, the most tokens of one request and the
     longest context).  A step of single tokens cuts its key rounds into shares, a CTA each, and a
-    second kernel merges them (`attention_window_set_splits`)."""
+    second kernel merges them (`attention_window_set_splits`).  ``out`` is bfloat16, or float32 for heads that are combined further."""
     _need(q, "attention_window.q", torch.bfloat16, 2)
-    _need(out, "attention_window.out", torch.bfloat16, 2)
+    _need(out, "attention_window.out", None if out.dtype == torch.float32 else torch.bfloat16, 2)
     _need(k_cache, "attention_window.k_cache", torch.bfloat16, 4)
     _need(v_cache, "attention_window.v_cache", torch.bfloat16, 4)
     _need(block_table, "attention_window.block_table", torch.int32, 2)
@@ -1080,8 +1103,8 @@ def attention_window(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     scratch = None
     if ksplit > 1:
         scratch = torch.empty(lib.kestrel_attention_window_scratch_floats(int(batch.num_seqs), int(batch.max_count), nq, nkv, hd, vd, ksplit), dtype=torch.float32, device=q.device)
-    _check(lib.kestrel_attention_window_biased(
-        q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), _p(gate), batch.cu_seqlens.data_ptr(), batch.kv_lens.data_ptr(),
+    _check(lib.kestrel_attention_window_to(
+        q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), 1 if out.dtype == torch.float32 else 0, _p(gate), batch.cu_seqlens.data_ptr(), batch.kv_lens.data_ptr(),
         block_table.data_ptr(), block_table.stride(0), int(page_size), int(batch.num_seqs), int(batch.max_count), nq, nkv, hd, vd, int(window),
         int(keep_first), float(scale), *(score or _NO_SCORE).args(nq), *(score or _NO_SCORE).rel_args(nq), int(v_ld), ksplit, _p(scratch), _stream()))
     if ksplit > 1:
@@ -1113,6 +1136,26 @@ def row_tiles(batch, rows_per_token: int, rows_per_tile: int = 256):
         t = torch.tensor([seq, row0], dtype=torch.int32).to(batch.device_buffer.device, non_blocking=True)
         kept[key] = (t[0], t[1])
     return kept[key]
+
+
+# ---- differential attention: two maps a head over the same values --------------------------------
+
+def differential_combine(a: torch.Tensor, lq1: torch.Tensor, lk1: torch.Tensor, lq2: torch.Tensor, lk2: torch.Tensor, diff: float, eps: float,
+                         out: torch.Tensor, H: int, vd: int) -> None:
+    """out = (a1 - lambda a2) / its root mean square over a head's ``vd`` values * (1 - diff), a [T, H, 2, vd] float32 the maps'
+    outputs, lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff."""
+    _need(a, "differential_combine.a", torch.float32, 2)
+    _need(out, "differential_combine.out", dims=2)
+    T = out.shape[0]
+    if a.shape != (T, 2 * H * vd) or out.shape[1] != H * vd:
+        raise KernelError("differential_combine: shapes differ")
+    dim = lq1.shape[0]
+    for t in (lq1, lk1, lq2, lk2):
+        _need(t, "differential_combine.lambda", torch.float32, 1)
+        if t.shape[0] != dim:
+            raise KernelError("differential_combine: the four vectors of lambda have one size")
+    _check(library().kestrel_differential_combine(a.data_ptr(), lq1.data_ptr(), lk1.data_ptr(), lq2.data_ptr(), lk2.data_ptr(), dim, float(diff),
+                                                  float(eps), out.data_ptr(), _code(out, "differential_combine.out"), T, H, vd, _stream()))
 
 
 # ---- attention over cached latents -----------------------------------------------------------
@@ -1329,23 +1372,52 @@ def recurrence_scan(r: torch.Tensor, w: torch.Tensor, k: torch.Tensor, v: torch.
     return out
 
 
-def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, eps: float, gate: Optional[Partials], gate_col0: int, out: torch.Tensor,
-                   H: int, dv: int) -> None:
+GATE_ACTS = {"sigmoid": 0, "silu": 1}
+
+
+def head_norm_gate(o: torch.Tensor, weight: Optional[torch.Tensor], eps: float, gate: Optional[Partials], gate_col0: int, out: torch.Tensor,
+                   H: int, dv: int, gate_act: str = "sigmoid") -> None:
     """out = o / sqrt(mean(o^2) + eps) per head, times ``weight`` ([dv]: shared by the heads; [H dv]: one per
-    head), times sigmoid of the columns [gate_col0, gate_col0 + H dv) of ``gate`` where given."""
+    head; None: no weight), times ``gate_act`` (a sigmoid, or silu) of the columns [gate_col0, gate_col0 + H dv) of ``gate`` where given."""
     _need(o, "head_norm_gate.o", torch.float32, 2)
-    _need(weight, "head_norm_gate.weight", torch.float32, 1)
+    if weight is not None:
+        _need(weight, "head_norm_gate.weight", torch.float32, 1)
     _need(out, "head_norm_gate.out", dims=2)
     T = o.shape[0]
-    if o.shape[1] != H * dv or out.shape != o.shape or weight.shape[0] not in (dv, H * dv):
+    if o.shape[1] != H * dv or out.shape != o.shape or (weight is not None and weight.shape[0] not in (dv, H * dv)):
         raise KernelError("head_norm_gate: shapes differ")
     if gate is not None and (gate.tokens != T or gate.bias is not None or gate_col0 + H * dv > gate.width):
         raise KernelError("head_norm_gate: the gate's product does not fit, or carries a bias")
-    w_stride = dv if (weight.shape[0] == H * dv and H > 1) else 0
-    _check(library().kestrel_head_norm_gate(o.data_ptr(), weight.data_ptr(), w_stride, float(eps), _p(gate.data) if gate is not None else None,
+    w_stride = dv if (weight is not None and weight.shape[0] == H * dv and H > 1) else 0
+    _check(library().kestrel_head_norm_act(o.data_ptr(), _p(weight), w_stride, float(eps), _p(gate.data) if gate is not None else None,
                                             gate.slices if gate is not None else 0, gate.slice_stride if gate is not None else 0,
-                                            gate.width if gate is not None else 0, int(gate_col0), out.data_ptr(), _code(out, "head_norm_gate.out"),
+                                            gate.width if gate is not None else 0, int(gate_col0), GATE_ACTS[gate_act], out.data_ptr(), _code(out, "head_norm_gate.out"),
                                             T, H, dv, _stream()))
+
+
+# ---- retention: linear attention with a fixed decay per head -----------------------------------------
+
+def retention_prepare(fused: Partials, positions: torch.Tensor, rotation, decay: torch.Tensor, dtype: torch.dtype, H: int, d: int, dv: int,
+                      with_decay: bool = True):
+    """(q, k, v, w) of a retention from the columns [q | k | v | ...] of a fused product: q and k turned by position where a
+    ``rotation`` is given (rotate-half pairs), k times d^-1/2 afterwards, in ``dtype``; w (None without ``with_decay``) the heads'
+    decays in every key channel, float32."""
+    T, dev = fused.tokens, fused.data.device
+    if fused.bias is not None or fused.width < H * (2 * d + dv):
+        raise KernelError("retention_prepare: the product does not fit the heads, or carries a bias")
+    _need(decay, "retention_prepare.decay", torch.float32, 1)
+    if decay.shape[0] != H:
+        raise KernelError("retention_prepare: a decay per head")
+    if rotation is not None and (rotation.mode != 0 or rotation.scale != 1.0):
+        raise KernelError("retention_prepare: rotate-half pairs without a factor")
+    q, k = (torch.empty((T, H * d), dtype=dtype, device=dev) for _ in range(2))
+    v = torch.empty((T, H * dv), dtype=dtype, device=dev)
+    w = torch.empty((T, H * d), dtype=torch.float32, device=dev) if with_decay else None
+    _check(library().kestrel_retention_prepare(fused.data.data_ptr(), fused.slices, fused.slice_stride, fused.width, positions.data_ptr(),
+                                               _p(rotation.inv_freq) if rotation is not None else None, rotation.dim if rotation is not None else 0,
+                                               decay.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), _p(w), _code(q, "retention_prepare.q"),
+                                               T, H, d, dv, _stream()))
+    return q, k, v, w
 
 
 # ---- routed feed-forward -----------------------------------------------------------------------
@@ -1396,6 +1468,29 @@ def moe_route_sigmoid(z: Partials, correction: Optional[torch.Tensor], top: int,
     w = torch.empty((T, top), dtype=torch.float32, device=z.data.device)
     _check(library().kestrel_moe_route_sigmoid(z.data.data_ptr(), z.slices, z.slice_stride, _p(correction), int(groups), int(keep), float(scale),
                                                ids.data_ptr(), w.data_ptr(), T, E, top, _stream()))
+    return ids, w
+
+
+def moe_route_scored(z: Partials, n: int, correction: Optional[torch.Tensor], top: int, groups: int = 1, keep: int = 1, scale: float = 1.0,
+                     scores: str = "softmax", group_score: str = "max", renorm: bool = False):
+    """(ids int32 [T, top], weights float32 [T, top]) of a router over the first ``n`` columns of a product: scores s = softmax over the n
+    outputs or their sigmoids; outputs are chosen by s + ``correction`` among the ``keep`` best of ``groups`` equal groups of neighbours (a
+    group's score: its largest choice score, or the sum of its two largest, "top2") and weighted by s, over the chosen s' sum with
+    ``renorm``, times ``scale``."""
+    T = z.tokens
+    if z.bias is not None or z.width < n:
+        raise KernelError("moe_route_scored: the product has too few columns, or a bias is pending")
+    if scores not in ("softmax", "sigmoid") or group_score not in ("max", "top2"):
+        raise KernelError(f"moe_route_scored: scores {scores!r}, group score {group_score!r}")
+    if correction is not None:
+        _need(correction, "moe_route_scored.correction", torch.float32, 1)
+        if correction.shape[0] != n:
+            raise KernelError("moe_route_scored: a correction per router output")
+    ids = torch.empty((T, top), dtype=torch.int32, device=z.data.device)
+    w = torch.empty((T, top), dtype=torch.float32, device=z.data.device)
+    _check(library().kestrel_moe_route_scored(z.data.data_ptr(), z.slices, z.slice_stride, z.width, _p(correction), int(groups), int(keep),
+                                              float(scale), 1 if scores == "softmax" else 0, 1 if group_score == "max" else 0, 1 if renorm else 0,
+                                              ids.data_ptr(), w.data_ptr(), T, int(n), top, _stream()))
     return ids, w
 
 
@@ -1506,10 +1601,22 @@ def rglru_scan(y: torch.Tensor, u: torch.Tensor, gr: torch.Tensor, gi: torch.Ten
                                         _code(out, "rglru_scan.out"), batch.num_seqs, C, _stream()))
 
 
+class MoeExtra:
+    """What a routed feed-forward adds beside its experts: ``identity`` router outputs behind the experts whose output is the token's
+    input itself; ``shared`` (Partials), the product of an expert that every token takes, times sigmoid(column ``gate_col`` of ``z``)
+    where that product is given."""
+
+    __slots__ = ("identity", "shared", "z", "gate_col")
+
+    def __init__(self, identity: int = 0, shared: Optional[Partials] = None, z: Optional[Partials] = None, gate_col: int = 0):
+        self.identity, self.shared, self.z, self.gate_col = int(identity), shared, z, int(gate_col)
+
+
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
-                limit: float) -> torch.Tensor:
+                limit: Optional[float], extra: Optional[MoeExtra] = None) -> torch.Tensor:
     """The chosen experts' outputs, weighted and summed per token: float32 [T, width].
-    w_gate_up [E, 2 ff, width] (gate rows, then up rows), w_down [E, width, ff]."""
+    w_gate_up [E, 2 ff, width] (gate rows, then up rows), w_down [E, width, ff].  ``limit`` clamps the activation
+    min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1); None: silu(g) u."""
     _need(x, "moe.x", dims=2)
     _need(w_gate_up, "moe.w_gate_up", x.dtype, 3)
     _need(w_down, "moe.w_down", x.dtype, 3)
@@ -1519,42 +1626,52 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     N = w_down.shape[1]
     if w_gate_up.shape[2] != K or w_down.shape != (E, N, ff) or ids.shape[0] != T:
         raise KernelError("moe_experts: shapes differ")
-    lib, dev, P = library(), x.device, T * top
+    lim = -1.0 if limit is None else float(limit)
+    lib, dev, P, outputs = library(), x.device, T * top, E + (extra.identity if extra is not None else 0)
     act = torch.empty((P, ff), dtype=x.dtype, device=dev)
     y = torch.empty((P, N), dtype=torch.float32, device=dev)
     out = torch.empty((T, N), dtype=torch.float32, device=dev)
+    xs = None
     if _moe_tc and x.dtype == torch.bfloat16 and P >= MOE_TC_MIN_PAIRS and x.stride(0) % 8 == 0:
         xs = torch.empty((P, K), dtype=x.dtype, device=dev)
-        if lib.kestrel_moe_tc_supported(xs.data_ptr(), act.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), ff, K):
-            rows = lib.kestrel_moe_tc_tile_rows()
-            max_tiles = lib.kestrel_moe_max_tiles(P, E, rows)
-            meta = torch.empty((E + 1) + 2 * P + 2 * max_tiles + 1, dtype=torch.int32, device=dev)
-            offsets, row_pair, pair_row = meta[:E + 1], meta[E + 1:E + 1 + P], meta[E + 1 + P:E + 1 + 2 * P]
-            o = E + 1 + 2 * P
-            tile_expert, tile_row0, n_tiles = meta[o:o + max_tiles], meta[o + max_tiles:o + 2 * max_tiles], meta[o + 2 * max_tiles:]
-            _check(lib.kestrel_moe_group(ids.data_ptr(), P, E, rows, offsets.data_ptr(), row_pair.data_ptr(), pair_row.data_ptr(),
-                                         tile_expert.data_ptr(), tile_row0.data_ptr(), n_tiles.data_ptr(), _stream()))
-            _check(lib.kestrel_moe_gather_rows(x.data_ptr(), x.stride(0), row_pair.data_ptr(), top, xs.data_ptr(), P, K, _stream()))
-            _check(lib.kestrel_moe_gate_up_tc(xs.data_ptr(), w_gate_up.data_ptr(), offsets.data_ptr(), tile_expert.data_ptr(), tile_row0.data_ptr(),
-                                              n_tiles.data_ptr(), max_tiles, float(limit), act.data_ptr(), P, E, ff, K, _stream()))
-            _check(lib.kestrel_moe_down_tc(act.data_ptr(), w_down.data_ptr(), offsets.data_ptr(), row_pair.data_ptr(), tile_expert.data_ptr(),
-                                           tile_row0.data_ptr(), n_tiles.data_ptr(), max_tiles, weights.data_ptr(), y.data_ptr(), P, E, N, ff, _stream()))
-            _check(lib.kestrel_moe_combine(y.data_ptr(), pair_row.data_ptr(), top, out.data_ptr(), T, N, _stream()))
-            return out
-    max_tiles = lib.kestrel_moe_max_tiles(P, E, MOE_TILE_ROWS)
-    meta = torch.empty((E + 1) + 2 * P + 2 * max_tiles + 1, dtype=torch.int32, device=dev)
-    offsets, row_pair, pair_row = meta[:E + 1], meta[E + 1:E + 1 + P], meta[E + 1 + P:E + 1 + 2 * P]
-    o = E + 1 + 2 * P
+        if not lib.kestrel_moe_tc_supported(xs.data_ptr(), act.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), ff, K):
+            xs = None
+    rows = lib.kestrel_moe_tc_tile_rows() if xs is not None else MOE_TILE_ROWS
+    max_tiles = lib.kestrel_moe_max_tiles(P, E, rows)
+    meta = torch.empty((outputs + 1) + 2 * P + 2 * max_tiles + 1, dtype=torch.int32, device=dev)
+    offsets, row_pair, pair_row = meta[:outputs + 1], meta[outputs + 1:outputs + 1 + P], meta[outputs + 1 + P:outputs + 1 + 2 * P]
+    o = outputs + 1 + 2 * P
     tile_expert, tile_row0, n_tiles = meta[o:o + max_tiles], meta[o + max_tiles:o + 2 * max_tiles], meta[o + 2 * max_tiles:]
-    _check(lib.kestrel_moe_group(ids.data_ptr(), P, E, MOE_TILE_ROWS, offsets.data_ptr(), row_pair.data_ptr(), pair_row.data_ptr(),
-                                 tile_expert.data_ptr(), tile_row0.data_ptr(), n_tiles.data_ptr(), _stream()))
-    _check(lib.kestrel_moe_gate_up(x.data_ptr(), x.stride(0), w_gate_up.data_ptr(), offsets.data_ptr(), row_pair.data_ptr(),
-                                   tile_expert.data_ptr(), tile_row0.data_ptr(), n_tiles.data_ptr(), max_tiles, top, float(limit),
-                                   act.data_ptr(), _code(x, "moe.x"), ff, K, _stream()))
-    _check(lib.kestrel_moe_down(act.data_ptr(), w_down.data_ptr(), offsets.data_ptr(), row_pair.data_ptr(), tile_expert.data_ptr(),
-                                tile_row0.data_ptr(), n_tiles.data_ptr(), max_tiles, weights.data_ptr(), y.data_ptr(), _code(x, "moe.x"), N, ff,
-                                _stream()))
-    _check(lib.kestrel_moe_combine(y.data_ptr(), pair_row.data_ptr(), top, out.data_ptr(), T, N, _stream()))
+    _check(lib.kestrel_moe_group_some(ids.data_ptr(), P, outputs, E, rows, offsets.data_ptr(), row_pair.data_ptr(), pair_row.data_ptr(),
+                                      tile_expert.data_ptr(), tile_row0.data_ptr(), n_tiles.data_ptr(), _stream()))
+    if xs is not None:
+        _check(lib.kestrel_moe_gather_rows(x.data_ptr(), x.stride(0), row_pair.data_ptr(), top, xs.data_ptr(), P, K, _stream()))
+        _check(lib.kestrel_moe_gate_up_tc(xs.data_ptr(), w_gate_up.data_ptr(), offsets.data_ptr(), tile_expert.data_ptr(), tile_row0.data_ptr(),
+                                          n_tiles.data_ptr(), max_tiles, lim, act.data_ptr(), P, E, ff, K, _stream()))
+        _check(lib.kestrel_moe_down_tc(act.data_ptr(), w_down.data_ptr(), offsets.data_ptr(), row_pair.data_ptr(), tile_expert.data_ptr(),
+                                       tile_row0.data_ptr(), n_tiles.data_ptr(), max_tiles, weights.data_ptr(), y.data_ptr(), P, E, N, ff, _stream()))
+    else:
+        _check(lib.kestrel_moe_gate_up(x.data_ptr(), x.stride(0), w_gate_up.data_ptr(), offsets.data_ptr(), row_pair.data_ptr(),
+                                       tile_expert.data_ptr(), tile_row0.data_ptr(), n_tiles.data_ptr(), max_tiles, top, lim,
+                                       act.data_ptr(), _code(x, "moe.x"), ff, K, _stream()))
+        _check(lib.kestrel_moe_down(act.data_ptr(), w_down.data_ptr(), offsets.data_ptr(), row_pair.data_ptr(), tile_expert.data_ptr(),
+                                    tile_row0.data_ptr(), n_tiles.data_ptr(), max_tiles, weights.data_ptr(), y.data_ptr(), _code(x, "moe.x"), N, ff,
+                                    _stream()))
+    if extra is None:
+        _check(lib.kestrel_moe_combine(y.data_ptr(), pair_row.data_ptr(), top, out.data_ptr(), T, N, _stream()))
+        return out
+    if extra.identity and N != K:
+        raise KernelError("moe_experts: identity experts need an output as wide as the input")
+    sh, z = extra.shared, extra.z
+    if sh is not None and (sh.tokens != T or sh.width != N or sh.bias is not None):
+        raise KernelError("moe_experts: the shared expert's product does not fit, or carries a bias")
+    if z is not None and (z.tokens != T or not 0 <= extra.gate_col < z.width or z.bias is not None):
+        raise KernelError("moe_experts: the shared expert's gate is no column of its product")
+    _check(lib.kestrel_moe_combine_with(y.data_ptr(), pair_row.data_ptr(), ids.data_ptr(), weights.data_ptr(), top, E, x.data_ptr(),
+                                        _code(x, "moe.x"), x.stride(0), _p(sh.data) if sh is not None else None, sh.slices if sh is not None else 0,
+                                        sh.slice_stride if sh is not None else 0, _p(z.data) if z is not None else None,
+                                        z.slices if z is not None else 0, z.slice_stride if z is not None else 0, z.width if z is not None else 1,
+                                        extra.gate_col, out.data_ptr(), T, N, _stream()))
     return out
 
 

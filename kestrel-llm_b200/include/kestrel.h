@@ -166,6 +166,8 @@ KESTREL_API int kestrel_add_normed(float *residual, const float *p, int S, long 
 KESTREL_API int kestrel_partial_columns(const float *p, int S, long long slice_stride, int ld, int col0, void *out, int dtype, int T, int n, kestrel_stream_t stream);
 /* the same with the product's bias (NULL: none; indexed like the product's columns) and an activation on the sum: 0 none, 1 relu squared, 2 tanh, 3 silu, 4 gelu (erf), 5 gelu (tanh form) */
 KESTREL_API int kestrel_partial_columns_act(const float *p, int S, long long slice_stride, int ld, int col0, const float *bias, int act, void *out, int dtype, int T, int n, kestrel_stream_t stream);
+/* the same; act 6: xIELU with its two numbers in act_p */
+KESTREL_API int kestrel_partial_columns_act_with(const float *p, int S, long long slice_stride, int ld, int col0, const float *bias, int act, const float *act_p, void *out, int dtype, int T, int n, kestrel_stream_t stream);
 /* residual += sum of a's + b's + c's slices (b, c may be NULL), (a + b) + c; cast = residual in the storage type (may be NULL) */
 KESTREL_API int kestrel_add_three(float *residual, const float *a, int Sa, long long stride_a, const float *b, int Sb, long long stride_b, const float *c, int Sc, long long stride_c, void *cast, int cast_dtype, int T, int d, kestrel_stream_t stream);
 /* x[t, i] *= sigmoid(sum of g's slices at [t, col0 + i] + bias[col0 + i]), i < n, in place in the storage type (bias may be NULL) */
@@ -176,7 +178,7 @@ KESTREL_API int kestrel_add_row(float *x, const float *row, int T, int d, kestre
 KESTREL_API int kestrel_embed_scaled(const void *table, int dtype, const int *ids, float *out, int T, int d, float scale, kestrel_stream_t stream);
 /* out[t] = mix (a / sqrt(mean(a^2) + eps) wa + b / sqrt(mean(b^2) + eps) wb), a and b the sums of two products' slices, float32 */
 KESTREL_API int kestrel_combine_normed(const float *a, int Sa, long long stride_a, const float *wa, const float *b, int Sb, long long stride_b, const float *wb, float eps, float mix, float *out, int T, int d, kestrel_stream_t stream);
-/* v = (sum of y's slices + y_bias) * sigmoid(sum of g's slices + g_bias) (g may be NULL: no gate); residual[t] += v / sqrt(mean(v^2) + eps) w; with next_w also next_out[t] = residual[t] / sqrt(mean(residual[t]^2) + eps_next) next_w in the storage type */
+/* v = (sum of y's slices + y_bias) * sigmoid(sum of g's slices + g_bias) (g may be NULL: no gate); residual[t] += v / sqrt(mean(v^2) + eps) w; with next_w also next_out[t] = residual[t] / sqrt(mean(residual[t]^2) + eps_next) next_w in the storage type, with next_out alone the stream itself in it */
 KESTREL_API int kestrel_add_gated_normed(float *residual, const float *y, int Sy, long long stride_y, const float *y_bias, const float *g, int Sg, long long stride_g, const float *g_bias, const float *w, float eps, const float *next_w, float eps_next, void *next_out, int next_dtype, int T, int d, kestrel_stream_t stream);
 /* x[t] += table[ids[t]] */
 KESTREL_API int kestrel_embed_add(const void *table, int dtype, const int *ids, float *x, int T, int d, kestrel_stream_t stream);
@@ -199,8 +201,12 @@ KESTREL_API int kestrel_attention_window(const void *q, const void *k_cache, con
 KESTREL_API int kestrel_attention_plain_scored(const void *q, const void *k_cache, const void *v_cache, const int *positions, const int *seq_of_token, const int *block_table, int table_stride, int page_size, void *out, int dtype, int T, int nq, int nkv, int hd, int vd, int window, int keep_first, const float *gate, float scale, float softcap, const float *r1, const float *r2, const float *head_bias, int weighting, const float *sink, kestrel_stream_t stream);
 /* the same with rel[bucket[min(i - j, rel_far)], head] added to the scores: rel float32 [buckets, nq], rel_bucket int32 [rel_far + 1] (rel may be NULL); v_ld > 0: the V plane's rows hold v_ld numbers, the first vd of them the value */
 KESTREL_API int kestrel_attention_plain_biased(const void *q, const void *k_cache, const void *v_cache, const int *positions, const int *seq_of_token, const int *block_table, int table_stride, int page_size, void *out, int dtype, int T, int nq, int nkv, int hd, int vd, int window, int keep_first, const float *gate, float scale, float softcap, const float *r1, const float *r2, const float *head_bias, int weighting, const float *sink, const float *rel, const int *rel_bucket, int rel_far, int v_ld, kestrel_stream_t stream);
+/* the same; out_f32: the output is float32 whatever the storage type */
+KESTREL_API int kestrel_attention_plain_to(const void *q, const void *k_cache, const void *v_cache, const int *positions, const int *seq_of_token, const int *block_table, int table_stride, int page_size, void *out, int dtype, int out_f32, int T, int nq, int nkv, int hd, int vd, int window, int keep_first, const float *gate, float scale, float softcap, const float *r1, const float *r2, const float *head_bias, int weighting, const float *sink, const float *rel, const int *rel_bucket, int rel_far, int v_ld, kestrel_stream_t stream);
 KESTREL_API int kestrel_attention_window_scored(const void *q, const void *k_cache, const void *v_cache, void *out, const float *gate, const int *cu_seqlens, const int *kv_lens, const int *block_table, int table_stride, int page_size, int nseq, int max_count, int nq, int nkv, int hd, int vd, int window, int keep_first, float scale, float softcap, const float *r1, const float *r2, const float *head_bias, int weighting, const float *sink, int ksplit, float *scratch, kestrel_stream_t stream);
 KESTREL_API int kestrel_attention_window_biased(const void *q, const void *k_cache, const void *v_cache, void *out, const float *gate, const int *cu_seqlens, const int *kv_lens, const int *block_table, int table_stride, int page_size, int nseq, int max_count, int nq, int nkv, int hd, int vd, int window, int keep_first, float scale, float softcap, const float *r1, const float *r2, const float *head_bias, int weighting, const float *sink, const float *rel, const int *rel_bucket, int rel_far, int v_ld, int ksplit, float *scratch, kestrel_stream_t stream);
+/* the same; out_f32: the output is float32 */
+KESTREL_API int kestrel_attention_window_to(const void *q, const void *k_cache, const void *v_cache, void *out, int out_f32, const float *gate, const int *cu_seqlens, const int *kv_lens, const int *block_table, int table_stride, int page_size, int nseq, int max_count, int nq, int nkv, int hd, int vd, int window, int keep_first, float scale, float softcap, const float *r1, const float *r2, const float *head_bias, int weighting, const float *sink, const float *rel, const int *rel_bucket, int rel_far, int v_ld, int ksplit, float *scratch, kestrel_stream_t stream);
 /* a step of single tokens may cut its key rounds into `ksplit` shares, a CTA each, merged by a second kernel; scratch of kestrel_attention_window_scratch_floats floats */
 KESTREL_API int kestrel_attention_window_splits(int nseq, int max_count, int nq, int nkv, int hd, int vd, int window, int max_kv_len);
 KESTREL_API long long kestrel_attention_window_scratch_floats(int nseq, int max_count, int nq, int nkv, int hd, int vd, int ksplit);
@@ -212,6 +218,8 @@ KESTREL_API int kestrel_attn_prepare_normed(const float *partial, int S, long lo
 KESTREL_API int kestrel_attn_prepare_rotated(const float *partial, int S, long long slice_stride, int ld, const float *bias, const float *q_norm_w, const float *k_norm_w, int qk_norm, int v_norm, float norm_eps, const float *inv_freq, int rot, int rot_mode, float rot_scale, const int *positions, const int *seq_of_token, const int *block_table, int table_stride, int page_size, void *k_cache, void *v_cache, void *q_out, float *gate_out, int dtype, int T, int nq, int nkv, int hd, int vd, int has_kv, kestrel_stream_t stream);
 /* the same with a query temperature: q times 1 + q_temp_coef ln(floor((position + 1) / q_temp_every) + 1); q_temp_every = 0: none */
 KESTREL_API int kestrel_attn_prepare_tempered(const float *partial, int S, long long slice_stride, int ld, const float *bias, const float *q_norm_w, const float *k_norm_w, int qk_norm, int v_norm, float norm_eps, const float *inv_freq, int rot, int rot_mode, float rot_scale, float q_temp_coef, int q_temp_every, const int *positions, const int *seq_of_token, const int *block_table, int table_stride, int page_size, void *k_cache, void *v_cache, void *q_out, float *gate_out, int dtype, int T, int nq, int nkv, int hd, int vd, int has_kv, kestrel_stream_t stream);
+/* the same for heads of `maps` queries and keys of size hd over one value, laid out [head][map]: columns [q: nq maps hd | k: nkv maps hd | v: nkv vd | gate: nq], K pages [page][kv head][slot][maps hd], q_out [T, nq maps, hd] or, with q_pad, [T, nq maps, maps hd] with zeros outside a row's own map */
+KESTREL_API int kestrel_attn_prepare_maps(const float *partial, int S, long long slice_stride, int ld, const float *bias, const float *q_norm_w, const float *k_norm_w, int qk_norm, int v_norm, float norm_eps, const float *inv_freq, int rot, int rot_mode, float rot_scale, float q_temp_coef, int q_temp_every, const int *positions, const int *seq_of_token, const int *block_table, int table_stride, int page_size, void *k_cache, void *v_cache, void *q_out, float *gate_out, int dtype, int T, int nq, int nkv, int hd, int vd, int has_kv, int maps, int q_pad, kestrel_stream_t stream);
 
 /* ---- attention over cached latents (attention_latent.cu) ---- */
 /* product columns [q latent: q_rank | kv latent: kv_rank | gate: n_gate]: both latents RMS-normed with their weights; the query latent to q_out [T, q_rank], the kv latent into the token's slot of latent_cache [pages, 1, page_size, kv_rank], sigmoid of the gate columns to gate_out [T, n_gate]; kv_out (may be NULL) receives the kv latents as rows [T, kv_rank] too */
@@ -249,14 +257,27 @@ KESTREL_API int kestrel_removal_gates(const float *partial, int S, long long sli
 KESTREL_API int kestrel_recurrence_scan(const float *r, const float *w, const float *k, const float *v, const float *a, const float *b, float *state, long long state_stride, long long state_off, const int *cu_seqlens, const int *slots, float *out, int nseq, int H, int d, int dv, kestrel_stream_t stream);
 /* out = o / sqrt(mean(o^2) + eps) per head, times w[h w_stride + i] (w_stride 0: one weight [dv] for all heads, dv: one per head), times sigmoid of the gate product's columns g_col0 + h dv + i where g_part is given; storage type */
 KESTREL_API int kestrel_head_norm_gate(const float *o, const float *w, int w_stride, float eps, const float *g_part, int Sg, long long g_stride, int g_ld, int g_col0, void *out, int dtype, int T, int H, int dv, kestrel_stream_t stream);
+/* the same; w may be NULL (no weight); g_act 0: sigmoid of the gate columns, 1: silu */
+KESTREL_API int kestrel_head_norm_act(const float *o, const float *w, int w_stride, float eps, const float *g_part, int Sg, long long g_stride, int g_ld, int g_col0, int g_act, void *out, int dtype, int T, int H, int dv, kestrel_stream_t stream);
+/* ---- retention: a fixed decay per head (retention.cu) ---- */
+/* product columns [q: H d | k: H d | v: H dv | ...]: q, k turned by position (first `rot` dimensions, rotate-half), k times d^-1/2; q_out, k_out [T, H d], v_out [T, H dv] in `dtype`; w_out (may be NULL) [T, H d] = the head's decay */
+KESTREL_API int kestrel_retention_prepare(const float *partial, int S, long long slice_stride, int ld, const int *positions, const float *inv_freq, int rot, const float *decay, void *q_out, void *k_out, void *v_out, float *w_out, int dtype, int T, int H, int d, int dv, kestrel_stream_t stream);
+
+/* ---- differential attention (differential.cu): a [T, H, 2, vd] the two maps' outputs; out = (a1 - lambda a2) / its root mean square (eps) * (1 - diff), lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff ---- */
+KESTREL_API int kestrel_differential_combine(const float *a, const float *lq1, const float *lk1, const float *lq2, const float *lk2, int dim, float diff, float eps, void *out, int dtype, int T, int H, int vd, kestrel_stream_t stream);
 
 /* ---- routed feed-forward (moe.cu) ---- */
 KESTREL_API int kestrel_moe_route(const float *z_part, int S, long long slice_stride, const float *bias, int *ids, float *weights, int T, int E, int top, kestrel_stream_t stream);
 /* scores sigmoid(z); chosen by score + correction[e] (may be NULL) among the experts of the `keep` best of `n_groups` groups of neighbours (a group's score: the sum of its two largest choice scores); weights = chosen scores / (their sum + 1e-20) * scale */
 KESTREL_API int kestrel_moe_route_sigmoid(const float *z_part, int S, long long slice_stride, const float *correction, int n_groups, int keep, float scale, int *ids, float *weights, int T, int E, int top, kestrel_stream_t stream);
+/* the general form: the first E of ld columns; softmax 1: scores are the softmax of z over all E, 0: sigmoid(z); group_max 1: a group's score is its largest choice score, 0: the sum of its two largest; renorm 0: weights are the chosen scores times scale */
+KESTREL_API int kestrel_moe_route_scored(const float *z_part, int S, long long slice_stride, int ld, const float *correction, int n_groups, int keep, float scale, int softmax, int group_max, int renorm, int *ids, float *weights, int T, int E, int top, kestrel_stream_t stream);
 KESTREL_API int kestrel_moe_max_tiles(int P, int E, int rows_per_tile);
 KESTREL_API void kestrel_moe_set_plain(int on);   /* 1: the bfloat16 grouped products take the CUDA-core kernel instead of the tensor-core one; for tests of both */
 KESTREL_API int kestrel_moe_group(const int *ids, int P, int E, int rows_per_tile, int *offsets, int *row_pair, int *pair_row, int *tile_expert, int *tile_row0, int *n_tiles, kestrel_stream_t stream);
+/* the same; only the first with_tiles router outputs get tiles (those behind them have no matrices) */
+KESTREL_API int kestrel_moe_group_some(const int *ids, int P, int E, int with_tiles, int rows_per_tile, int *offsets, int *row_pair, int *pair_row, int *tile_expert, int *tile_row0, int *n_tiles, kestrel_stream_t stream);
+/* limit < 0: the experts' activation is silu(g) u, without the clamp */
 KESTREL_API int kestrel_moe_gate_up(const void *x, long long ldx, const void *w, const int *offsets, const int *row_pair, const int *tile_expert, const int *tile_row0, const int *n_tiles, int max_tiles, int top, float limit, void *act, int dtype, int ff, int K, kestrel_stream_t stream);
 KESTREL_API int kestrel_moe_down(const void *act, const void *w, const int *offsets, const int *row_pair, const int *tile_expert, const int *tile_row0, const int *n_tiles, int max_tiles, const float *pair_weight, float *y, int dtype, int N, int ff, kestrel_stream_t stream);
 /* experts without a gate: act [P, ff] = activation(W_up[e] xs), xs [P, K] the pairs' input rows in sorted order, w [E, ff, K]; act_kind 1 gelu (erf), 2 gelu (tanh form), 3 silu, 4 relu squared */
@@ -272,6 +293,8 @@ KESTREL_API int kestrel_moe_up_act_tc(const void *xs, const void *w, const int *
 KESTREL_API int kestrel_moe_tc_error(void);
 KESTREL_API void kestrel_moe_tc_set_ring_kb(int kb);   /* shared memory of a CTA's stages in KB: 104 (default) lets two CTAs share an SM, 200 gives one all of it; for measurements */
 KESTREL_API int kestrel_moe_combine(const float *y, const int *pair_row, int top, float *out, int T, int N, kestrel_stream_t stream);
+/* the same with identity experts (choices with ids >= experts add their weight times x[t]) and, where `shared` is given, an expert every token takes: its slices' sum times sigmoid(column sg_col of z) where z_part is given */
+KESTREL_API int kestrel_moe_combine_with(const float *y, const int *pair_row, const int *ids, const float *weights, int top, int experts, const void *x, int dtype, long long ldx, const float *shared, int Ss, long long shared_stride, const float *z_part, int Sz, long long z_stride, int z_ld, int sg_col, float *out, int T, int N, kestrel_stream_t stream);
 
 /* ---- matrix products ---- */
 KESTREL_API int kestrel_gemm_plain(const void *x, const void *w, float *out, int dtype, int T, int N, int K, long long ldx, long long ldw, long long ldo, kestrel_stream_t stream);

@@ -4,5 +4,6 @@ from . import zidivik  # registers "Zidivik"
 from . import tidavik  # registers "Tidavik"
 from . import toredra  # registers "Toredra"
 from . import korirax  # registers "Korirax"
+from . import tuganex  # registers "Tuganex"
 
-__all__ = ["DecoderModel", "LayerCall", "qwen3", "zidivik", "tidavik", "toredra", "korirax"]
+__all__ = ["DecoderModel", "LayerCall", "qwen3", "zidivik", "tidavik", "toredra", "korirax", "tuganex"]

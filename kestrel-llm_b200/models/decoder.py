@@ -151,6 +151,8 @@ class DecoderModel(Part):
         """Layer calls order[lo:hi] on the residual stream ``x`` and the not yet added ``pending``."""
         for call in self.order[lo:hi]:
             lc = cache.layer(call.cache, call.writes_cache) if call.cache >= 0 else None
+            if (call.add_embedding or call.add_row >= 0) and isinstance(pending, ops.StreamCopy):
+                pending = None                  # a copy of the stream as it was: nothing to add, and about to be out of date
             if call.add_embedding:
                 if pending is not None:         # what the call before left unadded goes in first
                     ops.add_two(x, pending, None, None)
@@ -167,5 +169,7 @@ class DecoderModel(Part):
     def forward_head(self, x, pending, batch) -> Optional[torch.Tensor]:
         if batch.num_logit_rows == 0:
             return None
+        if isinstance(pending, ops.StreamCopy):
+            pending = None                      # the stream is complete
         n = self.final_norm.add_forward(x, pending, self.dtype, rows=batch.logit_rows)
         return self.lm_head.forward(n)

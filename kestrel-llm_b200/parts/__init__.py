@@ -7,13 +7,15 @@ from .attention import GroupedQueryAttention
 from .mlp import DenseMLP, GatedMLP
 from .attention_gated import GatedWindowAttention
 from .attention_latent import LatentAttention
+from .attention_differential import DifferentialAttention
 from .delta import ChannelDeltaMixer
 from .recurrence import ForgetGateRecurrence, RemovalDeltaMixer
+from .retention import RetentionMixer
 from .parallel import ParallelMixers
-from .moe import GroupRoutedExperts, RoutedExperts
+from .moe import GroupRoutedExperts, RoutedExperts, SoftmaxRoutedExperts
 from .rglru import GatedDiagonalRecurrence
 from .side_input import TokenSideInput, TokenTable
-from .block import ParallelBlock, PreNormBlock, SandwichBlock
+from .block import ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
 from .embedding import LMHead, StreamRows, TokenEmbedding
 
 __all__ = ["Block", "CacheSpec", "FeedForward", "FixedStateSpec", "Mixer", "Norm", "PagedKVSpec", "Part",
@@ -21,4 +23,5 @@ __all__ = ["Block", "CacheSpec", "FeedForward", "FixedStateSpec", "Mixer", "Norm
            "GroupedQueryAttention", "GatedMLP", "PreNormBlock", "LMHead", "TokenEmbedding", "SinusoidalPositions",
            "GatedWindowAttention", "LatentAttention", "ChannelDeltaMixer", "RoutedExperts", "TokenSideInput", "TokenTable", "ParallelBlock",
            "CombinedSpec", "FrequencyScaling", "DenseMLP", "ForgetGateRecurrence", "RemovalDeltaMixer", "ParallelMixers", "SandwichBlock",
-           "RampScaling", "GroupRoutedExperts", "GatedDiagonalRecurrence", "StreamRows"]
+           "RampScaling", "GroupRoutedExperts", "GatedDiagonalRecurrence", "StreamRows", "DifferentialAttention",
+           "RetentionMixer", "SoftmaxRoutedExperts", "PostNormBlock"]

@@ -133,3 +133,42 @@ class SandwichBlock(Block):
         g = self.gate2.forward(h) if self.gate2 is not None else None
         ops.add_gated_normed(residual, z, g, self.norm2b.weight, self.norm2b.eps)
         return residual, None
+
+
+class PostNormBlock(Block):
+    """A norm on each sublayer's result only; the sublayers read the stream itself:
+
+        x += norm1(mixer(x));  x += norm2(ffn(x))
+
+    (``ffn`` and ``norm2`` None: the first line alone.)  Norm and add are one kernel, which also leaves the stream in the storage
+    type for the sublayer that follows; the block hands that copy on to the next block."""
+
+    def __init__(self, mixer: Mixer, norm1: RMSNorm, ffn: Optional[FeedForward], norm2: Optional[RMSNorm], dtype: torch.dtype):
+        if (norm2 is None) != (ffn is None):
+            raise ValueError("the second norm and the feed-forward come together or not at all")
+        self.mixer, self.norm1, self.ffn, self.norm2 = mixer, norm1, ffn, norm2
+        self.dtype = dtype
+
+    def parts(self):
+        return [p for p in (self.mixer, self.norm1, self.ffn, self.norm2) if p is not None]
+
+    def weight_slots(self) -> List[WeightSlot]:
+        return [s for p in self.parts() for s in p.weight_slots()]
+
+    def _add(self, residual: torch.Tensor, y, norm: RMSNorm) -> torch.Tensor:
+        """The stream after residual += norm(y), in the storage type."""
+        h = torch.empty(residual.shape, dtype=self.dtype, device=residual.device) if self.dtype != torch.float32 else None
+        ops.add_gated_normed(residual, y, None, norm.weight, norm.eps, next_out=h)
+        return residual if h is None else h
+
+    def forward(self, residual: torch.Tensor, pending, batch, cache):
+        if isinstance(pending, ops.StreamCopy):
+            h = pending.data
+        else:
+            if pending is not None:
+                ops.add_two(residual, pending, None, None)
+            h = residual if self.dtype == torch.float32 else ops.Partials(residual).reduce(self.dtype)
+        h = self._add(residual, self.mixer.forward(h, batch, cache), self.norm1)
+        if self.ffn is not None:
+            h = self._add(residual, self.ffn.forward(h, batch), self.norm2)
+        return residual, ops.StreamCopy(h)

@@ -42,21 +42,33 @@ class GatedMLP(FeedForward):
 
 class DenseMLP(FeedForward):
     """Feed-forward without a gate: y = W_down act(W_up x), ``activation`` "relu2" (the square of
-    relu), "silu", "tanh", "gelu" (the exact one, with erf) or "gelu_tanh"."""
+    relu), "silu", "tanh", "gelu" (the exact one, with erf), "gelu_tanh" or "xielu" (z^2 above zero, exp(z) - 1 - z
+    below it, each times a learned number, plus z / 2; the checkpoint's two numbers are ``act_name``).  ``bias``: both projections
+    have one."""
     graph_safe = True
 
     def __init__(self, width: int, intermediate: int, dtype: torch.dtype, device, prefix: str, activation: str = "relu2",
-                 names=("up", "down")):
-        if activation not in ("relu2", "silu", "tanh", "gelu", "gelu_tanh"):
-            raise ValueError(f"activation '{activation}' has no kernel; one of 'relu2', 'silu', 'tanh', 'gelu', 'gelu_tanh'")
+                 names=("up", "down"), bias: bool = False, act_name: str = "act"):
+        if activation not in ("relu2", "silu", "tanh", "gelu", "gelu_tanh", "xielu"):
+            raise ValueError(f"activation '{activation}' has no kernel; one of 'relu2', 'silu', 'tanh', 'gelu', 'gelu_tanh', 'xielu'")
         self.width, self.intermediate, self.activation = width, intermediate, activation
         self.prefix, self.names, self.dtype = prefix, names, dtype
-        self.up = Linear(width, intermediate, dtype, device)
-        self.down = Linear(intermediate, width, dtype, device)
+        self.up = Linear(width, intermediate, dtype, device, bias=bias)
+        self.down = Linear(intermediate, width, dtype, device, bias=bias)
+        self.act_name = act_name
+        self.act_params = torch.empty((2,), dtype=torch.float32, device=device) if activation == "xielu" else None
 
     def weight_slots(self) -> List[WeightSlot]:
-        return [WeightSlot(self.prefix + self.names[0], self.up.weight), WeightSlot(self.prefix + self.names[1], self.down.weight)]
+        slots = []
+        for name, proj in zip(self.names, (self.up, self.down)):
+            slots.append(WeightSlot(self.prefix + name, proj.weight))
+            if proj.bias is not None:
+                slots.append(WeightSlot(self.prefix + name + ".b", proj.bias, "bias"))
+        if self.act_params is not None:
+            slots.append(WeightSlot(self.prefix + self.act_name, self.act_params, "bias"))
+        return slots
 
     def forward(self, x: torch.Tensor, batch) -> ops.Partials:
         # many tokens in bfloat16: the activation is the up product's epilogue; otherwise its slices are summed and activated
-        return self.down.forward(ops.linear_act(x, self.up.weight, self.activation, weights_static=True))
+        return self.down.forward(ops.linear_act(x, self.up.weight, self.activation, weights_static=True, bias=self.up.bias,
+                                               act_params=self.act_params))

@@ -16,6 +16,12 @@ group's score the sum of its two largest choice scores, only experts of the ``ke
 others count as minus infinity); weights = the chosen experts' s over their sum (+ 1e-20) times ``scale``; and optionally
 one more expert of the same form that every token takes (``shared_inner`` > 0), whose product is handed on beside the
 routed experts' so that the block adds both.
+
+`SoftmaxRoutedExperts` has gated experts, y = W_down (silu(W_gate h) * W_up h), and a softmax router in float32 over ``experts`` +
+``identity`` outputs: outputs are chosen by s + correction among the ``keep`` best of ``groups`` groups of neighbours (experts and identity
+outputs together; a group's score its largest choice score) and weighted by s as it is (or over the chosen scores' sum, ``renorm``).  An
+identity output's expert is h itself.  An expert that every token takes (``shared_inner`` > 0) is added times sigmoid(w_sg . h), one number
+a token, whose logit is one more row of the router's product.
 """
 from __future__ import annotations
 
@@ -26,7 +32,7 @@ import torch
 from ..csrc import ops
 from .base import FeedForward, WeightSlot
 from .linear import Linear
-from .mlp import DenseMLP
+from .mlp import DenseMLP, GatedMLP
 
 
 class RoutedExperts(FeedForward):
@@ -100,3 +106,49 @@ class GroupRoutedExperts(FeedForward):
         if self.shared is None:
             return routed
         return routed, self.shared.forward(x, batch)
+
+
+class SoftmaxRoutedExperts(FeedForward):
+    graph_safe = True          # forward launches kernels over device tensors of the batch only
+
+    def __init__(self, width: int, inner: int, experts: int, top: int, dtype: torch.dtype, device, prefix: str, identity: int = 0,
+                 groups: int = 1, keep: int = 1, renorm: bool = False, scale: float = 1.0, shared_inner: int = 0, shared_gate: bool = True,
+                 correction: bool = True, expert_name: str = "e{}.",
+                 names=("gate", "up", "down", "router", "correction", "shared.", "sg")):
+        n = experts + identity
+        if not 1 <= top <= min(n, 32):
+            raise ValueError(f"top = {top} of {n} router outputs: the router kernel takes 1 to min(outputs, 32)")
+        if n % groups or not 1 <= keep <= groups or top > keep * (n // groups):
+            raise ValueError(f"{n} router outputs in {groups} groups, {keep} kept, {top} chosen do not fit")
+        self.width, self.inner, self.experts, self.identity, self.top = width, inner, experts, identity, top
+        self.groups, self.keep, self.renorm, self.scale = groups, keep, bool(renorm), float(scale)
+        self.dtype, self.prefix, self.expert_name, self.names = dtype, prefix, expert_name, names
+        self.outputs = n
+        self.shared_gate = bool(shared_inner) and shared_gate
+        self.router = Linear(width, n + (1 if self.shared_gate else 0), dtype, device)      # rows: experts, identity outputs, the shared gate
+        self.correction: Optional[torch.Tensor] = torch.empty((n,), dtype=torch.float32, device=device) if correction else None
+        self.w_gate_up = torch.empty((experts, 2 * inner, width), dtype=dtype, device=device)
+        self.w_down = torch.empty((experts, width, inner), dtype=dtype, device=device)
+        self.shared = GatedMLP(width, shared_inner, dtype, device, prefix + names[5], names=names[:3]) if shared_inner else None
+
+    def weight_slots(self) -> List[WeightSlot]:
+        p, ff, (gate, up, down, router, correction, shared, sg) = self.prefix, self.inner, self.names
+        slots = [WeightSlot(p + router, self.router.weight[:self.outputs])]
+        if self.correction is not None:
+            slots.append(WeightSlot(p + correction, self.correction, "bias"))
+        for e in range(self.experts):
+            q = p + self.expert_name.format(e)
+            slots += [WeightSlot(q + gate, self.w_gate_up[e, :ff]), WeightSlot(q + up, self.w_gate_up[e, ff:]),
+                      WeightSlot(q + down, self.w_down[e])]
+        if self.shared is not None:
+            slots += self.shared.weight_slots()
+            if self.shared_gate:
+                slots.append(WeightSlot(p + shared + sg, self.router.weight[self.outputs:]))
+        return slots
+
+    def forward(self, x: torch.Tensor, batch) -> ops.Partials:
+        z = self.router.forward(x)
+        ids, weights = ops.moe_route_scored(z, self.outputs, self.correction, self.top, self.groups, self.keep, self.scale, renorm=self.renorm)
+        extra = ops.MoeExtra(self.identity, self.shared.forward(x, batch) if self.shared is not None else None,
+                             z if self.shared_gate else None, self.outputs)
+        return ops.Partials(ops.moe_experts(x, ids, weights, self.w_gate_up, self.w_down, None, extra))

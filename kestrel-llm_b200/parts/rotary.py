@@ -73,7 +73,8 @@ class RotaryHalf(PositionEncoding):
     pairing = "half"
 
     def __init__(self, head_dim: int, theta: float, device, rotary_dim: Optional[int] = None, scale: float = 1.0,
-                 scaling: Optional[FrequencyScaling] = None):
+                 scaling: Optional[FrequencyScaling] = None, exact: bool = False):
+        """``exact``: the frequencies are made in float64 and rounded once (a `FrequencyScaling` always does that)."""
         rot = head_dim if rotary_dim is None else rotary_dim
         if rot % 2 or rot <= 0 or rot > head_dim:
             raise ValueError(f"rotary size {rot} must be even and at most the head size {head_dim}")
@@ -82,7 +83,9 @@ class RotaryHalf(PositionEncoding):
         self.scale = float(scale)
         self.scaling = scaling
         half = rot // 2
-        if scaling is None:
+        if scaling is None and exact:
+            inv = np.power(float(theta), -np.arange(half, dtype=np.float64) / half)
+        elif scaling is None:
             j = np.arange(half, dtype=np.float32)
             inv = (np.float32(1.0) / np.power(np.float32(theta), j / np.float32(half), dtype=np.float32))
         else:       # the bands are decided on the frequencies in float64; the kernel gets them rounded to float32
