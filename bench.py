@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--impl ours|reference]
     python bench.py --workload mix14b | 32b
-    python bench.py --workload zidivik | tidavik | toredra | korirax [--size a|b]
+    python bench.py --workload zidivik | tidavik | toredra | korirax | tuganex [--size a|b]
 
 Default run (the headline): decode tokens a second at batch 8, at batch 1 and 64, prefill of
 2,048 tokens, and the same decode through the Python entry point with host tokens in and out.
@@ -354,12 +354,37 @@ def korirax_raw(z):
             "token_side": {"dim": z["side"]}, "max_positions": 8192, "layers": layers}
 
 
+TUGANEX_SIZES = {
+    # width, attention heads / kv heads x (map, value) sizes, rotated dimensions of a map, recurrence heads x key / value size, dense feed-forward
+    # (two matrices), experts x ff (top of experts + identity outputs in groups) and the shared expert, vocab
+    "a": dict(width=2048, heads=16, kv_heads=4, dim=64, vdim=128, rot=64, r_heads=16, r_dim=128, r_vdim=128, ff=9216, experts=32, identity=8, top=4,
+              e_ff=768, groups=4, keep=2, shared=768, vocab=32000),
+    "b": dict(width=4096, heads=32, kv_heads=8, dim=64, vdim=128, rot=64, r_heads=32, r_dim=128, r_vdim=128, ff=18432, experts=64, identity=16, top=4,
+              e_ff=1024, groups=8, keep=4, shared=1024, vocab=64000),
+}
+
+
+def tuganex_raw(z):
+    rot = {"dims": z["rot"], "base": 500000.0}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5, "diff": 0.5, "rot": rot}
+    # decays from a memory of 32 tokens to one of 4,096, as far apart as the heads are many
+    ret = {"heads": z["r_heads"], "dim": z["r_dim"], "vdim": z["r_vdim"], "decay": [1.0 - 2.0 ** (-5 - 7.0 * h / (z["r_heads"] - 1)) for h in range(z["r_heads"])],
+           "rot": {"dims": z["r_dim"], "base": 10000.0}}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["e_ff"]}, "router": {"experts": z["experts"], "identity": z["identity"], "top": z["top"],
+                                                                  "groups": {"count": z["groups"], "keep": z["keep"]}}, "shared": {"ff": z["shared"]}}
+    layers = [{"type": "attention", "mixer": att, "mlp": dense}, {"type": "attention", "mixer": att, "mlp": moe},
+              {"type": "retention", "mixer": ret, "mlp": dense}, {"type": "attention", "mixer": dict(att, kv_from=1), "mlp": moe}]
+    return {"architecture": "Tuganex", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "max_positions": 8192, "layers": layers}
+
+
 def run_zidivik(args) -> int:
-    """Prefill and decode of the Zidivik, the Tidavik, the Toredra or the Korirax decoder at real layer sizes, beside the Qwen3 dense decoder of equal size."""
+    """Prefill and decode of the Zidivik, the Tidavik, the Toredra, the Korirax or the Tuganex decoder at real layer sizes, beside the Qwen3 dense decoder of equal size."""
     import numpy as np
     import torch
     from kestrel_llm_b200.config import EngineOptions, Qwen3Config, TidavikConfig, ToredraConfig, ZidivikConfig
     from kestrel_llm_b200.config.korirax_config import KoriraxConfig
+    from kestrel_llm_b200.config.tuganex_config import TuganexConfig
     from kestrel_llm_b200.config.registry import resolve_architecture
     from kestrel_llm_b200.csrc import ops
     from kestrel_llm_b200.engine import Engine, Entry
@@ -368,7 +393,8 @@ def run_zidivik(args) -> int:
     dev = "cuda:0"
     torch.cuda.set_device(0)
     tidavik, toredra, korirax = args.workload == "tidavik", args.workload == "toredra", args.workload == "korirax"
-    z = (KORIRAX_SIZES if korirax else TOREDRA_SIZES if toredra else TIDAVIK_SIZES if tidavik else ZIDIVIK_SIZES)[args.size]
+    tuganex = args.workload == "tuganex"
+    z = (TUGANEX_SIZES if tuganex else KORIRAX_SIZES if korirax else TOREDRA_SIZES if toredra else TIDAVIK_SIZES if tidavik else ZIDIVIK_SIZES)[args.size]
     T, B, CTX = args.prefill_tokens, args.batch, 2048
     W, K = max(3, args.warmup), max(1, min(args.steps, 32))
     pk = peaks()
@@ -379,7 +405,8 @@ def run_zidivik(args) -> int:
                    "add_two", "gelu_table_mul", "add_normed", "embed", "add_sinusoid", "linear_add_into", "latent_prepare", "head_gemm", "attention_tc",
                    "forget_gates", "removal_gates", "recurrence_scan", "head_norm_gate", "combine_normed", "add_gated_normed", "partial_columns_act",
                    "embed_add", "logit_scale_cap", "linear_act", "rglru_branches", "rglru_scan", "moe_route_sigmoid", "moe_experts_ungated",
-                   "gate_columns_mul", "latent_rotate_queries", "add_row"]
+                   "gate_columns_mul", "latent_rotate_queries", "add_row", "differential_combine", "retention_prepare", "retention_step", "retention_chunks",
+                   "moe_route_scored", "attention_tc_maps", "reduce_partials"]
 
     def measure(cfg, label):
         model = resolve_architecture(cfg.architecture).build(cfg, torch.bfloat16, dev)
@@ -495,20 +522,46 @@ def run_zidivik(args) -> int:
                 "decode_batch": B, "decode_context": CTX, "decode_ms": round(1000 * dec, 4), "decode_tok_s": round(B / dec, 1),
                 "launches_per_decode_step": int(launches), "device_us_per_operation": split}
 
-    raw = korirax_raw(z) if korirax else toredra_raw(z) if toredra else tidavik_raw(z) if tidavik else zidivik_raw(z)
-    zc = (KoriraxConfig if korirax else ToredraConfig if toredra else TidavikConfig if tidavik else ZidivikConfig).from_dict(raw)
+    raw = tuganex_raw(z) if tuganex else korirax_raw(z) if korirax else toredra_raw(z) if toredra else tidavik_raw(z) if tidavik else zidivik_raw(z)
+    zc = (TuganexConfig if tuganex else KoriraxConfig if korirax else ToredraConfig if toredra else TidavikConfig if tidavik else ZidivikConfig).from_dict(raw)
     L = len(raw["layers"])
     dense_raw = dict(QWEN3_8B, num_hidden_layers=L, hidden_size=z["width"], num_attention_heads=z["heads"],
-                     num_key_value_heads=z["kv_heads"], head_dim=z["dim"],
-                     intermediate_size=(z["ff"] + (z["top"] * z["e_ff"] + z["shared"]) * 2 // 3) // 2 // 256 * 256 if korirax else
+                     num_key_value_heads=z["kv_heads"], head_dim=z["vdim"] if tuganex else z["dim"],
+                     intermediate_size=(z["ff"] * 2 // 3 + z["top"] * z["e_ff"] + z["shared"]) // 2 // 256 * 256 if tuganex else
+                     (z["ff"] + (z["top"] * z["e_ff"] + z["shared"]) * 2 // 3) // 2 // 256 * 256 if korirax else
                      z["ff"] * 2 // 3 if toredra else z["ff"] if tidavik else z["top"] * z["ff"],
                      vocab_size=z["vocab"], max_position_embeddings=8192)
     if tidavik:                              # the dense model's layers look through the same window
         dense_raw.update(sliding_window=z["window"], use_sliding_window=True, layer_types=["sliding_attention"] * L)
     qc = Qwen3Config.from_dict(dense_raw)
-    ours = measure(zc, "Korirax" if korirax else "Toredra" if toredra else "Tidavik" if tidavik else "Zidivik")
+    ours = measure(zc, "Tuganex" if tuganex else "Korirax" if korirax else "Toredra" if toredra else "Tidavik" if tidavik else "Zidivik")
     dense = measure(qc, "Qwen3 dense, equal size" + (" and window" if tidavik else ""))
     clocks.close()
+    if tuganex:
+        D, H, G, d, dv, ff, n = z["width"], z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["ff"], z["experts"] + z["identity"]
+        q_w, kv_w, o_w = D * H * 2 * d, D * G * (2 * d + dv), H * dv * D
+        rq, rv = z["r_heads"] * z["r_dim"], z["r_heads"] * z["r_vdim"]
+        mixers = 3 * (q_w + o_w) + 2 * kv_w + D * (2 * rq + 2 * rv) + rv * D
+        share = z["experts"] / n                 # of a token's choices, those that are experts with matrices (random router)
+        moe_fixed = 3 * z["shared"] * D + (n + 1) * D
+        active = mixers + 2 * 2 * ff * D + 2 * (3 * z["e_ff"] * D * z["top"] * share + moe_fixed)
+        touched = mixers + 2 * 2 * ff * D + 2 * (3 * z["e_ff"] * D * min(z["experts"], B * z["top"] * share) + moe_fixed) + z["vocab"] * D
+        # products, two causal maps a head over one value each (half of the T x T scores), three passes over a head's state a token
+        flops_prefill = 2.0 * T * active + 3 * 2.0 * H * (2 * d + 2 * dv) * T * T / 2 + T * 6.0 * rq * z["r_vdim"]
+        state_bytes, cache_bytes = 4.0 * B * rq * z["r_vdim"] * 2, 2.0 * B * CTX * 3 * G * (2 * d + dv)
+        rec = {"metric": f"Tuganex prefill tokens/s at size {args.size}, bf16, beside Qwen3 dense of equal size", "value": ours["prefill_tok_s"],
+               "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": W, "ms_per_step": ours["prefill_ms"], "higher_is_better": True,
+               "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "impl": "ours", "workload": "tuganex",
+               "data": "synthetic: random weights, uniform random token ids, cache of the context filled with random values",
+               "config": dict(z, layers=[l["type"] + ("/shared keys" if "kv_from" in l["mixer"] else "") + "+" + l["mlp"]["kind"] for l in raw["layers"]],
+                              page_size=args.page_size, peaks=pk["source"], parallelism="single GPU"),
+               "tuganex": ours, "dense": dense,
+               "ratio_to_dense": {"prefill": round(ours["prefill_tok_s"] / dense["prefill_tok_s"], 3), "decode": round(ours["decode_tok_s"] / dense["decode_tok_s"], 3)},
+               "prefill_flops_frac_of_peak": round(flops_prefill / (ours["prefill_ms"] / 1000.0) / (pk["bf16_tflops"] * 1e12), 4),
+               "decode_bytes_frac_of_hbm": round((2.0 * touched + state_bytes + cache_bytes) / (ours["decode_ms"] / 1000.0) / (pk["hbm_gbs"] * 1e9), 4),
+               "gpu_launches": ours["launches_per_decode_step"] * K, "clocks": clocks.summary()}
+        print(json.dumps(rec))
+        return 0
     if korirax:
         D, H, G, d, dv, ff = z["width"], z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["ff"]
         LH, ld, lr, lv, qr, kr, C = z["l_heads"], z["l_dim"], z["l_rot"], z["l_vdim"], z["q_rank"], z["kv_rank"], z["channels"]
@@ -614,10 +667,10 @@ def main() -> int:
     ap.add_argument("--page-size", type=int, default=16, help="tokens per cache page (default 16)")
     ap.add_argument("--context", type=int, default=CONTEXT, help="context length at which the decode steps end (default 4096)")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS, help="tokens of the prefill step (default 2048)")
-    ap.add_argument("--workload", default="decode8b", choices=["decode8b", "mix14b", "32b", "zidivik", "tidavik", "toredra", "korirax"],
-                    help="decode8b: the headline run; mix14b / 32b: whole workloads through the scheduler; zidivik / tidavik / toredra / korirax: that decoder "
+    ap.add_argument("--workload", default="decode8b", choices=["decode8b", "mix14b", "32b", "zidivik", "tidavik", "toredra", "korirax", "tuganex"],
+                    help="decode8b: the headline run; mix14b / 32b: whole workloads through the scheduler; zidivik / tidavik / toredra / korirax / tuganex: that decoder "
                          "at real layer sizes beside Qwen3 dense of equal size")
-    ap.add_argument("--size", default="a", choices=sorted(ZIDIVIK_SIZES), help="layer sizes of --workload zidivik / tidavik / toredra / korirax")
+    ap.add_argument("--size", default="a", choices=sorted(ZIDIVIK_SIZES), help="layer sizes of --workload zidivik / tidavik / toredra / korirax / tuganex")
     ap.add_argument("--requests", type=int, default=0, help="requests of a workload (0: 32 for mix14b, 16 for 32b)")
     ap.add_argument("--generate", type=int, default=0, help="tokens to generate per request of a workload (0: 256 / 128)")
     ap.add_argument("--step-tokens", type=int, default=2048,
@@ -629,7 +682,7 @@ def main() -> int:
     if args.gpus != 1:
         print(f"bench.py: this engine runs on ONE GPU; --gpus {args.gpus} is not supported (no multi-GPU path exists)")
         return 2
-    if args.workload in ("zidivik", "tidavik", "toredra", "korirax"):
+    if args.workload in ("zidivik", "tidavik", "toredra", "korirax", "tuganex"):
         return run_zidivik(args)
     if args.workload != "decode8b":
         return run_workload(args)

@@ -51,7 +51,7 @@ class DifferentialAttention(Mixer):
         f32 = dict(dtype=torch.float32, device=device)
         self.q_norm = torch.empty((dim,), **f32)
         self.k_norm = torch.empty((dim,), **f32) if own_kv else None
-        self.lam = [torch.empty((dim,), **f32) for _ in range(4)]           # lq1, lk1, lq2, lk2
+        self.lambdas = [torch.empty((dim,), **f32) for _ in range(4)]           # lq1, lk1, lq2, lk2
 
     def cache_spec(self) -> PagedKVSpec:
         return PagedKVSpec(self.kv_heads, 2 * self.dim, v_head_dim=self.v_dim)
@@ -64,7 +64,7 @@ class DifferentialAttention(Mixer):
             slots += [WeightSlot(p + nk, w[self.q_cols:k_end]), WeightSlot(p + nv, w[k_end:]),
                       WeightSlot(p + nk + self.norm_suffix, self.k_norm, "norm")]
         slots += [WeightSlot(p + nq + self.norm_suffix, self.q_norm, "norm"), WeightSlot(p + no, self.out.weight)]
-        return slots + [WeightSlot(p + n, t, "bias") for n, t in zip(self.lambda_names, self.lam)]
+        return slots + [WeightSlot(p + n, t, "bias") for n, t in zip(self.lambda_names, self.lambdas)]
 
     def forward(self, x: torch.Tensor, batch, cache) -> ops.Partials:
         if cache.writable != self.own_kv:
@@ -82,5 +82,5 @@ class DifferentialAttention(Mixer):
             ops.attention_plain_ex(q, cache.k, cache.v, batch.positions, batch.seq_of_token, table, cache.page_size, a, 2 * H, G, 2 * d, dv, 0, 0,
                                    None, self.scale)
         o = torch.empty((T, H * dv), dtype=self.dtype, device=x.device)
-        ops.differential_combine(a, *self.lam, self.diff, self.norm_eps, o, H, dv)
+        ops.differential_combine(a, *self.lambdas, self.diff, self.norm_eps, o, H, dv)
         return self.out.forward(o)

@@ -158,8 +158,8 @@ def _spike(layer, map_, i, j):
     return prepare
 
 
-SPIKES = {"first map": (U.attn(4, 2, 24, 40, 0.5, 0.4, (4, 1e6)), 0), "second map": (U.attn(4, 2, 24, 40, 0.5, 0.4, (4, 1e6)), 1),
-          "second map of 64": (U.attn(4, 2, 64, 128, 0.25, 0.4, (4, 1e6)), 1), "first map of 64": (U.attn(4, 2, 64, 128, 0.25, 0.4, (4, 1e6)), 0),
+SPIKES = {"first map": (U.attn(4, 2, 24, 40, 0.5, 0.4), 0), "second map": (U.attn(4, 2, 24, 40, 0.5, 0.4), 1),
+          "second map of 64": (U.attn(4, 2, 64, 128, 0.25, 0.4), 1), "first map of 64": (U.attn(4, 2, 64, 128, 0.25, 0.4), 0),
           "retention": (U.retention(2, 32, 24, (1.0, 1.0), (4, 1e6)), 0), "retention of 128": (U.retention(2, 128, 128, (1.0, 0.9998), (4, 1e6)), 0)}
 
 
