@@ -3,6 +3,7 @@
 #include <cuda_bf16.h>
 #include "common.cuh"
 #include "attention_score.cuh"
+#include "differential.cuh"
 
 struct AttnParams {
     const __nv_bfloat16 *q;         // [T, nq * hd]
@@ -24,6 +25,8 @@ struct AttnParams {
     float scale;
     ScoreOpts opts;
     int scored;
+    // two maps a head over the same values (differential attention); read by attention_tc.cu only
+    DifferentialOpts maps;
 };
 
 // Keys per slice.  A launch recorded for replay fixes the number of slices; their length then

@@ -64,6 +64,7 @@ attn_prepare_ex_kernel(const float *__restrict__ partial, int S, size_t slice_st
                        const float *__restrict__ inv_freq, int rot, int rot_mode, float rot_scale, float q_temp_coef, int q_temp_every,
                        int maps, int q_pad) {
     extern __shared__ float apx_ss[];              // qk_norm = 2: sum of squares of every q and k head, then (keep_x) their columns
+    __shared__ float apx_cs[16 * APX_PER_LANE], apx_sn[16 * APX_PER_LANE];      // the token's cosines and sines, made once a block
     __shared__ float apx_rot[APX_WARPS][32 * APX_PER_LANE];   // rotate-half pairing: a warp's head, so that a lane reaches its partner
     pdl_launch_dependents();
     pdl_wait();
@@ -98,6 +99,15 @@ attn_prepare_ex_kernel(const float *__restrict__ partial, int S, size_t slice_st
     }
     size_t slot_row = 0;
     const int pos = positions[t];
+    if (inv_freq) {
+        for (int j = threadIdx.x; j < rot / 2; j += APX_WARPS * 32) {
+            float sn, cs;
+            sincosf((float)pos * inv_freq[j], &sn, &cs);
+            apx_sn[j] = sn * rot_scale;
+            apx_cs[j] = cs * rot_scale;
+        }
+        __syncthreads();
+    }
     const float q_temp = q_temp_every > 0 ? 1.0f + q_temp_coef * logf((float)((pos + 1) / q_temp_every) + 1.0f) : 1.0f;
     if (has_kv) {
         const int page = block_table[(size_t)seq_of_token[t] * table_stride + pos / page_size];
@@ -167,10 +177,7 @@ attn_prepare_ex_kernel(const float *__restrict__ partial, int S, size_t slice_st
                 if (i < rot) {
                     const bool first = rot_mode == 0 ? i < half : (i & 1) == 0;
                     const int j = rot_mode == 0 ? (i < half ? i : i - half) : i >> 1;
-                    float sn, cs;
-                    sincosf((float)pos * inv_freq[j], &sn, &cs);
-                    sn *= rot_scale;
-                    cs *= rot_scale;
+                    const float sn = apx_sn[j], cs = apx_cs[j];
                     x[c] = first ? x[c] * cs - other * sn : x[c] * cs + other * sn;
                 }
             }
@@ -252,7 +259,9 @@ KESTREL_API int kestrel_attn_prepare_maps(const float *partial, int S, long long
     KESTREL_REQUIRE(ld >= need, "attn_prepare_ex: the product has %d columns, the heads need %d", ld, need);
     // few tokens: a block per four head rows, so that the step's few tokens still fill the device
     const int n_heads = nq * maps + (has_kv ? nkv * (maps + 1) : 0);
-    const int by = T >= 512 ? 1 : (n_heads + APX_WARPS - 1) / APX_WARPS;
+    // (many tokens: up to four head rows a warp, so that a row's round trips overlap other blocks'; the norm over a whole
+    // projection, whose blocks each sum all heads first, takes one block a token)
+    const int by = T >= 512 ? (qk_norm == 2 ? 1 : (n_heads + 4 * APX_WARPS - 1) / (4 * APX_WARPS)) : (n_heads + APX_WARPS - 1) / APX_WARPS;
     if (dtype == KESTREL_F32)
         kestrel_launch(attn_prepare_ex_kernel<float>, dim3(T, by), dim3(APX_WARPS * 32), smem, stream, partial, S, (size_t)slice_stride, ld, q_norm_w, k_norm_w, qk_norm, norm_eps,
                        positions, seq_of_token, block_table, table_stride, page_size, (float *)k_cache, (float *)v_cache, (float *)q_out, gate_out, nq, nkv, hd, vd, has_kv, bias, v_norm, keep_x, inv_freq, rot, rot_mode, rot_scale, q_temp_coef, q_temp_every, maps, q_pad);

@@ -29,7 +29,14 @@
 // term, sigmoid weights) are applied by the softmax threads on the scores in their registers, on
 // the special-function unit; with sigmoid weights there is no maximum, no sum and no rescaling, P is
 // the weights.  Shared memory per CTA is 193 KB: one CTA per SM; CTAs with the most
-// keys are launched first.  Every mbarrier wait is bounded; the error word is read by
+// keys are launched first.
+//
+// Differential attention (MAPS): a head has two queries and keys of 64 and one value of 128, and a cache row of K holds both
+// maps' keys, 64 numbers each.  The two row tiles are then the two MAPS of the same 128 (token, head) rows: S_A = Q_1 K_1^T
+// over the first panel of a K tile and S_B = Q_2 K_2^T over the second, half of the steps each, while P_A V and P_B V share the V
+// tile.  When both are done a row's two outputs lie in the same TMEM lane: the softmax threads of tile A take the first 64
+// columns of both, those of tile B the other 64, o = o_A / l_A - lambda o_B / l_B, exchange their parts of the sum of squares
+// through shared memory and write the normed head.  Every mbarrier wait is bounded; the error word is read by
 // kestrel_attention_tc_error.  Formulas as in attention_plain.cu (reference: st.c:10779-10911,
 // st.c:9762-9859).
 #include "attention_params.cuh"
@@ -116,6 +123,7 @@ enum {
 };
 #define AT_RESCALE_STEP 8.0f            // log2 units by which a row's maximum may outgrow its reference
 
+template <bool MAPS>
 __global__ void __launch_bounds__(AT_THREADS, 1)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                     const AttnParams p, int cache_pages, int rows_per_tile) {
@@ -173,9 +181,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
     const int n_tiles = k_hi > k_lo ? (k_hi - k_lo + AT_BN - 1) / AT_BN : 0;
     // row tile A ends earlier: it skips the key tiles beyond its last row
     const int rows_a = min(rows_here, AT_BM);
-    const bool has_b = rows_here > AT_BM;
-    const int k_hi_a = min(pos_begin + (row0 + rows_a - 1) / G + 1, (slice + 1) * slice_len);
-    const int n_tiles_a = has_b ? (k_hi_a > k_lo ? (k_hi_a - k_lo + AT_BN - 1) / AT_BN : 0) : n_tiles;
+    const bool has_b = MAPS || rows_here > AT_BM;
+    const int k_hi_a = MAPS ? k_hi : min(pos_begin + (row0 + rows_a - 1) / G + 1, (slice + 1) * slice_len);
+    const int n_tiles_a = MAPS ? n_tiles : has_b ? (k_hi_a > k_lo ? (k_hi_a - k_lo + AT_BN - 1) / AT_BN : 0) : n_tiles;
 
     if (warp == 8 || warp == 10) {
         // ------------------------------------------------------------------ loaders
@@ -216,8 +224,11 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
             auto issue_s = [&](int x, int t) {
                 const int b = t & 1;
 #pragma unroll
-                for (int ks = 0; ks < AT_HD / 16; ++ks) {
+                for (int ks = 0; ks < (MAPS ? AT_HD / 32 : AT_HD / 16); ++ks) {
                     uint32_t off = (ks >> 2) * AT_PANEL + (ks & 3) * 32;
+                    if (MAPS)           // map x: its own queries, panel x of the key tile
+                        tc_mma(tmem + x * 128, smem_desc(q_s + x * TILE_BYTES + off), smem_desc(k_s + b * TILE_BYTES + x * AT_PANEL + off), IDESC_S, ks > 0 ? 1u : 0u);
+                    else
                     tc_mma(tmem + x * 128, smem_desc(q_s + x * TILE_BYTES + off), smem_desc(k_s + b * TILE_BYTES + off), IDESC_S, ks > 0 ? 1u : 0u);
                 }
                 tc_commit(bar(B_S_FULL + x));
@@ -265,7 +276,29 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
         // ------------------------------------------------------------------ softmax
         // warps 0-3: row tile A, warps 4-7: row tile B; thread r of a tile owns row r (TMEM lane r)
         const int x = warp >> 2, r = tid & 127;
-        {
+        if (MAPS) {
+            // Q: thread t moves 16-byte chunk t % 8 of rows (t / 8) * 4 .. + 3 of both maps
+            const int ld_c = tid & 7, ld_r0 = (tid >> 3) * 4;
+#pragma unroll
+            for (int xt = 0; xt < 2; ++xt) {
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const int rr = ld_r0 + j;
+                    const bool valid = rr < rows_here;
+                    size_t off = 0;
+                    if (valid) {
+                        const int row = row0 + rr;
+                        off = (((size_t)(tok_begin + row / G) * p.nq + kvh * G + row % G) * 2 + xt) * (AT_HD / 2) + ld_c * 8;
+                    }
+                    at_cp_async16(q_s + xt * TILE_BYTES + swizzle128(rr, ld_c), p.q + off, valid);
+                }
+            }
+            asm volatile("cp.async.commit_group;" ::: "memory");
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // cp.async writes -> tensor-core reads
+            __syncwarp();
+            if (lane == 0) mbar_arrive(bar(B_Q_FULL));
+        } else {
             // Q: thread t moves 16-byte chunk t % 16 of rows (t / 16) * 8 .. + 7 of both row tiles
             const int ld_c = tid & 15, ld_r0 = (tid >> 4) * 8;
             const uint32_t ld_panel = (uint32_t)(ld_c >> 3) * AT_PANEL;
@@ -289,11 +322,12 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
             __syncwarp();
             if (lane == 0) mbar_arrive(bar(B_Q_FULL));
         }
-        const int rows_x = x == 0 ? rows_a : rows_here - AT_BM;          // rows of this row tile (<= 0: none)
+        const int tile_row = MAPS ? row0 : row0 + x * AT_BM;             // the tile's first row among the request's
+        const int rows_x = x == 0 || MAPS ? rows_a : rows_here - AT_BM;  // rows of this row tile (<= 0: none)
         const int n_tiles_x = x == 0 ? n_tiles_a : (has_b ? n_tiles : 0);
         const int k_hi_x = x == 0 ? k_hi_a : k_hi;
         const bool row_ok = r < rows_x;
-        const int my_pos = row_ok ? pos_begin + (row0 + x * AT_BM + r) / G : -1;
+        const int my_pos = row_ok ? pos_begin + (tile_row + r) / G : -1;
         const int my_lo = p.window > 0 ? max(0, my_pos - p.window + 1) : 0;
         // warps none of whose 32 rows exist (decode: a few rows per request) skip the arithmetic
         const bool warp_has_rows = 32 * (warp & 3) < rows_x;
@@ -302,7 +336,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
         float m_ref = -INFINITY, l_run = 0.f;       // the reference the output is accumulated against, and the row's sum
         const bool sigmoid = p.scored && p.opts.weighting == KESTREL_WEIGH_SIGMOID, sink = p.scored && p.opts.weighting == KESTREL_WEIGH_SOFTMAX_SINK;
         const ScoreOpts no_opts = {0.f, nullptr, nullptr, nullptr, 0};
-        const HeadScore hs(p.scored ? p.opts : no_opts, kvh * G + (row0 + x * AT_BM + (row_ok ? r : 0)) % G);
+        const HeadScore hs(p.scored ? p.opts : no_opts, kvh * G + (tile_row + (row_ok ? r : 0)) % G);
         const float eff_scale = p.scored ? 1.f : p.scale_log2;   // transformed scores are in base-2 units already
         bool ok = true;             // after a wait gave up the loop runs on without waiting, so that the warps still meet
 
@@ -453,10 +487,52 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
         // the last product of this row tile
         if (n_tiles_x > 0 && ok && !mbar_wait(bar(B_PV_DONE + x), (uint32_t)(n_tiles_x - 1) & 1u)) { atomicExch(&g_at_error, 9); ok = false; }
         tc_fence_after();
-        if (warp_has_rows) {
+        if (MAPS && p.slices == 1) {
+            // both maps' last products, then the two outputs of a row - one TMEM lane - as one head
+            if (ok && !mbar_wait(bar(B_PV_DONE + (x ^ 1)), (uint32_t)(n_tiles - 1) & 1u)) { atomicExch(&g_at_error, 9); ok = false; }
+            tc_fence_after();
+            const float lam = differential_lambda(p.maps, lane);
+            float *xch = reinterpret_cast<float *>(aligned);             // Q's memory: every product that read it is done
+            xch[x * 128 + r] = 1.0f / l_run;
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            const float inv_a = xch[r], inv_b = -lam * xch[128 + r];
+            float o[64], ss = 0.f;
+            if (warp_has_rows) {
+#pragma unroll
+                for (int c = 0; c < 64; c += 32) {
+                    uint32_t oa[32], ob[32];
+                    at_ld32(tmem + lane_base + 256 + x * 64 + c, oa);
+                    at_ld32(tmem + lane_base + 384 + x * 64 + c, ob);
+                    at_ld_wait();
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) {
+                        o[c + j] = fmaf(__uint_as_float(ob[j]), inv_b, __uint_as_float(oa[j]) * inv_a);
+                        ss = fmaf(o[c + j], o[c + j], ss);
+                    }
+                }
+            }
+            xch[256 + x * 128 + r] = ss;
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            if (row_ok && ok) {
+                const int row = tile_row + r;
+                const float mul = 1.0f / sqrtf((xch[256 + r] + xch[384 + r]) / (float)AT_HD + p.maps.eps) * (1.0f - p.maps.diff);
+                __nv_bfloat16 *po = p.out + ((size_t)(tok_begin + row / G) * p.nq + kvh * G + row % G) * AT_HD + x * 64;
+#pragma unroll
+                for (int j = 0; j < 64; j += 8) {
+                    uint32_t w[4];
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        __nv_bfloat162 b2 = __floats2bfloat162_rn(o[j + 2 * k] * mul, o[j + 2 * k + 1] * mul);
+                        w[k] = *reinterpret_cast<uint32_t *>(&b2);
+                    }
+                    *reinterpret_cast<uint4 *>(po + j) = make_uint4(w[0], w[1], w[2], w[3]);
+                }
+            }
+        } else if (warp_has_rows) {
             const bool write = row_ok && ok;
-            int row = row0 + x * AT_BM + r;
+            int row = tile_row + r;
             size_t qrow = write ? (size_t)(tok_begin + row / G) * p.nq + kvh * G + row % G : 0;
+            if (MAPS) qrow = qrow * 2 + x;
             float inv = p.slices > 1 ? 1.f : 1.0f / l_run;
             if (sigmoid) inv = 1.f;
             if (sink) inv = 1.0f / (l_run + at_exp2(hs.sink * 1.4426950408889634f - m_ref));     // one more term exp(sink), against the same reference
@@ -588,15 +664,61 @@ KESTREL_API int kestrel_attention_tc_biased(const void *q, const void *k_cache, 
     size_t smem = 12 * AT_PANEL + 8 * B_COUNT + 16 + 1024;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return kestrel_fail(-3, "attention_tc: cannot raise the shared-memory limit: %s", cudaGetErrorString(e));
         attr_set = true;
     }
-    kestrel_launch(attention_tc_kernel, dim3((unsigned)((long long)tiles * nkv), 1, slices), dim3(AT_THREADS), smem, stream, map_k, map_v, p, cache_pages, rows_per_tile);
+    kestrel_launch(attention_tc_kernel<false>, dim3((unsigned)((long long)tiles * nkv), 1, slices), dim3(AT_THREADS), smem, stream, map_k, map_v, p, cache_pages, rows_per_tile);
     rc = kestrel_check_launch("attention_tc");
     if (rc || slices == 1) return rc;
     return kestrel_attention_merge(part_o, part_ml, out, tile_seq, tile_row0, tiles, rows_per_tile, cu_seqlens, slices, hd, nq, nkv,
                                    scored && weighting == KESTREL_WEIGH_SOFTMAX_SINK ? sink : nullptr, stream);
+}
+
+// Differential attention on the same kernel: q [T, nq, 2, 64] (the two maps' queries of a head), K pages of rows [k_1 | k_2] of 2 * 64
+// numbers, V pages of rows of 128, out [T, nq, 128] = the combined and normed heads (differential.cuh).  Tiles of up to 128 rows
+// - (token, head of a kv group) pairs, both maps together.  With slices > 1 the scratch is part_o [T * nq * 2, slices, 128] and part_ml
+// [T * nq * 2, slices, 2], merged and combined by kestrel_differential_merge.
+KESTREL_API int kestrel_attention_tc_maps(const void *q, const void *k_cache, const void *v_cache, void *out, float *part_o, float *part_ml,
+                                          const int *tile_seq, const int *tile_row0, int tiles, int rows_per_tile, const int *cu_seqlens,
+                                          const int *kv_lens, const int *block_table, int table_width, int table_stride, int page_size,
+                                          int cache_pages, int T, int nq, int nkv, int dim, int vd, int window, int slices, int slice_len, float scale,
+                                          const float *lq1, const float *lk1, const float *lq2, const float *lk2, float diff, float eps,
+                                          cudaStream_t stream) {
+    if (T == 0 || tiles == 0) return 0;
+    KESTREL_REQUIRE(2 * dim == AT_HD && vd == AT_HD, "attention_tc_maps: maps of %d over values of %d; this kernel is built for %d and %d", dim, vd, AT_HD / 2, AT_HD);
+    KESTREL_REQUIRE(rows_per_tile >= 1 && rows_per_tile <= AT_BM, "attention_tc_maps: tiles of %d rows; a CTA takes up to %d of both maps", rows_per_tile, AT_BM);
+    KESTREL_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention_tc_maps: %d query heads over %d kv heads", nq, nkv);
+    KESTREL_REQUIRE(slices >= 1 && slice_len > 0 && slice_len % AT_BN == 0, "attention_tc_maps: slice length %d must be a positive multiple of %d", slice_len, AT_BN);
+    KESTREL_REQUIRE(slices == 1 || (part_o && part_ml), "attention_tc_maps: %d slices without scratch", slices);
+    KESTREL_REQUIRE((long long)tiles * nkv < (1ll << 31) && slices <= 65535, "attention_tc_maps: grid too large");
+    KESTREL_REQUIRE(kestrel_attention_tc_supported(AT_HD, page_size), "attention_tc_maps: pages of %d keys; the page size must be a multiple of 8 that divides 128 or is a multiple of it", page_size);
+    KESTREL_REQUIRE(cache_pages > 0 && (long long)cache_pages * nkv * page_size < (1ll << 31), "attention_tc_maps: a cache of %d pages is beyond the 32-bit row coordinate", cache_pages);
+    CUtensorMap map_k, map_v;
+    const long long cache_rows = (long long)cache_pages * nkv * page_size;
+    const int box = page_size < AT_BN ? page_size : AT_BN;
+    int rc = kestrel_tensor_map_bf16(&map_k, k_cache, cache_rows, AT_HD, AT_HD, box);
+    if (rc == 0) rc = kestrel_tensor_map_bf16(&map_v, v_cache, cache_rows, AT_HD, AT_HD, box);
+    if (rc) return rc;
+    AttnParams p = {};
+    p.q = (const __nv_bfloat16 *)q; p.k_cache = (const __nv_bfloat16 *)k_cache; p.v_cache = (const __nv_bfloat16 *)v_cache;
+    p.out = (__nv_bfloat16 *)out; p.part_o = part_o; p.part_ml = part_ml; p.tile_seq = tile_seq; p.tile_row0 = tile_row0;
+    p.cu_seqlens = cu_seqlens; p.kv_lens = kv_lens; p.block_table = block_table; p.table_width = table_width; p.table_stride = table_stride;
+    p.page_size = page_size; p.nq = nq; p.nkv = nkv; p.hd = AT_HD; p.window = window; p.slices = slices; p.slice_len = slice_len;
+    p.scale_log2 = scale * 1.4426950408889634f;
+    p.scale = scale;
+    p.maps = {lq1, lk1, lq2, lk2, dim, diff, eps};
+    const size_t smem = 12 * AT_PANEL + 8 * B_COUNT + 16 + 1024;
+    static bool attr_set = false;
+    if (!attr_set) {
+        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return kestrel_fail(-3, "attention_tc_maps: cannot raise the shared-memory limit: %s", cudaGetErrorString(e));
+        attr_set = true;
+    }
+    kestrel_launch(attention_tc_kernel<true>, dim3((unsigned)((long long)tiles * nkv), 1, slices), dim3(AT_THREADS), smem, stream, map_k, map_v, p, cache_pages, rows_per_tile);
+    rc = kestrel_check_launch("attention_tc_maps");
+    if (rc || slices == 1) return rc;
+    return kestrel_differential_merge(part_o, part_ml, slices, AT_HD, lq1, lk1, lq2, lk2, dim, diff, eps, out, T, nq, vd, stream);
 }
 
 // Error word of the kernel's bounded waits: 0 = none, else the number of the wait that gave up

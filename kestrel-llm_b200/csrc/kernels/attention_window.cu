@@ -36,6 +36,7 @@
 #include "common.cuh"
 #include "mma_sync.cuh"
 #include "attention_score.cuh"
+#include "differential.cuh"
 #include <math.h>
 
 #define AW_THREADS 128
@@ -56,6 +57,8 @@ struct AwParams {
     ScoreOpts opts;
     int scored;                     // any of the options is on
     float *part_o, *part_ml;        // KW = 4 with several CTAs a row tile: [seq, kv head, row tile, split, 16, D] and [.., 16, 2]
+    int to_scratch;                 // KW = 4: leave the merged state in scratch even if one CTA has all of a row tile's keys
+    DifferentialOpts maps;          // differential attention: the merge combines the maps of a head (attention_window_merge_maps_kernel)
     int ksplit, row_tiles;          // KW = 4: shares of the key rounds a row tile, and row tiles of 16 a request (the grid's x is their product)
 };
 
@@ -320,7 +323,7 @@ attention_window_kernel(const AwParams p) {
             }
         }
         __syncthreads();
-        if (ksplit > 1) {
+        if (ksplit > 1 || p.to_scratch) {
             // this CTA's share of the keys as one state: the warps' states merged in warp order, not normalised
             const size_t base = ((((size_t)seq * p.nkv + kvh) * p.row_tiles + rt_idx) * ksplit + split) * 16;
             for (int idx = tid; idx < rows_here * (vd + 1); idx += AW_THREADS) {
@@ -408,6 +411,55 @@ attention_window_merge_kernel(const AwParams p, int ksplit, int D) {
     }
 }
 
+// Differential attention: query heads 2 n and 2 n + 1 are the two maps of head n.  A block takes one (token, head): 64 threads a
+// map merge its shares as above, then o = a1 - lambda a2 is normed over the head (differential.cuh) and written.
+__global__ void __launch_bounds__(AW_THREADS)
+attention_window_merge_maps_kernel(const AwParams p, int ksplit, int D) {
+    pdl_launch_dependents();
+    __shared__ float a_s[2][256], f_s[2][33], red[AW_THREADS / 32];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, map = tid >> 6;
+    const float lam = differential_lambda(p.maps, lane);
+    pdl_wait();
+    const int kvh = blockIdx.x, seq = blockIdx.y, row = 2 * blockIdx.z, G = p.nq / p.nkv, vd = p.vd;      // the first map's row; G is even
+    const int tok_begin = p.cu_seqlens[seq];
+    if (row >= (p.cu_seqlens[seq + 1] - tok_begin) * G) return;
+    const size_t base = (((size_t)seq * p.nkv + kvh) * p.row_tiles + row / 16) * ksplit * 16 + row % 16 + map;      // + s * 16
+    if ((warp & 1) == 0) {
+        const float m = lane < ksplit ? p.part_ml[(base + (size_t)lane * 16) * 2] : -INFINITY;
+        const float l = lane < ksplit ? p.part_ml[(base + (size_t)lane * 16) * 2 + 1] : 0.f;
+        const float M = warp_max(m), f = m == -INFINITY ? 0.f : fast_exp2(m - M);
+        float L = 0.f;
+        for (int k = 0; k < ksplit; ++k) L += __shfl_sync(0xffffffffu, l * f, k);
+        if (lane < ksplit) f_s[map][lane] = f;
+        if (lane == 0) f_s[map][32] = 1.0f / L;
+    }
+    __syncthreads();
+    for (int col = tid & 63; col < vd; col += 64) {
+        float acc = 0.f;
+#pragma unroll 8
+        for (int s = 0; s < ksplit; ++s) acc = fmaf(p.part_o[(base + (size_t)s * 16) * D + col], f_s[map][s], acc);
+        a_s[map][col] = acc * f_s[map][32];
+    }
+    __syncthreads();
+    float o[2], ss = 0.f;                             // vd <= 256
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int col = tid + AW_THREADS * k;
+        o[k] = col < vd ? a_s[0][col] - lam * a_s[1][col] : 0.f;
+        ss = fmaf(o[k], o[k], ss);
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    const float mul = 1.0f / sqrtf(((red[0] + red[1]) + (red[2] + red[3])) / (float)vd + p.maps.eps) * (1.0f - p.maps.diff);
+    const int tok = tok_begin + row / G, head = (kvh * G + row % G) / 2;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int col = tid + AW_THREADS * k;
+        if (col < vd) p.out[((size_t)tok * (p.nq / 2) + head) * vd + col] = __float2bfloat16_rn(o[k] * mul);
+    }
+}
+
 template <int D, int KW>
 static int aw_launch(const AwParams &p, int nseq, int max_count, int ksplit, cudaStream_t stream) {
     constexpr int BM = 16 * (4 / KW), AW_BN = KW == 1 ? (D > 128 ? AW_BN_ROWS / 2 : AW_BN_ROWS) : (D > 128 ? AW_BN_KEYS / 2 : AW_BN_KEYS);
@@ -422,7 +474,12 @@ static int aw_launch(const AwParams &p, int nseq, int max_count, int ksplit, cud
     dim3 grid(KW == 4 ? ksplit * p.row_tiles : ((size_t)max_count * G + BM - 1) / BM, p.nkv, nseq);
     kestrel_launch(attention_window_kernel<D, KW>, grid, dim3(AW_THREADS), smem, stream, p);
     int rc = kestrel_check_launch("attention_window");
-    if (rc || KW != 4 || ksplit == 1) return rc;
+    if (rc || KW != 4) return rc;
+    if (p.to_scratch) {
+        kestrel_launch(attention_window_merge_maps_kernel, dim3(p.nkv, nseq, 8 * p.row_tiles), dim3(AW_THREADS), 0, stream, p, ksplit, D);
+        return kestrel_check_launch("attention_window_merge_maps");
+    }
+    if (ksplit == 1) return rc;
     kestrel_launch(attention_window_merge_kernel, dim3(p.nkv, nseq, 16 * p.row_tiles), dim3(AW_THREADS), 0, stream, p, ksplit, D);
     return kestrel_check_launch("attention_window_merge");
 }
@@ -500,7 +557,7 @@ KESTREL_API int kestrel_attention_window_to(const void *q, const void *k_cache, 
     KESTREL_REQUIRE(weighting >= 0 && weighting <= 2 && softcap >= 0.f && (r1 == nullptr) == (r2 == nullptr), "attention_window: bad score options");
     KESTREL_REQUIRE(kestrel_attention_window_supported(hd, vd, nq, nkv), "attention_window: head sizes %d / %d, heads %d / %d are not taken", hd, vd, nq, nkv);
     KESTREL_REQUIRE(nseq > 0 && nseq <= 65535 && nkv <= 65535 && max_count > 0 && window >= 0 && keep_first >= 0, "attention_window: bad sizes");
-    AwParams p;
+    AwParams p = {};
     p.q = (const __nv_bfloat16 *)q;
     p.k_cache = (const __nv_bfloat16 *)k_cache;
     p.v_cache = (const __nv_bfloat16 *)v_cache;
@@ -540,4 +597,48 @@ KESTREL_API int kestrel_attention_window_to(const void *q, const void *k_cache, 
     if (D <= 128) { AW_CASE(128); }
     AW_CASE(256);
 #undef AW_CASE
+}
+
+// rows a request may bring for the kernel's tiling of few rows (tokens x heads of a group)
+KESTREL_API int kestrel_attention_window_keys_rows(void) { return AW_KEYS_MODE_ROWS; }
+
+// Differential attention of steps of few tokens: 2 nq query heads of 2 dim padded numbers (attention_prepare_ex.cu, `maps`) over nkv
+// key heads; the merge of the keys' shares combines and norms the heads.
+KESTREL_API int kestrel_attention_window_maps(const void *q, const void *k_cache, const void *v_cache, void *out, const int *cu_seqlens,
+                                              const int *kv_lens, const int *block_table, int table_stride, int page_size, int nseq, int max_count,
+                                              int nq, int nkv, int dim, int vd, float scale, int ksplit, float *scratch, const float *lq1,
+                                              const float *lk1, const float *lq2, const float *lk2, float diff, float eps, cudaStream_t stream) {
+    if (nseq == 0 || max_count == 0) return 0;
+    const int hd = 2 * dim;
+    KESTREL_REQUIRE(scratch && ksplit >= 1 && ksplit <= 32, "attention_window_maps: %d shares of the keys, scratch %p", ksplit, (void *)scratch);
+    KESTREL_REQUIRE(kestrel_attention_window_supported(hd, vd, 2 * nq, nkv), "attention_window_maps: maps of %d, values of %d, heads %d / %d are not taken", dim, vd, nq, nkv);
+    KESTREL_REQUIRE(nseq > 0 && nseq <= 65535 && nkv <= 65535 && max_count > 0 && (long long)max_count * (2 * nq / nkv) <= AW_KEYS_MODE_ROWS,
+                    "attention_window_maps: %d tokens a request bring more rows than this tiling takes", max_count);
+    AwParams p = {};
+    p.q = (const __nv_bfloat16 *)q;
+    p.k_cache = (const __nv_bfloat16 *)k_cache;
+    p.v_cache = (const __nv_bfloat16 *)v_cache;
+    p.out = (__nv_bfloat16 *)out;
+    p.cu_seqlens = cu_seqlens;
+    p.kv_lens = kv_lens;
+    p.block_table = block_table;
+    p.table_stride = table_stride;
+    p.page_size = page_size;
+    p.nq = 2 * nq;
+    p.nkv = nkv;
+    p.hd = hd;
+    p.vd = p.v_ld = vd;
+    p.scale_log2 = scale * 1.4426950408889634f;
+    p.scale = scale;
+    p.to_scratch = 1;
+    p.maps = {lq1, lk1, lq2, lk2, dim, diff, eps};
+    p.ksplit = ksplit;
+    p.row_tiles = (max_count * (2 * nq / nkv) + 15) / 16;
+    const int D = max(hd, vd), Dt = D <= 32 ? 32 : (D <= 64 ? 64 : (D <= 128 ? 128 : 256));
+    p.part_o = scratch;
+    p.part_ml = scratch + (size_t)nseq * nkv * p.row_tiles * ksplit * 16 * Dt;
+    if (Dt == 32) return aw_launch<32, 4>(p, nseq, max_count, ksplit, stream);
+    if (Dt == 64) return aw_launch<64, 4>(p, nseq, max_count, ksplit, stream);
+    if (Dt == 128) return aw_launch<128, 4>(p, nseq, max_count, ksplit, stream);
+    return aw_launch<256, 4>(p, nseq, max_count, ksplit, stream);
 }

@@ -6,20 +6,10 @@
 // The maps' outputs arrive in float32, [T, heads, 2, vd], as the attention kernels write them for 2 * heads query heads whose
 // rows are zero outside their own map's part of a cache row (attention_prepare_ex.cu, `maps`).
 #include "common.cuh"
+#include "differential.cuh"
 #include <math.h>
 
 #define DC_WARPS 4
-
-// lambda, the same bits in every warp: the sums run over the lanes' elements in ascending order, then a shuffle tree
-__device__ __forceinline__ float differential_lambda(const float *lq1, const float *lk1, const float *lq2, const float *lk2, int dim, float diff,
-                                                     int lane) {
-    float a = 0.f, b = 0.f;
-    for (int i = lane; i < dim; i += 32) {
-        a = fmaf(lq1[i], lk1[i], a);
-        b = fmaf(lq2[i], lk2[i], b);
-    }
-    return expf(warp_sum(a)) - expf(warp_sum(b)) + diff;
-}
 
 template <typename T>
 __global__ void __launch_bounds__(DC_WARPS * 32)
@@ -62,4 +52,63 @@ KESTREL_API int kestrel_differential_combine(const float *a, const float *lq1, c
     else
         return kestrel_fail(-2, "differential_combine: unknown dtype %d", dtype);
     return kestrel_check_launch("differential_combine");
+}
+
+// The maps' outputs as key-range slices: part_o [T * H * 2, slices, ld] unnormalised, part_ml [T * H * 2, slices, 2] the slices' (maximum
+// in base-2 units, sum).  Slices in ascending order, then the head as above.  A block of four warps a (token, head): warps 0, 1
+// first merge map 1, warps 2, 3 map 2, each its half of the columns.
+__global__ void __launch_bounds__(128)
+differential_merge_kernel(const float *__restrict__ part_o, const float *__restrict__ part_ml, int slices, int ld, const DifferentialOpts opts,
+                          __nv_bfloat16 *__restrict__ out, int vd) {
+    pdl_launch_dependents();
+    __shared__ float a_s[2][256];
+    __shared__ float red[4];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const float lam = differential_lambda(opts, lane);
+    pdl_wait();
+    const size_t h = blockIdx.x;                      // (token, head)
+    const int map = tid >> 6;
+    const size_t row = (h * 2 + map) * slices;
+    float M = -INFINITY, L = 0.f;
+    for (int s = 0; s < slices; ++s) M = fmaxf(M, part_ml[(row + s) * 2]);
+    for (int s = 0; s < slices; ++s) {
+        const float m = part_ml[(row + s) * 2];
+        if (m != -INFINITY) L = fmaf(part_ml[(row + s) * 2 + 1], exp2f(m - M), L);
+    }
+    const float inv = 1.0f / L;
+    for (int c = tid & 63; c < vd; c += 64) {
+        float acc = 0.f;
+        for (int s = 0; s < slices; ++s) {
+            const float m = part_ml[(row + s) * 2];
+            if (m != -INFINITY) acc = fmaf(part_o[(row + s) * ld + c], exp2f(m - M), acc);
+        }
+        a_s[map][c] = acc * inv;
+    }
+    __syncthreads();
+    float o[2], ss = 0.f;                             // vd <= 256
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int c = tid + 128 * k;
+        o[k] = c < vd ? a_s[0][c] - lam * a_s[1][c] : 0.f;
+        ss = fmaf(o[k], o[k], ss);
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    const float mul = 1.0f / sqrtf(((red[0] + red[1]) + (red[2] + red[3])) / (float)vd + opts.eps) * (1.0f - opts.diff);
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int c = tid + 128 * k;
+        if (c < vd) out[h * vd + c] = __float2bfloat16_rn(o[k] * mul);
+    }
+}
+
+KESTREL_API int kestrel_differential_merge(const float *part_o, const float *part_ml, int slices, int ld, const float *lq1, const float *lk1,
+                                           const float *lq2, const float *lk2, int dim, float diff, float eps, void *out, int T, int H, int vd,
+                                           cudaStream_t stream) {
+    if (T == 0) return 0;
+    KESTREL_REQUIRE(T > 0 && H > 0 && slices > 0 && dim > 0 && vd > 0 && vd <= 256 && ld >= vd && (long long)T * H < (1ll << 31), "differential_merge: bad sizes");
+    const DifferentialOpts opts = {lq1, lk1, lq2, lk2, dim, diff, eps};
+    kestrel_launch(differential_merge_kernel, dim3(T * H), dim3(128), 0, stream, part_o, part_ml, slices, ld, opts, (__nv_bfloat16 *)out, vd);
+    return kestrel_check_launch("differential_merge");
 }

@@ -22,6 +22,7 @@
 // (TMA); N, T and K need not be multiples of the tile - TMA fills out-of-range rows and
 // columns with zeros and stores are predicated.  Anything else is refused
 // (kestrel_gemm_tc_supported) and takes the CUDA-core kernel.
+#include "xielu.cuh"
 #include "tcgen05.cuh"
 #include <mutex>
 #include <unordered_map>
@@ -35,7 +36,8 @@ enum { TC_PARTIAL = 0, TC_SWIGLU = 1, TC_PARTIAL2 = 2, TC_SWIGLU_T = 3, TC_QKV_P
 // and writes the storage type, out bf16 [T, N] = act(x w^T) - a feed-forward's first product without
 // a gate: the float32 plane is neither written nor read back.  The kernel's `up_row_offset` argument
 // carries the activation: 1 the square of relu, 2 tanh, 3 silu, 4 gelu (erf), 5 gelu (tanh form) (the numbering and the arithmetic of
-// the elementwise kernel that serves the product when it comes as slices: same bits).
+// the elementwise kernel that serves the product when it comes as slices: same bits); 6 is xIELU, whose two numbers come in
+// `prep.act_p` (xielu.cuh).  A bias per feature (`prep.bias`) is added before the activation.
 __device__ __forceinline__ float tc_act(float z, int act) {
     if (act == 4) return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
     if (act == 5) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
@@ -67,6 +69,7 @@ struct QkvPrepParams {
     int table_stride, page_size;
     __nv_bfloat16 *k_cache, *v_cache, *q_out;
     int nq, nkv, write_kv;
+    const float *act_p;              // ACT: the numbers of an activation that has any
 };
 
 // ------------------------------------------------------------------------------- kernel
@@ -727,6 +730,10 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
             }
             int valid = min(TCP_BN, T - t0);
             const int c_begin = ((warp - 2) >> 2) * (TCP_BN / TCP_EPI_GROUPS);      // each group of four warps its columns
+            Xielu xielu;
+            float act_bias = 0.f;
+            if (MODE == TC_ACT && up_row_offset == 6) xielu = Xielu(prep.act_p);
+            if (MODE == TC_ACT && prep.bias && n < N) act_bias = prep.bias[n];
 #pragma unroll 1
             for (int c = c_begin; c < c_begin + TCP_BN / TCP_EPI_GROUPS; c += 16) {
                 if (c >= valid) break;
@@ -746,7 +753,15 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                     }
                 } else if (MODE == TC_ACT) {
                     __nv_bfloat16 *o = (__nv_bfloat16 *)out;
-                    if (n < N) {
+                    if (prep.bias) {
+#pragma unroll
+                        for (int jj = 0; jj < 16; ++jj) g[jj] += act_bias;
+                    }
+                    if (n < N && up_row_offset == 6) {
+#pragma unroll
+                        for (int jj = 0; jj < 16; ++jj)
+                            if (c + jj < valid) o[(size_t)(t0 + c + jj) * ldo + n] = __float2bfloat16_rn(xielu(g[jj]));
+                    } else if (n < N) {
 #pragma unroll
                         for (int jj = 0; jj < 16; ++jj)
                             if (c + jj < valid) o[(size_t)(t0 + c + jj) * ldo + n] = __float2bfloat16_rn(tc_act(g[jj], up_row_offset));
@@ -1141,8 +1156,14 @@ KESTREL_API int kestrel_gemm_tc_add(const void *x, const void *w, float *residua
 // product as slices and lets an elementwise kernel apply the activation.
 KESTREL_API int kestrel_gemm_tc_act(const void *x, const void *w, void *out, int act, int T, int N, int K, long long ldx, long long ldw,
                                     long long ldo, cudaStream_t stream) {
+    return kestrel_gemm_tc_act_with(x, w, nullptr, out, act, nullptr, T, N, K, ldx, ldw, ldo, stream);
+}
+
+// the same with a bias [N] (may be null) and, for activation 6 (xIELU), its two numbers
+KESTREL_API int kestrel_gemm_tc_act_with(const void *x, const void *w, const float *bias, void *out, int act, const float *act_p, int T, int N, int K,
+                                         long long ldx, long long ldw, long long ldo, cudaStream_t stream) {
     if (T == 0) return 0;
-    KESTREL_REQUIRE(act >= 1 && act <= 5, "gemm_tc_act: unknown activation %d", act);
+    KESTREL_REQUIRE(act >= 1 && act <= 6 && (act == 6) == (act_p != nullptr), "gemm_tc_act: unknown activation %d, or its numbers are missing", act);
     if (T <= g_pair_min_tokens || !g_persistent || !g_pairs || !kestrel_gemm_tc_supported(x, w, T, N, K, ldx, ldw)) return 1;
     if (kestrel_gemm_tc_splits(T, N, K) > 1) return 1;
     CUtensorMap mw, mx;
@@ -1150,7 +1171,10 @@ KESTREL_API int kestrel_gemm_tc_act(const void *x, const void *w, void *out, int
     if (rc) return rc;
     rc = kestrel_tensor_map_bf16(&mx, x, T, K, ldx, TCP_BN / 2);
     if (rc) return rc;
-    return launch_tc_pair<TC_ACT>(mw, mx, out, T, N, K, ldo, act, 0, 1, 0, stream);
+    QkvPrepParams prep = {};
+    prep.bias = bias;
+    prep.act_p = act_p;
+    return launch_tc_pair<TC_ACT>(mw, mx, out, T, N, K, ldo, act, 0, 1, 0, stream, prep);
 }
 
 // The q, k, v product of a prompt portion and everything between it and attention in one kernel

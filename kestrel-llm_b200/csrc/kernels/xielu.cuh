@@ -7,6 +7,7 @@ __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + 
 
 struct Xielu {
     float up, down;
+    __device__ __forceinline__ Xielu() : up(0.f), down(0.f) {}
     __device__ __forceinline__ explicit Xielu(const float *pq) : up(softplus_f32(pq[0])), down(0.5f + softplus_f32(pq[1])) {}
     __device__ __forceinline__ float operator()(float z) const {
         const float curved = z > 0.f ? up * z * z : down * (expm1f(z) - z);

@@ -512,11 +512,10 @@ def linear_act(x: torch.Tensor, w: torch.Tensor, act: str, weights_static: bool 
     product's epilogue and the float32 product never reaches memory; otherwise the product comes as slices and
     `partial_columns_act` sums and activates them.  Both ways give the same bits where the product is one slice."""
     T, N = x.shape[0], w.shape[0]
-    if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.dim() == 2 and w.dim() == 2 and linear_act_fused and \
-            bias is None and act_params is None:
+    if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.dim() == 2 and w.dim() == 2 and linear_act_fused:
         out = torch.empty((T, N), dtype=torch.bfloat16, device=x.device)
-        rc = library().kestrel_gemm_tc_act(x.data_ptr(), w.data_ptr(), out.data_ptr(), COLUMN_ACTS[act], T, N, x.shape[1], x.stride(0),
-                                           w.stride(0), out.stride(0), _stream())
+        rc = library().kestrel_gemm_tc_act_with(x.data_ptr(), w.data_ptr(), _p(bias), out.data_ptr(), COLUMN_ACTS[act], _p(act_params), T, N,
+                                                x.shape[1], x.stride(0), w.stride(0), out.stride(0), _stream())
         if rc != 1:
             _check(rc)
             return out
@@ -1158,6 +1157,66 @@ def differential_combine(a: torch.Tensor, lq1: torch.Tensor, lk1: torch.Tensor, 
                                                   float(eps), out.data_ptr(), _code(out, "differential_combine.out"), T, H, vd, _stream()))
 
 
+def attention_tc_maps(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, batch, block_table: torch.Tensor,
+                      page_size: int, nq: int, nkv: int, dim: int, vd: int, scale: float, lambdas, diff: float, eps: float,
+                      slices: int = 1, slice_len: int = 1 << 30) -> None:
+    """Differential attention of a step with prompt portions on the tcgen05 kernel (maps of 64, values of 128): both maps, their
+    combination and the head's norm in one kernel; with ``slices`` of the key range a second one merges them."""
+    _need(q, "attention_tc_maps.q", torch.bfloat16, 2)
+    _need(out, "attention_tc_maps.out", torch.bfloat16, 2)
+    _need(k_cache, "attention_tc_maps.k_cache", torch.bfloat16, 4)
+    _need(v_cache, "attention_tc_maps.v_cache", torch.bfloat16, 4)
+    _need(block_table, "attention_tc_maps.block_table", torch.int32, 2)
+    T = q.shape[0]
+    if q.shape[1] != nq * 2 * dim or out.shape != (T, nq * vd) or T != batch.num_tokens:
+        raise KernelError("attention_tc_maps: shapes differ")
+    if tuple(k_cache.shape[1:]) != (nkv, page_size, 2 * dim) or tuple(v_cache.shape[1:]) != (nkv, page_size, vd):
+        raise KernelError("attention_tc_maps: the cache planes do not fit the heads")
+    tile_seq, tile_row0 = row_tiles(batch, nq // nkv, 128)
+    part_o = part_ml = None
+    if slices > 1:
+        part_o = torch.empty((T * nq * 2, slices, 128), dtype=torch.float32, device=q.device)
+        part_ml = torch.empty((T * nq * 2, slices, 2), dtype=torch.float32, device=q.device)
+    slice_len = min(int(slice_len), (1 << 30) // 128 * 128)
+    for t in lambdas:
+        _need(t, "attention_tc_maps.lambda", torch.float32, 1)
+    _check(library().kestrel_attention_tc_maps(
+        q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), _p(part_o), _p(part_ml), tile_seq.data_ptr(), tile_row0.data_ptr(),
+        tile_seq.shape[0], 128, batch.cu_seqlens.data_ptr(), batch.kv_lens.data_ptr(), block_table.data_ptr(), block_table.shape[1],
+        block_table.stride(0), int(page_size), int(k_cache.shape[0]), T, nq, nkv, dim, vd, 0, int(slices), slice_len, float(scale),
+        *(t.data_ptr() for t in lambdas), float(diff), float(eps), _stream()))
+    if slices > 1:
+        global launches
+        launches += 1          # the merge kernel
+
+
+def attention_window_maps(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch, block_table: torch.Tensor, page_size: int,
+                          out: torch.Tensor, nq: int, nkv: int, dim: int, vd: int, scale: float, lambdas, diff: float, eps: float) -> bool:
+    """Differential attention of a step of few tokens on the kernel of `attention_window`, whose merge of the keys' shares combines and
+    norms the heads.  ``q`` has padded rows [T, 2 nq, 2 dim].  False if the step brings too many rows; nothing has run then."""
+    lib = library()
+    if batch.max_count * (2 * nq // nkv) > lib.kestrel_attention_window_keys_rows():
+        return False
+    _need(q, "attention_window_maps.q", torch.bfloat16, 2)
+    _need(out, "attention_window_maps.out", torch.bfloat16, 2)
+    _need(k_cache, "attention_window_maps.k_cache", torch.bfloat16, 4)
+    _need(v_cache, "attention_window_maps.v_cache", torch.bfloat16, 4)
+    T = q.shape[0]
+    if q.shape[1] != 2 * nq * 2 * dim or out.shape != (T, nq * vd) or tuple(k_cache.shape[1:]) != (nkv, page_size, 2 * dim) or \
+            tuple(v_cache.shape[1:]) != (nkv, page_size, vd):
+        raise KernelError("attention_window_maps: shapes differ")
+    sizes = (int(batch.num_seqs), int(batch.max_count), 2 * nq, nkv, 2 * dim, vd)
+    ksplit = lib.kestrel_attention_window_splits(*sizes, 0, int(batch.max_kv_len)) if _window_splits else 1
+    scratch = torch.empty(lib.kestrel_attention_window_scratch_floats(*sizes, ksplit), dtype=torch.float32, device=q.device)
+    _check(lib.kestrel_attention_window_maps(
+        q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), batch.cu_seqlens.data_ptr(), batch.kv_lens.data_ptr(),
+        block_table.data_ptr(), block_table.stride(0), int(page_size), int(batch.num_seqs), int(batch.max_count), nq, nkv, dim, vd, float(scale),
+        ksplit, scratch.data_ptr(), *(t.data_ptr() for t in lambdas), float(diff), float(eps), _stream()))
+    global launches
+    launches += 1              # the merge kernel
+    return True
+
+
 # ---- attention over cached latents -----------------------------------------------------------
 
 def latent_prepare(fused: Partials, q_norm_w: torch.Tensor, kv_norm_w: torch.Tensor, norm_eps: float, positions: torch.Tensor,
@@ -1418,6 +1477,55 @@ def retention_prepare(fused: Partials, positions: torch.Tensor, rotation, decay:
                                                decay.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), _p(w), _code(q, "retention_prepare.q"),
                                                T, H, d, dv, _stream()))
     return q, k, v, w
+
+
+def retention_step(fused: Partials, positions: torch.Tensor, rotation, decay: torch.Tensor, state: torch.Tensor, batch, eps: float,
+                   out: torch.Tensor, H: int, d: int, dv: int) -> None:
+    """Steps of few tokens per request: from the columns [q | k | v | gate] of a fused product to out = (S^T q), normed per head, times
+    silu(gate), in one kernel; S [H, d, dv] at the start of each request's state slot."""
+    _need(state, "retention_step.state", torch.float32, 2)
+    _need(out, "retention_step.out", dims=2)
+    if fused.bias is not None or fused.tokens != out.shape[0] or fused.width < 2 * H * (d + dv) or out.shape[1] != H * dv or \
+            state.shape[1] < H * d * dv:
+        raise KernelError("retention_step: shapes differ, or a bias is pending")
+    _check(library().kestrel_retention_step(fused.data.data_ptr(), fused.slices, fused.slice_stride, fused.width, positions.data_ptr(),
+                                            _p(rotation.inv_freq) if rotation is not None else None, rotation.dim if rotation is not None else 0,
+                                            decay.data_ptr(), state.data_ptr(), state.stride(0), 0, batch.cu_seqlens.data_ptr(),
+                                            batch.slots.data_ptr(), float(eps), out.data_ptr(), _code(out, "retention_step.out"), batch.num_seqs,
+                                            H, d, dv, _stream()))
+
+
+def retention_chunks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, powers: torch.Tensor, fused: Partials, gate_col0: int,
+                     state: torch.Tensor, batch, eps: float, out: torch.Tensor, H: int, d: int, dv: int) -> None:
+    """Prompt portions in chunks on the tensor cores: q, k, v bfloat16 as `retention_prepare` leaves them, ``powers`` [H, chunk + 1] the
+    decays' powers; out = (S^T q), normed per head, times silu of the gate's columns.  Three kernels; the states in front of the chunks
+    pass through a scratch of one state per chunk."""
+    _need(state, "retention_chunks.state", torch.float32, 2)
+    _need(powers, "retention_chunks.powers", torch.float32, 2)
+    for t, name, n in ((q, "q", H * d), (k, "k", H * d), (v, "v", H * dv), (out, "out", H * dv)):
+        _need(t, f"retention_chunks.{name}", torch.bfloat16, 2)
+        if t.shape != (q.shape[0], n):
+            raise KernelError(f"retention_chunks.{name}: shape {tuple(t.shape)}")
+    lib = library()
+    chunk = lib.kestrel_retention_chunk_tokens()
+    if fused.bias is not None or fused.tokens != q.shape[0] or state.shape[1] < H * d * dv or powers.shape != (H, chunk + 1):
+        raise KernelError("retention_chunks: shapes differ, or a bias is pending")
+    tile_seq, tile_row0 = row_tiles(batch, 1, chunk)
+    kept = batch.__dict__.setdefault("_row_tiles", {})
+    if ("first", chunk) not in kept:
+        first = [0]
+        for n in batch.counts:
+            first.append(first[-1] + -(-n // chunk))
+        kept[("first", chunk)] = torch.tensor(first, dtype=torch.int32).to(q.device, non_blocking=True)
+    tiles = tile_seq.shape[0]
+    scratch = torch.empty((tiles * H * d * dv,), dtype=torch.float32, device=q.device)
+    _check(lib.kestrel_retention_chunks(q.data_ptr(), k.data_ptr(), v.data_ptr(), powers.data_ptr(), fused.data.data_ptr(), fused.slices,
+                                        fused.slice_stride, fused.width, int(gate_col0), state.data_ptr(), state.stride(0), 0,
+                                        batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), tile_seq.data_ptr(), tile_row0.data_ptr(),
+                                        kept[("first", chunk)].data_ptr(), tiles, scratch.data_ptr(), float(eps), out.data_ptr(), batch.num_seqs,
+                                        H, d, dv, _stream()))
+    global launches
+    launches += 2
 
 
 # ---- routed feed-forward -----------------------------------------------------------------------

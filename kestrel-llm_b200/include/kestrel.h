@@ -262,9 +262,21 @@ KESTREL_API int kestrel_head_norm_act(const float *o, const float *w, int w_stri
 /* ---- retention: a fixed decay per head (retention.cu) ---- */
 /* product columns [q: H d | k: H d | v: H dv | ...]: q, k turned by position (first `rot` dimensions, rotate-half), k times d^-1/2; q_out, k_out [T, H d], v_out [T, H dv] in `dtype`; w_out (may be NULL) [T, H d] = the head's decay */
 KESTREL_API int kestrel_retention_prepare(const float *partial, int S, long long slice_stride, int ld, const int *positions, const float *inv_freq, int rot, const float *decay, void *q_out, void *k_out, void *v_out, float *w_out, int dtype, int T, int H, int d, int dv, kestrel_stream_t stream);
+/* steps of few tokens per request, everything between the fused product (columns [q | k | v | gate]) and the output product in one kernel: out [T, H dv] = (S^T q) / its root mean square (eps) per head * silu(gate), S float32 at state_off of the requests' slots; d, dv <= 256 */
+KESTREL_API int kestrel_retention_step(const float *partial, int S, long long slice_stride, int ld, const int *positions, const float *inv_freq, int rot, const float *decay, float *state, long long state_stride, long long state_off, const int *cu_seqlens, const int *slots, float eps, void *out, int dtype, int nseq, int H, int d, int dv, kestrel_stream_t stream);
+/* prompt portions in chunks of kestrel_retention_chunk_tokens() tokens on the tensor cores (bfloat16 q, k, v as kestrel_retention_prepare leaves them; d, dv multiples of 8 up to 256): tiles list the chunks (request, first token among the request's), first_tile [nseq + 1] each request's first; powers [H, chunk + 1] = decay^n; scratch of tiles * H * d * dv floats; gate columns at gate_col0 of the fused product */
+KESTREL_API int kestrel_retention_chunk_tokens(void);
+KESTREL_API int kestrel_retention_chunks(const void *q, const void *k, const void *v, const float *powers, const float *partial, int S, long long slice_stride, int ld, int gate_col0, float *state, long long state_stride, long long state_off, const int *cu_seqlens, const int *slots, const int *tile_seq, const int *tile_row0, const int *first_tile, int tiles, float *scratch, float eps, void *out, int nseq, int H, int d, int dv, kestrel_stream_t stream);
 
 /* ---- differential attention (differential.cu): a [T, H, 2, vd] the two maps' outputs; out = (a1 - lambda a2) / its root mean square (eps) * (1 - diff), lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff ---- */
 KESTREL_API int kestrel_differential_combine(const float *a, const float *lq1, const float *lk1, const float *lq2, const float *lk2, int dim, float diff, float eps, void *out, int dtype, int T, int H, int vd, kestrel_stream_t stream);
+/* the same from key-range slices: part_o [T H 2, slices, ld] unnormalised outputs, part_ml [T H 2, slices, 2] their maxima (base-2 units) and sums; bfloat16 out */
+KESTREL_API int kestrel_differential_merge(const float *part_o, const float *part_ml, int slices, int ld, const float *lq1, const float *lk1, const float *lq2, const float *lk2, int dim, float diff, float eps, void *out, int T, int H, int vd, kestrel_stream_t stream);
+/* prompt portions on the tcgen05 attention kernel: q [T, nq, 2, dim], K pages of rows of 2 dim, V pages of rows of vd (dim 64, vd 128), tiles of up to 128 (token, head) rows; out [T, nq, vd] the combined, normed heads; slices > 1 needs part_o [T nq 2, slices, 128] and part_ml [T nq 2, slices, 2] */
+KESTREL_API int kestrel_attention_tc_maps(const void *q, const void *k_cache, const void *v_cache, void *out, float *part_o, float *part_ml, const int *tile_seq, const int *tile_row0, int tiles, int rows_per_tile, const int *cu_seqlens, const int *kv_lens, const int *block_table, int table_width, int table_stride, int page_size, int cache_pages, int T, int nq, int nkv, int dim, int vd, int window, int slices, int slice_len, float scale, const float *lq1, const float *lk1, const float *lq2, const float *lk2, float diff, float eps, kestrel_stream_t stream);
+/* few rows a request (at most kestrel_attention_window_keys_rows() rows of 2 nq / nkv a token): q [T, 2 nq, 2 dim] padded rows; the kernel of kestrel_attention_window over shares of the keys, whose merge combines and norms the heads; scratch of kestrel_attention_window_scratch_floats(nseq, max_count, 2 nq, nkv, 2 dim, vd, ksplit) floats; bfloat16 out [T, nq, vd] */
+KESTREL_API int kestrel_attention_window_keys_rows(void);
+KESTREL_API int kestrel_attention_window_maps(const void *q, const void *k_cache, const void *v_cache, void *out, const int *cu_seqlens, const int *kv_lens, const int *block_table, int table_stride, int page_size, int nseq, int max_count, int nq, int nkv, int dim, int vd, float scale, int ksplit, float *scratch, const float *lq1, const float *lk1, const float *lq2, const float *lk2, float diff, float eps, kestrel_stream_t stream);
 
 /* ---- routed feed-forward (moe.cu) ---- */
 KESTREL_API int kestrel_moe_route(const float *z_part, int S, long long slice_stride, const float *bias, int *ids, float *weights, int T, int E, int top, kestrel_stream_t stream);
@@ -305,6 +317,8 @@ KESTREL_API int kestrel_gemm_tc_w(const void *x, const void *w, float *out, int 
 KESTREL_API int kestrel_gemm_tc(const void *x, const void *w, float *out, int T, int N, int K, long long ldx, long long ldw, long long ldo, int splits, long long slice_stride, kestrel_stream_t stream);
 KESTREL_API int kestrel_gemm_tc_add(const void *x, const void *w, float *residual, int T, int N, int K, long long ldx, long long ldw, long long ldo, kestrel_stream_t stream);
 KESTREL_API int kestrel_gemm_tc_act(const void *x, const void *w, void *out, int act, int T, int N, int K, long long ldx, long long ldw, long long ldo, kestrel_stream_t stream);
+/* the same with a bias [N] (may be NULL) before the activation; act 6: xIELU with its two numbers in act_p (NULL for the others) */
+KESTREL_API int kestrel_gemm_tc_act_with(const void *x, const void *w, const float *bias, void *out, int act, const float *act_p, int T, int N, int K, long long ldx, long long ldw, long long ldo, kestrel_stream_t stream);
 KESTREL_API int kestrel_gemm_tc_swiglu_w(const void *x, const void *w, void *out, int T, int ff, int K, long long ldx, long long ldw, long long ldo, int weights_static, kestrel_stream_t stream);
 KESTREL_API int kestrel_gemm_tc_swiglu(const void *x, const void *w, void *out, int T, int ff, int K, long long ldx, long long ldw, long long ldo, kestrel_stream_t stream);
 /* the q, k, v product of many tokens with the prepare kernel's work in its epilogue (head size 128, rotate-half over the whole head); 0 done, 1 this form does not apply and nothing ran */

@@ -11,7 +11,11 @@ own, over the same values, and the second is subtracted from the first.
 A token's cache row holds both maps' keys, [k_1 | k_2], as ONE key of 2 d numbers, so a layer's pages are those of any grouped
 attention with head sizes (2 d, dv).  A query of map i is that long too, zero in the other map's half: its dot product with a row is
 its own map's score, and 2 H query heads over G key/value heads run on the attention kernels as they are - keys and values are read
-once for both maps.  Their float32 outputs are combined by `ops.differential_combine`.
+once for both maps.  Their float32 outputs are combined by `ops.differential_combine`.  Steps with prompt portions of maps of 64
+over values of 128 take the tcgen05 kernel (`ops.attention_tc_maps`), which works on the two maps as two row tiles, multiplies each
+with its own half of the keys, and combines and norms the heads itself; a long key range is cut into slices there so that the few
+tiles of a portion far into a context fill the chip.  Steps of few tokens share the keys out over CTAs; the kernel that merges the
+shares combines and norms the heads.
 
 A mixer built with ``own_kv=False`` has no key and value projections and attends over the pages that an earlier layer of the same
 step wrote, with its own queries, lambda and scale.
@@ -29,6 +33,10 @@ from .linear import Linear
 
 class DifferentialAttention(Mixer):
     force_plain = False        # tests: bfloat16 through the plain kernel too, the twin of the tensor-core one
+    tcgen05 = True             # tests: off, portions of maps of 64 over values of 128 stay on the mma.sync kernel
+    TC_MIN_ROWS = 64           # a step whose longest portion has more rows (tokens x heads of a group) takes the tcgen05 kernel
+    TC_SLICE = 512             # fewest keys a slice where a portion's key range is cut
+    TC_SLICE_FILL = 148        # CTAs that the cut should reach: one an SM
     graph_safe = True          # forward launches kernels over device tensors of the batch only
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, v_dim: int, dtype: torch.dtype, device, prefix: str, scale: float,
@@ -72,15 +80,33 @@ class DifferentialAttention(Mixer):
         T, H, G, d, dv = x.shape[0], self.heads, self.kv_heads, self.dim, self.v_dim
         fused = self.proj.forward(x)
         table = batch.block_table(cache.group)
-        q = torch.empty((T, 2 * H * 2 * d), dtype=self.dtype, device=x.device)
+        o = torch.empty((T, H * dv), dtype=self.dtype, device=x.device)
+        fast = self.dtype == torch.bfloat16 and not self.force_plain
+        tc = fast and self.tcgen05 and (d, dv) == (64, 128) and not batch.captured and batch.max_count * (H // G) > self.TC_MIN_ROWS and \
+            ops.attention_tc_supported(128, cache.page_size)
+        q = torch.empty((T, 2 * H * d * (1 if tc else 2)), dtype=self.dtype, device=x.device)
         ops.attn_prepare_ex(fused, self.q_norm, self.k_norm, "head", self.norm_eps, batch.positions, batch.seq_of_token, table, cache.page_size,
-                            cache.k, cache.v, q, None, H, G, d, dv, self.own_kv, rotation=self.rotation, maps=2, q_pad=True)
+                            cache.k, cache.v, q, None, H, G, d, dv, self.own_kv, rotation=self.rotation, maps=2, q_pad=not tc)
+        if tc:
+            # few tiles far into a long context: as many slices of the keys as fill the chip
+            tiles = sum(-(-n * (H // G) // 128) for n in batch.counts)
+            fill, slices, slice_len = self.TC_SLICE_FILL // max(1, tiles * G), 1, 1 << 30
+            if fill >= 2 and batch.max_kv_len > 2 * self.TC_SLICE:
+                per = -(-batch.max_kv_len // min(32, fill))
+                slice_len = max(self.TC_SLICE, (per + 127) // 128 * 128)
+                slices = -(-batch.max_kv_len // slice_len)
+            ops.attention_tc_maps(q, cache.k, cache.v, o, batch, table, cache.page_size, H, G, d, dv, self.scale, self.lambdas, self.diff,
+                                  self.norm_eps, slices, slice_len)
+            return self.out.forward(o)
+        window = fast and ops.attention_window_supported(2 * d, dv, 2 * H, G)
+        if window and ops.attention_window_maps(q, cache.k, cache.v, batch, table, cache.page_size, o, H, G, d, dv, self.scale, self.lambdas,
+                                                self.diff, self.norm_eps):
+            return self.out.forward(o)
         a = torch.empty((T, 2 * H * dv), dtype=torch.float32, device=x.device)
-        if self.dtype == torch.bfloat16 and not self.force_plain and ops.attention_window_supported(2 * d, dv, 2 * H, G):
+        if window:
             ops.attention_window(q, cache.k, cache.v, batch, table, cache.page_size, a, 2 * H, G, 2 * d, dv, 0, 0, None, self.scale)
         else:           # float32, sizes that are no multiple of 8, and maps of more than 128
             ops.attention_plain_ex(q, cache.k, cache.v, batch.positions, batch.seq_of_token, table, cache.page_size, a, 2 * H, G, 2 * d, dv, 0, 0,
                                    None, self.scale)
-        o = torch.empty((T, H * dv), dtype=self.dtype, device=x.device)
         ops.differential_combine(a, *self.lambdas, self.diff, self.norm_eps, o, H, dv)
         return self.out.forward(o)

@@ -139,7 +139,7 @@ def _spike(layer, map_, i, j):
         p, half = "l0.mix.", h.shape[1] // 2
         if layer["type"] == "retention":
             other = h.copy()
-            h[j] *= 40.0
+            h[j] *= 6.0
             return other
         H, G, d = m["heads"], m["kv_heads"], m["dim"]
         W[p + "k"][:, half:] = 0.0
@@ -258,6 +258,42 @@ def test_retention_in_chunks_of_unequal_requests(dtype):
         o2 = hs.step([(3, hs_[2][2:5]), (1, hs_[0][400:430]), (2, hs_[1][129:140])])
         for r, (a, b) in enumerate(((o1[0], o2[1]), (o1[1], o2[2]), (o1[2], o2[0]))):
             _close(np.concatenate([a, b]), want[r], dtype, f"request {r}", tol=1e-4 if dtype == "float32" else None)
+
+
+@pytest.mark.parametrize("which", [7, 9, 10, 11, 12])
+def test_retention_forms_against_each_other(which):
+    """One kernel for few tokens, chunks, and the sequential scan: the same portions through each form that takes them."""
+    from kestrel_llm_b200.parts import RetentionMixer
+    label, layer = MIXERS[which]
+    for dtype, cuts in (("bfloat16", [100, 1, 2, 200, 64, 4, 129]), ("float32", [3, 1, 2, 4, 30, 1, 1])):
+        both, want, _ = _mixer_case(layer, dtype, 16, sum(cuts), cuts, seed=which)
+        RetentionMixer.chunked = RetentionMixer.one_kernel = False
+        try:
+            scan, _, _ = _mixer_case(layer, dtype, 16, sum(cuts), cuts, seed=which)
+        finally:
+            RetentionMixer.chunked = RetentionMixer.one_kernel = True
+        scale = float(np.abs(want).max())
+        _close(both, scan, dtype, f"{label}, forms", scale=scale, tol={"float32": 1e-5, "bfloat16": 2e-2}[dtype])
+
+
+@pytest.mark.parametrize("cuts", [[130, 1, 1, 70], [33, 20, 500, 2, 90]])
+@pytest.mark.parametrize("which", [0, 3, 4])
+def test_attention_kernels_against_their_plain_twin(which, cuts):
+    """bfloat16: the tcgen05 kernel, the mma.sync kernel's two tilings and its shares of the keys against the plain kernel."""
+    from kestrel_llm_b200.csrc import ops
+    from kestrel_llm_b200.parts import DifferentialAttention
+    label, layer = MIXERS[which]
+    runs = {}
+    for name, plain, tc, splits in (("default", False, True, True), ("mma", False, False, True), ("one share", False, False, False), ("plain", True, True, True)):
+        DifferentialAttention.force_plain, DifferentialAttention.tcgen05 = plain, tc
+        ops.attention_window_set_splits(splits)
+        try:
+            runs[name], want, _ = _mixer_case(layer, "bfloat16", 16, sum(cuts), cuts, seed=which)
+        finally:
+            DifferentialAttention.force_plain, DifferentialAttention.tcgen05 = False, True
+            ops.attention_window_set_splits(True)
+    for name in ("default", "mma", "one share"):
+        _close(runs[name], runs["plain"], "bfloat16", f"{label}, {name}", scale=float(np.abs(want).max()), tol=2e-2)
 
 
 def _ffn_case(mlp, dtype, n, seed=0, width=48, prepare=None, h_scale=1.0):
