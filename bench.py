@@ -406,7 +406,7 @@ def run_zidivik(args) -> int:
                    "forget_gates", "removal_gates", "recurrence_scan", "head_norm_gate", "combine_normed", "add_gated_normed", "partial_columns_act",
                    "embed_add", "logit_scale_cap", "linear_act", "rglru_branches", "rglru_scan", "moe_route_sigmoid", "moe_experts_ungated",
                    "gate_columns_mul", "latent_rotate_queries", "add_row", "differential_combine", "retention_prepare", "retention_step", "retention_chunks",
-                   "moe_route_scored", "attention_tc_maps", "attention_window_maps", "reduce_partials"]
+                   "moe_route_scored", "attention_tc_maps", "attention_window_maps", "attention_decode_maps", "post_norm_add", "embed_copy"]
 
     def measure(cfg, label):
         model = resolve_architecture(cfg.architecture).build(cfg, torch.bfloat16, dev)

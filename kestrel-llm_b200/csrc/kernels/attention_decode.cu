@@ -313,7 +313,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             if (d0 == 0) { finml[2 * r] = M; finml[2 * r + 1] = L; }
         } else if (!ok) {
             // a wait gave up: nothing is written
-        } else if (p.slices > 1) {
+        } else if (p.slices > 1 || p.partial_only) {
             float *po = p.part_o + (qrow * p.slices + slice) * HD + d0;
             *reinterpret_cast<float4 *>(po) = make_float4(acc[0], acc[1], acc[2], acc[3]);
             *reinterpret_cast<float4 *>(po + 4) = make_float4(acc[4], acc[5], acc[6], acc[7]);
@@ -452,6 +452,40 @@ KESTREL_API int kestrel_attention_decode(const void *q, const void *k_cache, con
     else rc = hd == 64 ? launch_decode<64, false>(mk, mv, p, tiles, cache_pages, stream) : launch_decode<128, false>(mk, mv, p, tiles, cache_pages, stream);
     if (rc || slices == 1 || cluster) return rc;
     return kestrel_attention_merge(part_o, part_ml, out, tile_seq, tile_row0, tiles, 16, cu_seqlens, slices, hd, nq, nkv, nullptr, stream);
+}
+
+// Differential attention of decode tokens on the same kernel: q [T, 2 nq, 2 dim] padded rows (attention_prepare_ex.cu, `maps`) over
+// nkv key heads whose cache rows of K hold both maps' keys and whose values are as long (2 dim = vd = 64 or 128), at most 8 heads a
+// group; every slice leaves its outputs in scratch (part_o [T * 2 nq, slices, vd], part_ml [T * 2 nq, slices, 2]) and
+// kestrel_differential_merge merges the slices, combines the maps and norms the heads.
+KESTREL_API int kestrel_attention_decode_maps(const void *q, const void *k_cache, const void *v_cache, void *out, float *part_o, float *part_ml,
+                                              const int *tile_seq, const int *tile_row0, int tiles, const int *cu_seqlens, const int *kv_lens,
+                                              const int *block_table, int table_width, int table_stride, int page_size, int cache_pages, int T, int nq,
+                                              int nkv, int dim, int vd, int slices, int slice_len, const int *max_kv_ptr, float scale, const float *lq1,
+                                              const float *lk1, const float *lq2, const float *lk2, float diff, float eps, cudaStream_t stream) {
+    if (T == 0 || tiles == 0) return 0;
+    const int hd = 2 * dim;
+    KESTREL_REQUIRE(hd == vd && kestrel_attention_decode_supported(hd, page_size), "attention_decode_maps: maps of %d over values of %d with pages of %d keys are not taken", dim, vd, page_size);
+    KESTREL_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0 && 2 * nq / nkv <= 16, "attention_decode_maps: %d query heads over %d kv heads", nq, nkv);
+    KESTREL_REQUIRE(slices >= 1 && slice_len > 0 && slice_len % AD_BN == 0 && part_o && part_ml, "attention_decode_maps: slice length %d must be a positive multiple of %d", slice_len, AD_BN);
+    KESTREL_REQUIRE(nkv <= 65535 && slices <= 65535, "attention_decode_maps: grid too large");
+    KESTREL_REQUIRE(cache_pages > 0 && (long long)cache_pages * nkv * page_size < (1ll << 31), "attention_decode_maps: a cache of %d pages is beyond the 32-bit row coordinate", cache_pages);
+    CUtensorMap mk, mv;
+    const long long cache_rows = (long long)cache_pages * nkv * page_size;
+    const int box_rows = page_size < AD_BN ? page_size : AD_BN;
+    int rc = kestrel_tensor_map_bf16(&mk, k_cache, cache_rows, hd, hd, box_rows);
+    if (rc == 0) rc = kestrel_tensor_map_bf16(&mv, v_cache, cache_rows, hd, hd, box_rows);
+    if (rc) return rc;
+    AttnParams p = {};
+    p.q = (const __nv_bfloat16 *)q; p.k_cache = (const __nv_bfloat16 *)k_cache; p.v_cache = (const __nv_bfloat16 *)v_cache;
+    p.out = (__nv_bfloat16 *)out; p.part_o = part_o; p.part_ml = part_ml; p.tile_seq = tile_seq; p.tile_row0 = tile_row0;
+    p.cu_seqlens = cu_seqlens; p.kv_lens = kv_lens; p.block_table = block_table; p.table_width = table_width;
+    p.table_stride = table_stride; p.page_size = page_size; p.nq = 2 * nq; p.nkv = nkv; p.hd = hd;
+    p.slices = slices; p.slice_len = slice_len; p.max_kv_ptr = max_kv_ptr; p.partial_only = 1;
+    p.scale_log2 = scale * 1.4426950408889634f;
+    rc = hd == 64 ? launch_decode<64, false>(mk, mv, p, tiles, cache_pages, stream) : launch_decode<128, false>(mk, mv, p, tiles, cache_pages, stream);
+    if (rc) return rc;
+    return kestrel_differential_merge(part_o, part_ml, slices, hd, lq1, lk1, lq2, lk2, dim, diff, eps, out, T, nq, vd, stream);
 }
 
 // Error word of the kernel's bounded waits: 0 = none, 1 = the loader waited for a free stage,

@@ -25,6 +25,7 @@ struct AttnParams {
     float scale;
     ScoreOpts opts;
     int scored;
+    int partial_only;               // attention_decode.cu: the unnormalised outputs go to part_o / part_ml even from one slice
     // two maps a head over the same values (differential attention); read by attention_tc.cu only
     DifferentialOpts maps;
 };

@@ -199,6 +199,113 @@ attn_prepare_ex_kernel(const float *__restrict__ partial, int S, size_t slice_st
     }
 }
 
+// The same work for the common case of rotated, normed heads in a fast form: heads (maps) of HD numbers, all of them turned in
+// rotate-half pairs, a norm per head with a weight, no bias, no gate, values in multiples of HD.  HD / 8 lanes take a head row, a
+// lane the numbers 4 j .. 4 j + 3 and their partners HD / 2 + 4 j .., so that loads and stores are vectors and a pair is turned
+// inside a lane; a value row counts as vd / HD rows that are copied.  A row's sum of squares is a shuffle tree over its lanes:
+// its bits depend on nothing else in the step.
+#define APR_THREADS 128
+__device__ __forceinline__ void apr_store4(float *dst, const float (&x)[4]) { *reinterpret_cast<float4 *>(dst) = make_float4(x[0], x[1], x[2], x[3]); }
+__device__ __forceinline__ void apr_store4(__nv_bfloat16 *dst, const float (&x)[4]) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(x[0], x[1]), hi = __floats2bfloat162_rn(x[2], x[3]);
+    *reinterpret_cast<uint2 *>(dst) = make_uint2(*reinterpret_cast<uint32_t *>(&lo), *reinterpret_cast<uint32_t *>(&hi));
+}
+
+template <typename T, int HD>
+__global__ void __launch_bounds__(APR_THREADS)
+attn_prepare_rows_kernel(const float *__restrict__ partial, int S, size_t slice_stride, int ld, const float *__restrict__ q_w,
+                         const float *__restrict__ k_w, float eps, const int *__restrict__ positions, const int *__restrict__ seq_of_token,
+                         const int *__restrict__ block_table, int table_stride, int page_size, T *__restrict__ k_cache, T *__restrict__ v_cache,
+                         T *__restrict__ q_out, int nq, int nkv, int vd, int has_kv, const float *__restrict__ inv_freq, float rot_scale, int maps,
+                         int q_pad) {
+    constexpr int LANES = HD / 8, ROWS = APR_THREADS / LANES, HALF = HD / 2;
+    __shared__ float cs_s[HALF], sn_s[HALF];
+    pdl_launch_dependents();
+    // the step's description and the weights are not the predecessor's output
+    const int t = blockIdx.x, tid = threadIdx.x, j = tid % LANES, r = blockIdx.y * ROWS + tid / LANES;
+    const int pos = positions[t];
+    for (int i = tid; i < HALF; i += APR_THREADS) {
+        float sn, cs;
+        sincosf((float)pos * inv_freq[i], &sn, &cs);
+        sn_s[i] = sn * rot_scale;
+        cs_s[i] = cs * rot_scale;
+    }
+    const int nqm = nq * maps, nkm = nkv * maps, vr = vd / HD, n_rows = nqm + (has_kv ? nkm + nkv * vr : 0);
+    const int kind = r < nqm ? 0 : (r < nqm + nkm ? 1 : 2);
+    const bool live = r < n_rows;
+    size_t slot_row = 0;
+    if (live && kind != 0) {
+        const int page = block_table[(size_t)seq_of_token[t] * table_stride + pos / page_size];
+        slot_row = (size_t)page * nkv * page_size + (pos % page_size);
+    }
+    float w0[4] = {1.f, 1.f, 1.f, 1.f}, w1[4] = {1.f, 1.f, 1.f, 1.f};
+    const float *w = kind == 0 ? q_w : (kind == 1 ? k_w : nullptr);
+    if (live && w) {
+#pragma unroll
+        for (int c = 0; c < 4; ++c) { w0[c] = w[4 * j + c]; w1[c] = w[HALF + 4 * j + c]; }
+    }
+    __syncthreads();
+    pdl_wait();
+    float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
+    if (live) {
+        const float *src = partial + (size_t)t * ld + (size_t)r * HD + 4 * j;          // q, k and v rows follow each other in the columns
+#pragma unroll 4
+        for (int s = 0; s < S; ++s) {
+            const float4 x = *reinterpret_cast<const float4 *>(src + (size_t)s * slice_stride), y = *reinterpret_cast<const float4 *>(src + (size_t)s * slice_stride + HALF);
+            a[0] += x.x; a[1] += x.y; a[2] += x.z; a[3] += x.w;
+            b[0] += y.x; b[1] += y.y; b[2] += y.z; b[3] += y.w;
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < 4; ++c) ss = fmaf(a[c], a[c], fmaf(b[c], b[c], ss));
+#pragma unroll
+    for (int sh = 1; sh < LANES; sh <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, sh);
+    if (!live) return;
+    T *dst;
+    if (kind == 2) {
+        const int u = r - nqm - nkm;
+        dst = v_cache + (slot_row + (size_t)(u / vr) * page_size) * vd + (u % vr) * HD;
+    } else {
+        const float mul = 1.0f / sqrtf(ss / (float)HD + eps);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            const float x = a[c] * mul * w0[c], y = b[c] * mul * w1[c];
+            const float cs = cs_s[4 * j + c], sn = sn_s[4 * j + c];
+            a[c] = x * cs - y * sn;
+            b[c] = y * cs + x * sn;
+        }
+        const int head = kind == 0 ? r : r - nqm, own = head % maps * HD;
+        if (kind == 1) {
+            dst = k_cache + (slot_row + (size_t)(head / maps) * page_size) * (maps * HD) + own;
+        } else {
+            dst = q_out + ((size_t)t * nqm + head) * (q_pad ? maps * HD : HD);
+            if (q_pad) {
+                const float zero[4] = {0.f, 0.f, 0.f, 0.f};
+                for (int m = 0; m < maps; ++m)
+                    if (m * HD != own) {
+                        apr_store4(dst + m * HD + 4 * j, zero);
+                        apr_store4(dst + m * HD + HALF + 4 * j, zero);
+                    }
+                dst += own;
+            }
+        }
+    }
+    apr_store4(dst + 4 * j, a);
+    apr_store4(dst + HALF + 4 * j, b);
+}
+
+template <typename T, int HD>
+static int apr_launch(const float *partial, int S, long long slice_stride, int ld, const float *q_w, const float *k_w, float eps, const int *positions,
+                      const int *seq_of_token, const int *block_table, int table_stride, int page_size, void *k_cache, void *v_cache, void *q_out,
+                      int n_tokens, int nq, int nkv, int vd, int has_kv, const float *inv_freq, float rot_scale, int maps, int q_pad, cudaStream_t stream) {
+    const int rows = nq * maps + (has_kv ? nkv * (maps + vd / HD) : 0), per = APR_THREADS / (HD / 8);
+    kestrel_launch(attn_prepare_rows_kernel<T, HD>, dim3(n_tokens, (rows + per - 1) / per), dim3(APR_THREADS), 0, stream, partial, S, (size_t)slice_stride, ld, q_w, k_w,
+                   eps, positions, seq_of_token, block_table, table_stride, page_size, (T *)k_cache, (T *)v_cache, (T *)q_out, nq, nkv, vd, has_kv, inv_freq,
+                   rot_scale, maps, q_pad);
+    return kestrel_check_launch("attn_prepare_rows");
+}
+
 KESTREL_API int kestrel_attn_prepare_normed(const float *partial, int S, long long slice_stride, int ld, const float *bias, const float *q_norm_w,
                                             const float *k_norm_w, int qk_norm, int v_norm, float norm_eps, const int *positions,
                                             const int *seq_of_token, const int *block_table, int table_stride, int page_size,
@@ -257,6 +364,21 @@ KESTREL_API int kestrel_attn_prepare_maps(const float *partial, int S, long long
     KESTREL_REQUIRE(hd <= 32 * APX_PER_LANE && vd <= 32 * APX_PER_LANE, "attn_prepare_ex: head size %d / %d exceeds %d", hd, vd, 32 * APX_PER_LANE);
     const int need = nq * maps * hd + (has_kv ? nkv * (maps * hd + vd) : 0) + (gate_out ? nq : 0);
     KESTREL_REQUIRE(ld >= need, "attn_prepare_ex: the product has %d columns, the heads need %d", ld, need);
+    // the fast form for heads of several maps (those of one keep the kernel, and the bits, they have)
+    if (maps > 1 && inv_freq && rot == hd && rot_mode == 0 && qk_norm == 1 && !bias && !v_norm && q_temp_every == 0 && !gate_out && nq > 0 && vd % hd == 0 &&
+        (hd == 32 || hd == 64 || hd == 128) && ld % 4 == 0 && slice_stride % 4 == 0 && ((uintptr_t)partial & 15) == 0 && (dtype == KESTREL_F32 || dtype == KESTREL_BF16)) {
+#define APR_CASE(TT, H_) return apr_launch<TT, H_>(partial, S, slice_stride, ld, q_norm_w, k_norm_w, norm_eps, positions, seq_of_token, block_table, table_stride, page_size, \
+                                                  k_cache, v_cache, q_out, T, nq, nkv, vd, has_kv, inv_freq, rot_scale, maps, q_pad, stream)
+        if (dtype == KESTREL_F32) {
+            if (hd == 32) APR_CASE(float, 32);
+            if (hd == 64) APR_CASE(float, 64);
+            APR_CASE(float, 128);
+        }
+        if (hd == 32) APR_CASE(__nv_bfloat16, 32);
+        if (hd == 64) APR_CASE(__nv_bfloat16, 64);
+        APR_CASE(__nv_bfloat16, 128);
+#undef APR_CASE
+    }
     // few tokens: a block per four head rows, so that the step's few tokens still fill the device
     const int n_heads = nq * maps + (has_kv ? nkv * (maps + 1) : 0);
     // (many tokens: up to four head rows a warp, so that a row's round trips overlap other blocks'; the norm over a whole

@@ -57,11 +57,12 @@ KESTREL_API int kestrel_differential_combine(const float *a, const float *lq1, c
 // The maps' outputs as key-range slices: part_o [T * H * 2, slices, ld] unnormalised, part_ml [T * H * 2, slices, 2] the slices' (maximum
 // in base-2 units, sum).  Slices in ascending order, then the head as above.  A block of four warps a (token, head): warps 0, 1
 // first merge map 1, warps 2, 3 map 2, each its half of the columns.
+#define DM_SLICES 64
 __global__ void __launch_bounds__(128)
 differential_merge_kernel(const float *__restrict__ part_o, const float *__restrict__ part_ml, int slices, int ld, const DifferentialOpts opts,
                           __nv_bfloat16 *__restrict__ out, int vd) {
     pdl_launch_dependents();
-    __shared__ float a_s[2][256];
+    __shared__ float a_s[2][256], f_s[2][DM_SLICES + 1];
     __shared__ float red[4];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const float lam = differential_lambda(opts, lane);
@@ -69,20 +70,27 @@ differential_merge_kernel(const float *__restrict__ part_o, const float *__restr
     const size_t h = blockIdx.x;                      // (token, head)
     const int map = tid >> 6;
     const size_t row = (h * 2 + map) * slices;
-    float M = -INFINITY, L = 0.f;
-    for (int s = 0; s < slices; ++s) M = fmaxf(M, part_ml[(row + s) * 2]);
-    for (int s = 0; s < slices; ++s) {
-        const float m = part_ml[(row + s) * 2];
-        if (m != -INFINITY) L = fmaf(part_ml[(row + s) * 2 + 1], exp2f(m - M), L);
+    if ((warp & 1) == 0) {
+        // the slices' factors 2^(m_s - M), a lane a slice (further ones in rounds), and the row's sum in ascending order
+        float M = -INFINITY, L = 0.f;
+        for (int s = lane; s < slices; s += 32) M = fmaxf(M, part_ml[(row + s) * 2]);
+        M = warp_max(M);
+        for (int s0 = 0; s0 < slices; s0 += 32) {
+            const int s = s0 + lane;
+            const float m = s < slices ? part_ml[(row + s) * 2] : -INFINITY, f = m == -INFINITY ? 0.f : exp2f(m - M);
+            const float l = s < slices && f > 0.f ? part_ml[(row + s) * 2 + 1] * f : 0.f;
+            if (s < slices && s < DM_SLICES) f_s[map][s] = f;
+            for (int k = 0; k < min(32, slices - s0); ++k) L += __shfl_sync(0xffffffffu, l, k);
+        }
+        if (lane == 0) f_s[map][DM_SLICES] = 1.0f / L;
     }
-    const float inv = 1.0f / L;
+    __syncthreads();
     for (int c = tid & 63; c < vd; c += 64) {
         float acc = 0.f;
-        for (int s = 0; s < slices; ++s) {
-            const float m = part_ml[(row + s) * 2];
-            if (m != -INFINITY) acc = fmaf(part_o[(row + s) * ld + c], exp2f(m - M), acc);
-        }
-        a_s[map][c] = acc * inv;
+#pragma unroll 8
+        for (int s = 0; s < slices; ++s)
+            if (f_s[map][s] > 0.f) acc = fmaf(part_o[(row + s) * ld + c], f_s[map][s], acc);
+        a_s[map][c] = acc * f_s[map][DM_SLICES];
     }
     __syncthreads();
     float o[2], ss = 0.f;                             // vd <= 256
@@ -107,7 +115,7 @@ KESTREL_API int kestrel_differential_merge(const float *part_o, const float *par
                                            const float *lq2, const float *lk2, int dim, float diff, float eps, void *out, int T, int H, int vd,
                                            cudaStream_t stream) {
     if (T == 0) return 0;
-    KESTREL_REQUIRE(T > 0 && H > 0 && slices > 0 && dim > 0 && vd > 0 && vd <= 256 && ld >= vd && (long long)T * H < (1ll << 31), "differential_merge: bad sizes");
+    KESTREL_REQUIRE(T > 0 && H > 0 && slices > 0 && slices <= DM_SLICES && dim > 0 && vd > 0 && vd <= 256 && ld >= vd && (long long)T * H < (1ll << 31), "differential_merge: bad sizes");
     const DifferentialOpts opts = {lq1, lk1, lq2, lk2, dim, diff, eps};
     kestrel_launch(differential_merge_kernel, dim3(T * H), dim3(128), 0, stream, part_o, part_ml, slices, ld, opts, (__nv_bfloat16 *)out, vd);
     return kestrel_check_launch("differential_merge");

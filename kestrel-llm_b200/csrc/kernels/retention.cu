@@ -58,12 +58,79 @@ retention_prepare_kernel(const float *__restrict__ p, int S, size_t slice_stride
     }
 }
 
+// The same where all of a head is turned and the sizes are multiples of 8: a thread takes eight numbers, four of a head's first half
+// with their partners, or eight of the values.  Same bits.
+__device__ __forceinline__ void rp_store4(float *dst, const float (&x)[4]) { *reinterpret_cast<float4 *>(dst) = make_float4(x[0], x[1], x[2], x[3]); }
+__device__ __forceinline__ void rp_store4(__nv_bfloat16 *dst, const float (&x)[4]) { *reinterpret_cast<uint2 *>(dst) = make_uint2(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3])); }
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+retention_prepare_rows_kernel(const float *__restrict__ p, int S, size_t slice_stride, int ld, const int *__restrict__ positions,
+                              const float *__restrict__ inv_freq, const float *__restrict__ decay, T *__restrict__ q_out, T *__restrict__ k_out,
+                              T *__restrict__ v_out, float *__restrict__ w_out, int H, int d, int dv) {
+    __shared__ float cs_s[128], sn_s[128];
+    pdl_launch_dependents();
+    const int t = blockIdx.x, tid = threadIdx.x, half = d / 2, per = d / 8, n_qk = H * per, n = 2 * n_qk + H * dv / 8;
+    const float pos = (float)positions[t], k_scale = 1.0f / sqrtf((float)d);
+    for (int i = tid; i < half; i += 256) sincosf(pos * inv_freq[i], &sn_s[i], &cs_s[i]);
+    __syncthreads();
+    pdl_wait();
+    for (int u = tid; u < n; u += 256) {
+        const bool is_v = u >= 2 * n_qk, is_k = !is_v && u >= n_qk;
+        const int w = is_k ? u - n_qk : u, h = is_v ? 0 : w / per, j = is_v ? 0 : w % per;
+        const size_t col = is_v ? 2 * (size_t)H * d + (size_t)(u - 2 * n_qk) * 8 : (is_k ? (size_t)H * d : 0) + (size_t)h * d + 4 * j;
+        const int other = is_v ? 4 : half;
+        float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
+        const float *src = p + (size_t)t * ld + col;
+#pragma unroll 4
+        for (int s = 0; s < S; ++s) {
+            const float4 x = *reinterpret_cast<const float4 *>(src + (size_t)s * slice_stride), y = *reinterpret_cast<const float4 *>(src + (size_t)s * slice_stride + other);
+            a[0] += x.x; a[1] += x.y; a[2] += x.z; a[3] += x.w;
+            b[0] += y.x; b[1] += y.y; b[2] += y.z; b[3] += y.w;
+        }
+        if (is_v) {
+            T *dst = v_out + (size_t)t * H * dv + (size_t)(u - 2 * n_qk) * 8;
+            rp_store4(dst, a);
+            rp_store4(dst + 4, b);
+            continue;
+        }
+        const float mul = is_k ? k_scale : 1.0f;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            const float x = a[c], y = b[c], cs = cs_s[4 * j + c], sn = sn_s[4 * j + c];
+            a[c] = (x * cs - y * sn) * mul;
+            b[c] = (y * cs + x * sn) * mul;
+        }
+        T *dst = (is_k ? k_out : q_out) + ((size_t)t * H + h) * d + 4 * j;
+        rp_store4(dst, a);
+        rp_store4(dst + half, b);
+        if (w_out && !is_k) {
+            const float g = decay[h];
+            float *wd = w_out + ((size_t)t * H + h) * d + 4 * j;
+            const float gg[4] = {g, g, g, g};
+            rp_store4(wd, gg);
+            rp_store4(wd + half, gg);
+        }
+    }
+}
+
 KESTREL_API int kestrel_retention_prepare(const float *partial, int S, long long slice_stride, int ld, const int *positions, const float *inv_freq,
                                           int rot, const float *decay, void *q_out, void *k_out, void *v_out, float *w_out, int dtype, int T, int H,
                                           int d, int dv, cudaStream_t stream) {
     if (T == 0) return 0;
     KESTREL_REQUIRE(T > 0 && S > 0 && H > 0 && d > 0 && dv > 0 && ld >= H * (2 * d + dv), "retention_prepare: bad sizes");
     KESTREL_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= d && (rot == 0 || inv_freq), "retention_prepare: %d rotated dimensions of a head of %d", rot, d);
+    if (rot == d && d % 8 == 0 && d <= 256 && dv % 8 == 0 && ld % 4 == 0 && slice_stride % 4 == 0 && ((uintptr_t)partial & 15) == 0) {
+        if (dtype == KESTREL_F32)
+            kestrel_launch(retention_prepare_rows_kernel<float>, dim3(T), dim3(256), 0, stream, partial, S, (size_t)slice_stride, ld, positions, inv_freq, decay,
+                           (float *)q_out, (float *)k_out, (float *)v_out, w_out, H, d, dv);
+        else if (dtype == KESTREL_BF16)
+            kestrel_launch(retention_prepare_rows_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, partial, S, (size_t)slice_stride, ld, positions, inv_freq,
+                           decay, (__nv_bfloat16 *)q_out, (__nv_bfloat16 *)k_out, (__nv_bfloat16 *)v_out, w_out, H, d, dv);
+        else
+            return kestrel_fail(-2, "retention_prepare: unknown dtype %d", dtype);
+        return kestrel_check_launch("retention_prepare");
+    }
     const int by = T >= 512 ? 1 : (3 * H + RT_WARPS - 1) / RT_WARPS;
     if (dtype == KESTREL_F32)
         kestrel_launch(retention_prepare_kernel<float>, dim3(T, by), dim3(RT_WARPS * 32), 0, stream, partial, S, (size_t)slice_stride, ld, positions, inv_freq,
@@ -209,7 +276,8 @@ struct RetentionChunkParams {
     const __nv_bfloat16 *q, *k, *v;      // [T, H d], [T, H d], [T, H dv]
     const float *powers;                 // [H, RC_C + 1]
     const int *cu_seqlens, *slots, *tile_seq, *tile_row0, *first_tile;
-    float *state, *scratch;              // scratch [tiles, H, d, dv]
+    float *state, *scratch;              // scratch [tiles, H, d, dv]: the chunks' sums
+    __nv_bfloat16 *before;               // [tiles, H, 2, d, dv]: the states in front of the chunks, as two terms
     size_t state_stride, state_off;
     const float *gate;                   // the fused product
     int gate_slices, gate_ld, gate_col0;
@@ -231,14 +299,18 @@ __device__ __forceinline__ uint32_t rc_bits(__nv_bfloat16 a, __nv_bfloat16 b) {
     return *reinterpret_cast<uint32_t *>(&v);
 }
 
+__device__ __forceinline__ void rc_cp16(__nv_bfloat16 *dst, const __nv_bfloat16 *src, bool valid) {
+    const int sz = valid ? 16 : 0;                    // 0: sixteen zero bytes
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(sz) : "memory");
+}
+
 // a chunk's rows of a head into shared memory [RC_C][D + 8], zero beyond its tokens and channels
 template <int D>
 __device__ __forceinline__ void rc_load_rows(__nv_bfloat16 *dst, const __nv_bfloat16 *src, size_t row_stride, int n, int d, int tid) {
     for (int idx = tid; idx < RC_C * (D / 8); idx += 128) {
         const int r = idx / (D / 8), c = idx % (D / 8) * 8;
-        uint4 x = make_uint4(0, 0, 0, 0);
-        if (r < n && c < d) x = *reinterpret_cast<const uint4 *>(src + (size_t)r * row_stride + c);
-        *reinterpret_cast<uint4 *>(dst + r * (D + 8) + c) = x;
+        const bool ok = r < n && c < d;
+        rc_cp16(dst + r * (D + 8) + c, src + (ok ? (size_t)r * row_stride + c : 0), ok);
     }
 }
 
@@ -268,6 +340,7 @@ retention_chunk_kv_kernel(const RetentionChunkParams p) {
         *reinterpret_cast<uint32_t *>(Vh + r * RC_LDN + c) = rc_bits(h0, h1);
         *reinterpret_cast<uint32_t *>(Vl + r * RC_LDN + c) = rc_bits(l0, l1);
     }
+    asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     const int g = lane >> 2, tq = lane & 3;
     const int v_row = (lane & 7) + ((lane >> 3) & 1) * 8, v_col = (lane >> 4) * 8;
@@ -307,7 +380,7 @@ retention_chunk_kv_kernel(const RetentionChunkParams p) {
     }
 }
 
-// Per request and head: the state in front of every chunk in place of the chunk's own sum, then the state after the last one.
+// Per request and head: the state in front of every chunk, as the two terms its product takes, then the state after the last one.
 __global__ void __launch_bounds__(256)
 retention_chunk_scan_kernel(const RetentionChunkParams p) {
     pdl_launch_dependents();
@@ -318,7 +391,8 @@ retention_chunk_scan_kernel(const RetentionChunkParams p) {
     if (lo == hi) return;
     const float *pw = p.powers + (size_t)h * (RC_C + 1);
     float4 *st = reinterpret_cast<float4 *>(p.state + (size_t)p.slots[seq] * p.state_stride + p.state_off + (size_t)h * p.d * p.dv) + i;
-    float4 *sc = reinterpret_cast<float4 *>(p.scratch) + ((size_t)lo * p.H + h) * n4 + i;
+    const float4 *sc = reinterpret_cast<const float4 *>(p.scratch) + ((size_t)lo * p.H + h) * n4 + i;
+    uint2 *bf = reinterpret_cast<uint2 *>(p.before) + ((size_t)lo * p.H + h) * 2 * n4 + i;
     const size_t step = (size_t)p.H * n4;
     float4 s = *st;
     const float full = pw[RC_C];
@@ -331,7 +405,13 @@ retention_chunk_scan_kernel(const RetentionChunkParams p) {
         for (int u = 0; u < 8; ++u) {
             if (c + u >= hi) break;
             const float g = c + u + 1 < hi ? full : pw[tokens - (hi - 1 - lo) * RC_C];
-            sc[(size_t)(c - lo + u) * step] = s;
+            __nv_bfloat16 hi4[4], lo4[4];
+            rc_split(s.x, hi4[0], lo4[0]);
+            rc_split(s.y, hi4[1], lo4[1]);
+            rc_split(s.z, hi4[2], lo4[2]);
+            rc_split(s.w, hi4[3], lo4[3]);
+            bf[(size_t)(c - lo + u) * 2 * step] = make_uint2(rc_bits(hi4[0], hi4[1]), rc_bits(hi4[2], hi4[3]));
+            bf[(size_t)(c - lo + u) * 2 * step + n4] = make_uint2(rc_bits(lo4[0], lo4[1]), rc_bits(lo4[2], lo4[3]));
             s.x = fmaf(g, s.x, kv[u].x);
             s.y = fmaf(g, s.y, kv[u].y);
             s.z = fmaf(g, s.z, kv[u].z);
@@ -355,9 +435,28 @@ retention_chunk_out_kernel(const RetentionChunkParams p) {
     const int seq = p.tile_seq[tile], row0 = p.tile_row0[tile], tb = p.cu_seqlens[seq], n = min(RC_C, p.cu_seqlens[seq + 1] - tb - row0);
     const int d = p.d, dv = p.dv, k_steps = (d + 15) / 16;
     const size_t t0 = (size_t)tb + row0;
-    for (int i = tid; i <= RC_C; i += 128) pw[i] = p.powers[(size_t)h * (RC_C + 1) + i];
+    const __nv_bfloat16 *st = p.before + ((size_t)tile * p.H + h) * 2 * d * dv;
+    auto load_slice = [&](int n0) {
+        for (int idx = tid; idx < RC_C * (RC_N / 8); idx += 128) {
+            const int r = idx / (RC_N / 8), c = idx % (RC_N / 8) * 8;
+            const bool ok = r < n && n0 + c < dv;
+            rc_cp16(Vs + r * RC_LDN + c, p.v + (ok ? ((t0 + r) * p.H + h) * dv + n0 + c : 0), ok);
+        }
+        for (int idx = tid; idx < D * (RC_N / 8); idx += 128) {
+            const int i = idx / (RC_N / 8), c = idx % (RC_N / 8) * 8;
+            const bool ok = i < d && n0 + c < dv;
+            const size_t off = ok ? (size_t)i * dv + n0 + c : 0;
+            rc_cp16(Sh + i * RC_LDN + c, st + off, ok);
+            rc_cp16(Sl + i * RC_LDN + c, st + (size_t)d * dv + off, ok);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
     rc_load_rows<D>(Qs, p.q + (t0 * p.H + h) * d, (size_t)p.H * d, n, d, tid);
     rc_load_rows<D>(Ks, p.k + (t0 * p.H + h) * d, (size_t)p.H * d, n, d, tid);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    load_slice(0);                                    // under the scores
+    for (int i = tid; i <= RC_C; i += 128) pw[i] = p.powers[(size_t)h * (RC_C + 1) + i];
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
     __syncthreads();
     const int g = lane >> 2, tq = lane & 3;
     const int a_row = warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, a_k = (lane >> 4) * 8;
@@ -398,29 +497,13 @@ retention_chunk_out_kernel(const RetentionChunkParams p) {
             }
     }
     float o[NS][RC_N / 8][4];
-    const float *st = p.scratch + ((size_t)tile * p.H + h) * d * dv;
 #pragma unroll
     for (int ns = 0; ns < NS; ++ns) {
-        const int n0 = ns * RC_N;
-        if (ns > 0) __syncthreads();
-        for (int idx = tid; idx < RC_C * (RC_N / 8); idx += 128) {
-            const int r = idx / (RC_N / 8), c = idx % (RC_N / 8) * 8;
-            uint4 x = make_uint4(0, 0, 0, 0);
-            if (r < n && n0 + c < dv) x = *reinterpret_cast<const uint4 *>(p.v + ((t0 + r) * p.H + h) * dv + n0 + c);
-            *reinterpret_cast<uint4 *>(Vs + r * RC_LDN + c) = x;
+        if (ns > 0) {
+            __syncthreads();                          // everyone has left the slice before
+            load_slice(ns * RC_N);
         }
-        for (int idx = tid; idx < D * (RC_N / 4); idx += 128) {
-            const int i = idx / (RC_N / 4), c = idx % (RC_N / 4) * 4;
-            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (i < d && n0 + c < dv) x = *reinterpret_cast<const float4 *>(st + (size_t)i * dv + n0 + c);
-            __nv_bfloat16 hi[4], lo[4];
-            rc_split(x.x, hi[0], lo[0]);
-            rc_split(x.y, hi[1], lo[1]);
-            rc_split(x.z, hi[2], lo[2]);
-            rc_split(x.w, hi[3], lo[3]);
-            *reinterpret_cast<uint2 *>(Sh + i * RC_LDN + c) = make_uint2(rc_bits(hi[0], hi[1]), rc_bits(hi[2], hi[3]));
-            *reinterpret_cast<uint2 *>(Sl + i * RC_LDN + c) = make_uint2(rc_bits(lo[0], lo[1]), rc_bits(lo[2], lo[3]));
-        }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         float (&oo)[RC_N / 8][4] = o[ns];
 #pragma unroll
@@ -481,17 +564,29 @@ retention_chunk_out_kernel(const RetentionChunkParams p) {
         const float rn = 1.0f / sqrtf(ss / (float)dv + p.eps);
         const size_t gate_row = (t0 + i) * p.gate_ld + p.gate_col0 + (size_t)h * dv;
         __nv_bfloat16 *dst = p.out + ((t0 + i) * p.H + h) * dv;
+        float2 z[NS][RC_N / 8];                       // all of a row's gate logits in flight at once
+#pragma unroll
+        for (int ns = 0; ns < NS; ++ns)
+#pragma unroll
+            for (int j = 0; j < RC_N / 8; ++j) z[ns][j] = make_float2(0.f, 0.f);
+        for (int s = 0; s < p.gate_slices; ++s)
+#pragma unroll
+            for (int ns = 0; ns < NS; ++ns)
+#pragma unroll
+                for (int j = 0; j < RC_N / 8; ++j) {
+                    const int col = ns * RC_N + j * 8 + 2 * tq;
+                    if (col >= dv) continue;
+                    const float2 x = *reinterpret_cast<const float2 *>(p.gate + (size_t)s * p.gate_stride + gate_row + col);
+                    z[ns][j].x += x.x;
+                    z[ns][j].y += x.y;
+                }
 #pragma unroll
         for (int ns = 0; ns < NS; ++ns)
 #pragma unroll
             for (int j = 0; j < RC_N / 8; ++j) {
                 const int col = ns * RC_N + j * 8 + 2 * tq;
                 if (col >= dv) continue;
-                float z0 = 0.f, z1 = 0.f;
-                for (int s = 0; s < p.gate_slices; ++s) {
-                    z0 += p.gate[(size_t)s * p.gate_stride + gate_row + col];
-                    z1 += p.gate[(size_t)s * p.gate_stride + gate_row + col + 1];
-                }
+                const float z0 = z[ns][j].x, z1 = z[ns][j].y;
                 *reinterpret_cast<uint32_t *>(dst + col) = pack_bf16(o[ns][j][2 * hf] * rn * (z0 / (1.0f + expf(-z0))), o[ns][j][2 * hf + 1] * rn * (z1 / (1.0f + expf(-z1))));
             }
     }
@@ -525,12 +620,12 @@ KESTREL_API int kestrel_retention_chunks(const void *q, const void *k, const voi
     if (nseq == 0 || tiles == 0) return 0;
     KESTREL_REQUIRE(nseq > 0 && nseq <= 65535 && tiles > 0 && H > 0 && H <= 65535 && d > 0 && dv > 0 && d % 8 == 0 && dv % 8 == 0 && d <= 256 && dv <= 256,
                     "retention_chunks: bad sizes H=%d d=%d dv=%d", H, d, dv);
-    KESTREL_REQUIRE(S > 0 && gate_col0 >= 0 && gate_col0 + H * dv <= ld && state_stride % 4 == 0 && state_off % 4 == 0 && ((uintptr_t)state & 15) == 0,
+    KESTREL_REQUIRE(S > 0 && gate_col0 >= 0 && gate_col0 + H * dv <= ld && state_stride % 4 == 0 && state_off % 4 == 0 && ((uintptr_t)state & 15) == 0 && ld % 2 == 0 && gate_col0 % 2 == 0 && slice_stride % 2 == 0,
                     "retention_chunks: the gate's columns or the state's place do not fit");
     RetentionChunkParams p = {};
     p.q = (const __nv_bfloat16 *)q; p.k = (const __nv_bfloat16 *)k; p.v = (const __nv_bfloat16 *)v;
     p.powers = powers; p.cu_seqlens = cu_seqlens; p.slots = slots; p.tile_seq = tile_seq; p.tile_row0 = tile_row0; p.first_tile = first_tile;
-    p.state = state; p.scratch = scratch; p.state_stride = (size_t)state_stride; p.state_off = (size_t)state_off;
+    p.state = state; p.scratch = scratch; p.before = (__nv_bfloat16 *)(scratch + (size_t)tiles * H * d * dv); p.state_stride = (size_t)state_stride; p.state_off = (size_t)state_off;
     p.gate = partial; p.gate_slices = S; p.gate_ld = ld; p.gate_col0 = gate_col0; p.gate_stride = (size_t)slice_stride;
     p.eps = eps; p.out = (__nv_bfloat16 *)out; p.H = H; p.d = d; p.dv = dv;
 #define RC_CASE(D)                                                              \

@@ -741,7 +741,7 @@ def attention(planner: Optional[AttentionPlanner], q: torch.Tensor, k_cache: tor
     the tiling of their rows and the cutting of key ranges into slices are decided natively
     (csrc/kernels/attention_dispatch.cu); float32 always takes the plain kernel."""
     _need(q, "attention.q", dims=2)
-    _need(out, "attention.out", None if out.dtype == torch.float32 else q.dtype, 2)
+    _need(out, "attention.out", q.dtype, 2)
     _need(k_cache, "attention.k_cache", q.dtype, 4)
     _need(v_cache, "attention.v_cache", q.dtype, 4)
     if q.shape[1] != nq * hd or out.shape != q.shape:
@@ -894,6 +894,52 @@ def add_gated_normed(residual: torch.Tensor, y: Partials, gate: Optional[Partial
         gate.slices if gate is not None else 0, gate.slice_stride if gate is not None else 0, _p(gate.bias) if gate is not None else None,
         weight.data_ptr(), float(eps), _p(next_weight), float(next_eps), _p(next_out),
         _code(next_out, "add_gated_normed.next_out") if next_out is not None else F32, T, d, _stream()))
+
+
+def post_norm_add(residual: torch.Tensor, y, weight: torch.Tensor, eps: float, copy: Optional[torch.Tensor] = None) -> None:
+    """residual += y / sqrt(mean(y^2) + eps) * weight over the row, y a product (`Partials`) or a routed feed-forward's sum that was not
+    written out (`MoeSum`); ``copy`` = the new residual in its own dtype."""
+    _need(residual, "post_norm_add.residual", torch.float32, 2)
+    _need(weight, "post_norm_add.weight", torch.float32, 1)
+    T, d = residual.shape
+    lib = library()
+    if not lib.kestrel_post_norm_takes(d):
+        add_gated_normed(residual, y.combine() if isinstance(y, MoeSum) else y, None, weight, eps, next_out=copy)
+        return
+    if y.tokens != T or y.width != d or weight.shape[0] != d:
+        raise KernelError("post_norm_add: shapes differ")
+    if copy is not None:
+        _need(copy, "post_norm_add.copy", dims=2)
+        if copy.shape != residual.shape:
+            raise KernelError("post_norm_add: the copy's shape differs")
+    if isinstance(y, MoeSum):
+        sh, z = y.extra.shared, y.extra.z
+        if copy is not None and copy.dtype != y.x.dtype:
+            raise KernelError("post_norm_add: the copy and the experts' input differ in dtype")
+        _check(lib.kestrel_post_norm_add_moe(
+            residual.data_ptr(), y.rows.data_ptr(), y.pair_row.data_ptr(), y.ids.data_ptr(), y.weights.data_ptr(), y.ids.shape[1], y.experts,
+            y.x.data_ptr(), y.x.stride(0), _p(sh.data) if sh is not None else None, sh.slices if sh is not None else 0,
+            sh.slice_stride if sh is not None else 0, _p(z.data) if z is not None else None, z.slices if z is not None else 0,
+            z.slice_stride if z is not None else 0, z.width if z is not None else 1, y.extra.gate_col, weight.data_ptr(), float(eps), _p(copy),
+            _code(y.x, "post_norm_add.x"), T, d, _stream()))
+        return
+    if y.bias is not None and y.bias.shape[0] != d:
+        raise KernelError("post_norm_add: the bias does not fit the row")
+    _check(lib.kestrel_post_norm_add(residual.data_ptr(), y.data.data_ptr(), y.slices, y.slice_stride, _p(y.bias), weight.data_ptr(), float(eps),
+                                     _p(copy), _code(copy, "post_norm_add.copy") if copy is not None else F32, T, d, _stream()))
+
+
+def embed_copy(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out[t] = table[ids[t]] widened to float32; returns the same rows in the table's own bfloat16."""
+    _need(table, "embed_copy.table", torch.bfloat16, 2)
+    _need(ids, "embed_copy.ids", torch.int32, 1)
+    _need(out, "embed_copy.out", torch.float32, 2)
+    T, d = out.shape
+    if ids.shape[0] != T or table.shape[1] != d:
+        raise KernelError("embed_copy: shapes differ")
+    copy = torch.empty((T, d), dtype=torch.bfloat16, device=out.device)
+    _check(library().kestrel_embed_copy(table.data_ptr(), ids.data_ptr(), out.data_ptr(), copy.data_ptr(), T, d, _stream()))
+    return copy
 
 
 def embed_add(table: torch.Tensor, ids: torch.Tensor, x: torch.Tensor) -> None:
@@ -1188,6 +1234,51 @@ def attention_tc_maps(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     if slices > 1:
         global launches
         launches += 1          # the merge kernel
+
+
+_decode_tiles: dict = {}
+
+
+def _single_token_tiles(n: int, device):
+    """Tile lists (request i, row 0) of a step of one token per request, made once per device and size."""
+    key = (str(device), n)
+    if key not in _decode_tiles:
+        _decode_tiles[key] = (torch.arange(n, dtype=torch.int32, device=device), torch.zeros((n,), dtype=torch.int32, device=device))
+    return _decode_tiles[key]
+
+
+def attention_decode_maps(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch, block_table: torch.Tensor, page_size: int,
+                          out: torch.Tensor, nq: int, nkv: int, dim: int, vd: int, scale: float, lambdas, diff: float, eps: float) -> bool:
+    """Differential attention of a step of one token per request on the TMA decode kernel (2 ``dim`` = ``vd`` = 64 or 128, at most 8 heads a
+    group), keys cut into slices that fill the device; the merge of the slices combines and norms the heads.  ``q`` has padded rows
+    [T, 2 nq, 2 dim].  False if the step or the sizes are not taken; nothing has run then."""
+    lib = library()
+    if batch.max_count != 1 or 2 * dim != vd or 2 * nq // nkv > 16 or not lib.kestrel_attention_decode_supported(vd, int(page_size)):
+        return False
+    _need(q, "attention_decode_maps.q", torch.bfloat16, 2)
+    _need(out, "attention_decode_maps.out", torch.bfloat16, 2)
+    _need(k_cache, "attention_decode_maps.k_cache", torch.bfloat16, 4)
+    _need(v_cache, "attention_decode_maps.v_cache", torch.bfloat16, 4)
+    T = q.shape[0]
+    if q.shape[1] != 2 * nq * 2 * dim or out.shape != (T, nq * vd) or tuple(k_cache.shape[1:]) != (nkv, page_size, 2 * dim) or \
+            tuple(v_cache.shape[1:]) != (nkv, page_size, vd):
+        raise KernelError("attention_decode_maps: shapes differ")
+    n, max_kv = int(batch.num_seqs), max(1, int(batch.max_kv_len))
+    tile_seq, tile_row0 = _single_token_tiles(n, q.device)
+    cand = max(1, min(lib.kestrel_attention_decode_slots(vd) // max(1, n * nkv), -(-max_kv // 128), 32))
+    slice_len = (-(-max_kv // cand) + 127) // 128 * 128
+    slices = -(-max_kv // slice_len)
+    # a recorded step fixes the number of slices; their length follows the longest request on the device
+    follow = batch.device_buffer.data_ptr() + 4 * int(batch.layout[_cdecl.constants()["KB_O_MAX_KV"]]) if batch.captured else None
+    part = torch.empty((T * 2 * nq * slices * (vd + 2),), dtype=torch.float32, device=q.device)
+    _check(lib.kestrel_attention_decode_maps(
+        q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), part.data_ptr(), part.data_ptr() + 4 * T * 2 * nq * slices * vd,
+        tile_seq.data_ptr(), tile_row0.data_ptr(), n, batch.cu_seqlens.data_ptr(), batch.kv_lens.data_ptr(), block_table.data_ptr(),
+        block_table.shape[1], block_table.stride(0), int(page_size), int(k_cache.shape[0]), T, nq, nkv, dim, vd, slices, slice_len, follow,
+        float(scale), *(t.data_ptr() for t in lambdas), float(diff), float(eps), _stream()))
+    global launches
+    launches += 1              # the merge kernel
+    return True
 
 
 def attention_window_maps(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch, block_table: torch.Tensor, page_size: int,
@@ -1498,8 +1589,8 @@ def retention_step(fused: Partials, positions: torch.Tensor, rotation, decay: to
 def retention_chunks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, powers: torch.Tensor, fused: Partials, gate_col0: int,
                      state: torch.Tensor, batch, eps: float, out: torch.Tensor, H: int, d: int, dv: int) -> None:
     """Prompt portions in chunks on the tensor cores: q, k, v bfloat16 as `retention_prepare` leaves them, ``powers`` [H, chunk + 1] the
-    decays' powers; out = (S^T q), normed per head, times silu of the gate's columns.  Three kernels; the states in front of the chunks
-    pass through a scratch of one state per chunk."""
+    decays' powers; out = (S^T q), normed per head, times silu of the gate's columns.  Three kernels; the chunks' sums and the states in
+    front of the chunks pass through a scratch of two states per chunk."""
     _need(state, "retention_chunks.state", torch.float32, 2)
     _need(powers, "retention_chunks.powers", torch.float32, 2)
     for t, name, n in ((q, "q", H * d), (k, "k", H * d), (v, "v", H * dv), (out, "out", H * dv)):
@@ -1518,7 +1609,7 @@ def retention_chunks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, powers: 
             first.append(first[-1] + -(-n // chunk))
         kept[("first", chunk)] = torch.tensor(first, dtype=torch.int32).to(q.device, non_blocking=True)
     tiles = tile_seq.shape[0]
-    scratch = torch.empty((tiles * H * d * dv,), dtype=torch.float32, device=q.device)
+    scratch = torch.empty((2 * tiles * H * d * dv,), dtype=torch.float32, device=q.device)
     _check(lib.kestrel_retention_chunks(q.data_ptr(), k.data_ptr(), v.data_ptr(), powers.data_ptr(), fused.data.data_ptr(), fused.slices,
                                         fused.slice_stride, fused.width, int(gate_col0), state.data_ptr(), state.stride(0), 0,
                                         batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), tile_seq.data_ptr(), tile_row0.data_ptr(),
@@ -1720,9 +1811,41 @@ class MoeExtra:
         self.identity, self.shared, self.z, self.gate_col = int(identity), shared, z, int(gate_col)
 
 
+class MoeSum:
+    """A routed feed-forward's result before its last sum: the experts' weighted rows, where each (token, choice) pair's row lies, and
+    what is added beside them.  A consumer sums while it reads (`post_norm_add`); ``combine`` writes the sum out."""
+
+    __slots__ = ("rows", "pair_row", "ids", "weights", "experts", "x", "extra")
+
+    def __init__(self, rows, pair_row, ids, weights, experts, x, extra):
+        self.rows, self.pair_row, self.ids, self.weights, self.experts, self.x, self.extra = rows, pair_row, ids, weights, experts, x, extra
+
+    @property
+    def tokens(self) -> int:
+        return self.x.shape[0]
+
+    @property
+    def width(self) -> int:
+        return self.rows.shape[1]
+
+    def combine(self) -> Partials:
+        sh, z, x, top = self.extra.shared, self.extra.z, self.x, self.ids.shape[1]
+        out = torch.empty((self.tokens, self.width), dtype=torch.float32, device=x.device)
+        _check(library().kestrel_moe_combine_with(
+            self.rows.data_ptr(), self.pair_row.data_ptr(), self.ids.data_ptr(), self.weights.data_ptr(), top, self.experts, x.data_ptr(),
+            _code(x, "moe.x"), x.stride(0), _p(sh.data) if sh is not None else None, sh.slices if sh is not None else 0,
+            sh.slice_stride if sh is not None else 0, _p(z.data) if z is not None else None, z.slices if z is not None else 0,
+            z.slice_stride if z is not None else 0, z.width if z is not None else 1, self.extra.gate_col, out.data_ptr(), self.tokens, self.width,
+            _stream()))
+        return Partials(out)
+
+    def reduce(self, dtype: torch.dtype) -> torch.Tensor:
+        return self.combine().reduce(dtype)
+
+
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
-                limit: Optional[float], extra: Optional[MoeExtra] = None) -> torch.Tensor:
-    """The chosen experts' outputs, weighted and summed per token: float32 [T, width].
+                limit: Optional[float], extra: Optional[MoeExtra] = None):
+    """The chosen experts' outputs, weighted and summed per token: float32 [T, width], or with ``extra`` a `MoeSum` still to be summed.
     w_gate_up [E, 2 ff, width] (gate rows, then up rows), w_down [E, width, ff].  ``limit`` clamps the activation
     min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1); None: silu(g) u."""
     _need(x, "moe.x", dims=2)
@@ -1738,7 +1861,6 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     lib, dev, P, outputs = library(), x.device, T * top, E + (extra.identity if extra is not None else 0)
     act = torch.empty((P, ff), dtype=x.dtype, device=dev)
     y = torch.empty((P, N), dtype=torch.float32, device=dev)
-    out = torch.empty((T, N), dtype=torch.float32, device=dev)
     xs = None
     if _moe_tc and x.dtype == torch.bfloat16 and P >= MOE_TC_MIN_PAIRS and x.stride(0) % 8 == 0:
         xs = torch.empty((P, K), dtype=x.dtype, device=dev)
@@ -1766,6 +1888,7 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
                                     tile_row0.data_ptr(), n_tiles.data_ptr(), max_tiles, weights.data_ptr(), y.data_ptr(), _code(x, "moe.x"), N, ff,
                                     _stream()))
     if extra is None:
+        out = torch.empty((T, N), dtype=torch.float32, device=dev)
         _check(lib.kestrel_moe_combine(y.data_ptr(), pair_row.data_ptr(), top, out.data_ptr(), T, N, _stream()))
         return out
     if extra.identity and N != K:
@@ -1775,12 +1898,7 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
         raise KernelError("moe_experts: the shared expert's product does not fit, or carries a bias")
     if z is not None and (z.tokens != T or not 0 <= extra.gate_col < z.width or z.bias is not None):
         raise KernelError("moe_experts: the shared expert's gate is no column of its product")
-    _check(lib.kestrel_moe_combine_with(y.data_ptr(), pair_row.data_ptr(), ids.data_ptr(), weights.data_ptr(), top, E, x.data_ptr(),
-                                        _code(x, "moe.x"), x.stride(0), _p(sh.data) if sh is not None else None, sh.slices if sh is not None else 0,
-                                        sh.slice_stride if sh is not None else 0, _p(z.data) if z is not None else None,
-                                        z.slices if z is not None else 0, z.slice_stride if z is not None else 0, z.width if z is not None else 1,
-                                        extra.gate_col, out.data_ptr(), T, N, _stream()))
-    return out
+    return MoeSum(y, pair_row, ids, weights, E, x, extra)
 
 
 # ---- the step program and its runner ---------------------------------------------------------

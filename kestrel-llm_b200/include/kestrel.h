@@ -264,7 +264,7 @@ KESTREL_API int kestrel_head_norm_act(const float *o, const float *w, int w_stri
 KESTREL_API int kestrel_retention_prepare(const float *partial, int S, long long slice_stride, int ld, const int *positions, const float *inv_freq, int rot, const float *decay, void *q_out, void *k_out, void *v_out, float *w_out, int dtype, int T, int H, int d, int dv, kestrel_stream_t stream);
 /* steps of few tokens per request, everything between the fused product (columns [q | k | v | gate]) and the output product in one kernel: out [T, H dv] = (S^T q) / its root mean square (eps) per head * silu(gate), S float32 at state_off of the requests' slots; d, dv <= 256 */
 KESTREL_API int kestrel_retention_step(const float *partial, int S, long long slice_stride, int ld, const int *positions, const float *inv_freq, int rot, const float *decay, float *state, long long state_stride, long long state_off, const int *cu_seqlens, const int *slots, float eps, void *out, int dtype, int nseq, int H, int d, int dv, kestrel_stream_t stream);
-/* prompt portions in chunks of kestrel_retention_chunk_tokens() tokens on the tensor cores (bfloat16 q, k, v as kestrel_retention_prepare leaves them; d, dv multiples of 8 up to 256): tiles list the chunks (request, first token among the request's), first_tile [nseq + 1] each request's first; powers [H, chunk + 1] = decay^n; scratch of tiles * H * d * dv floats; gate columns at gate_col0 of the fused product */
+/* prompt portions in chunks of kestrel_retention_chunk_tokens() tokens on the tensor cores (bfloat16 q, k, v as kestrel_retention_prepare leaves them; d, dv multiples of 8 up to 256): tiles list the chunks (request, first token among the request's), first_tile [nseq + 1] each request's first; powers [H, chunk + 1] = decay^n; scratch of 2 * tiles * H * d * dv floats; gate columns at gate_col0 of the fused product */
 KESTREL_API int kestrel_retention_chunk_tokens(void);
 KESTREL_API int kestrel_retention_chunks(const void *q, const void *k, const void *v, const float *powers, const float *partial, int S, long long slice_stride, int ld, int gate_col0, float *state, long long state_stride, long long state_off, const int *cu_seqlens, const int *slots, const int *tile_seq, const int *tile_row0, const int *first_tile, int tiles, float *scratch, float eps, void *out, int nseq, int H, int d, int dv, kestrel_stream_t stream);
 
@@ -274,6 +274,17 @@ KESTREL_API int kestrel_differential_combine(const float *a, const float *lq1, c
 KESTREL_API int kestrel_differential_merge(const float *part_o, const float *part_ml, int slices, int ld, const float *lq1, const float *lk1, const float *lq2, const float *lk2, int dim, float diff, float eps, void *out, int T, int H, int vd, kestrel_stream_t stream);
 /* prompt portions on the tcgen05 attention kernel: q [T, nq, 2, dim], K pages of rows of 2 dim, V pages of rows of vd (dim 64, vd 128), tiles of up to 128 (token, head) rows; out [T, nq, vd] the combined, normed heads; slices > 1 needs part_o [T nq 2, slices, 128] and part_ml [T nq 2, slices, 2] */
 KESTREL_API int kestrel_attention_tc_maps(const void *q, const void *k_cache, const void *v_cache, void *out, float *part_o, float *part_ml, const int *tile_seq, const int *tile_row0, int tiles, int rows_per_tile, const int *cu_seqlens, const int *kv_lens, const int *block_table, int table_width, int table_stride, int page_size, int cache_pages, int T, int nq, int nkv, int dim, int vd, int window, int slices, int slice_len, float scale, const float *lq1, const float *lk1, const float *lq2, const float *lk2, float diff, float eps, kestrel_stream_t stream);
+/* decode tokens on the kernel of kestrel_attention_decode: q [T, 2 nq, 2 dim] padded rows, 2 dim = vd = 64 or 128, tiles of at most 16 rows (2 nq / nkv a token); part_o [T 2 nq, slices, vd], part_ml [T 2 nq, slices, 2]; the merge combines and norms the heads */
+KESTREL_API int kestrel_attention_decode_maps(const void *q, const void *k_cache, const void *v_cache, void *out, float *part_o, float *part_ml, const int *tile_seq, const int *tile_row0, int tiles, const int *cu_seqlens, const int *kv_lens, const int *block_table, int table_width, int table_stride, int page_size, int cache_pages, int T, int nq, int nkv, int dim, int vd, int slices, int slice_len, const int *max_kv_ptr, float scale, const float *lq1, const float *lk1, const float *lq2, const float *lk2, float diff, float eps, kestrel_stream_t stream);
+
+/* ---- a norm on a sublayer's result and the add to the stream (post_norm.cu); rows of a multiple of 4 numbers (kestrel_post_norm_takes) ---- */
+KESTREL_API int kestrel_post_norm_takes(int d);
+/* residual[t] += y / sqrt(mean(y^2) + eps) w, y the sum of the slices plus the bias (may be NULL); copy[t] = residual[t] in `dtype` (may be NULL) */
+KESTREL_API int kestrel_post_norm_add(float *residual, const float *y, int S, long long stride, const float *bias, const float *w, float eps, void *copy, int dtype, int T, int d, kestrel_stream_t stream);
+/* the same where y is a routed feed-forward's sum, as kestrel_moe_combine_with would write it; x in `dtype` too */
+KESTREL_API int kestrel_post_norm_add_moe(float *residual, const float *y, const int *pair_row, const int *ids, const float *weights, int top, int experts, const void *x, long long ldx, const float *shared, int Ss, long long shared_stride, const float *z, int Sz, long long z_stride, int z_ld, int sg_col, const float *w, float eps, void *copy, int dtype, int T, int d, kestrel_stream_t stream);
+/* x[t] = table[ids[t]] in float32, copy[t] = the bfloat16 row itself */
+KESTREL_API int kestrel_embed_copy(const void *table, const int *ids, float *x, void *copy, int T, int d, kestrel_stream_t stream);
 /* few rows a request (at most kestrel_attention_window_keys_rows() rows of 2 nq / nkv a token): q [T, 2 nq, 2 dim] padded rows; the kernel of kestrel_attention_window over shares of the keys, whose merge combines and norms the heads; scratch of kestrel_attention_window_scratch_floats(nseq, max_count, 2 nq, nkv, 2 dim, vd, ksplit) floats; bfloat16 out [T, nq, vd] */
 KESTREL_API int kestrel_attention_window_keys_rows(void);
 KESTREL_API int kestrel_attention_window_maps(const void *q, const void *k_cache, const void *v_cache, void *out, const int *cu_seqlens, const int *kv_lens, const int *block_table, int table_stride, int page_size, int nseq, int max_count, int nq, int nkv, int dim, int vd, float scale, int ksplit, float *scratch, const float *lq1, const float *lk1, const float *lq2, const float *lk2, float diff, float eps, kestrel_stream_t stream);

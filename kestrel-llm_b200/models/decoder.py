@@ -70,6 +70,9 @@ class DecoderModel(Part):
                 elif c.cache not in seen:
                     raise ValueError(f"cache layer {c.cache} is read before it is written")
         self._cache_owner = owners
+        # the first block reads the stream unnormed, and the stream starts as rows of the table: the table's rows are that copy
+        self._starts_with_copy = bool(self.order) and getattr(self.blocks[self.order[0].block], "reads_stream_copy", False) and \
+            position is None and embedding_norm is None and self.order[0].add_row < 0 and embedding.copies_rows
         if any(c.add_embedding for c in self.order) and (embedding_norm is not None or (
                 position is not None and type(position).add_to_embedding is not PositionEncoding.add_to_embedding)):
             raise ValueError("feeding the embedded tokens in again is built for models whose stream starts as the table's rows alone")
@@ -140,6 +143,8 @@ class DecoderModel(Part):
     # The three stages of `forward`, for callers that run a step in pieces (a captured decode
     # step is two graphs, so that the second is submitted while the first already runs).
     def forward_embed(self, batch):
+        if self._starts_with_copy:
+            return self.embedding.forward_with_copy(batch.token_ids)
         x = self.embedding.forward(batch.token_ids)
         if self.position is not None:
             self.position.add_to_embedding(x, batch)

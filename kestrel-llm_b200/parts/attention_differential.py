@@ -34,6 +34,7 @@ from .linear import Linear
 class DifferentialAttention(Mixer):
     force_plain = False        # tests: bfloat16 through the plain kernel too, the twin of the tensor-core one
     tcgen05 = True             # tests: off, portions of maps of 64 over values of 128 stay on the mma.sync kernel
+    decode = True              # tests: off, single tokens of 2 x 32 / 64 and 2 x 64 / 128 stay on the kernel of every other size
     TC_MIN_ROWS = 64           # a step whose longest portion has more rows (tokens x heads of a group) takes the tcgen05 kernel
     TC_SLICE = 512             # fewest keys a slice where a portion's key range is cut
     TC_SLICE_FILL = 148        # CTAs that the cut should reach: one an SM
@@ -97,6 +98,9 @@ class DifferentialAttention(Mixer):
                 slices = -(-batch.max_kv_len // slice_len)
             ops.attention_tc_maps(q, cache.k, cache.v, o, batch, table, cache.page_size, H, G, d, dv, self.scale, self.lambdas, self.diff,
                                   self.norm_eps, slices, slice_len)
+            return self.out.forward(o)
+        if fast and self.decode and ops.attention_decode_maps(q, cache.k, cache.v, batch, table, cache.page_size, o, H, G, d, dv, self.scale,
+                                                              self.lambdas, self.diff, self.norm_eps):
             return self.out.forward(o)
         window = fast and ops.attention_window_supported(2 * d, dv, 2 * H, G)
         if window and ops.attention_window_maps(q, cache.k, cache.v, batch, table, cache.page_size, o, H, G, d, dv, self.scale, self.lambdas,

@@ -143,6 +143,8 @@ class PostNormBlock(Block):
     (``ffn`` and ``norm2`` None: the first line alone.)  Norm and add are one kernel, which also leaves the stream in the storage
     type for the sublayer that follows; the block hands that copy on to the next block."""
 
+    reads_stream_copy = True        # a model whose stream starts as table rows may hand this block those rows as the copy
+
     def __init__(self, mixer: Mixer, norm1: RMSNorm, ffn: Optional[FeedForward], norm2: Optional[RMSNorm], dtype: torch.dtype):
         if (norm2 is None) != (ffn is None):
             raise ValueError("the second norm and the feed-forward come together or not at all")
@@ -158,7 +160,7 @@ class PostNormBlock(Block):
     def _add(self, residual: torch.Tensor, y, norm: RMSNorm) -> torch.Tensor:
         """The stream after residual += norm(y), in the storage type."""
         h = torch.empty(residual.shape, dtype=self.dtype, device=residual.device) if self.dtype != torch.float32 else None
-        ops.add_gated_normed(residual, y, None, norm.weight, norm.eps, next_out=h)
+        ops.post_norm_add(residual, y, norm.weight, norm.eps, copy=h)
         return residual if h is None else h
 
     def forward(self, residual: torch.Tensor, pending, batch, cache):

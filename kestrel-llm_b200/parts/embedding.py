@@ -33,6 +33,16 @@ class TokenEmbedding(Part):
         ops.embed(self.weight, token_ids, out, self.scale)
         return out
 
+    @property
+    def copies_rows(self) -> bool:
+        """Whether `forward_with_copy` serves this table: bfloat16 rows without a factor."""
+        return self.weight.dtype == torch.bfloat16 and self.scale == 1.0 and self.width % 4 == 0
+
+    def forward_with_copy(self, token_ids: torch.Tensor):
+        """The stream and, as what a block before would have handed on, its copy in the storage type: the table's own rows."""
+        out = torch.empty((token_ids.shape[0], self.width), dtype=torch.float32, device=token_ids.device)
+        return out, ops.StreamCopy(ops.embed_copy(self.weight, token_ids, out))
+
     def add_forward(self, token_ids: torch.Tensor, x: torch.Tensor) -> None:
         """x += E[token]: the embedded tokens fed into the stream once more."""
         ops.embed_add(self.weight, token_ids, x)

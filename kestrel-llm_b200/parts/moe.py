@@ -146,9 +146,9 @@ class SoftmaxRoutedExperts(FeedForward):
                 slots.append(WeightSlot(p + shared + sg, self.router.weight[self.outputs:]))
         return slots
 
-    def forward(self, x: torch.Tensor, batch) -> ops.Partials:
+    def forward(self, x: torch.Tensor, batch) -> ops.MoeSum:
         z = self.router.forward(x)
         ids, weights = ops.moe_route_scored(z, self.outputs, self.correction, self.top, self.groups, self.keep, self.scale, renorm=self.renorm)
         extra = ops.MoeExtra(self.identity, self.shared.forward(x, batch) if self.shared is not None else None,
                              z if self.shared_gate else None, self.outputs)
-        return ops.Partials(ops.moe_experts(x, ids, weights, self.w_gate_up, self.w_down, None, extra))
+        return ops.moe_experts(x, ids, weights, self.w_gate_up, self.w_down, None, extra)

@@ -92,6 +92,7 @@ MIXERS = [
     ("attention 5/1 x 10/14 (no multiples of 8)", U.attn(5, 1, 10, 14, 0.4, 0.2, (6, 20.0))),
     ("attention 4/2 x 64/128", U.attn(4, 2, 64, 128, 0.125, 0.35, (64, 10000.0))),
     ("attention 2/1 x 128/64", U.attn(2, 1, 128, 64, 0.1, 0.6, (32, 10000.0))),
+    ("attention 4/1 x 32/64, all turned", U.attn(4, 1, 32, 64, 0.18, 0.45, (32, 10000.0))),
     ("attention 8/1 x 8/24", U.attn(8, 1, 8, 24, 0.5, 0.1, (8, 10.0))),
     ("attention 2/1 x 144/32 (maps beyond the tensor-core kernels' sizes)", U.attn(2, 1, 144, 32, 0.08, 0.5, (144, 1000.0))),
     ("retention 3 x 40/24, 16 of 40 turned", U.retention(3, 40, 24, (0.75, 0.99, 1.0), (16, 50.0))),
@@ -119,7 +120,7 @@ def test_mixer_alone_whole_and_cut(dtype, label, layer):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("cuts", [[700], [1, 299, 400], [64, 65, 63, 508], [520, 2, 178], [900, 400]])
-@pytest.mark.parametrize("which", [3, 9, 10, 7])
+@pytest.mark.parametrize("which", [3, 10, 11, 8])
 def test_mixers_in_long_portions(which, dtype, cuts):
     """Portions long enough for the kernels of many tokens: the tcgen05 attention (also over key ranges in slices) and the
     recurrence in chunks, whose first chunk starts from the state an earlier portion left and whose last is cut short."""
@@ -245,7 +246,7 @@ def test_positions_turn_queries_and_keys_far_out(dtype):
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_retention_in_chunks_of_unequal_requests(dtype):
     """Three requests in one step, 400, 129 and 2 tokens: the grid is sized by the longest, the others' chunks end early."""
-    for layer in (MIXERS[7][1], MIXERS[9][1]):
+    for layer in (MIXERS[8][1], MIXERS[10][1]):
         rng = np.random.default_rng(3)
         model, W, _ = _model_of([U.layer(layer, None)], 48, dtype, seed=3)
         mixer = model.blocks[0].mixer
@@ -260,7 +261,7 @@ def test_retention_in_chunks_of_unequal_requests(dtype):
             _close(np.concatenate([a, b]), want[r], dtype, f"request {r}", tol=1e-4 if dtype == "float32" else None)
 
 
-@pytest.mark.parametrize("which", [7, 9, 10, 11, 12])
+@pytest.mark.parametrize("which", [8, 10, 11, 12, 13])
 def test_retention_forms_against_each_other(which):
     """One kernel for few tokens, chunks, and the sequential scan: the same portions through each form that takes them."""
     from kestrel_llm_b200.parts import RetentionMixer
@@ -277,7 +278,7 @@ def test_retention_forms_against_each_other(which):
 
 
 @pytest.mark.parametrize("cuts", [[130, 1, 1, 70], [33, 20, 500, 2, 90]])
-@pytest.mark.parametrize("which", [0, 3, 4])
+@pytest.mark.parametrize("which", [0, 3, 4, 5])
 def test_attention_kernels_against_their_plain_twin(which, cuts):
     """bfloat16: the tcgen05 kernel, the mma.sync kernel's two tilings and its shares of the keys against the plain kernel."""
     from kestrel_llm_b200.csrc import ops
@@ -285,12 +286,12 @@ def test_attention_kernels_against_their_plain_twin(which, cuts):
     label, layer = MIXERS[which]
     runs = {}
     for name, plain, tc, splits in (("default", False, True, True), ("mma", False, False, True), ("one share", False, False, False), ("plain", True, True, True)):
-        DifferentialAttention.force_plain, DifferentialAttention.tcgen05 = plain, tc
+        DifferentialAttention.force_plain, DifferentialAttention.tcgen05, DifferentialAttention.decode = plain, tc, tc
         ops.attention_window_set_splits(splits)
         try:
             runs[name], want, _ = _mixer_case(layer, "bfloat16", 16, sum(cuts), cuts, seed=which)
         finally:
-            DifferentialAttention.force_plain, DifferentialAttention.tcgen05 = False, True
+            DifferentialAttention.force_plain, DifferentialAttention.tcgen05, DifferentialAttention.decode = False, True, True
             ops.attention_window_set_splits(True)
     for name in ("default", "mma", "one share"):
         _close(runs[name], runs["plain"], "bfloat16", f"{label}, {name}", scale=float(np.abs(want).max()), tol=2e-2)
@@ -420,7 +421,7 @@ def test_block_norms_each_sublayers_result(dtype):
 # ---- requests beside each other, memory used again --------------------------------------------------
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("which", [0, 2, 3, 4, 7, 8, 9, 12])
+@pytest.mark.parametrize("which", [0, 2, 3, 4, 5, 8, 9, 10, 13])
 def test_requests_beside_each_other_and_memory_used_again(dtype, which):
     """Three requests of unequal length in one step, portions beside single tokens, against each alone; then two are given
     back and a new request runs on their pages and slot."""
