@@ -55,60 +55,70 @@ KESTREL_API int kestrel_differential_combine(const float *a, const float *lq1, c
 }
 
 // The maps' outputs as key-range slices: part_o [T * H * 2, slices, ld] unnormalised, part_ml [T * H * 2, slices, 2] the slices' (maximum
-// in base-2 units, sum).  Slices in ascending order, then the head as above.  A block of four warps a (token, head): warps 0, 1
-// first merge map 1, warps 2, 3 map 2, each its half of the columns.
+// in base-2 units, sum); a slice without visible keys holds zeros, minus infinity and a sum of zero.  Slices in ascending order,
+// then the head as above.  A block of 256 threads a (token, head), 128 a map; a column's slices are fetched before their factors
+// are known, so that the two round trips overlap.
 #define DM_SLICES 64
-__global__ void __launch_bounds__(128)
+#define DM_AHEAD 16
+__global__ void __launch_bounds__(256)
 differential_merge_kernel(const float *__restrict__ part_o, const float *__restrict__ part_ml, int slices, int ld, const DifferentialOpts opts,
                           __nv_bfloat16 *__restrict__ out, int vd) {
     pdl_launch_dependents();
     __shared__ float a_s[2][256], f_s[2][DM_SLICES + 1];
-    __shared__ float red[4];
+    __shared__ float red[8];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const float lam = differential_lambda(opts, lane);
     pdl_wait();
     const size_t h = blockIdx.x;                      // (token, head)
-    const int map = tid >> 6;
+    const int map = tid >> 7, c0 = tid & 127;
     const size_t row = (h * 2 + map) * slices;
-    if ((warp & 1) == 0) {
-        // the slices' factors 2^(m_s - M), a lane a slice (further ones in rounds), and the row's sum in ascending order
-        float M = -INFINITY, L = 0.f;
-        for (int s = lane; s < slices; s += 32) M = fmaxf(M, part_ml[(row + s) * 2]);
-        M = warp_max(M);
-        for (int s0 = 0; s0 < slices; s0 += 32) {
-            const int s = s0 + lane;
-            const float m = s < slices ? part_ml[(row + s) * 2] : -INFINITY, f = m == -INFINITY ? 0.f : exp2f(m - M);
-            const float l = s < slices && f > 0.f ? part_ml[(row + s) * 2 + 1] * f : 0.f;
-            if (s < slices && s < DM_SLICES) f_s[map][s] = f;
-            for (int k = 0; k < min(32, slices - s0); ++k) L += __shfl_sync(0xffffffffu, l, k);
+    float x[DM_AHEAD];
+#pragma unroll
+    for (int s = 0; s < DM_AHEAD; ++s) x[s] = s < slices && c0 < vd ? part_o[(row + s) * ld + c0] : 0.f;
+    if ((warp & 3) == 0) {
+        // the slices' factors 2^(m_s - M), a lane a slice and another 32 further on, and the row's sum
+        float m[2], l[2];
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int s = lane + 32 * k;
+            const float2 ml = s < slices ? *reinterpret_cast<const float2 *>(part_ml + (row + s) * 2) : make_float2(-INFINITY, 0.f);
+            m[k] = ml.x;
+            l[k] = ml.y;
         }
+        const float M = warp_max(fmaxf(m[0], m[1]));
+        float L = 0.f;
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const float f = m[k] == -INFINITY ? 0.f : exp2f(m[k] - M);
+            f_s[map][lane + 32 * k] = f;
+            L = fmaf(l[k], f, L);
+        }
+        L = warp_sum(L);
         if (lane == 0) f_s[map][DM_SLICES] = 1.0f / L;
     }
     __syncthreads();
-    for (int c = tid & 63; c < vd; c += 64) {
+    for (int c = c0; c < vd; c += 128) {
         float acc = 0.f;
+        if (c == c0) {
+#pragma unroll
+            for (int s = 0; s < DM_AHEAD; ++s) acc = fmaf(x[s], s < slices ? f_s[map][s] : 0.f, acc);
+#pragma unroll 4
+            for (int s = DM_AHEAD; s < slices; ++s) acc = fmaf(part_o[(row + s) * ld + c], f_s[map][s], acc);
+        } else {
 #pragma unroll 8
-        for (int s = 0; s < slices; ++s)
-            if (f_s[map][s] > 0.f) acc = fmaf(part_o[(row + s) * ld + c], f_s[map][s], acc);
+            for (int s = 0; s < slices; ++s) acc = fmaf(part_o[(row + s) * ld + c], f_s[map][s], acc);
+        }
         a_s[map][c] = acc * f_s[map][DM_SLICES];
     }
     __syncthreads();
-    float o[2], ss = 0.f;                             // vd <= 256
-#pragma unroll
-    for (int k = 0; k < 2; ++k) {
-        const int c = tid + 128 * k;
-        o[k] = c < vd ? a_s[0][c] - lam * a_s[1][c] : 0.f;
-        ss = fmaf(o[k], o[k], ss);
-    }
-    ss = warp_sum(ss);
+    const float o = tid < vd ? a_s[0][tid] - lam * a_s[1][tid] : 0.f;      // vd <= 256
+    const float ss = warp_sum(o * o);
     if (lane == 0) red[warp] = ss;
     __syncthreads();
-    const float mul = 1.0f / sqrtf(((red[0] + red[1]) + (red[2] + red[3])) / (float)vd + opts.eps) * (1.0f - opts.diff);
+    float tot = 0.f;
 #pragma unroll
-    for (int k = 0; k < 2; ++k) {
-        const int c = tid + 128 * k;
-        if (c < vd) out[h * vd + c] = __float2bfloat16_rn(o[k] * mul);
-    }
+    for (int k = 0; k < 8; ++k) tot += red[k];
+    if (tid < vd) out[h * vd + tid] = __float2bfloat16_rn(o * (1.0f / sqrtf(tot / (float)vd + opts.eps) * (1.0f - opts.diff)));
 }
 
 KESTREL_API int kestrel_differential_merge(const float *part_o, const float *part_ml, int slices, int ld, const float *lq1, const float *lk1,
@@ -117,6 +127,6 @@ KESTREL_API int kestrel_differential_merge(const float *part_o, const float *par
     if (T == 0) return 0;
     KESTREL_REQUIRE(T > 0 && H > 0 && slices > 0 && slices <= DM_SLICES && dim > 0 && vd > 0 && vd <= 256 && ld >= vd && (long long)T * H < (1ll << 31), "differential_merge: bad sizes");
     const DifferentialOpts opts = {lq1, lk1, lq2, lk2, dim, diff, eps};
-    kestrel_launch(differential_merge_kernel, dim3(T * H), dim3(128), 0, stream, part_o, part_ml, slices, ld, opts, (__nv_bfloat16 *)out, vd);
+    kestrel_launch(differential_merge_kernel, dim3(T * H), dim3(256), 0, stream, part_o, part_ml, slices, ld, opts, (__nv_bfloat16 *)out, vd);
     return kestrel_check_launch("differential_merge");
 }

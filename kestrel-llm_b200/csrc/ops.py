@@ -525,10 +525,14 @@ def linear_act(x: torch.Tensor, w: torch.Tensor, act: str, weights_static: bool 
 linear_act_fused = True          # tests switch the epilogue form off to hold both forms against each other
 
 
-def gate_up_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, ff: int, weights_static: bool = False) -> torch.Tensor:
+def gate_up_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, ff: int, weights_static: bool = False, cut_few: bool = False) -> torch.Tensor:
     """silu(x Wg^T) * (x Wu^T) in x's dtype, Wg and Wu being the two halves of w_gate_up's rows.
-    ``weights_static`` as in `gemm_tc`."""
+    ``weights_static`` as in `gemm_tc`.  ``cut_few``: with few tokens the product may be cut along K and activated by a second
+    kernel, for a feed-forward so narrow that the uncut product would leave most of the device idle."""
     out = torch.empty((x.shape[0], ff), dtype=x.dtype, device=x.device)
+    if cut_few and x.shape[0] <= 64 and ff <= 128 * 37:
+        swiglu(Partials(linear(x, w_gate_up, weights_static=weights_static)), out)
+        return out
     if gemm_tc_supported(x, w_gate_up):
         # the activation is the product's epilogue: the K range is not split, whatever the number of
         # tokens, and the gate/up product never reaches memory

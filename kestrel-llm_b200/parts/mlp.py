@@ -16,12 +16,15 @@ class GatedMLP(FeedForward):
     graph_safe = True
 
     def __init__(self, width: int, intermediate: int, dtype: torch.dtype, device, prefix: str,
-                 activation: str = "silu", names=("gate_proj.weight", "up_proj.weight", "down_proj.weight")):
+                 activation: str = "silu", names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), cut_few: bool = False):
         if activation != "silu":
             raise ValueError(f"activation '{activation}' has no kernel; only 'silu'")
         self.width, self.intermediate = width, intermediate
         self.prefix, self.names = prefix, names
         self.dtype = dtype
+        self.cut_few = cut_few               # a narrow one beside routed experts: few tokens take the product cut along K
+        if cut_few:
+            self.emit = None                 # the step program has the uncut form
         self.gate_up = Linear(width, 2 * intermediate, dtype, device)
         self.down = Linear(intermediate, width, dtype, device)
 
@@ -32,7 +35,7 @@ class GatedMLP(FeedForward):
                 WeightSlot(p + down, self.down.weight)]
 
     def forward(self, x: torch.Tensor, batch, residual: Optional[torch.Tensor] = None) -> Optional[ops.Partials]:
-        act = ops.gate_up_swiglu(x, self.gate_up.weight, self.intermediate, weights_static=True)
+        act = ops.gate_up_swiglu(x, self.gate_up.weight, self.intermediate, weights_static=True, cut_few=self.cut_few)
         return self.down.forward(act, residual=residual)
 
     def emit(self, prog, x: int, residual: Optional[int]) -> int:

@@ -129,7 +129,7 @@ class SoftmaxRoutedExperts(FeedForward):
         self.correction: Optional[torch.Tensor] = torch.empty((n,), dtype=torch.float32, device=device) if correction else None
         self.w_gate_up = torch.empty((experts, 2 * inner, width), dtype=dtype, device=device)
         self.w_down = torch.empty((experts, width, inner), dtype=dtype, device=device)
-        self.shared = GatedMLP(width, shared_inner, dtype, device, prefix + names[5], names=names[:3]) if shared_inner else None
+        self.shared = GatedMLP(width, shared_inner, dtype, device, prefix + names[5], names=names[:3], cut_few=True) if shared_inner else None
 
     def weight_slots(self) -> List[WeightSlot]:
         p, ff, (gate, up, down, router, correction, shared, sg) = self.prefix, self.inner, self.names
