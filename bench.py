@@ -43,6 +43,10 @@ element; attention over cached latents with a rotated key part that all heads sh
 gated feed-forward and routed experts with a sigmoid router, groups and a shared expert; a token input per layer) the same
 way, beside the Qwen3 dense decoder of equal width, heads, depth, vocabulary and active feed-forward weights.
 
+`--workload tuganex`: the Tuganex decoder (differential attention, also on another layer's keys; retention; a dense feed-forward
+with xIELU and routed experts with a softmax router, groups, identity experts and a gated shared expert; norms on the
+sublayers' results only) the same way.
+
 Timing: CUDA events on the launching stream around exactly K steps after W warm-up steps, with
 a synchronize on both sides.  Every step streams all weights (15 GB) and the live requests'
 cache from HBM, far more than the 126 MB of L2, so nothing a step reads is still cached from

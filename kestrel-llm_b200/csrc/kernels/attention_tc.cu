@@ -229,7 +229,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
                     if (MAPS)           // map x: its own queries, panel x of the key tile
                         tc_mma(tmem + x * 128, smem_desc(q_s + x * TILE_BYTES + off), smem_desc(k_s + b * TILE_BYTES + x * AT_PANEL + off), IDESC_S, ks > 0 ? 1u : 0u);
                     else
-                    tc_mma(tmem + x * 128, smem_desc(q_s + x * TILE_BYTES + off), smem_desc(k_s + b * TILE_BYTES + off), IDESC_S, ks > 0 ? 1u : 0u);
+                        tc_mma(tmem + x * 128, smem_desc(q_s + x * TILE_BYTES + off), smem_desc(k_s + b * TILE_BYTES + off), IDESC_S, ks > 0 ? 1u : 0u);
                 }
                 tc_commit(bar(B_S_FULL + x));
             };

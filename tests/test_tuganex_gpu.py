@@ -92,7 +92,7 @@ MIXERS = [
     ("attention 5/1 x 10/14 (no multiples of 8)", U.attn(5, 1, 10, 14, 0.4, 0.2, (6, 20.0))),
     ("attention 4/2 x 64/128", U.attn(4, 2, 64, 128, 0.125, 0.35, (64, 10000.0))),
     ("attention 2/1 x 128/64", U.attn(2, 1, 128, 64, 0.1, 0.6, (32, 10000.0))),
-    ("attention 4/1 x 32/64, all turned", U.attn(4, 1, 32, 64, 0.18, 0.45, (32, 10000.0))),
+    ("attention 6/2 x 32/64, all turned", U.attn(6, 2, 32, 64, 0.19, 0.45, (32, 10000.0))),
     ("attention 8/1 x 8/24", U.attn(8, 1, 8, 24, 0.5, 0.1, (8, 10.0))),
     ("attention 2/1 x 144/32 (maps beyond the tensor-core kernels' sizes)", U.attn(2, 1, 144, 32, 0.08, 0.5, (144, 1000.0))),
     ("retention 3 x 40/24, 16 of 40 turned", U.retention(3, 40, 24, (0.75, 0.99, 1.0), (16, 50.0))),
