@@ -405,7 +405,7 @@ def run_zidivik(args) -> int:
     clocks = ClockSampler(0)
     rng = np.random.default_rng(0)
     timed_names = ["linear", "add_rmsnorm", "attn_prepare", "attn_prepare_ex", "attention", "attention_plain_ex", "attention_window", "qkv_prepare_fused",
-                   "gate_up_swiglu", "moe_route", "moe_experts", "delta_conv_silu", "delta_gates", "delta_scan", "delta_out", "partial_columns",
+                   "gate_up_swiglu", "moe_route", "moe_experts", "short_conv", "delta_gates", "delta_scan", "delta_out", "partial_columns",
                    "add_two", "gelu_table_mul", "add_normed", "embed", "add_sinusoid", "linear_add_into", "latent_prepare", "head_gemm", "attention_tc",
                    "forget_gates", "removal_gates", "recurrence_scan", "head_norm_gate", "combine_normed", "add_gated_normed", "partial_columns_act",
                    "embed_add", "logit_scale_cap", "linear_act", "rglru_branches", "rglru_scan", "moe_route_sigmoid", "moe_experts_ungated",

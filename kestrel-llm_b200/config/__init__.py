@@ -6,8 +6,9 @@ from .tidavik_config import TidavikConfig
 from .toredra_config import ToredraConfig
 from .korirax_config import KoriraxConfig
 from .tuganex_config import TuganexConfig
+from .fasanex_config import FasanexConfig
 from .engine_options import EngineOptions
 
-__all__ = ["ConfigError", "ModelConfig", "Qwen3Config", "ZidivikConfig", "TidavikConfig", "ToredraConfig", "KoriraxConfig", "TuganexConfig", "read_config_json", "Architecture",
+__all__ = ["ConfigError", "ModelConfig", "Qwen3Config", "ZidivikConfig", "TidavikConfig", "ToredraConfig", "KoriraxConfig", "TuganexConfig", "FasanexConfig", "read_config_json", "Architecture",
            "architecture_of", "known_architectures", "load_config", "register_architecture",
            "resolve_architecture", "EngineOptions"]

@@ -1,5 +1,4 @@
-// A recurrent mixer: the gated delta rule with one decay per key channel, and the short causal
-// convolutions in front of it.  Per head, with a state S [d, dv] that starts at zero and is
+// A recurrent mixer: the gated delta rule with one decay per key channel, or one per head.  Per head, with a state S [d, dv] that starts at zero and is
 // carried from token to token of a request (float32, in the request's state slot):
 //
 //     S <- diag(a_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t
@@ -7,12 +6,10 @@
 // The read-out sees the token's own write.  Everything that enters the recurrence is float32.
 //
 // Kernels, in the order of a step:
-//   conv_silu     y[t, c] = silu(sum_j w[c, j] x[t - (taps-1) + j, c]) per channel of the fused
-//                 q|k|v product; inputs before this step's first token of a request come from the
-//                 request's state slot (the last taps-1 inputs; zeros for a new request)
-//   conv_tail     writes the last taps-1 inputs back to the slot
+//   (short_conv.cu) q, k, v out of the fused product through a causal convolution and silu
 //   gates         q, k made unit vectors per head (x / sqrt(sum x^2 + 1e-6)), q scaled by d^-1/2;
-//                 beta = sigmoid(.); a = exp(-exp(A_log[h]) softplus(. + dt_bias))
+//                 beta = sigmoid(.); a = exp(-exp(A_log[h]) softplus(. + dt_bias)),
+//                 the dot a column per key channel, or one per head that all of its channels take
 //   scan          the recurrence; a value column of S stays in the registers of eight lanes (an
 //                 eighth of the key channels each), so S^T k and S^T q are sums inside a thread
 //                 and one fixed shuffle tree - a token's result does not depend on how the
@@ -21,64 +18,15 @@
 #include "common.cuh"
 #include <math.h>
 
-#define DR_MAX_TAPS 8
-
 // sum of a product's slices at (token, column)
 __device__ __forceinline__ float slices_at(const float *p, int S, size_t slice_stride, size_t off) {
     return sum_slices(p, S, slice_stride, off);
 }
 
-__global__ void delta_conv_silu_kernel(const float *__restrict__ partial, int S, size_t slice_stride, int ld, const float *__restrict__ w,
-                                       int taps, const float *__restrict__ state, size_t state_stride, size_t tail_off,
-                                       const int *__restrict__ seq_of_token, const int *__restrict__ cu_seqlens,
-                                       const int *__restrict__ slots, float *__restrict__ out, int C) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const int t = blockIdx.x;
-    const int seq = seq_of_token[t];
-    const int first = cu_seqlens[seq];
-    const int i = t - first;
-    const float *tail = state + (size_t)slots[seq] * state_stride + tail_off;     // [taps - 1][C], oldest first
-    for (int c = threadIdx.x; c < C; c += blockDim.x) {
-        float y = 0.f;
-        for (int j = 0; j < taps; ++j) {
-            const int n = i - (taps - 1) + j;          // input index among this step's tokens of the request
-            const float x = n >= 0 ? slices_at(partial, S, slice_stride, (size_t)(first + n) * ld + c)
-                                   : tail[(size_t)(taps - 1 + n) * C + c];
-            y = fmaf(w[(size_t)c * taps + j], x, y);
-        }
-        out[(size_t)t * C + c] = y / (1.0f + expf(-y));
-    }
-}
-
-__global__ void delta_conv_tail_kernel(const float *__restrict__ partial, int S, size_t slice_stride, int ld, int taps,
-                                       float *__restrict__ state, size_t state_stride, size_t tail_off,
-                                       const int *__restrict__ cu_seqlens, const int *__restrict__ slots, int C) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const int seq = blockIdx.x;
-    const int first = cu_seqlens[seq], n_tok = cu_seqlens[seq + 1] - first;
-    float *tail = state + (size_t)slots[seq] * state_stride + tail_off;
-    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
-        float keep[DR_MAX_TAPS];
-#pragma unroll
-        for (int r = 0; r < DR_MAX_TAPS; ++r) {
-            if (r < taps - 1) {
-                const int n = n_tok - (taps - 1) + r;
-                keep[r] = n >= 0 ? slices_at(partial, S, slice_stride, (size_t)(first + n) * ld + c)
-                                 : tail[(size_t)(taps - 1 + n) * C + c];
-            }
-        }
-#pragma unroll
-        for (int r = 0; r < DR_MAX_TAPS; ++r)
-            if (r < taps - 1) tail[(size_t)r * C + c] = keep[r];
-    }
-}
-
 // act [T, C] = q (G*d) | k (G*d) | v (H*dv) after convolution and silu
 __global__ void __launch_bounds__(128)
 delta_gates_kernel(const float *__restrict__ act, int C, const float *__restrict__ partial, int S, size_t slice_stride, int ld, int col_beta,
-                   const float *__restrict__ a_part, int Sa, size_t a_stride, const float *__restrict__ A_log,
+                   const float *__restrict__ a_part, int Sa, size_t a_stride, int a_ld, int col_a, int per_head, const float *__restrict__ A_log,
                    const float *__restrict__ dt_bias, float *__restrict__ qn, float *__restrict__ kn, float *__restrict__ decay,
                    float *__restrict__ beta, int H, int G, int d) {
     pdl_launch_dependents();
@@ -96,7 +44,8 @@ delta_gates_kernel(const float *__restrict__ act, int C, const float *__restrict
     }
     for (int idx = threadIdx.x; idx < H * d; idx += 128) {
         const int h = idx / d;
-        const float a = slices_at(a_part, Sa, a_stride, (size_t)t * H * d + idx) + dt_bias[idx];
+        const int c = per_head ? h : idx;
+        const float a = slices_at(a_part, Sa, a_stride, (size_t)t * a_ld + col_a + c) + dt_bias[c];
         const float sp = a > 20.f ? a : log1pf(expf(a));
         decay[(size_t)t * H * d + idx] = expf(-expf(A_log[h]) * sp);
     }
@@ -247,27 +196,13 @@ delta_out_kernel(const float *__restrict__ o, const float *__restrict__ w, float
     }
 }
 
-KESTREL_API int kestrel_delta_conv_silu(const float *partial, int S, long long slice_stride, int ld, const float *w, int taps, float *state,
-                                        long long state_stride, long long tail_off, const int *seq_of_token, const int *cu_seqlens,
-                                        const int *slots, float *out, int T, int nseq, int C, cudaStream_t stream) {
-    if (T == 0) return 0;
-    KESTREL_REQUIRE(T > 0 && nseq > 0 && C > 0 && S > 0 && taps >= 1 && taps <= DR_MAX_TAPS + 1, "delta_conv_silu: bad sizes (taps %d)", taps);
-    kestrel_launch(delta_conv_silu_kernel, dim3(T), dim3(256), 0, stream, partial, S, (size_t)slice_stride, ld, w, taps, (const float *)state,
-                   (size_t)state_stride, (size_t)tail_off, seq_of_token, cu_seqlens, slots, out, C);
-    int rc = kestrel_check_launch("delta_conv_silu");
-    if (rc != 0 || taps == 1) return rc;
-    kestrel_launch(delta_conv_tail_kernel, dim3(nseq, (C + 255) / 256), dim3(256), 0, stream, partial, S, (size_t)slice_stride, ld, taps, state,
-                   (size_t)state_stride, (size_t)tail_off, cu_seqlens, slots, C);
-    return kestrel_check_launch("delta_conv_tail");
-}
-
 KESTREL_API int kestrel_delta_gates(const float *act, int C, const float *partial, int S, long long slice_stride, int ld, int col_beta,
-                                    const float *a_part, int Sa, long long a_stride, const float *A_log, const float *dt_bias, float *qn,
-                                    float *kn, float *decay, float *beta, int T, int H, int G, int d, cudaStream_t stream) {
+                                    const float *a_part, int Sa, long long a_stride, int a_ld, int col_a, int per_head, const float *A_log,
+                                    const float *dt_bias, float *qn, float *kn, float *decay, float *beta, int T, int H, int G, int d, cudaStream_t stream) {
     if (T == 0) return 0;
-    KESTREL_REQUIRE(T > 0 && H > 0 && G > 0 && H % G == 0 && d > 0, "delta_gates: bad sizes");
+    KESTREL_REQUIRE(T > 0 && H > 0 && G > 0 && H % G == 0 && d > 0 && Sa > 0 && col_a >= 0 && col_a + (per_head ? H : H * d) <= a_ld, "delta_gates: bad sizes");
     kestrel_launch(delta_gates_kernel, dim3(T), dim3(128), 0, stream, act, C, partial, S, (size_t)slice_stride, ld, col_beta, a_part, Sa,
-                   (size_t)a_stride, A_log, dt_bias, qn, kn, decay, beta, H, G, d);
+                   (size_t)a_stride, a_ld, col_a, per_head, A_log, dt_bias, qn, kn, decay, beta, H, G, d);
     return kestrel_check_launch("delta_gates");
 }
 

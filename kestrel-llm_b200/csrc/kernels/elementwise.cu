@@ -9,6 +9,7 @@
 // RMSNorm st.c:8811-8827, per-head norm st.c:9541-9561, rotation st.c:8950-8991, SiLU
 // st.c:3605-3607 (st.c = src/model/vllm_safetensors.c).
 #include "common.cuh"
+#include "gated_act.cuh"
 
 // ------------------------------------------------------------------------------------------
 // embedding: out[t, :] = table[ids[t], :] widened to float32 (st.c:16392-16393)
@@ -331,11 +332,11 @@ KESTREL_API int kestrel_add_rmsnorm(float *residual, const float *partial, int S
 }
 
 // ------------------------------------------------------------------------------------------
-// gated activation: out[t, i] = silu(g) * u,  g = sum_s P[s, t, i],  u = sum_s P[s, t, ff + i]
+// gated activation: out[t, i] = silu(g) * u (or its bounded form, gated_act.cuh),  g = sum_s P[s, t, i],  u = sum_s P[s, t, ff + i]
 // ------------------------------------------------------------------------------------------
 template <typename TOut>
 __global__ void swiglu_kernel(const float *__restrict__ partial, int S, size_t slice_stride,
-                              TOut *__restrict__ out, int T, int ff) {
+                              TOut *__restrict__ out, int T, int ff, float limit) {
     pdl_launch_dependents();
     pdl_wait();
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -347,20 +348,24 @@ __global__ void swiglu_kernel(const float *__restrict__ partial, int S, size_t s
         g += row[(size_t)s * slice_stride + i];
         u += row[(size_t)s * slice_stride + ff + i];
     }
-    float a = g / (1.0f + expf(-g));
-    out[idx] = from_f32<TOut>(a * u);
+    out[idx] = from_f32<TOut>(gated_act(g, u, limit));
 }
 
 KESTREL_API int kestrel_swiglu(const float *partial, int S, long long slice_stride, void *out,
                                int out_dtype, int T, int ff, cudaStream_t stream) {
+    return kestrel_gated_act(partial, S, slice_stride, 0.f, out, out_dtype, T, ff, stream);
+}
+
+KESTREL_API int kestrel_gated_act(const float *partial, int S, long long slice_stride, float limit, void *out,
+                                  int out_dtype, int T, int ff, cudaStream_t stream) {
     if (T == 0) return 0;
     KESTREL_REQUIRE(T > 0 && ff > 0, "swiglu: bad sizes T=%d ff=%d", T, ff);
     size_t n = (size_t)T * ff;
     unsigned blocks = (unsigned)((n + 255) / 256);
     if (out_dtype == KESTREL_F32)
-        kestrel_launch(swiglu_kernel<float>, dim3(blocks), dim3(256), 0, stream, partial, S, (size_t)slice_stride, (float *)out, T, ff);
+        kestrel_launch(swiglu_kernel<float>, dim3(blocks), dim3(256), 0, stream, partial, S, (size_t)slice_stride, (float *)out, T, ff, limit);
     else if (out_dtype == KESTREL_BF16)
-        kestrel_launch(swiglu_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, partial, S, (size_t)slice_stride, (__nv_bfloat16 *)out, T, ff);
+        kestrel_launch(swiglu_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, partial, S, (size_t)slice_stride, (__nv_bfloat16 *)out, T, ff, limit);
     else
         return kestrel_fail(-2, "swiglu: unknown dtype %d", out_dtype);
     return kestrel_check_launch("swiglu");

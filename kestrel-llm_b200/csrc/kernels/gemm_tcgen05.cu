@@ -22,6 +22,7 @@
 // (TMA); N, T and K need not be multiples of the tile - TMA fills out-of-range rows and
 // columns with zeros and stores are predicated.  Anything else is refused
 // (kestrel_gemm_tc_supported) and takes the CUDA-core kernel.
+#include "gated_act.cuh"
 #include "xielu.cuh"
 #include "tcgen05.cuh"
 #include <mutex>
@@ -70,6 +71,7 @@ struct QkvPrepParams {
     __nv_bfloat16 *k_cache, *v_cache, *q_out;
     int nq, nkv, write_kv;
     const float *act_p;              // ACT: the numbers of an activation that has any
+    float act_limit;                 // the gated forms: the bound of gated_act.cuh (0: none, SiLU)
 };
 
 // ------------------------------------------------------------------------------- kernel
@@ -77,7 +79,7 @@ template <int BN, int MODE>
 __global__ void __launch_bounds__(TC_THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                void *__restrict__ out, int T, int N, int K, int kb_per_split, long long slice_stride,
-               long long ldo, int stages, int up_row_offset, int early_w) {
+               long long ldo, int stages, int up_row_offset, int early_w, float act_limit) {
     pdl_launch_dependents();
     constexpr int A_TILES = MODE == TC_PARTIAL ? 1 : 2;
     constexpr uint32_t A_BYTES = TC_BM * TC_BK * 2;
@@ -200,8 +202,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                         for (int j = 0; j < 16; ++j)
                             if (c + j < valid) {
-                                float a = __fdividef(g[j], 1.0f + __expf(-g[j]));     // bfloat16 output: 2-ulp float32 intrinsics
-                                o[(size_t)(t0 + c + j) * ldo + n] = __float2bfloat16_rn(a * u[j]);
+                                o[(size_t)(t0 + c + j) * ldo + n] = __float2bfloat16_rn(gated_act_fast(g[j], u[j], act_limit));
                             }
                     }
                 } else {
@@ -244,7 +245,7 @@ template <int BN, int MODE>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                           void *__restrict__ out, int T, int N, int K, long long ldo, int stages, int up_row_offset,
-                          int tiles_n, int tiles_total) {
+                          int tiles_n, int tiles_total, float act_limit) {
     pdl_launch_dependents();
     constexpr int A_TILES = MODE == TC_SWIGLU ? 2 : 1;
     constexpr uint32_t A_BYTES = TC_BM * TC_BK * 2;
@@ -366,8 +367,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
 #pragma unroll
                         for (int jj = 0; jj < 16; ++jj)
                             if (c + jj < valid) {
-                                float a = __fdividef(g[jj], 1.0f + __expf(-g[jj]));   // bfloat16 output: 2-ulp float32 intrinsics
-                                o[(size_t)(t0 + c + jj) * ldo + n] = __float2bfloat16_rn(a * u[jj]);
+                                o[(size_t)(t0 + c + jj) * ldo + n] = __float2bfloat16_rn(gated_act_fast(g[jj], u[jj], act_limit));
                             }
                     }
                 } else {
@@ -705,9 +705,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                             uint32_t pk[8];
 #pragma unroll
                             for (int jj = 0; jj < 8; ++jj) {
-                                float a0 = __fdividef(g[2 * jj], 1.0f + __expf(-g[2 * jj])) * u[2 * jj];
-                                float a1 = __fdividef(g[2 * jj + 1], 1.0f + __expf(-g[2 * jj + 1])) * u[2 * jj + 1];
-                                __nv_bfloat162 h = __floats2bfloat162_rn(a0, a1);
+                                __nv_bfloat162 h = __floats2bfloat162_rn(gated_act_fast(g[2 * jj], u[2 * jj], prep.act_limit),
+                                                                         gated_act_fast(g[2 * jj + 1], u[2 * jj + 1], prep.act_limit));
                                 pk[jj] = *reinterpret_cast<uint32_t *>(&h);
                             }
                             uint4 *dst = reinterpret_cast<uint4 *>(o + c);
@@ -717,8 +716,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 #pragma unroll
                             for (int jj = 0; jj < 16; ++jj)
                                 if (f0 + c + jj < N) {
-                                    float a = __fdividef(g[jj], 1.0f + __expf(-g[jj]));
-                                    o[c + jj] = __float2bfloat16_rn(a * u[jj]);
+                                    o[c + jj] = __float2bfloat16_rn(gated_act_fast(g[jj], u[jj], prep.act_limit));
                                 }
                         }
                     }
@@ -747,8 +745,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 #pragma unroll
                         for (int jj = 0; jj < 16; ++jj)
                             if (c + jj < valid) {
-                                float a = __fdividef(g[jj], 1.0f + __expf(-g[jj]));
-                                o[(size_t)(t0 + c + jj) * ldo + n] = __float2bfloat16_rn(a * u[jj]);
+                                o[(size_t)(t0 + c + jj) * ldo + n] = __float2bfloat16_rn(gated_act_fast(g[jj], u[jj], prep.act_limit));
                             }
                     }
                 } else if (MODE == TC_ACT) {
@@ -960,7 +957,7 @@ KESTREL_API int kestrel_gemm_tc_plan(const void *x, const void *w, int T, int N,
 
 template <int BN, int MODE>
 static int launch_tc(const CUtensorMap &mw, const CUtensorMap &mx, void *out, int T, int N, int K, int splits,
-                     long long slice_stride, long long ldo, int up_off, int early_w, cudaStream_t stream) {
+                     long long slice_stride, long long ldo, int up_off, int early_w, float act_limit, cudaStream_t stream) {
     constexpr int A_TILES = MODE == TC_PARTIAL ? 1 : 2;
     constexpr int STAGE_BYTES = A_TILES * TC_BM * TC_BK * 2 + BN * TC_BK * 2;
     int total_kb = (K + TC_BK - 1) / TC_BK;
@@ -980,13 +977,13 @@ static int launch_tc(const CUtensorMap &mw, const CUtensorMap &mx, void *out, in
     }
     dim3 grid((N + TC_BM - 1) / TC_BM, (T + BN - 1) / BN, splits);
     if (grid.y > 65535) return kestrel_fail(-2, "gemm_tc: T=%d needs more than 65535 token tiles", T);
-    kestrel_launch(gemm_tc_kernel<BN, MODE>, dim3(grid), dim3(TC_THREADS), smem, stream, mw, mx, out, T, N, K, per, slice_stride, ldo, stages, up_off, early_w);
+    kestrel_launch(gemm_tc_kernel<BN, MODE>, dim3(grid), dim3(TC_THREADS), smem, stream, mw, mx, out, T, N, K, per, slice_stride, ldo, stages, up_off, early_w, act_limit);
     return kestrel_check_launch("gemm_tc");
 }
 
 template <int BN, int MODE>
 static int launch_tc_persistent(const CUtensorMap &mw, const CUtensorMap &mx, void *out, int T, int N, int K,
-                                long long ldo, int up_off, cudaStream_t stream) {
+                                long long ldo, int up_off, float act_limit, cudaStream_t stream) {
     constexpr int A_TILES = MODE == TC_SWIGLU ? 2 : 1;
     constexpr int STAGE_BYTES = A_TILES * TC_BM * TC_BK * 2 + BN * TC_BK * 2;
     int stages = (200 * 1024) / STAGE_BYTES;
@@ -1004,7 +1001,7 @@ static int launch_tc_persistent(const CUtensorMap &mw, const CUtensorMap &mx, vo
     const int sms = kestrel_sms();
     int grid = total < sms ? (int)total : sms;
     kestrel_launch(gemm_tc_persistent_kernel<BN, MODE>, dim3(grid), dim3(TC_THREADS), smem, stream, mw, mx, out, T, N, K, ldo,
-                   stages, up_off, tiles_n, (int)total);
+                   stages, up_off, tiles_n, (int)total, act_limit);
     return kestrel_check_launch("gemm_tc_persistent");
 }
 
@@ -1077,7 +1074,7 @@ static bool swiglu_swapped_wins(int T, int ff) {
 
 template <int MODE>
 static int dispatch_tc(const void *x, const void *w, void *out, int T, int N, int w_rows, int K, long long ldx, long long ldw,
-                       long long ldo, int splits, long long slice_stride, int up_off, int early_w, cudaStream_t stream) {
+                       long long ldo, int splits, long long slice_stride, int up_off, int early_w, cudaStream_t stream, float act_limit = 0.f) {
     int bn = T <= 16 ? 16 : T <= 32 ? 32 : T <= 64 ? 64 : T <= 128 ? 128 : 256;
     bool persistent = T > g_pair_min_tokens && g_persistent && (splits == 1 || (g_pairs && MODE == TC_PARTIAL));
     if (persistent && MODE == TC_SWIGLU) bn = g_swiglu_bn;
@@ -1085,31 +1082,33 @@ static int dispatch_tc(const void *x, const void *w, void *out, int T, int N, in
     int rc = kestrel_tensor_map_bf16(&mw, w, w_rows, K, ldw, TC_BM);
     if (rc) return rc;
     if (persistent && g_pairs) {
+        QkvPrepParams prep = {};
+        prep.act_limit = act_limit;
         rc = kestrel_tensor_map_bf16(&mx, x, T, K, ldx, TCP_BN / 2);
         if (rc) return rc;
         if (MODE == TC_SWIGLU && swiglu_swapped_wins(T, N) && ((uintptr_t)out & 15) == 0 && ldo % 8 == 0)
-            rc = launch_tc_pair<TC_SWIGLU_T>(mw, mx, out, T, N, K, ldo, up_off, 0, 1, 0, stream);
+            rc = launch_tc_pair<TC_SWIGLU_T>(mw, mx, out, T, N, K, ldo, up_off, 0, 1, 0, stream, prep);
         else
-            rc = launch_tc_pair<MODE>(mw, mx, out, T, N, K, ldo, up_off, 0, splits, slice_stride, stream);
+            rc = launch_tc_pair<MODE>(mw, mx, out, T, N, K, ldo, up_off, 0, splits, slice_stride, stream, prep);
         if (rc <= 0) return rc;            // 1 = pairs cannot be scheduled: go on with one CTA per tile
     }
     if (splits > 1) persistent = false;    // the one-CTA persistent kernel does not cut K
     rc = kestrel_tensor_map_bf16(&mx, x, T, K, ldx, bn);
     if (rc) return rc;
     if (persistent) {
-        if (MODE == TC_SWIGLU && bn == 128) return launch_tc_persistent<128, TC_SWIGLU>(mw, mx, out, T, N, K, ldo, up_off, stream);
-        if (MODE == TC_SWIGLU) return launch_tc_persistent<256, TC_SWIGLU>(mw, mx, out, T, N, K, ldo, up_off, stream);
-        return launch_tc_persistent<256, TC_PARTIAL>(mw, mx, out, T, N, K, ldo, up_off, stream);
+        if (MODE == TC_SWIGLU && bn == 128) return launch_tc_persistent<128, TC_SWIGLU>(mw, mx, out, T, N, K, ldo, up_off, act_limit, stream);
+        if (MODE == TC_SWIGLU) return launch_tc_persistent<256, TC_SWIGLU>(mw, mx, out, T, N, K, ldo, up_off, act_limit, stream);
+        return launch_tc_persistent<256, TC_PARTIAL>(mw, mx, out, T, N, K, ldo, up_off, act_limit, stream);
     }
     if (MODE == TC_PARTIAL && tc_wide(T, N))
-        return bn == 128 ? launch_tc<128, TC_PARTIAL2>(mw, mx, out, T, N / 2, K, splits, slice_stride, ldo, N / 2, early_w, stream)
-                         : launch_tc<64, TC_PARTIAL2>(mw, mx, out, T, N / 2, K, splits, slice_stride, ldo, N / 2, early_w, stream);
+        return bn == 128 ? launch_tc<128, TC_PARTIAL2>(mw, mx, out, T, N / 2, K, splits, slice_stride, ldo, N / 2, early_w, act_limit, stream)
+                         : launch_tc<64, TC_PARTIAL2>(mw, mx, out, T, N / 2, K, splits, slice_stride, ldo, N / 2, early_w, act_limit, stream);
     switch (bn) {
-        case 16: return launch_tc<16, MODE>(mw, mx, out, T, N, K, splits, slice_stride, ldo, up_off, early_w, stream);
-        case 32: return launch_tc<32, MODE>(mw, mx, out, T, N, K, splits, slice_stride, ldo, up_off, early_w, stream);
-        case 64: return launch_tc<64, MODE>(mw, mx, out, T, N, K, splits, slice_stride, ldo, up_off, early_w, stream);
-        case 128: return launch_tc<128, MODE>(mw, mx, out, T, N, K, splits, slice_stride, ldo, up_off, early_w, stream);
-        default: return launch_tc<256, MODE>(mw, mx, out, T, N, K, splits, slice_stride, ldo, up_off, early_w, stream);
+        case 16: return launch_tc<16, MODE>(mw, mx, out, T, N, K, splits, slice_stride, ldo, up_off, early_w, act_limit, stream);
+        case 32: return launch_tc<32, MODE>(mw, mx, out, T, N, K, splits, slice_stride, ldo, up_off, early_w, act_limit, stream);
+        case 64: return launch_tc<64, MODE>(mw, mx, out, T, N, K, splits, slice_stride, ldo, up_off, early_w, act_limit, stream);
+        case 128: return launch_tc<128, MODE>(mw, mx, out, T, N, K, splits, slice_stride, ldo, up_off, early_w, act_limit, stream);
+        default: return launch_tc<256, MODE>(mw, mx, out, T, N, K, splits, slice_stride, ldo, up_off, early_w, act_limit, stream);
     }
 }
 
@@ -1226,6 +1225,14 @@ KESTREL_API int kestrel_gemm_tc_swiglu_w(const void *x, const void *w, void *out
     if (T == 0) return 0;
     KESTREL_REQUIRE(kestrel_gemm_tc_supported(x, w, T, ff, K, ldx, ldw), "gemm_tc_swiglu: sizes T=%d ff=%d K=%d do not fit the TMA rules", T, ff, K);
     return dispatch_tc<TC_SWIGLU>(x, w, out, T, ff, 2 * ff, K, ldx, ldw, ldo, 1, 0, ff, weights_static ? 1 : 0, stream);
+}
+
+// the same with the bounded activation of gated_act.cuh where `limit` > 0
+KESTREL_API int kestrel_gemm_tc_gated_w(const void *x, const void *w, void *out, int T, int ff, int K, long long ldx, long long ldw, long long ldo,
+                                        float limit, int weights_static, cudaStream_t stream) {
+    if (T == 0) return 0;
+    KESTREL_REQUIRE(kestrel_gemm_tc_supported(x, w, T, ff, K, ldx, ldw), "gemm_tc_gated: sizes T=%d ff=%d K=%d do not fit the TMA rules", T, ff, K);
+    return dispatch_tc<TC_SWIGLU>(x, w, out, T, ff, 2 * ff, K, ldx, ldw, ldo, 1, 0, ff, weights_static ? 1 : 0, stream, limit);
 }
 
 KESTREL_API int kestrel_gemm_tc_swiglu(const void *x, const void *w, void *out, int T, int ff, int K, long long ldx,

@@ -5,7 +5,11 @@
 //
 //     S_t = diag(w_t) S_{t-1} + a_t (b_t^T S_{t-1}) + k_t v_t^T,      o_t = S_t^T r_t
 //
-// w, a, b, k, r are vectors over the d key channels of a head, v over its dv value channels.
+// or, in a second form, a read-out of the OLD state with a bonus for the token's own write,
+//
+//     o_t = (S_{t-1} + diag(u) k_t v_t^T)^T r_t,      S_t = diag(w_t) S_{t-1} + k_t v_t^T
+//
+// w, a, b, k, r are vectors over the d key channels of a head, v over its dv value channels; u is a weight per head and channel.
 //   * a gated linear recurrence whose forget gate also sets what is written (HGRN2 style):
 //       w = f, k = 1 - f, no correction, r = silu(query);  f = lower + (1 - lower) sigmoid(z)
 //   * a generalised delta rule: with u the unit key k / sqrt(sum k^2 + 1e-6),
@@ -155,8 +159,9 @@ __device__ __forceinline__ void lr_cp_async(float *dst, const float *src, bool v
     else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src) : "memory");
 }
 
-// D: key channels padded to 32, 64, 128 or 256; RANK1: the correction a (b^T S) is present
-template <int D, bool RANK1>
+// D: key channels padded to 32, 64, 128 or 256
+enum { LR_PLAIN = 0, LR_RANK1 = 1, LR_BONUS = 2 };          // RANK1: the correction a (b^T S) is present; BONUS: the second form, `a` holds u [H, d]
+template <int D, int MODE>
 __global__ void __launch_bounds__(128)
 recurrence_scan_kernel(const float *__restrict__ r, const float *__restrict__ w, const float *__restrict__ k, const float *__restrict__ v,
                        const float *__restrict__ a, const float *__restrict__ b, float *__restrict__ state, size_t state_stride,
@@ -164,6 +169,7 @@ recurrence_scan_kernel(const float *__restrict__ r, const float *__restrict__ w,
                        int H, int d, int dv) {
     pdl_launch_dependents();
     pdl_wait();
+    constexpr bool RANK1 = MODE == LR_RANK1, BONUS = MODE == LR_BONUS;
     constexpr int NV = RANK1 ? 5 : 3;                        // vectors over key channels per token: k, r, w (, a, b)
     constexpr int STAGE = LR_TC * (NV * D + 32);             // floats; v [TC][32, LR_COLS used]
     constexpr int M = D / (4 * LR_LPC);                      // float4s of a thread's part
@@ -184,6 +190,16 @@ recurrence_scan_kernel(const float *__restrict__ r, const float *__restrict__ w,
             const int i = 4 * (LR_LPC * m + part) + c;
             Sc[m][c] = (i < d && live) ? Sg[(size_t)i * dv + j] : 0.f;
         }
+    float U[BONUS ? M : 1][4];
+    if (BONUS) {
+#pragma unroll
+        for (int m = 0; m < M; ++m)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const int i = 4 * (LR_LPC * m + part) + c;
+                U[m][c] = i < d ? a[(size_t)h * d + i] : 0.f;
+            }
+    }
     for (int idx = tid; idx < 2 * STAGE; idx += 128) sm[idx] = 0.f;       // the padded channels stay zero
     __syncthreads();
 
@@ -249,6 +265,13 @@ recurrence_scan_kernel(const float *__restrict__ r, const float *__restrict__ w,
                     const float4 aa = a4[LR_LPC * m + part];
                     e0 = fmaf(aa.x, held, e0); e1 = fmaf(aa.y, held, e1); e2 = fmaf(aa.z, held, e2); e3 = fmaf(aa.w, held, e3);
                 }
+                if (BONUS) {
+                    s0 = fmaf(fmaf(U[m][0], e0, Sc[m][0]), rr.x, s0); Sc[m][0] = fmaf(ww.x, Sc[m][0], e0);
+                    s1 = fmaf(fmaf(U[m][1], e1, Sc[m][1]), rr.y, s1); Sc[m][1] = fmaf(ww.y, Sc[m][1], e1);
+                    s2 = fmaf(fmaf(U[m][2], e2, Sc[m][2]), rr.z, s2); Sc[m][2] = fmaf(ww.z, Sc[m][2], e2);
+                    s3 = fmaf(fmaf(U[m][3], e3, Sc[m][3]), rr.w, s3); Sc[m][3] = fmaf(ww.w, Sc[m][3], e3);
+                    continue;
+                }
                 Sc[m][0] = fmaf(ww.x, Sc[m][0], e0); s0 = fmaf(Sc[m][0], rr.x, s0);
                 Sc[m][1] = fmaf(ww.y, Sc[m][1], e1); s1 = fmaf(Sc[m][1], rr.y, s1);
                 Sc[m][2] = fmaf(ww.z, Sc[m][2], e2); s2 = fmaf(Sc[m][2], rr.z, s2);
@@ -291,6 +314,14 @@ recurrence_scan_kernel(const float *__restrict__ r, const float *__restrict__ w,
                 float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
 #pragma unroll
                 for (int m = 0; m < M; ++m) {
+                    if (BONUS) {
+                        const float e0 = K[m].x * vj, e1 = K[m].y * vj, e2 = K[m].z * vj, e3 = K[m].w * vj;
+                        s0 = fmaf(fmaf(U[m][0], e0, Sc[m][0]), R[m].x, s0); Sc[m][0] = fmaf(W[m].x, Sc[m][0], e0);
+                        s1 = fmaf(fmaf(U[m][1], e1, Sc[m][1]), R[m].y, s1); Sc[m][1] = fmaf(W[m].y, Sc[m][1], e1);
+                        s2 = fmaf(fmaf(U[m][2], e2, Sc[m][2]), R[m].z, s2); Sc[m][2] = fmaf(W[m].z, Sc[m][2], e2);
+                        s3 = fmaf(fmaf(U[m][3], e3, Sc[m][3]), R[m].w, s3); Sc[m][3] = fmaf(W[m].w, Sc[m][3], e3);
+                        continue;
+                    }
                     Sc[m][0] = fmaf(W[m].x, Sc[m][0], K[m].x * vj); s0 = fmaf(Sc[m][0], R[m].x, s0);
                     Sc[m][1] = fmaf(W[m].y, Sc[m][1], K[m].y * vj); s1 = fmaf(Sc[m][1], R[m].y, s1);
                     Sc[m][2] = fmaf(W[m].z, Sc[m][2], K[m].z * vj); s2 = fmaf(Sc[m][2], R[m].z, s2);
@@ -413,7 +444,7 @@ recurrence_scan_kernel(const float *__restrict__ r, const float *__restrict__ w,
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float *__restrict__ o, const float *__restrict__ w, int w_stride, float eps, const float *__restrict__ g_part,
-                      int Sg, size_t g_stride, int g_ld, int g_col0, int g_act, T *__restrict__ out, int H, int dv) {
+                      int Sg, size_t g_stride, int g_ld, int g_col0, int g_act, T *__restrict__ out, long long ldo, float scale, int H, int dv) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -430,7 +461,7 @@ head_norm_gate_kernel(const float *__restrict__ o, const float *__restrict__ w, 
                 const float z = sum_slices(g_part, Sg, g_stride, (size_t)t * g_ld + g_col0 + (size_t)h * dv + i);
                 y *= g_act == 1 ? z * lr_sigmoid(z) : lr_sigmoid(z);
             }
-            out[base + i] = from_f32<T>(y);
+            out[(size_t)t * ldo + (size_t)h * dv + i] = from_f32<T>(y * scale);
         }
     }
 }
@@ -470,39 +501,53 @@ KESTREL_API int kestrel_removal_gates(const float *partial, int S, long long sli
     return kestrel_check_launch("removal_gates");
 }
 
-template <int D, bool RANK1>
+template <int D, int MODE>
 static int lr_launch(dim3 grid, cudaStream_t stream, const float *r, const float *w, const float *k, const float *v, const float *a,
                      const float *b, float *state, size_t state_stride, size_t state_off, const int *cu_seqlens, const int *slots, float *out,
                      int H, int d, int dv) {
-    constexpr size_t smem_need = (size_t)2 * LR_TC * ((RANK1 ? 5 : 3) * D + 32) * sizeof(float);
+    constexpr size_t smem_need = (size_t)2 * LR_TC * ((MODE == LR_RANK1 ? 5 : 3) * D + 32) * sizeof(float);
     static bool attr_set = false;
-    if (!attr_set && cudaFuncSetAttribute(recurrence_scan_kernel<D, RANK1>, cudaFuncAttributeMaxDynamicSharedMemorySize, KESTREL_SMEM_MAX_DYNAMIC) != cudaSuccess)
+    if (!attr_set && cudaFuncSetAttribute(recurrence_scan_kernel<D, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, KESTREL_SMEM_MAX_DYNAMIC) != cudaSuccess)
         return kestrel_fail(-3, "recurrence_scan: cannot set the shared memory size");
     attr_set = true;
     // a prompt's scan is few CTAs that run for hundreds of microseconds: one SM each (kestrel_spread_smem)
     const size_t smem = kestrel_spread_smem((long)grid.x * grid.y * grid.z, smem_need);
-    kestrel_launch(recurrence_scan_kernel<D, RANK1>, grid, dim3(128), smem, stream, r, w, k, v, a, b, state, state_stride, state_off, cu_seqlens,
+    kestrel_launch(recurrence_scan_kernel<D, MODE>, grid, dim3(128), smem, stream, r, w, k, v, a, b, state, state_stride, state_off, cu_seqlens,
                    slots, out, H, d, dv);
     return kestrel_check_launch("recurrence_scan");
+}
+
+template <int MODE>
+static int lr_dispatch(const float *r, const float *w, const float *k, const float *v, const float *a, const float *b, float *state,
+                       long long state_stride, long long state_off, const int *cu_seqlens, const int *slots, float *out, int nseq, int H, int d, int dv,
+                       cudaStream_t stream) {
+    if (nseq == 0) return 0;
+    KESTREL_REQUIRE(nseq > 0 && H > 0 && d > 0 && dv > 0 && state_off >= 0, "recurrence_scan: bad sizes");
+    KESTREL_REQUIRE(d <= 256, "recurrence_scan: key size %d exceeds 256", d);
+    KESTREL_REQUIRE(H <= 65535 && nseq <= 65535, "recurrence_scan: grid too large");
+    dim3 grid((dv + LR_COLS - 1) / LR_COLS, H, nseq);
+#define LR_CASE(D) return lr_launch<D, MODE>(grid, stream, r, w, k, v, a, b, state, (size_t)state_stride, (size_t)state_off, cu_seqlens, slots, out, H, d, dv)
+    if (d <= 32) LR_CASE(32);
+    if (d <= 64) LR_CASE(64);
+    if (d <= 128) LR_CASE(128);
+    LR_CASE(256);
+#undef LR_CASE
 }
 
 KESTREL_API int kestrel_recurrence_scan(const float *r, const float *w, const float *k, const float *v, const float *a, const float *b,
                                         float *state, long long state_stride, long long state_off, const int *cu_seqlens, const int *slots,
                                         float *out, int nseq, int H, int d, int dv, cudaStream_t stream) {
-    if (nseq == 0) return 0;
-    KESTREL_REQUIRE(nseq > 0 && H > 0 && d > 0 && dv > 0 && state_off >= 0, "recurrence_scan: bad sizes");
     KESTREL_REQUIRE((a == nullptr) == (b == nullptr), "recurrence_scan: the correction needs both of its vectors");
-    KESTREL_REQUIRE(d <= 256, "recurrence_scan: key size %d exceeds 256", d);
-    KESTREL_REQUIRE(H <= 65535 && nseq <= 65535, "recurrence_scan: grid too large");
-    dim3 grid((dv + LR_COLS - 1) / LR_COLS, H, nseq);
-#define LR_CASE(D)                                                                                                                            \
-    return a ? lr_launch<D, true>(grid, stream, r, w, k, v, a, b, state, (size_t)state_stride, (size_t)state_off, cu_seqlens, slots, out, H, d, dv) \
-             : lr_launch<D, false>(grid, stream, r, w, k, v, a, b, state, (size_t)state_stride, (size_t)state_off, cu_seqlens, slots, out, H, d, dv)
-    if (d <= 32) { LR_CASE(32); }
-    if (d <= 64) { LR_CASE(64); }
-    if (d <= 128) { LR_CASE(128); }
-    LR_CASE(256);
-#undef LR_CASE
+    return a ? lr_dispatch<LR_RANK1>(r, w, k, v, a, b, state, state_stride, state_off, cu_seqlens, slots, out, nseq, H, d, dv, stream)
+             : lr_dispatch<LR_PLAIN>(r, w, k, v, a, b, state, state_stride, state_off, cu_seqlens, slots, out, nseq, H, d, dv, stream);
+}
+
+// the read-out of the old state with the bonus u [H, d] for the token's own write
+KESTREL_API int kestrel_recurrence_scan_bonus(const float *r, const float *w, const float *k, const float *v, const float *u, float *state,
+                                              long long state_stride, long long state_off, const int *cu_seqlens, const int *slots, float *out,
+                                              int nseq, int H, int d, int dv, cudaStream_t stream) {
+    KESTREL_REQUIRE(nseq == 0 || u, "recurrence_scan_bonus: the bonus is missing");
+    return lr_dispatch<LR_BONUS>(r, w, k, v, u, nullptr, state, state_stride, state_off, cu_seqlens, slots, out, nseq, H, d, dv, stream);
 }
 
 KESTREL_API int kestrel_head_norm_gate(const float *o, const float *w, int w_stride, float eps, const float *g_part, int Sg, long long g_stride,
@@ -512,16 +557,23 @@ KESTREL_API int kestrel_head_norm_gate(const float *o, const float *w, int w_str
 
 KESTREL_API int kestrel_head_norm_act(const float *o, const float *w, int w_stride, float eps, const float *g_part, int Sg, long long g_stride,
                                       int g_ld, int g_col0, int g_act, void *out, int dtype, int T, int H, int dv, cudaStream_t stream) {
+    return kestrel_head_norm_act_to(o, w, w_stride, eps, g_part, Sg, g_stride, g_ld, g_col0, g_act, 1.0f, out, (long long)H * dv, dtype, T, H, dv, stream);
+}
+
+// the same times `scale`, into rows of ldo numbers (a place inside a wider matrix)
+KESTREL_API int kestrel_head_norm_act_to(const float *o, const float *w, int w_stride, float eps, const float *g_part, int Sg, long long g_stride,
+                                         int g_ld, int g_col0, int g_act, float scale, void *out, long long ldo, int dtype, int T, int H, int dv,
+                                         cudaStream_t stream) {
     if (T == 0) return 0;
     KESTREL_REQUIRE(T > 0 && H > 0 && dv > 0 && (g_act == 0 || g_act == 1) && (w_stride == 0 || w_stride == dv) && (!g_part || (Sg > 0 && g_col0 >= 0 && g_col0 + H * dv <= g_ld)),
                     "head_norm_gate: bad sizes");
     const int by = T >= 512 ? 1 : (H + 3) / 4;
     if (dtype == KESTREL_F32)
         kestrel_launch(head_norm_gate_kernel<float>, dim3(T, by), dim3(128), 0, stream, o, w, w_stride, eps, g_part, Sg, (size_t)g_stride, g_ld, g_col0,
-                       g_act, (float *)out, H, dv);
+                       g_act, (float *)out, ldo, scale, H, dv);
     else if (dtype == KESTREL_BF16)
         kestrel_launch(head_norm_gate_kernel<__nv_bfloat16>, dim3(T, by), dim3(128), 0, stream, o, w, w_stride, eps, g_part, Sg, (size_t)g_stride, g_ld,
-                       g_col0, g_act, (__nv_bfloat16 *)out, H, dv);
+                       g_col0, g_act, (__nv_bfloat16 *)out, ldo, scale, H, dv);
     else
         return kestrel_fail(-2, "head_norm_gate: unknown dtype %d", dtype);
     return kestrel_check_launch("head_norm_gate");

@@ -463,8 +463,8 @@ KESTREL_API int kestrel_add_three(float *residual, const float *a, int Sa, long 
 // mixer's output, its logits columns of a product of the mixer's input.  The sigmoid is float32.
 // ------------------------------------------------------------------------------------------
 template <typename T>
-__global__ void gate_columns_mul_kernel(T *__restrict__ x, const float *__restrict__ g, int S, size_t slice_stride, int ld, int col0,
-                                        const float *__restrict__ bias, int n, size_t total) {
+__global__ void gate_columns_mul_kernel(const T *x, const float *__restrict__ g, int S, size_t slice_stride, int ld, int col0,
+                                        const float *__restrict__ bias, float scale, T *out, long long ldo, int n, size_t total) {
     pdl_launch_dependents();
     pdl_wait();
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -473,19 +473,27 @@ __global__ void gate_columns_mul_kernel(T *__restrict__ x, const float *__restri
     int i = (int)(idx % n);
     float z = sum_slices(g, S, slice_stride, t * ld + col0 + i);
     if (bias) z += bias[col0 + i];
-    x[idx] = from_f32<T>(to_f32<T>(x[idx]) * (1.0f / (1.0f + expf(-z))));
+    out[t * ldo + i] = from_f32<T>(to_f32<T>(x[idx]) * (1.0f / (1.0f + expf(-z))) * scale);
 }
 
 KESTREL_API int kestrel_gate_columns_mul(void *x, int dtype, const float *g, int S, long long slice_stride, int ld, int col0, const float *bias,
                                          int T, int n, cudaStream_t stream) {
+    return kestrel_gate_columns_mul_to(x, dtype, g, S, slice_stride, ld, col0, bias, 1.0f, x, n, T, n, stream);
+}
+
+// the same times `scale`, into rows of ldo numbers (a place inside a wider matrix; x itself is left as it is unless it is the output)
+KESTREL_API int kestrel_gate_columns_mul_to(const void *x, int dtype, const float *g, int S, long long slice_stride, int ld, int col0, const float *bias,
+                                            float scale, void *out, long long ldo, int T, int n, cudaStream_t stream) {
     if (T == 0) return 0;
-    KESTREL_REQUIRE(T > 0 && n > 0 && S > 0 && col0 >= 0 && col0 + n <= ld, "gate_columns_mul: bad sizes");
+    KESTREL_REQUIRE(T > 0 && n > 0 && S > 0 && col0 >= 0 && col0 + n <= ld && ldo >= n, "gate_columns_mul: bad sizes");
     size_t total = (size_t)T * n;
     unsigned blocks = (unsigned)((total + 255) / 256);
     if (dtype == KESTREL_F32)
-        kestrel_launch(gate_columns_mul_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float *)x, g, S, (size_t)slice_stride, ld, col0, bias, n, total);
+        kestrel_launch(gate_columns_mul_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float *)x, g, S, (size_t)slice_stride, ld, col0, bias, scale,
+                       (float *)out, ldo, n, total);
     else if (dtype == KESTREL_BF16)
-        kestrel_launch(gate_columns_mul_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (__nv_bfloat16 *)x, g, S, (size_t)slice_stride, ld, col0, bias, n, total);
+        kestrel_launch(gate_columns_mul_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16 *)x, g, S, (size_t)slice_stride, ld,
+                       col0, bias, scale, (__nv_bfloat16 *)out, ldo, n, total);
     else
         return kestrel_fail(-2, "gate_columns_mul: unknown dtype %d", dtype);
     return kestrel_check_launch("gate_columns_mul");

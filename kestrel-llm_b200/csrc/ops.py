@@ -211,13 +211,14 @@ def add_rmsnorm(residual: torch.Tensor, delta: Optional[Partials], weight: torch
         1 if (write_back and delta is not None) else 0, _stream()))
 
 
-def swiglu(gate_up: Partials, out: torch.Tensor) -> None:
-    """out[t, i] = silu(g[t, i]) * u[t, i] with g, u the two halves of gate_up's width."""
+def swiglu(gate_up: Partials, out: torch.Tensor, limit: float = 0.0) -> None:
+    """out[t, i] = silu(g[t, i]) * u[t, i] with g, u the two halves of gate_up's width; ``limit`` > 0: the bounded form of
+    `gate_up_swiglu`."""
     _need(out, "swiglu.out", dims=2)
     T, ff = out.shape
     if gate_up.tokens != T or gate_up.width != 2 * ff or gate_up.bias is not None:
         raise KernelError("swiglu: shapes differ, or a bias is pending")
-    _check(library().kestrel_swiglu(gate_up.data.data_ptr(), gate_up.slices, gate_up.slice_stride,
+    _check(library().kestrel_gated_act(gate_up.data.data_ptr(), gate_up.slices, gate_up.slice_stride, float(limit),
                                     out.data_ptr(), _code(out, "swiglu.out"), T, ff, _stream()))
 
 
@@ -403,8 +404,9 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None
     return out
 
 
-def gemm_tc_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, weights_static: bool = False) -> None:
-    """out = silu(x Wg^T) * (x Wu^T) in one tcgen05 kernel with two accumulators."""
+def gemm_tc_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, weights_static: bool = False,
+                   limit: float = 0.0) -> None:
+    """out = silu(x Wg^T) * (x Wu^T), or its bounded form (`gate_up_swiglu`), in one tcgen05 kernel with two accumulators."""
     _need(x, "gemm_tc_swiglu.x", torch.bfloat16, 2)
     _need(w_gate_up, "gemm_tc_swiglu.w", torch.bfloat16, 2)
     _need(out, "gemm_tc_swiglu.out", torch.bfloat16, 2)
@@ -412,9 +414,9 @@ def gemm_tc_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, 
     ff = out.shape[1]
     if w_gate_up.shape != (2 * ff, K) or out.shape[0] != T:
         raise KernelError("gemm_tc_swiglu: shapes differ")
-    _check(library().kestrel_gemm_tc_swiglu_w(x.data_ptr(), w_gate_up.data_ptr(), out.data_ptr(), T, ff, K,
-                                              x.stride(0), w_gate_up.stride(0), out.stride(0),
-                                              1 if weights_static else 0, _stream()))
+    _check(library().kestrel_gemm_tc_gated_w(x.data_ptr(), w_gate_up.data_ptr(), out.data_ptr(), T, ff, K,
+                                              x.stride(0), w_gate_up.stride(0), out.stride(0), float(limit),
+                                             1 if weights_static else 0, _stream()))
 
 
 def gemm_tc_set_tuning(overhead_kb: int = -1, ctas_per_sm: int = 0) -> None:
@@ -485,6 +487,31 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None,
     return out
 
 
+def linear_groups(x: torch.Tensor, w: torch.Tensor, groups: int) -> Partials:
+    """``groups`` products of equal size over inputs of their own: columns [s n, (s + 1) n) of the result are x[s] times rows
+    [s n, (s + 1) n) of w, transposed; x [>= groups, T, K] contiguous, w [groups n, K].  The weights are a model's (`gemm_tc`)."""
+    _need(x, "linear_groups.x", dims=3)
+    _need(w, "linear_groups.w", x.dtype, 2)
+    T, K = x.shape[1:]
+    N = w.shape[0]
+    n = N // groups
+    if x.shape[0] < groups or w.shape[1] != K or N != groups * n:
+        raise KernelError(f"linear_groups: x {tuple(x.shape)}, w {tuple(w.shape)}, {groups} groups")
+    lib = library()
+    plan = lib.kestrel_gemm_tc_plan(x.data_ptr(), w.data_ptr(), T, n, K, K, w.stride(0)) if x.dtype == torch.bfloat16 else 0
+    if plan > 0 and (T * K * x.element_size()) % 16 == 0 and (n * w.stride(0) * w.element_size()) % 16 == 0:
+        out = torch.empty((plan, T, N), dtype=torch.float32, device=x.device)
+        for s in range(groups):
+            _check(lib.kestrel_gemm_tc_w(x[s].data_ptr(), w[s * n:].data_ptr(), out[0, 0, s * n:].data_ptr(), T, n, K, K, w.stride(0), N, plan, T * N, 1,
+                                         _stream()))
+        return Partials(out)
+    out = torch.empty((1, T, N), dtype=torch.float32, device=x.device)
+    for s in range(groups):
+        _check(lib.kestrel_gemm_plain(x[s].data_ptr(), w[s * n:].data_ptr(), out[0, 0, s * n:].data_ptr(), _code(x, "linear_groups.x"), T, n, K, K,
+                                      w.stride(0), N, _stream()))
+    return Partials(out)
+
+
 def linear_add_into(x: torch.Tensor, w: torch.Tensor, residual: torch.Tensor) -> bool:
     """residual += x w^T inside the product's epilogue, where the product can do that (bfloat16,
     many tokens, one pass over K); False if it cannot - nothing has run then and the caller takes
@@ -525,20 +552,19 @@ def linear_act(x: torch.Tensor, w: torch.Tensor, act: str, weights_static: bool 
 linear_act_fused = True          # tests switch the epilogue form off to hold both forms against each other
 
 
-def gate_up_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, ff: int, weights_static: bool = False, cut_few: bool = False) -> torch.Tensor:
-    """silu(x Wg^T) * (x Wu^T) in x's dtype, Wg and Wu being the two halves of w_gate_up's rows.
+def gate_up_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, ff: int, weights_static: bool = False, cut_few: bool = False,
+                   limit: float = 0.0) -> torch.Tensor:
+    """silu(x Wg^T) * (x Wu^T) in x's dtype, Wg and Wu being the two halves of w_gate_up's rows; with ``limit`` > 0 the bounded
+    form: g <- min(g, limit), u <- clamp(u, -limit, limit), g * sigmoid(1.702 g) * (u + 1).
     ``weights_static`` as in `gemm_tc`.  ``cut_few``: with few tokens the product may be cut along K and activated by a second
     kernel, for a feed-forward so narrow that the uncut product would leave most of the device idle."""
     out = torch.empty((x.shape[0], ff), dtype=x.dtype, device=x.device)
-    if cut_few and x.shape[0] <= 64 and ff <= 128 * 37:
-        swiglu(Partials(linear(x, w_gate_up, weights_static=weights_static)), out)
-        return out
-    if gemm_tc_supported(x, w_gate_up):
+    if not (cut_few and x.shape[0] <= 64 and ff <= 128 * 37) and gemm_tc_supported(x, w_gate_up):
         # the activation is the product's epilogue: the K range is not split, whatever the number of
         # tokens, and the gate/up product never reaches memory
-        gemm_tc_swiglu(x, w_gate_up, out, weights_static=weights_static)
+        gemm_tc_swiglu(x, w_gate_up, out, weights_static=weights_static, limit=limit)
     else:
-        swiglu(Partials(linear(x, w_gate_up, weights_static=weights_static)), out)
+        swiglu(Partials(linear(x, w_gate_up, weights_static=weights_static)), out, limit)
     return out
 
 
@@ -957,15 +983,17 @@ def embed_add(table: torch.Tensor, ids: torch.Tensor, x: torch.Tensor) -> None:
                                        _stream()))
 
 
-def gate_columns_mul(x: torch.Tensor, g: Partials, col0: int) -> None:
-    """x[t, i] *= sigmoid(columns [col0, col0 + x.shape[1]) of a product, summed over its slices, plus its bias), in place:
-    a gate per element of a mixer's output."""
+def gate_columns_mul(x: torch.Tensor, g: Partials, col0: int, out: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
+    """x[t, i] *= sigmoid(columns [col0, col0 + x.shape[1]) of a product, summed over its slices, plus its bias): a gate per element of a
+    mixer's output.  In place, or into ``out``, which may be a place inside a wider matrix; times ``scale``."""
     _need(x, "gate_columns_mul.x", dims=2)
     T, n = x.shape
-    if g.tokens != T or col0 < 0 or col0 + n > g.width or (g.bias is not None and g.bias.shape[0] != g.width):
+    out = x if out is None else out
+    _need_rows(out, "gate_columns_mul.out", T, n)
+    if g.tokens != T or col0 < 0 or col0 + n > g.width or (g.bias is not None and g.bias.shape[0] != g.width) or out.dtype != x.dtype:
         raise KernelError("gate_columns_mul: shapes differ")
-    _check(library().kestrel_gate_columns_mul(x.data_ptr(), _code(x, "gate_columns_mul.x"), g.data.data_ptr(), g.slices, g.slice_stride, g.width,
-                                              int(col0), _p(g.bias), T, n, _stream()))
+    _check(library().kestrel_gate_columns_mul_to(x.data_ptr(), _code(x, "gate_columns_mul.x"), g.data.data_ptr(), g.slices, g.slice_stride, g.width,
+                                                 int(col0), _p(g.bias), float(scale), out.data_ptr(), out.stride(0), T, n, _stream()))
 
 
 def add_row(x: torch.Tensor, row: torch.Tensor) -> None:
@@ -1043,6 +1071,43 @@ def attn_prepare_ex(qkv: Partials, q_norm_w: Optional[torch.Tensor], k_norm_w: O
         float(norm_eps), _p(inv_freq), rot or 0, rot_mode or 0, float(rotation.scale) if rotation is not None else 1.0, t_coef, t_every, positions.data_ptr(), seq_of_token.data_ptr(), block_table.data_ptr(), block_table.stride(0), int(page_size),
         k_cache.data_ptr(), v_cache.data_ptr(), q_out.data_ptr(), _p(gate_out), _code(q_out, "attn_prepare_ex.q_out"), T, nq, nkv, hd, vd,
         1 if has_kv else 0, int(maps), 1 if q_pad else 0, _stream()))
+
+
+def attn_prepare_conv(qk: Partials, conv_w: torch.Tensor, q_norm_w: Optional[torch.Tensor], k_norm_w: Optional[torch.Tensor], norm_eps: float,
+                      rotation, state: torch.Tensor, tail_off: int, batch, block_table: torch.Tensor, page_size: int, k_cache: torch.Tensor,
+                      v_cache: torch.Tensor, q_out: torch.Tensor, nq: int, nkv: int, hd: int) -> None:
+    """Columns [q | k | ...] of a product for a mixer whose values are its keys: q and k through a causal convolution over time
+    (``conv_w`` [(nq + nkv) hd, taps]; earlier inputs from, the last ones to, the slot at ``tail_off``), k as it then is into the V
+    pages; q and k divided by their root mean square per head, times weights [hd] where given, turned by position (rotate-half pairs);
+    q to ``q_out``, k into the K pages."""
+    _need(q_out, "attn_prepare_conv.q_out", dims=2)
+    _need(conv_w, "attn_prepare_conv.conv_w", torch.float32, 2)
+    _need(state, "attn_prepare_conv.state", torch.float32, 2)
+    _need(block_table, "attn_prepare_conv.block_table", torch.int32, 2)
+    _need(k_cache, "attn_prepare_conv.k_cache", q_out.dtype, 4)
+    _need(v_cache, "attn_prepare_conv.v_cache", q_out.dtype, 4)
+    T, C = q_out.shape[0], (nq + nkv) * hd
+    taps = conv_w.shape[1]
+    if qk.tokens != T or qk.width < C or qk.bias is not None or q_out.shape[1] != nq * hd or conv_w.shape[0] != C or \
+            tail_off + (taps - 1) * C > state.shape[1]:
+        raise KernelError("attn_prepare_conv: shapes differ, or a bias is pending")
+    for c in (k_cache, v_cache):
+        if tuple(c.shape[1:]) != (nkv, page_size, hd):
+            raise KernelError("attn_prepare_conv: the cache planes do not fit the heads")
+    for w in (q_norm_w, k_norm_w):
+        if w is not None and (w.dtype != torch.float32 or w.numel() != hd):
+            raise KernelError(f"attn_prepare_conv: the norm per head takes a float32 weight of {hd} entries")
+    if rotation is not None and rotation.mode != 0:
+        raise KernelError("attn_prepare_conv: rotate-half pairs only")
+    _check(library().kestrel_attn_prepare_conv(
+        qk.data.data_ptr(), qk.slices, qk.slice_stride, qk.width, conv_w.data_ptr(), taps, _p(q_norm_w), _p(k_norm_w), float(norm_eps),
+        _p(rotation.inv_freq) if rotation is not None else None, int(rotation.dim) if rotation is not None else 0,
+        float(rotation.scale) if rotation is not None else 1.0, state.data_ptr(), state.stride(0), int(tail_off), batch.positions.data_ptr(),
+        batch.seq_of_token.data_ptr(), batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), block_table.data_ptr(), block_table.stride(0),
+        int(page_size), k_cache.data_ptr(), v_cache.data_ptr(), q_out.data_ptr(), _code(q_out, "attn_prepare_conv.q_out"), T, batch.num_seqs,
+        nq, nkv, hd, _stream()))
+    global launches
+    launches += 1 if taps > 1 else 0
 
 
 WEIGHTINGS = {"softmax": 0, "softmax_sink": 1, "sigmoid": 2}
@@ -1420,34 +1485,38 @@ def head_gemm_set_plain(on: bool = True) -> None:
 
 # ---- gated delta rule ------------------------------------------------------------------------
 
-def delta_conv_silu(x: Partials, conv_w: torch.Tensor, state: torch.Tensor, tail_off: int, batch, out: torch.Tensor) -> None:
-    """out[t, c] = silu(causal convolution over time of x's first C columns), C = conv_w.shape[0];
-    inputs before the step come from, and the last taps - 1 inputs go to, each request's state slot
-    (``state`` float32 [slots, size], the tail [taps - 1, C] at ``tail_off``)."""
-    _need(conv_w, "delta_conv.w", torch.float32, 2)
-    _need(state, "delta_conv.state", torch.float32, 2)
-    _need(out, "delta_conv.out", torch.float32, 2)
+def short_conv(x: Partials, conv_w: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, tail_off: int, batch, out: torch.Tensor,
+               col0: int = 0, silu: bool = True) -> None:
+    """out[t, c] = act(causal convolution over time of x's columns col0 .. col0 + C, plus ``bias``), C = conv_w.shape[0], act silu or
+    nothing; inputs before the step come from, and the last taps - 1 inputs go to, each request's state slot (``state`` float32
+    [slots, size], the tail [taps - 1, C] at ``tail_off``)."""
+    _need(conv_w, "short_conv.w", torch.float32, 2)
+    _need(state, "short_conv.state", torch.float32, 2)
+    _need(out, "short_conv.out", dims=2)
     C, taps = conv_w.shape
     T = out.shape[0]
-    if x.tokens != T or x.width < C or out.shape[1] != C or x.bias is not None:
-        raise KernelError("delta_conv_silu: shapes differ")
-    _check(library().kestrel_delta_conv_silu(x.data.data_ptr(), x.slices, x.slice_stride, x.width, conv_w.data_ptr(), taps, state.data_ptr(),
-                                             state.stride(0), int(tail_off), batch.seq_of_token.data_ptr(), batch.cu_seqlens.data_ptr(),
-                                             batch.slots.data_ptr(), out.data_ptr(), T, batch.num_seqs, C, _stream()))
+    if x.tokens != T or x.width < col0 + C or out.shape[1] != C or x.bias is not None or tail_off + (taps - 1) * C > state.shape[1]:
+        raise KernelError("short_conv: shapes differ")
+    _check(library().kestrel_short_conv(x.data.data_ptr(), x.slices, x.slice_stride, x.width, int(col0), conv_w.data_ptr(), _p(bias), taps,
+                                        1 if silu else 0, state.data_ptr(), state.stride(0), int(tail_off), batch.seq_of_token.data_ptr(),
+                                        batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), out.data_ptr(), _code(out, "short_conv.out"), T,
+                                        batch.num_seqs, C, _stream()))
     global launches
     launches += 1 if taps > 1 else 0
 
 
 def delta_gates(act: torch.Tensor, x: Partials, col_beta: int, a: Partials, A_log: torch.Tensor, dt_bias: torch.Tensor,
-                qn: torch.Tensor, kn: torch.Tensor, decay: torch.Tensor, beta: torch.Tensor, H: int, G: int, d: int) -> None:
-    """Unit query and key vectors (queries scaled by d^-1/2), beta = sigmoid, decay = exp(-exp(A_log) softplus(a + dt_bias))."""
+                qn: torch.Tensor, kn: torch.Tensor, decay: torch.Tensor, beta: torch.Tensor, H: int, G: int, d: int, col_a: int = 0,
+                per_head: bool = False) -> None:
+    """Unit query and key vectors (queries scaled by d^-1/2), beta = sigmoid, decay = exp(-exp(A_log) softplus(a + dt_bias)), a the
+    columns of ``a`` from ``col_a``: one per head and key channel, or (``per_head``) one per head for all of its channels."""
     for t, n in ((act, "act"), (qn, "qn"), (kn, "kn"), (decay, "decay"), (beta, "beta")):
         _need(t, f"delta_gates.{n}", torch.float32, 2)
     T = act.shape[0]
-    if a.tokens != T or a.width != H * d or qn.shape != (T, G * d) or decay.shape != (T, H * d) or beta.shape != (T, H):
+    if a.tokens != T or a.width < col_a + (H if per_head else H * d) or qn.shape != (T, G * d) or decay.shape != (T, H * d) or beta.shape != (T, H):
         raise KernelError("delta_gates: shapes differ")
     _check(library().kestrel_delta_gates(act.data_ptr(), act.shape[1], x.data.data_ptr(), x.slices, x.slice_stride, x.width, int(col_beta),
-                                         a.data.data_ptr(), a.slices, a.slice_stride, A_log.data_ptr(), dt_bias.data_ptr(), qn.data_ptr(),
+                                         a.data.data_ptr(), a.slices, a.slice_stride, a.width, int(col_a), 1 if per_head else 0, A_log.data_ptr(), dt_bias.data_ptr(), qn.data_ptr(),
                                          kn.data_ptr(), decay.data_ptr(), beta.data_ptr(), T, H, G, d, _stream()))
 
 
@@ -1526,27 +1595,121 @@ def recurrence_scan(r: torch.Tensor, w: torch.Tensor, k: torch.Tensor, v: torch.
     return out
 
 
+def recurrence_scan_bonus(r: torch.Tensor, w: torch.Tensor, k: torch.Tensor, v: torch.Tensor, u: torch.Tensor, state: torch.Tensor,
+                          state_off: int, batch, H: int, d: int, dv: int) -> torch.Tensor:
+    """o = (S + diag(u) k v^T)^T r of the OLD state, then S <- diag(w) S + k v^T, per head; otherwise as `recurrence_scan`."""
+    _need(state, "recurrence_scan_bonus.state", torch.float32, 2)
+    T = r.shape[0]
+    for t, name, n in ((r, "r", H * d), (w, "w", H * d), (k, "k", H * d), (v, "v", H * dv)):
+        _need(t, f"recurrence_scan_bonus.{name}", torch.float32, 2)
+        if t.shape != (T, n):
+            raise KernelError(f"recurrence_scan_bonus.{name}: shape {tuple(t.shape)}, expected ({T}, {n})")
+    _need(u, "recurrence_scan_bonus.u", torch.float32)
+    if u.numel() != H * d or state_off < 0 or state_off + H * d * dv > state.shape[1]:
+        raise KernelError("recurrence_scan_bonus: the bonus does not fit the heads, or the state not the slot")
+    out = torch.empty((T, H * dv), dtype=torch.float32, device=r.device)
+    _check(library().kestrel_recurrence_scan_bonus(r.data_ptr(), w.data_ptr(), k.data_ptr(), v.data_ptr(), u.data_ptr(), state.data_ptr(),
+                                                   state.stride(0), int(state_off), batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(),
+                                                   out.data_ptr(), batch.num_seqs, H, d, dv, _stream()))
+    return out
+
+
 GATE_ACTS = {"sigmoid": 0, "silu": 1}
 
 
+def _need_rows(t: torch.Tensor, name: str, T: int, n: int) -> None:
+    """A [T, n] place for results inside a matrix: unit stride along a row, any row length."""
+    if not t.is_cuda or t.dim() != 2 or tuple(t.shape) != (T, n) or t.stride(1) != 1:
+        raise KernelError(f"{name}: shape {tuple(t.shape)} with strides {t.stride()}, expected ({T}, {n}) with unit column stride on a CUDA device")
+
+
 def head_norm_gate(o: torch.Tensor, weight: Optional[torch.Tensor], eps: float, gate: Optional[Partials], gate_col0: int, out: torch.Tensor,
-                   H: int, dv: int, gate_act: str = "sigmoid") -> None:
+                   H: int, dv: int, gate_act: str = "sigmoid", scale: float = 1.0) -> None:
     """out = o / sqrt(mean(o^2) + eps) per head, times ``weight`` ([dv]: shared by the heads; [H dv]: one per
-    head; None: no weight), times ``gate_act`` (a sigmoid, or silu) of the columns [gate_col0, gate_col0 + H dv) of ``gate`` where given."""
+    head; None: no weight), times ``gate_act`` (a sigmoid, or silu) of the columns [gate_col0, gate_col0 + H dv) of ``gate`` where given, times ``scale``.
+    ``out`` may be a place inside a wider matrix."""
     _need(o, "head_norm_gate.o", torch.float32, 2)
     if weight is not None:
         _need(weight, "head_norm_gate.weight", torch.float32, 1)
-    _need(out, "head_norm_gate.out", dims=2)
     T = o.shape[0]
-    if o.shape[1] != H * dv or out.shape != o.shape or (weight is not None and weight.shape[0] not in (dv, H * dv)):
+    _need_rows(out, "head_norm_gate.out", T, H * dv)
+    if o.shape[1] != H * dv or (weight is not None and weight.shape[0] not in (dv, H * dv)):
         raise KernelError("head_norm_gate: shapes differ")
     if gate is not None and (gate.tokens != T or gate.bias is not None or gate_col0 + H * dv > gate.width):
         raise KernelError("head_norm_gate: the gate's product does not fit, or carries a bias")
     w_stride = dv if (weight is not None and weight.shape[0] == H * dv and H > 1) else 0
-    _check(library().kestrel_head_norm_act(o.data_ptr(), _p(weight), w_stride, float(eps), _p(gate.data) if gate is not None else None,
+    _check(library().kestrel_head_norm_act_to(o.data_ptr(), _p(weight), w_stride, float(eps), _p(gate.data) if gate is not None else None,
                                             gate.slices if gate is not None else 0, gate.slice_stride if gate is not None else 0,
-                                            gate.width if gate is not None else 0, int(gate_col0), GATE_ACTS[gate_act], out.data_ptr(), _code(out, "head_norm_gate.out"),
+                                            gate.width if gate is not None else 0, int(gate_col0), GATE_ACTS[gate_act], float(scale), out.data_ptr(), out.stride(0), _code(out, "head_norm_gate.out"),
                                             T, H, dv, _stream()))
+
+
+# ---- a recurrence whose projections read each token blended with the one before it ------------------
+
+def token_shift(h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, state_off: int, batch) -> torch.Tensor:
+    """[n, T, d] in h's dtype: h[t] + (h[t - 1] - h[t]) * mu[s] for every row s of ``mu`` [n, d]; the token before a request's first one
+    of this step comes from its slot (float32 [d] at ``state_off``)."""
+    _need(h, "token_shift.h", dims=2)
+    _need(mu, "token_shift.mu", torch.float32, 2)
+    _need(state, "token_shift.state", torch.float32, 2)
+    T, d = h.shape
+    if mu.shape[1] != d or state_off < 0 or state_off + d > state.shape[1]:
+        raise KernelError("token_shift: shapes differ")
+    out = torch.empty((mu.shape[0], T, d), dtype=h.dtype, device=h.device)
+    _check(library().kestrel_token_shift(h.data_ptr(), mu.data_ptr(), mu.shape[0], state.data_ptr(), state.stride(0), int(state_off),
+                                         batch.seq_of_token.data_ptr(), batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), out.data_ptr(),
+                                         _code(h, "token_shift.h"), T, d, _stream()))
+    return out
+
+
+def time_mix_gates(p: Partials, z: Partials, w0: torch.Tensor, n: int, h: torch.Tensor, state: torch.Tensor, state_off: int, batch):
+    """(r, w, k, v) float32 [T, n] for `recurrence_scan_bonus`: r, k, v the columns 0, n, 2 n of ``p``, w = exp(-exp(z + w0)); every
+    request's last row of ``h`` goes into its slot at ``state_off``."""
+    T, dev = p.tokens, p.data.device
+    _need(h, "time_mix_gates.h", dims=2)
+    _need(w0, "time_mix_gates.w0", torch.float32, 1)
+    if p.bias is not None or z.bias is not None or z.tokens != T or z.width != n or p.width < 3 * n or w0.shape[0] != n or h.shape[0] != T or \
+            state_off + h.shape[1] > state.shape[1]:
+        raise KernelError("time_mix_gates: shapes differ, or a bias is pending")
+    r, w, k, v = (torch.empty((T, n), dtype=torch.float32, device=dev) for _ in range(4))
+    _check(library().kestrel_time_mix_gates(p.data.data_ptr(), p.slices, p.slice_stride, p.width, z.data.data_ptr(), z.slices, z.slice_stride,
+                                            w0.data_ptr(), r.data_ptr(), k.data_ptr(), v.data_ptr(), w.data_ptr(), int(n), h.data_ptr(),
+                                            _code(h, "time_mix_gates.h"), h.shape[1], state.data_ptr(), state.stride(0), int(state_off),
+                                            batch.seq_of_token.data_ptr(), batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), T, _stream()))
+    return r, w, k, v
+
+
+# ---- a state-space mixer with a scalar decay per head -----------------------------------------------
+
+def ssm_expand(act: torch.Tensor, fused: Partials, col_dt: int, dt_bias: torch.Tensor, A_log: torch.Tensor, H: int, G: int, N: int, P: int):
+    """(r, w, k, v) float32 for `recurrence_scan` from act = [x: H P | B: G N | C: G N] (float32, after the convolution) and the step sizes'
+    columns of the fused product: dt = softplus(. + dt_bias), r = C and k = B of the head's group, v = dt x, w = exp(-exp(A_log) dt)."""
+    _need(act, "ssm_expand.act", torch.float32, 2)
+    T, dev = act.shape[0], act.device
+    if act.shape[1] != H * P + 2 * G * N or fused.tokens != T or fused.bias is not None or col_dt + H > fused.width or dt_bias.shape[0] != H or A_log.shape[0] != H:
+        raise KernelError("ssm_expand: shapes differ, or a bias is pending")
+    r, w, k = (torch.empty((T, H * N), dtype=torch.float32, device=dev) for _ in range(3))
+    v = torch.empty((T, H * P), dtype=torch.float32, device=dev)
+    _check(library().kestrel_ssm_expand(act.data_ptr(), fused.data.data_ptr(), fused.slices, fused.slice_stride, fused.width, int(col_dt),
+                                        dt_bias.data_ptr(), A_log.data_ptr(), r.data_ptr(), w.data_ptr(), k.data_ptr(), v.data_ptr(), T, H, G, N, P,
+                                        _stream()))
+    return r, w, k, v
+
+
+def ssm_out(o: torch.Tensor, act: torch.Tensor, D: torch.Tensor, fused: Partials, col_z: int, weight: torch.Tensor, eps: float, out: torch.Tensor,
+            H: int, G: int, N: int, P: int, parts: int) -> None:
+    """out = (o + D x) * silu(z), normed in ``parts`` equal parts of its columns, times ``weight``; x the first columns of ``act``, z the
+    columns of the fused product from ``col_z``."""
+    _need(o, "ssm_out.o", torch.float32, 2)
+    _need(act, "ssm_out.act", torch.float32, 2)
+    _need(out, "ssm_out.out", dims=2)
+    T, inner = o.shape
+    if inner != H * P or act.shape != (T, inner + 2 * G * N) or out.shape != o.shape or fused.tokens != T or fused.bias is not None or \
+            weight.shape[0] != inner or D.shape[0] != H or inner % parts or col_z + inner > fused.width:
+        raise KernelError("ssm_out: shapes differ, or a bias is pending")
+    _check(library().kestrel_ssm_out(o.data_ptr(), act.data_ptr(), D.data_ptr(), fused.data.data_ptr(), fused.slices, fused.slice_stride, fused.width,
+                                     int(col_z), weight.data_ptr(), float(eps), out.data_ptr(), _code(out, "ssm_out.out"), T, H, G, N, P, int(parts),
+                                     _stream()))
 
 
 # ---- retention: linear attention with a fixed decay per head -----------------------------------------

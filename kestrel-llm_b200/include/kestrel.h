@@ -149,6 +149,8 @@ KESTREL_API int kestrel_embed(const void *table, int dtype, const int *ids, floa
 KESTREL_API void kestrel_set_norm_warp_rows(int rows, int with_slices);   /* rows from which a norm that only reads the stream takes a warp a row (0: the default), and whether one that adds slices does too; for tests of both kernels */
 KESTREL_API int kestrel_add_rmsnorm(float *residual, const float *partial, int S, long long slice_stride, const float *bias, const int *rows, const float *w, float eps, void *out, int out_dtype, int R, int d, int write_back, kestrel_stream_t stream);
 KESTREL_API int kestrel_swiglu(const float *partial, int S, long long slice_stride, void *out, int out_dtype, int T, int ff, kestrel_stream_t stream);
+/* the same with the activation bounded where limit > 0: g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(1.702 g) (u + 1) */
+KESTREL_API int kestrel_gated_act(const float *partial, int S, long long slice_stride, float limit, void *out, int out_dtype, int T, int ff, kestrel_stream_t stream);
 /* rot_mode: 0 pairs dimension j with j + rot/2 (rotate-half), 1 pairs 2j with 2j + 1 (interleaved); rot_scale multiplies cos and sin */
 KESTREL_API int kestrel_attn_prepare(const float *partial, int S, long long slice_stride, const float *bias, const float *q_norm_w, const float *k_norm_w, float norm_eps, const float *inv_freq, int rot, int rot_mode, float rot_scale, const int *positions, const int *seq_of_token, const int *block_table, int table_stride, int page_size, void *k_cache, void *v_cache, void *q_out, int dtype, int T, int nq, int nkv, int hd, int write_kv, kestrel_stream_t stream);
 KESTREL_API int kestrel_reduce_partials(const float *partial, int S, long long slice_stride, const float *bias, void *out, int out_dtype, int T, int width, kestrel_stream_t stream);
@@ -172,6 +174,8 @@ KESTREL_API int kestrel_partial_columns_act_with(const float *p, int S, long lon
 KESTREL_API int kestrel_add_three(float *residual, const float *a, int Sa, long long stride_a, const float *b, int Sb, long long stride_b, const float *c, int Sc, long long stride_c, void *cast, int cast_dtype, int T, int d, kestrel_stream_t stream);
 /* x[t, i] *= sigmoid(sum of g's slices at [t, col0 + i] + bias[col0 + i]), i < n, in place in the storage type (bias may be NULL) */
 KESTREL_API int kestrel_gate_columns_mul(void *x, int dtype, const float *g, int S, long long slice_stride, int ld, int col0, const float *bias, int T, int n, kestrel_stream_t stream);
+/* the same times `scale`, into rows of ldo numbers; x is left as it is unless it is the output */
+KESTREL_API int kestrel_gate_columns_mul_to(const void *x, int dtype, const float *g, int S, long long slice_stride, int ld, int col0, const float *bias, float scale, void *out, long long ldo, int T, int n, kestrel_stream_t stream);
 /* x[t, :] += row[:] */
 KESTREL_API int kestrel_add_row(float *x, const float *row, int T, int d, kestrel_stream_t stream);
 /* out[t, :] = table[ids[t], :] * scale, float32 */
@@ -236,9 +240,8 @@ KESTREL_API int kestrel_head_gemm(const void *x, int ldx, const void *w, int ldw
 KESTREL_API int kestrel_head_gemm_strided(const void *x, int ldx, int hsx, const void *w, int ldw, int w_kn, void *out, int ldo, int hso, int out_f32, int dtype, int T, int H, int N, int K, kestrel_stream_t stream);
 KESTREL_API void kestrel_head_gemm_set_plain(int on);   /* 1: bfloat16 head-wise products take the CUDA-core kernel too; for tests of both */
 
-/* ---- gated delta rule with a decay per key channel (delta_rule.cu); state slot = [S: H d dv | tail: (taps - 1) C] float32 ---- */
-KESTREL_API int kestrel_delta_conv_silu(const float *partial, int S, long long slice_stride, int ld, const float *w, int taps, float *state, long long state_stride, long long tail_off, const int *seq_of_token, const int *cu_seqlens, const int *slots, float *out, int T, int nseq, int C, kestrel_stream_t stream);
-KESTREL_API int kestrel_delta_gates(const float *act, int C, const float *partial, int S, long long slice_stride, int ld, int col_beta, const float *a_part, int Sa, long long a_stride, const float *A_log, const float *dt_bias, float *qn, float *kn, float *decay, float *beta, int T, int H, int G, int d, kestrel_stream_t stream);
+/* ---- gated delta rule with a decay per key channel or per head (delta_rule.cu); a: the product a_part's columns from col_a, H d of them or (per_head) H; state slot = [S: H d dv | tail: (taps - 1) C] float32 ---- */
+KESTREL_API int kestrel_delta_gates(const float *act, int C, const float *partial, int S, long long slice_stride, int ld, int col_beta, const float *a_part, int Sa, long long a_stride, int a_ld, int col_a, int per_head, const float *A_log, const float *dt_bias, float *qn, float *kn, float *decay, float *beta, int T, int H, int G, int d, kestrel_stream_t stream);
 KESTREL_API int kestrel_delta_scan(const float *qn, const float *kn, const float *decay, const float *act, int C, int col_v, const float *beta, float *state, long long state_stride, const int *cu_seqlens, const int *slots, float *out, int nseq, int H, int G, int d, int dv, kestrel_stream_t stream);
 KESTREL_API int kestrel_delta_out(const float *o, const float *w, float eps, const float *g_part, int Sg, long long g_stride, void *out, int dtype, int T, int H, int dv, kestrel_stream_t stream);
 
@@ -259,6 +262,29 @@ KESTREL_API int kestrel_recurrence_scan(const float *r, const float *w, const fl
 KESTREL_API int kestrel_head_norm_gate(const float *o, const float *w, int w_stride, float eps, const float *g_part, int Sg, long long g_stride, int g_ld, int g_col0, void *out, int dtype, int T, int H, int dv, kestrel_stream_t stream);
 /* the same; w may be NULL (no weight); g_act 0: sigmoid of the gate columns, 1: silu */
 KESTREL_API int kestrel_head_norm_act(const float *o, const float *w, int w_stride, float eps, const float *g_part, int Sg, long long g_stride, int g_ld, int g_col0, int g_act, void *out, int dtype, int T, int H, int dv, kestrel_stream_t stream);
+/* the same times `scale`, into rows of ldo numbers */
+KESTREL_API int kestrel_head_norm_act_to(const float *o, const float *w, int w_stride, float eps, const float *g_part, int Sg, long long g_stride, int g_ld, int g_col0, int g_act, float scale, void *out, long long ldo, int dtype, int T, int H, int dv, kestrel_stream_t stream);
+/* o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t, then S_t = diag(w_t) S_(t-1) + k_t v_t^T; u [H, d] */
+KESTREL_API int kestrel_recurrence_scan_bonus(const float *r, const float *w, const float *k, const float *v, const float *u, float *state, long long state_stride, long long state_off, const int *cu_seqlens, const int *slots, float *out, int nseq, int H, int d, int dv, kestrel_stream_t stream);
+
+/* ---- short causal convolutions per channel (short_conv.cu): out[t, c] = act(sum_j w[c, j] u[t - (taps - 1) + j, c] + bias[c]), u the product's columns col0 .. col0 + C, act silu or none; inputs before the step from, and the last taps - 1 inputs to, the request's state slot (float32 [taps - 1, C] at tail_off) ---- */
+KESTREL_API int kestrel_short_conv(const float *partial, int S, long long slice_stride, int ld, int col0, const float *w, const float *bias, int taps, int silu, float *state, long long state_stride, long long tail_off, const int *seq_of_token, const int *cu_seqlens, const int *slots, void *out, int dtype, int T, int nseq, int C, kestrel_stream_t stream);
+/* the second half alone: the last taps - 1 inputs into the slot */
+KESTREL_API int kestrel_short_conv_tail(const float *partial, int S, long long slice_stride, int ld, int col0, int taps, float *state, long long state_stride, long long tail_off, const int *cu_seqlens, const int *slots, int nseq, int C, kestrel_stream_t stream);
+/* between a product [q: nq hd | k: nkv hd | ...] and attention whose values are its keys (attention_prepare_conv.cu): both through such a convolution, k as it is into the V pages, then norm per head with weights [hd], rotation of the first `rot` dimensions (rotate-half), q to q_out, k into the K pages */
+KESTREL_API int kestrel_attn_prepare_conv(const float *partial, int S, long long slice_stride, int ld, const float *conv_w, int taps, const float *q_norm_w, const float *k_norm_w, float norm_eps, const float *inv_freq, int rot, float rot_scale, float *state, long long state_stride, long long tail_off, const int *positions, const int *seq_of_token, const int *cu_seqlens, const int *slots, const int *block_table, int table_stride, int page_size, void *k_cache, void *v_cache, void *q_out, int dtype, int T, int nseq, int nq, int nkv, int hd, kestrel_stream_t stream);
+
+/* ---- a recurrence whose projections read each token blended with the one before it (time_mix.cu) ---- */
+/* out[s, t] = h[t] + (h[t - 1] - h[t]) mu[s], s < n; the token before a request's first one of this step is float32 [d] at state_off of its slot */
+KESTREL_API int kestrel_token_shift(const void *h, const float *mu, int n, const float *state, long long state_stride, long long state_off, const int *seq_of_token, const int *cu_seqlens, const int *slots, void *out, int dtype, int T, int d, kestrel_stream_t stream);
+/* r, k, v = the product's columns 0, n, 2 n; w = exp(-exp(z + w0)), z a product [T, n]; every request's last h goes into its slot */
+KESTREL_API int kestrel_time_mix_gates(const float *partial, int S, long long slice_stride, int ld, const float *z, int Sz, long long z_stride, const float *w0, float *r_out, float *k_out, float *v_out, float *w_out, int n, const void *h, int dtype, int d, float *state, long long state_stride, long long state_off, const int *seq_of_token, const int *cu_seqlens, const int *slots, int T, kestrel_stream_t stream);
+
+/* ---- a state-space mixer with a scalar decay per head (ssm.cu); act [T, H P + 2 G N] = x | B | C ---- */
+/* dt = softplus(column col_dt + h of the product + dt_bias): r = C, k = B of the head's group, v = dt x, w = exp(-exp(A_log) dt), as the scan of linear_recurrence.cu takes them */
+KESTREL_API int kestrel_ssm_expand(const float *act, const float *partial, int S, long long slice_stride, int ld, int col_dt, const float *dt_bias, const float *A_log, float *r_out, float *w_out, float *k_out, float *v_out, int T, int H, int G, int N, int P, kestrel_stream_t stream);
+/* out = (o + D x) silu(z), normed (eps) in `parts` equal parts of the H P columns, times w; z the product's columns from col_z */
+KESTREL_API int kestrel_ssm_out(const float *o, const float *act, const float *D, const float *partial, int S, long long slice_stride, int ld, int col_z, const float *w, float eps, void *out, int dtype, int T, int H, int G, int N, int P, int parts, kestrel_stream_t stream);
 /* ---- retention: a fixed decay per head (retention.cu) ---- */
 /* product columns [q: H d | k: H d | v: H dv | ...]: q, k turned by position (first `rot` dimensions, rotate-half), k times d^-1/2; q_out, k_out [T, H d], v_out [T, H dv] in `dtype`; w_out (may be NULL) [T, H d] = the head's decay */
 KESTREL_API int kestrel_retention_prepare(const float *partial, int S, long long slice_stride, int ld, const int *positions, const float *inv_freq, int rot, const float *decay, void *q_out, void *k_out, void *v_out, float *w_out, int dtype, int T, int H, int d, int dv, kestrel_stream_t stream);
@@ -331,6 +357,8 @@ KESTREL_API int kestrel_gemm_tc_act(const void *x, const void *w, void *out, int
 /* the same with a bias [N] (may be NULL) before the activation; act 6: xIELU with its two numbers in act_p (NULL for the others) */
 KESTREL_API int kestrel_gemm_tc_act_with(const void *x, const void *w, const float *bias, void *out, int act, const float *act_p, int T, int N, int K, long long ldx, long long ldw, long long ldo, kestrel_stream_t stream);
 KESTREL_API int kestrel_gemm_tc_swiglu_w(const void *x, const void *w, void *out, int T, int ff, int K, long long ldx, long long ldw, long long ldo, int weights_static, kestrel_stream_t stream);
+/* the same with the bounded activation of kestrel_gated_act where limit > 0 */
+KESTREL_API int kestrel_gemm_tc_gated_w(const void *x, const void *w, void *out, int T, int ff, int K, long long ldx, long long ldw, long long ldo, float limit, int weights_static, kestrel_stream_t stream);
 KESTREL_API int kestrel_gemm_tc_swiglu(const void *x, const void *w, void *out, int T, int ff, int K, long long ldx, long long ldw, long long ldo, kestrel_stream_t stream);
 /* the q, k, v product of many tokens with the prepare kernel's work in its epilogue (head size 128, rotate-half over the whole head); 0 done, 1 this form does not apply and nothing ran */
 KESTREL_API int kestrel_gemm_tc_qkv_prepare(const void *x, const void *w, int T, int K, long long ldx, long long ldw, const float *bias, const float *q_norm_w, const float *k_norm_w, float norm_eps, const float *inv_freq, int rot, int rot_mode, float rot_scale, const int *positions, const int *seq_of_token, const int *block_table, int table_stride, int page_size, void *k_cache, void *v_cache, void *q_out, int nq, int nkv, int hd, int write_kv, kestrel_stream_t stream);

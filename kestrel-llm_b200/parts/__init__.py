@@ -8,10 +8,12 @@ from .mlp import DenseMLP, GatedMLP
 from .attention_gated import GatedWindowAttention
 from .attention_latent import LatentAttention
 from .attention_differential import DifferentialAttention
-from .delta import ChannelDeltaMixer
+from .delta import ChannelDeltaMixer, HeadDeltaMixer
 from .recurrence import ForgetGateRecurrence, RemovalDeltaMixer
 from .retention import RetentionMixer
-from .parallel import ParallelMixers
+from .parallel import JoinedMixers, ParallelMixers
+from .ssm import StateSpaceMixer
+from .time_mix import TimeMixRecurrence
 from .moe import GroupRoutedExperts, RoutedExperts, SoftmaxRoutedExperts
 from .rglru import GatedDiagonalRecurrence
 from .side_input import TokenSideInput, TokenTable
@@ -24,4 +26,4 @@ __all__ = ["Block", "CacheSpec", "FeedForward", "FixedStateSpec", "Mixer", "Norm
            "GatedWindowAttention", "LatentAttention", "ChannelDeltaMixer", "RoutedExperts", "TokenSideInput", "TokenTable", "ParallelBlock",
            "CombinedSpec", "FrequencyScaling", "DenseMLP", "ForgetGateRecurrence", "RemovalDeltaMixer", "ParallelMixers", "SandwichBlock",
            "RampScaling", "GroupRoutedExperts", "GatedDiagonalRecurrence", "StreamRows", "DifferentialAttention",
-           "RetentionMixer", "SoftmaxRoutedExperts", "PostNormBlock"]
+           "RetentionMixer", "SoftmaxRoutedExperts", "PostNormBlock", "HeadDeltaMixer", "JoinedMixers", "StateSpaceMixer", "TimeMixRecurrence"]

@@ -27,7 +27,13 @@ a learned table [rows, heads] of terms added to the scores by the bucket of the 
 rows / 2, beyond that min(rows - 1, rows / 2 + floor(ln(n / (rows / 2)) / ln(far / (rows / 2)) * (rows - rows / 2))), made
 once on the host in float64 for the distances 0 .. far.  ``element_gate``: the gate is a number per ELEMENT of the
 concatenated heads (heads * v_head_dim logits of the mixer's input, further columns of the fused product) instead of
-one per head.
+one per head.  ``conv_taps`` > 0: q and k pass a causal convolution over time per channel, directly after their projection; its last
+conv_taps - 1 inputs are state of the request.  ``values_from_keys`` (with ``conv_taps``): there is no value projection, a key as it
+leaves the convolution - before norm and rotation - is its own value.
+
+`heads_into` runs everything in front of the output projection and leaves the gated heads, times a factor, in a place inside a
+wider matrix: for a container that projects the heads of two mixers by one product (``out_proj=False``: the mixer has no output
+projection of its own).
 
 Kernels: float32 and head sizes that are no multiples of 8 run on the plain kernel; bfloat16 on the
 ``mma.sync`` kernel of `ops.attention_window` (single-token steps share their keys out over CTAs),
@@ -42,7 +48,7 @@ from typing import List, Optional
 import torch
 
 from ..csrc import ops
-from .base import Mixer, PagedKVSpec, PositionEncoding, WeightSlot
+from .base import CacheSpec, CombinedSpec, FixedStateSpec, Mixer, PagedKVSpec, PositionEncoding, WeightSlot
 from .linear import Linear
 
 
@@ -61,7 +67,7 @@ class GatedWindowAttention(Mixer):
                  softcap: float = 0.0, distance_bias: bool = False, weighting: str = "softmax", head_bias: bool = False,
                  extra_names=None, position: Optional[PositionEncoding] = None, head_sink: bool = False,
                  out_bias: Optional[bool] = None, head_norm_weight: bool = False, q_temp=None, distance_table=None,
-                 element_gate: bool = False):
+                 element_gate: bool = False, conv_taps: int = 0, values_from_keys: bool = False, out_proj: bool = True):
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads are not a multiple of {kv_heads} kv heads")
         if max(head_dim, v_head_dim) > 256:
@@ -75,13 +81,24 @@ class GatedWindowAttention(Mixer):
         self.own_kv, self.head_gate = own_kv, head_gate
         self.prefix, self.names, self.dtype = prefix, names, dtype
         self.q_cols = heads * head_dim
-        self.kv_cols = kv_heads * (head_dim + v_head_dim) if own_kv else 0
+        self.conv_taps, self.values_from_keys = int(conv_taps), bool(values_from_keys)
+        if values_from_keys and v_head_dim != head_dim:
+            raise ValueError(f"values that are keys have their size: {v_head_dim} is not {head_dim}")
+        if bool(conv_taps) != bool(values_from_keys) or (conv_taps and (not own_kv or bias or v_norm or q_temp or head_gate or qk_norm != "head")):
+            raise ValueError("the convolution in front of attention is built for keys that are values, normed per head, without biases")
+        if not 0 <= conv_taps <= 9:
+            raise ValueError(f"{conv_taps} taps: the convolution takes 1 to 9")
+        self.kv_cols = kv_heads * (head_dim + (0 if values_from_keys else v_head_dim)) if own_kv else 0
         if element_gate and head_gate:
             raise ValueError("a gate per head or a gate per element, not both")
         self.element_gate = bool(element_gate)
         self.gate_cols = heads if head_gate else (heads * v_head_dim if element_gate else 0)
         self.proj = Linear(width, self.q_cols + self.kv_cols + self.gate_cols, dtype, device, bias=bias)
-        self.out = Linear(heads * v_head_dim, width, dtype, device, bias=bias if out_bias is None else bool(out_bias))
+        self.out_features = heads * v_head_dim
+        self.out = Linear(heads * v_head_dim, width, dtype, device, bias=bias if out_bias is None else bool(out_bias)) if out_proj else None
+        self.conv_w = torch.empty((self.q_cols + self.kv_cols, conv_taps), dtype=torch.float32, device=device) if conv_taps else None
+        self.state_off = 0         # where the mixer's own state starts in the request's slot (a container of two mixers moves it)
+        self.state_size = max(4, (conv_taps - 1) * (self.q_cols + self.kv_cols)) if conv_taps else 0
         self.rotation = position.rotary() if position is not None else None
         if self.rotation is not None and self.rotation.dim > head_dim:
             raise ValueError(f"{self.rotation.dim} rotated dimensions exceed the head size {head_dim}")
@@ -127,8 +144,9 @@ class GatedWindowAttention(Mixer):
                                 sink="sink", rel="rel")
         self.extra_names.update(extra_names or {})
 
-    def cache_spec(self) -> PagedKVSpec:
-        return PagedKVSpec(self.kv_heads, self.head_dim, self.cache_window, self.cache_keep_first, self.v_head_dim)
+    def cache_spec(self) -> CacheSpec:
+        pages = PagedKVSpec(self.kv_heads, self.head_dim, self.cache_window, self.cache_keep_first, self.v_head_dim)
+        return CombinedSpec(pages, FixedStateSpec((self.state_size,), torch.float32)) if self.state_size else pages
 
     def weight_slots(self) -> List[WeightSlot]:
         p, (nq, nk, nv, ng, no) = self.prefix, self.names
@@ -136,10 +154,15 @@ class GatedWindowAttention(Mixer):
         slots = [WeightSlot(p + nq, w[:self.q_cols])]
         if self.own_kv:
             k_end = self.q_cols + self.kv_heads * self.head_dim
-            slots += [WeightSlot(p + nk, w[self.q_cols:k_end]), WeightSlot(p + nv, w[k_end:self.q_cols + self.kv_cols])]
+            slots.append(WeightSlot(p + nk, w[self.q_cols:k_end]))
+            if not self.values_from_keys:
+                slots.append(WeightSlot(p + nv, w[k_end:self.q_cols + self.kv_cols]))
         if self.gate_cols:
             slots.append(WeightSlot(p + ng, w[self.q_cols + self.kv_cols:]))
-        slots.append(WeightSlot(p + no, self.out.weight))
+        if self.out is not None:
+            slots.append(WeightSlot(p + no, self.out.weight))
+        if self.conv_w is not None:
+            slots += [WeightSlot(p + nq + ".conv", self.conv_w[:self.q_cols], "bias"), WeightSlot(p + nk + ".conv", self.conv_w[self.q_cols:], "bias")]
         x = self.extra_names
         if self.proj.bias is not None:
             b = self.proj.bias
@@ -148,7 +171,7 @@ class GatedWindowAttention(Mixer):
                 k_end = self.q_cols + self.kv_heads * self.head_dim
                 slots += [WeightSlot(p + nk + x["bias"], b[self.q_cols:k_end], "bias"),
                           WeightSlot(p + nv + x["bias"], b[k_end:self.q_cols + self.kv_cols], "bias")]
-        if self.out.bias is not None:
+        if self.out is not None and self.out.bias is not None:
             slots.append(WeightSlot(p + no + x["bias"], self.out.bias, "bias"))
         if self.q_norm_w is not None:
             slots.append(WeightSlot(p + x["q_norm"], self.q_norm_w, "norm"))
@@ -165,6 +188,20 @@ class GatedWindowAttention(Mixer):
         return slots
 
     def forward(self, x: torch.Tensor, batch, cache, residual: Optional[torch.Tensor] = None) -> Optional[ops.Partials]:
+        a, fused = self._heads(x, batch, cache)
+        if self.element_gate:
+            ops.gate_columns_mul(a, fused, self.q_cols + self.kv_cols)
+        return self.out.forward(a, residual=residual)      # without bias and with many tokens the product adds itself to the stream
+
+    def heads_into(self, x: torch.Tensor, batch, cache, out: torch.Tensor, scale: float) -> None:
+        """The concatenated heads in front of the output projection, gated, times ``scale``, into ``out`` [T, heads * v_head_dim]."""
+        if not self.element_gate:
+            raise ValueError("heads are handed over by their gate per element")
+        a, fused = self._heads(x, batch, cache)
+        ops.gate_columns_mul(a, fused, self.q_cols + self.kv_cols, out=out, scale=scale)
+
+    def _heads(self, x: torch.Tensor, batch, cache):
+        """(heads' outputs [T, heads * v_head_dim] with a gate per head applied, the fused product)."""
         if cache.writable != self.own_kv:
             raise ValueError("a mixer with key and value projections writes its cache layer; one without reads another's")
         T = x.shape[0]
@@ -172,9 +209,20 @@ class GatedWindowAttention(Mixer):
         q = torch.empty((T, self.q_cols), dtype=self.dtype, device=x.device)
         gate = torch.empty((T, self.heads), dtype=torch.float32, device=x.device) if self.head_gate else None
         table = batch.block_table(cache.group)
+        if self.conv_w is not None:
+            ops.attn_prepare_conv(fused, self.conv_w, self.q_norm_w, self.k_norm_w, self.norm_eps, self.rotation, cache.state, self.state_off, batch,
+                                  table, cache.page_size, cache.k, cache.v, q, self.heads, self.kv_heads, self.head_dim)
+        else:
+            self._prepare(fused, batch, cache, table, q, gate)
+        return self._attend(q, gate, batch, cache, table), fused
+
+    def _prepare(self, fused, batch, cache, table, q, gate) -> None:
         ops.attn_prepare_ex(fused, self.q_norm_w, self.k_norm_w, self.qk_norm, self.norm_eps, batch.positions, batch.seq_of_token, table,
                             cache.page_size, cache.k, cache.v, q, gate, self.heads, self.kv_heads, self.head_dim, self.v_head_dim,
                             self.own_kv, v_norm=self.v_norm, rotation=self.rotation, q_temp=self.q_temp)
+
+    def _attend(self, q: torch.Tensor, gate, batch, cache, table) -> torch.Tensor:
+        T, x = q.shape[0], q
         score = self.score if self._scored else None
         a = torch.empty((T, self.heads * self.v_head_dim), dtype=self.dtype, device=x.device)
         G = self.heads // self.kv_heads
@@ -204,6 +252,4 @@ class GatedWindowAttention(Mixer):
         else:           # float32, and head sizes that are no multiple of 8
             ops.attention_plain_ex(q, cache.k, cache.v, batch.positions, batch.seq_of_token, table, cache.page_size, a, self.heads,
                                    self.kv_heads, self.head_dim, self.v_head_dim, self.window, self.keep_first, gate, self.scale, score)
-        if self.element_gate:
-            ops.gate_columns_mul(a, fused, self.q_cols + self.kv_cols)
-        return self.out.forward(a, residual=residual)      # without bias and with many tokens the product adds itself to the stream
+        return a

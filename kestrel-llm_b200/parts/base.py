@@ -26,10 +26,12 @@ class WeightSlot:
 
     ``dest`` may be a slice of a larger fused tensor (rows of a fused QKV matrix).  ``init`` is
     the distribution used by the random-weights mode: "linear" N(0, 0.02), "norm"
-    1 + N(0, 0.02), "bias" N(0, 0.02), "positive" |N(0, 0.02)|, "unit" uniform in [0, 1)."""
+    1 + N(0, 0.02), "bias" N(0, 0.02), "positive" |N(0, 0.02)|, "unit" uniform in [0, 1).  ``add`` is added to the stored
+    numbers once they are in place (a norm weight that a checkpoint keeps as its distance from one)."""
     name: str
     dest: torch.Tensor
     init: str = "linear"
+    add: float = 0.0
 
 
 @dataclass(frozen=True)

@@ -1,4 +1,4 @@
-"""A recurrent mixer: the gated delta rule with one decay per head and key channel.
+"""A recurrent mixer: the gated delta rule with one decay per head and key channel, or one per head.
 
 With h the mixer's input, G key heads of size d and H value heads of size dv (value head n
 uses key head n // (H / G)):
@@ -13,6 +13,9 @@ uses key head n // (H / G)):
 The state S and the last taps - 1 inputs of the convolutions live in the request's state slot,
 in float32; everything between the products and the output norm is float32.  W_q, W_k, W_v,
 W_b, W_a1 and W_g1 are one fused product.
+
+`ChannelDeltaMixer` is the layer above; `HeadDeltaMixer` has one decay per value head, a = exp(-exp(A_log[n]) softplus(W_a h + dt_bias))
+for all of a head's key channels, and the gate silu(W_g h) without the step through a low rank; everything it reads h with is one product.
 """
 from __future__ import annotations
 
@@ -73,7 +76,7 @@ class ChannelDeltaMixer(Mixer):
         H, G, d, dv = self.H, self.G, self.d, self.dv
         fused = self.in_proj.forward(x)
         act = torch.empty((T, self.C), dtype=f32, device=dev)
-        ops.delta_conv_silu(fused, self.conv_w, cache.state, self.tail_off, batch, act)
+        ops.short_conv(fused, self.conv_w, None, cache.state, self.tail_off, batch, act)
         a = self.a2.forward(ops.partial_columns(fused, self.col_a1, self.ra, self.dtype))
         g = self.g2.forward(ops.partial_columns(fused, self.col_g1, self.rg, self.dtype))
         qn = torch.empty((T, G * d), dtype=f32, device=dev)
@@ -85,4 +88,56 @@ class ChannelDeltaMixer(Mixer):
         ops.delta_scan(qn, kn, decay, act, self.col_v, beta, cache.state, batch, o, H, G, d, dv)
         y = torch.empty((T, H * dv), dtype=self.dtype, device=dev)
         ops.delta_out(o, self.norm_w, self.eps, g, y, H, dv)
+        return self.out.forward(y)
+
+
+class HeadDeltaMixer(Mixer):
+    graph_safe = True          # forward launches kernels over device tensors of the batch only
+
+    def __init__(self, width: int, heads: int, kv_heads: int, key_dim: int, value_dim: int, taps: int, norm_eps: float, dtype: torch.dtype,
+                 device, prefix: str):
+        if heads % kv_heads:
+            raise ValueError(f"{heads} value heads are not a multiple of {kv_heads} key heads")
+        if key_dim > 256:
+            raise ValueError(f"key size {key_dim}: the recurrence kernel holds up to 256 key channels a thread")
+        if not 1 <= taps <= 9:
+            raise ValueError(f"{taps} taps: the convolution kernel takes 1 to 9")
+        self.width, self.H, self.G, self.d, self.dv, self.taps = width, heads, kv_heads, key_dim, value_dim, taps
+        self.eps, self.dtype, self.prefix = float(norm_eps), dtype, prefix
+        qk, vv = kv_heads * key_dim, heads * value_dim
+        self.C = 2 * qk + vv                                   # channels that pass a convolution: q | k | v
+        self.col_v, self.col_g, self.col_beta, self.col_a = 2 * qk, self.C, self.C + vv, self.C + vv + heads
+        self.in_proj = Linear(width, self.C + vv + 2 * heads, dtype, device)
+        self.out = Linear(vv, width, dtype, device)
+        f32 = dict(dtype=torch.float32, device=device)
+        self.conv_w = torch.empty((self.C, taps), **f32)
+        self.A_log, self.dt_bias = torch.empty((heads,), **f32), torch.empty((heads,), **f32)
+        self.norm_w = torch.empty((value_dim,), **f32)
+        self.tail_off = (heads * key_dim * value_dim + 3) // 4 * 4     # the slot: S [H, d, dv], then the convolutions' tail [taps - 1, C]
+        self.state_size = (self.tail_off + (taps - 1) * self.C + 3) // 4 * 4
+
+    def cache_spec(self) -> FixedStateSpec:
+        return FixedStateSpec((self.state_size,), torch.float32)
+
+    def weight_slots(self) -> List[WeightSlot]:
+        p, w, qk = self.prefix, self.in_proj.weight, self.G * self.d
+        return [WeightSlot(p + "q", w[:qk]), WeightSlot(p + "k", w[qk:2 * qk]), WeightSlot(p + "v", w[2 * qk:self.C]),
+                WeightSlot(p + "g", w[self.col_g:self.col_beta]), WeightSlot(p + "b", w[self.col_beta:self.col_a]), WeightSlot(p + "a", w[self.col_a:]),
+                WeightSlot(p + "q.conv", self.conv_w[:qk], "bias"), WeightSlot(p + "k.conv", self.conv_w[qk:2 * qk], "bias"),
+                WeightSlot(p + "v.conv", self.conv_w[2 * qk:], "bias"), WeightSlot(p + "o", self.out.weight),
+                WeightSlot(p + "A_log", self.A_log, "bias"), WeightSlot(p + "dt_bias", self.dt_bias, "bias"), WeightSlot(p + "norm", self.norm_w, "norm")]
+
+    def forward(self, x: torch.Tensor, batch, cache) -> ops.Partials:
+        T, dev, f32 = x.shape[0], x.device, torch.float32
+        H, G, d, dv = self.H, self.G, self.d, self.dv
+        fused = self.in_proj.forward(x)
+        y = torch.empty((T, H * dv), dtype=self.dtype, device=dev)
+        act = torch.empty((T, self.C), dtype=f32, device=dev)
+        ops.short_conv(fused, self.conv_w, None, cache.state, self.tail_off, batch, act)
+        qn, kn = (torch.empty((T, G * d), dtype=f32, device=dev) for _ in range(2))
+        decay, beta = torch.empty((T, H * d), dtype=f32, device=dev), torch.empty((T, H), dtype=f32, device=dev)
+        ops.delta_gates(act, fused, self.col_beta, fused, self.A_log, self.dt_bias, qn, kn, decay, beta, H, G, d, col_a=self.col_a, per_head=True)
+        o = torch.empty((T, H * dv), dtype=f32, device=dev)
+        ops.delta_scan(qn, kn, decay, act, self.col_v, beta, cache.state, batch, o, H, G, d, dv)
+        ops.head_norm_gate(o, self.norm_w, self.eps, fused, self.col_g, y, H, dv, gate_act="silu")
         return self.out.forward(y)

@@ -1,5 +1,6 @@
 """Gated feed-forward: y = W_down (silu(W_gate x) * W_up x), silu(z) = z / (1 + exp(-z))
-(reference: st.c:8904-8914, st.c:3605-3607).  Gate and up are one fused product.
+(reference: st.c:8904-8914, st.c:3605-3607); with a ``limit`` L the bounded form W_down (g sigmoid(1.702 g) (u + 1)),
+g = min(W_gate x, L), u = clamp(W_up x, -L, L).  Gate and up are one fused product.
 """
 from __future__ import annotations
 
@@ -16,15 +17,19 @@ class GatedMLP(FeedForward):
     graph_safe = True
 
     def __init__(self, width: int, intermediate: int, dtype: torch.dtype, device, prefix: str,
-                 activation: str = "silu", names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), cut_few: bool = False):
+                 activation: str = "silu", names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), cut_few: bool = False,
+                 limit: float = 0.0):
         if activation != "silu":
             raise ValueError(f"activation '{activation}' has no kernel; only 'silu'")
         self.width, self.intermediate = width, intermediate
         self.prefix, self.names = prefix, names
         self.dtype = dtype
         self.cut_few = cut_few               # a narrow one beside routed experts: few tokens take the product cut along K
-        if cut_few:
-            self.emit = None                 # the step program has the uncut form
+        self.limit = float(limit)            # 0: none
+        if self.limit < 0:
+            raise ValueError("a bound on the gate and the up values is positive, or 0 for none")
+        if cut_few or self.limit:
+            self.emit = None                 # the step program has the uncut, unbounded form
         self.gate_up = Linear(width, 2 * intermediate, dtype, device)
         self.down = Linear(intermediate, width, dtype, device)
 
@@ -35,7 +40,8 @@ class GatedMLP(FeedForward):
                 WeightSlot(p + down, self.down.weight)]
 
     def forward(self, x: torch.Tensor, batch, residual: Optional[torch.Tensor] = None) -> Optional[ops.Partials]:
-        act = ops.gate_up_swiglu(x, self.gate_up.weight, self.intermediate, weights_static=True, cut_few=self.cut_few)
+        act = ops.gate_up_swiglu(x, self.gate_up.weight, self.intermediate, weights_static=True, cut_few=self.cut_few,
+                                 limit=self.limit)
         return self.down.forward(act, residual=residual)
 
     def emit(self, prog, x: int, residual: Optional[int]) -> int:

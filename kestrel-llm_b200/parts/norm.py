@@ -1,7 +1,7 @@
 """RMSNorm over the model width, fused with the residual add that precedes it.
 
 out = (x * 1/sqrt(mean(x^2) + eps)) * w with the sum and the scaling in float32
-(reference: st.c:8811-8827).
+(reference: st.c:8811-8827).  ``around_zero``: the checkpoint stores w - 1; the weight kept here is w.
 """
 from __future__ import annotations
 
@@ -16,13 +16,16 @@ from .base import Norm, WeightSlot
 class RMSNorm(Norm):
     graph_safe = True
 
-    def __init__(self, width: int, eps: float, device, weight_name: str):
+    def __init__(self, width: int, eps: float, device, weight_name: str, around_zero: bool = False):
         self.width = width
         self.eps = float(eps)
         self.weight = torch.empty((width,), dtype=torch.float32, device=device)
         self.weight_name = weight_name
+        self.around_zero = around_zero
 
     def weight_slots(self) -> List[WeightSlot]:
+        if self.around_zero:
+            return [WeightSlot(self.weight_name, self.weight, "bias", add=1.0)]
         return [WeightSlot(self.weight_name, self.weight, "norm")]
 
     def add_forward(self, residual: torch.Tensor, delta, out_dtype: torch.dtype,

@@ -81,6 +81,8 @@ def fill_from_folder(model, folder: ModelFolder) -> None:
         src = folder.tensor(present[name])
         with torch.no_grad():
             slot.dest.copy_(src.to(slot.dest.dtype) if src.dtype != slot.dest.dtype else src)
+            if slot.add:
+                slot.dest.add_(slot.add)
 
 
 def load_model(model_dir: str, dtype: str = "bfloat16", device="cuda:0"):

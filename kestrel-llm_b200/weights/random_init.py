@@ -79,6 +79,8 @@ def fill_random_(model, seed: int) -> None:
                 elif slot.init == "unit":
                     tmp.uniform_(0.0, 1.0, generator=gen)
                 slot.dest.copy_(tmp)
+                if slot.add:
+                    slot.dest.add_(slot.add)
             else:
                 rows = slot.dest.shape[0]
                 step = max(1, (1 << 26) // max(1, slot.dest[0].numel()))

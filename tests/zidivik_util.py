@@ -253,6 +253,8 @@ def load_part(part, W: Dict[str, np.ndarray]):
     for s in part.weight_slots():
         with torch.no_grad():
             s.dest.copy_(torch.from_numpy(W[s.name]).to(torch.bfloat16).to(s.dest.dtype))
+            if s.add:
+                s.dest.add_(s.add)
         names.add(s.name)
     return names
 
