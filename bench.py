@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--impl ours|reference]
     python bench.py --workload mix14b | 32b
-    python bench.py --workload zidivik | tidavik | toredra | korirax | tuganex [--size a|b]
+    python bench.py --workload zidivik | tidavik | toredra | korirax | tuganex | fasanex [--size a|b]
 
 Default run (the headline): decode tokens a second at batch 8, at batch 1 and 64, prefill of
 2,048 tokens, and the same decode through the Python entry point with host tokens in and out.
@@ -46,6 +46,10 @@ way, beside the Qwen3 dense decoder of equal width, heads, depth, vocabulary and
 `--workload tuganex`: the Tuganex decoder (differential attention, also on another layer's keys; retention; a dense feed-forward
 with xIELU and routed experts with a softmax router, groups, identity experts and a gated shared expert; norms on the
 sublayers' results only) the same way.
+
+`--workload fasanex`: the Fasanex decoder (a state-space mixer with a scalar decay per head; window attention whose values are its keys
+beside time mixing; a delta rule with one decay per head; a bounded gated feed-forward; twice-normed sublayers) the same way, beside the
+Qwen3 dense decoder of equal width, heads, depth, feed-forward, vocabulary and window.
 
 Timing: CUDA events on the launching stream around exactly K steps after W warm-up steps, with
 a synchronize on both sides.  Every step streams all weights (15 GB) and the live requests'
@@ -382,13 +386,37 @@ def tuganex_raw(z):
     return {"architecture": "Tuganex", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "max_positions": 8192, "layers": layers}
 
 
+FASANEX_SIZES = {
+    # width, attention heads / kv heads x size and window, time-mixing heads x size and decay rank, state-space heads x value size, state, groups,
+    # delta heads / key heads x key / value size, feed-forward, vocab
+    "a": dict(width=2048, heads=16, kv_heads=4, dim=128, window=1024, t_heads=32, t_dim=64, rank=64, s_heads=64, s_vdim=64, s_state=128, s_groups=8,
+              d_heads=16, d_kv=8, d_dim=128, d_vdim=128, ff=6144, vocab=32000),
+    "b": dict(width=4096, heads=32, kv_heads=8, dim=128, window=2048, t_heads=64, t_dim=64, rank=128, s_heads=128, s_vdim=64, s_state=128, s_groups=8,
+              d_heads=32, d_kv=16, d_dim=128, d_vdim=128, ff=12288, vocab=64000),
+}
+
+
+def fasanex_raw(z):
+    left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "conv": 4, "scale": z["dim"] ** -0.5, "softcap": 30.0,
+            "mask": {"size": z["window"]}, "rot": {"dims": z["dim"], "base": 500000.0, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+    par = {"left": left, "right": {"heads": z["t_heads"], "dim": z["t_dim"], "decay_rank": z["rank"]}, "left_scale": 0.8, "right_scale": 1.1}
+    ssm = {"heads": z["s_heads"], "vdim": z["s_vdim"], "state": z["s_state"], "groups": z["s_groups"], "norm_groups": z["s_groups"], "conv": 4}
+    dlt = {"heads": z["d_heads"], "kv_heads": z["d_kv"], "dim": z["d_dim"], "vdim": z["d_vdim"], "conv": 4}
+    mlp = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    layers = [{"type": "mamba2", "mixer": ssm, "mlp": mlp}, {"type": "parallel", "mixer": par, "mlp": mlp}, {"type": "delta", "mixer": dlt, "mlp": mlp},
+              {"type": "parallel", "mixer": par, "mlp": mlp}]
+    return {"architecture": "Fasanex", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 12.0}, "max_positions": 8192,
+            "layers": layers}
+
+
 def run_zidivik(args) -> int:
-    """Prefill and decode of the Zidivik, the Tidavik, the Toredra, the Korirax or the Tuganex decoder at real layer sizes, beside the Qwen3 dense decoder of equal size."""
+    """Prefill and decode of the Zidivik, the Tidavik, the Toredra, the Korirax, the Tuganex or the Fasanex decoder at real layer sizes, beside the Qwen3 dense decoder of equal size."""
     import numpy as np
     import torch
     from kestrel_llm_b200.config import EngineOptions, Qwen3Config, TidavikConfig, ToredraConfig, ZidivikConfig
     from kestrel_llm_b200.config.korirax_config import KoriraxConfig
     from kestrel_llm_b200.config.tuganex_config import TuganexConfig
+    from kestrel_llm_b200.config.fasanex_config import FasanexConfig
     from kestrel_llm_b200.config.registry import resolve_architecture
     from kestrel_llm_b200.csrc import ops
     from kestrel_llm_b200.engine import Engine, Entry
@@ -398,7 +426,8 @@ def run_zidivik(args) -> int:
     torch.cuda.set_device(0)
     tidavik, toredra, korirax = args.workload == "tidavik", args.workload == "toredra", args.workload == "korirax"
     tuganex = args.workload == "tuganex"
-    z = (TUGANEX_SIZES if tuganex else KORIRAX_SIZES if korirax else TOREDRA_SIZES if toredra else TIDAVIK_SIZES if tidavik else ZIDIVIK_SIZES)[args.size]
+    fasanex = args.workload == "fasanex"
+    z = (FASANEX_SIZES if fasanex else TUGANEX_SIZES if tuganex else KORIRAX_SIZES if korirax else TOREDRA_SIZES if toredra else TIDAVIK_SIZES if tidavik else ZIDIVIK_SIZES)[args.size]
     T, B, CTX = args.prefill_tokens, args.batch, 2048
     W, K = max(3, args.warmup), max(1, min(args.steps, 32))
     pk = peaks()
@@ -410,7 +439,8 @@ def run_zidivik(args) -> int:
                    "forget_gates", "removal_gates", "recurrence_scan", "head_norm_gate", "combine_normed", "add_gated_normed", "partial_columns_act",
                    "embed_add", "logit_scale_cap", "linear_act", "rglru_branches", "rglru_scan", "moe_route_sigmoid", "moe_experts_ungated",
                    "gate_columns_mul", "latent_rotate_queries", "add_row", "differential_combine", "retention_prepare", "retention_step", "retention_chunks",
-                   "moe_route_scored", "attention_tc_maps", "attention_window_maps", "attention_decode_maps", "post_norm_add", "embed_copy"]
+                   "moe_route_scored", "attention_tc_maps", "attention_window_maps", "attention_decode_maps", "post_norm_add", "embed_copy",
+                   "attn_prepare_conv", "token_shift", "linear_groups", "time_mix_gates", "recurrence_scan_bonus", "ssm_expand", "ssm_out"]
 
     def measure(cfg, label):
         model = resolve_architecture(cfg.architecture).build(cfg, torch.bfloat16, dev)
@@ -526,21 +556,47 @@ def run_zidivik(args) -> int:
                 "decode_batch": B, "decode_context": CTX, "decode_ms": round(1000 * dec, 4), "decode_tok_s": round(B / dec, 1),
                 "launches_per_decode_step": int(launches), "device_us_per_operation": split}
 
-    raw = tuganex_raw(z) if tuganex else korirax_raw(z) if korirax else toredra_raw(z) if toredra else tidavik_raw(z) if tidavik else zidivik_raw(z)
-    zc = (TuganexConfig if tuganex else KoriraxConfig if korirax else ToredraConfig if toredra else TidavikConfig if tidavik else ZidivikConfig).from_dict(raw)
+    raw = fasanex_raw(z) if fasanex else tuganex_raw(z) if tuganex else korirax_raw(z) if korirax else toredra_raw(z) if toredra else tidavik_raw(z) if tidavik else zidivik_raw(z)
+    zc = (FasanexConfig if fasanex else TuganexConfig if tuganex else KoriraxConfig if korirax else ToredraConfig if toredra else TidavikConfig if tidavik else ZidivikConfig).from_dict(raw)
     L = len(raw["layers"])
     dense_raw = dict(QWEN3_8B, num_hidden_layers=L, hidden_size=z["width"], num_attention_heads=z["heads"],
                      num_key_value_heads=z["kv_heads"], head_dim=z["vdim"] if tuganex else z["dim"],
                      intermediate_size=(z["ff"] * 2 // 3 + z["top"] * z["e_ff"] + z["shared"]) // 2 // 256 * 256 if tuganex else
                      (z["ff"] + (z["top"] * z["e_ff"] + z["shared"]) * 2 // 3) // 2 // 256 * 256 if korirax else
-                     z["ff"] * 2 // 3 if toredra else z["ff"] if tidavik else z["top"] * z["ff"],
+                     z["ff"] * 2 // 3 if toredra else z["ff"] if tidavik or fasanex else z["top"] * z["ff"],
                      vocab_size=z["vocab"], max_position_embeddings=8192)
-    if tidavik:                              # the dense model's layers look through the same window
+    if tidavik or fasanex:                   # the dense model's layers look through the same window
         dense_raw.update(sliding_window=z["window"], use_sliding_window=True, layer_types=["sliding_attention"] * L)
     qc = Qwen3Config.from_dict(dense_raw)
-    ours = measure(zc, "Tuganex" if tuganex else "Korirax" if korirax else "Toredra" if toredra else "Tidavik" if tidavik else "Zidivik")
-    dense = measure(qc, "Qwen3 dense, equal size" + (" and window" if tidavik else ""))
+    ours = measure(zc, "Fasanex" if fasanex else "Tuganex" if tuganex else "Korirax" if korirax else "Toredra" if toredra else "Tidavik" if tidavik else "Zidivik")
+    dense = measure(qc, "Qwen3 dense, equal size" + (" and window" if tidavik or fasanex else ""))
     clocks.close()
+    if fasanex:
+        D, H, G, d, ff = z["width"], z["heads"], z["kv_heads"], z["dim"], z["ff"]
+        inner, gn, tn, dq, dvv = z["s_heads"] * z["s_vdim"], z["s_groups"] * z["s_state"], z["t_heads"] * z["t_dim"], z["d_kv"] * z["d_dim"], z["d_heads"] * z["d_vdim"]
+        ssm_w = D * (2 * inner + 2 * gn + z["s_heads"]) + inner * D
+        par_w = D * (2 * H * d + G * d) + 4 * D * tn + z["rank"] * (D + tn) + (H * d + tn) * D
+        dlt_w = D * (2 * dq + 2 * dvv + 2 * z["d_heads"]) + dvv * D
+        active = ssm_w + 2 * par_w + dlt_w + L * 3 * ff * D
+        win = min(z["window"], T)
+        pairs = win * (win + 1) / 2 + (T - win) * win           # (query, key) pairs inside the window
+        state = z["s_heads"] * z["s_state"] * z["s_vdim"] + 2 * tn * z["t_dim"] + z["d_heads"] * z["d_dim"] * z["d_vdim"]
+        # products, attention, and the recurrences' three passes over their states a token
+        flops_prefill = 2.0 * T * active + 2 * 4.0 * H * d * pairs + 6.0 * T * state
+        cache_bytes = 2.0 * B * min(CTX, z["window"]) * 2 * G * 2 * d
+        rec = {"metric": f"Fasanex prefill tokens/s at size {args.size}, bf16, beside Qwen3 dense of equal size", "value": ours["prefill_tok_s"],
+               "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": W, "ms_per_step": ours["prefill_ms"], "higher_is_better": True,
+               "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "impl": "ours", "workload": "fasanex",
+               "data": "synthetic: random weights, uniform random token ids, cache of the context filled with random values",
+               "config": dict(z, layers=[l["type"] + "+" + l["mlp"]["kind"] for l in raw["layers"]], page_size=args.page_size, peaks=pk["source"],
+                              parallelism="single GPU"),
+               "fasanex": ours, "dense": dense,
+               "ratio_to_dense": {"prefill": round(ours["prefill_tok_s"] / dense["prefill_tok_s"], 3), "decode": round(ours["decode_tok_s"] / dense["decode_tok_s"], 3)},
+               "prefill_flops_frac_of_peak": round(flops_prefill / (ours["prefill_ms"] / 1000.0) / (pk["bf16_tflops"] * 1e12), 4),
+               "decode_bytes_frac_of_hbm": round((2.0 * (active + z["vocab"] * D) + 8.0 * B * state + cache_bytes) / (ours["decode_ms"] / 1000.0) / (pk["hbm_gbs"] * 1e9), 4),
+               "gpu_launches": ours["launches_per_decode_step"] * K, "clocks": clocks.summary()}
+        print(json.dumps(rec))
+        return 0
     if tuganex:
         D, H, G, d, dv, ff, n = z["width"], z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["ff"], z["experts"] + z["identity"]
         q_w, kv_w, o_w = D * H * 2 * d, D * G * (2 * d + dv), H * dv * D
@@ -671,10 +727,10 @@ def main() -> int:
     ap.add_argument("--page-size", type=int, default=16, help="tokens per cache page (default 16)")
     ap.add_argument("--context", type=int, default=CONTEXT, help="context length at which the decode steps end (default 4096)")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS, help="tokens of the prefill step (default 2048)")
-    ap.add_argument("--workload", default="decode8b", choices=["decode8b", "mix14b", "32b", "zidivik", "tidavik", "toredra", "korirax", "tuganex"],
-                    help="decode8b: the headline run; mix14b / 32b: whole workloads through the scheduler; zidivik / tidavik / toredra / korirax / tuganex: that decoder "
+    ap.add_argument("--workload", default="decode8b", choices=["decode8b", "mix14b", "32b", "zidivik", "tidavik", "toredra", "korirax", "tuganex", "fasanex"],
+                    help="decode8b: the headline run; mix14b / 32b: whole workloads through the scheduler; zidivik / tidavik / toredra / korirax / tuganex / fasanex: that decoder "
                          "at real layer sizes beside Qwen3 dense of equal size")
-    ap.add_argument("--size", default="a", choices=sorted(ZIDIVIK_SIZES), help="layer sizes of --workload zidivik / tidavik / toredra / korirax / tuganex")
+    ap.add_argument("--size", default="a", choices=sorted(ZIDIVIK_SIZES), help="layer sizes of --workload zidivik / tidavik / toredra / korirax / tuganex / fasanex")
     ap.add_argument("--requests", type=int, default=0, help="requests of a workload (0: 32 for mix14b, 16 for 32b)")
     ap.add_argument("--generate", type=int, default=0, help="tokens to generate per request of a workload (0: 256 / 128)")
     ap.add_argument("--step-tokens", type=int, default=2048,
@@ -686,7 +742,7 @@ def main() -> int:
     if args.gpus != 1:
         print(f"bench.py: this engine runs on ONE GPU; --gpus {args.gpus} is not supported (no multi-GPU path exists)")
         return 2
-    if args.workload in ("zidivik", "tidavik", "toredra", "korirax", "tuganex"):
+    if args.workload in ("zidivik", "tidavik", "toredra", "korirax", "tuganex", "fasanex"):
         return run_zidivik(args)
     if args.workload != "decode8b":
         return run_workload(args)
