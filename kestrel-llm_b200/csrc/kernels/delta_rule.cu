@@ -16,6 +16,7 @@
 //                 request was cut into steps or on the batch
 //   out_norm_gate o / sqrt(mean(o^2) + eps) * w * sigmoid(gate) per head, in the storage type
 #include "common.cuh"
+#include "recurrence_step.cuh"
 #include <math.h>
 
 // sum of a product's slices at (token, column)
@@ -244,4 +245,147 @@ KESTREL_API int kestrel_delta_out(const float *o, const float *w, float eps, con
     else
         return kestrel_fail(-2, "delta_out: unknown dtype %d", dtype);
     return kestrel_check_launch("delta_out");
+}
+
+// ---- one decay per head, a step of few tokens: everything between the fused product and the output product --------------------
+// columns [q: G d | k: G d | v: H dv] through the convolution, gate logits at col_g, beta and decay logits a head at col_beta, col_a
+template <typename T, int VEC, int ROWS>
+__global__ void __launch_bounds__(RST_THREADS)
+delta_head_step_kernel(const float *__restrict__ p, int S, size_t slice_stride, int ld, int col_g, int col_beta, int col_a, const float *__restrict__ conv_w,
+                       int taps, const float *__restrict__ A_log, const float *__restrict__ dt_bias, const float *__restrict__ norm_w, float eps,
+                       float *__restrict__ state, size_t state_stride, size_t tail_off, const int *__restrict__ cu_seqlens, const int *__restrict__ slots,
+                       T *__restrict__ out, int H, int G, int d, int dv) {
+    __shared__ float q_s[256], k_s[256], v_s[256], g_s[256], u_s[256], part_s[RST_THREADS * VEC], red[RST_THREADS / 32], sc[4];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, hk = h / (H / G), C = 2 * G * d + H * dv;
+    const int t0 = cu_seqlens[seq], t1 = cu_seqlens[seq + 1];
+    if (t0 == t1) return;
+    float *slot = state + (size_t)slots[seq] * state_stride, *Sg = slot + (size_t)h * d * dv;
+    const float *tail = slot + tail_off;
+    const RstLayout l = rst_layout<VEC>(dv);
+    float s[ROWS][VEC];
+    const bool mine = l.rg < l.groups;
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        const int i = l.rg + r * l.groups;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) s[r][e] = 0.f;
+        if (mine && i < d) rst_load<VEC>(s[r], Sg + (size_t)i * dv + l.c0);
+    }
+    for (int t = t0; t < t1; ++t) {
+        for (int u = tid; u < 2 * d + 2 * dv + 2; u += RST_THREADS) {
+            if (u < 2 * d + dv) {
+                const int c = u < d ? hk * d + u : (u < 2 * d ? (G + hk) * d + u - d : 2 * G * d + h * dv + u - 2 * d);
+                const float a = rst_conv(p, S, slice_stride, ld, c, conv_w, taps, tail, C, c, t0, t), y = a / (1.0f + expf(-a));
+                if (u < d) q_s[u] = y;
+                else if (u < 2 * d) k_s[u - d] = y;
+                else v_s[u - 2 * d] = y;
+            } else if (u < 2 * d + 2 * dv) {
+                const int i = u - 2 * d - dv;
+                g_s[i] = sum_slices(p, S, slice_stride, (size_t)t * ld + col_g + h * dv + i);
+            } else if (u == 2 * d + 2 * dv) {
+                sc[0] = 1.0f / (1.0f + expf(-sum_slices(p, S, slice_stride, (size_t)t * ld + col_beta + h)));
+            } else {
+                const float a = sum_slices(p, S, slice_stride, (size_t)t * ld + col_a + h) + dt_bias[h];
+                sc[1] = expf(-expf(A_log[h]) * (a > 20.f ? a : log1pf(expf(a))));
+            }
+        }
+        __syncthreads();
+        if (warp < 2) {                               // q's and k's unit factors
+            const float *x = warp == 0 ? q_s : k_s;
+            float ss = 0.f;
+            for (int i = lane; i < d; i += 32) ss = fmaf(x[i], x[i], ss);
+            ss = warp_sum(ss);
+            if (lane == 0) sc[2 + warp] = (1.0f / sqrtf(ss + 1e-6f)) * (warp == 0 ? 1.0f / sqrtf((float)d) : 1.0f);
+        }
+        __syncthreads();
+        const float beta = sc[0], dec = sc[1], qf = sc[2], kf = sc[3];
+        float acc[VEC];
+        if (mine) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+#pragma unroll
+            for (int r = 0; r < ROWS; ++r) {
+                const int i = l.rg + r * l.groups;
+                const float k = i < d ? k_s[i] : 0.f;
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) {
+                    s[r][e] *= dec;
+                    acc[e] = fmaf(s[r][e], k, acc[e]);
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) part_s[l.rg * dv + l.c0 + e] = acc[e];
+        }
+        __syncthreads();
+        if (tid < dv) {                               // dv <= RST_THREADS: a thread a value channel
+            float held = 0.f;
+            for (int r = 0; r < l.groups; ++r) held += part_s[r * dv + tid];
+            u_s[tid] = beta * (v_s[tid] - held * kf) * kf;      // times k's factor: the write is k_s * this
+        }
+        __syncthreads();
+        if (mine) {
+            float u[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) { acc[e] = 0.f; u[e] = u_s[l.c0 + e]; }
+#pragma unroll
+            for (int r = 0; r < ROWS; ++r) {
+                const int i = l.rg + r * l.groups;
+                const float k = i < d ? k_s[i] : 0.f, q = i < d ? q_s[i] : 0.f;
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) {
+                    s[r][e] = fmaf(k, u[e], s[r][e]);
+                    acc[e] = fmaf(s[r][e], q, acc[e]);
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) part_s[l.rg * dv + l.c0 + e] = acc[e];
+        }
+        __syncthreads();
+        float o = 0.f;
+        if (tid < dv)
+            for (int r = 0; r < l.groups; ++r) o += part_s[r * dv + tid];
+        o *= qf;
+        const float tot = rst_block_sum(o * o, red);
+        if (tid < dv) {
+            const float z = g_s[tid];
+            out[((size_t)t * H + h) * dv + tid] = from_f32<T>(o * (1.0f / sqrtf(tot / (float)dv + eps)) * norm_w[tid] * (z / (1.0f + expf(-z))));
+        }
+        __syncthreads();                              // the next token overwrites the shared rows
+    }
+    if (mine) {
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            const int i = l.rg + r * l.groups;
+            if (i < d) rst_store<VEC>(Sg + (size_t)i * dv + l.c0, s[r]);
+        }
+    }
+}
+
+// whether the kernel holds a head's state: rows of a thread
+static int dh_rows(int d, int dv, int vec) { return (d + RST_THREADS / (dv / vec) - 1) / (RST_THREADS / (dv / vec)); }
+
+KESTREL_API int kestrel_delta_head_step_takes(int d, int dv) { return d > 0 && dv > 0 && d <= 256 && dv <= 256 && dv % 4 == 0 && dh_rows(d, dv, 4) <= 32; }
+
+KESTREL_API int kestrel_delta_head_step(const float *partial, int S, long long slice_stride, int ld, int col_g, int col_beta, int col_a, const float *conv_w,
+                                        int taps, const float *A_log, const float *dt_bias, const float *norm_w, float eps, float *state,
+                                        long long state_stride, long long tail_off, const int *cu_seqlens, const int *slots, void *out, int dtype, int nseq,
+                                        int H, int G, int d, int dv, cudaStream_t stream) {
+    if (nseq == 0) return 0;
+    KESTREL_REQUIRE(nseq > 0 && nseq <= 65535 && S > 0 && H > 0 && G > 0 && H % G == 0 && kestrel_delta_head_step_takes(d, dv) && taps >= 1 && taps <= 9 &&
+                    tail_off >= (long long)H * d * dv && state_stride % 4 == 0 && ((uintptr_t)state & 15) == 0, "delta_head_step: bad sizes H=%d d=%d dv=%d", H, d, dv);
+    const int rows = dh_rows(d, dv, 4);
+#define DH_GO(TT, R) kestrel_launch(delta_head_step_kernel<TT, 4, R>, dim3(H, nseq), dim3(RST_THREADS), 0, stream, partial, S, (size_t)slice_stride, ld, col_g, \
+                                    col_beta, col_a, conv_w, taps, A_log, dt_bias, norm_w, eps, state, (size_t)state_stride, (size_t)tail_off, cu_seqlens, slots, \
+                                    (TT *)out, H, G, d, dv)
+#define DH_ROWS(TT) { if (rows <= 4) DH_GO(TT, 4); else if (rows <= 8) DH_GO(TT, 8); else if (rows <= 16) DH_GO(TT, 16); else DH_GO(TT, 32); }
+    if (dtype == KESTREL_F32) DH_ROWS(float)
+    else if (dtype == KESTREL_BF16) DH_ROWS(__nv_bfloat16)
+    else return kestrel_fail(-2, "delta_head_step: unknown dtype %d", dtype);
+#undef DH_ROWS
+#undef DH_GO
+    int rc = kestrel_check_launch("delta_head_step");
+    if (rc) return rc;
+    return kestrel_short_conv_tail(partial, S, slice_stride, ld, 0, taps, state, state_stride, tail_off, cu_seqlens, slots, nseq, 2 * G * d + H * dv, stream);
 }

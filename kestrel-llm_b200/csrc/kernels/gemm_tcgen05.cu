@@ -72,6 +72,7 @@ struct QkvPrepParams {
     int nq, nkv, write_kv;
     const float *act_p;              // ACT: the numbers of an activation that has any
     float act_limit;                 // the gated forms: the bound of gated_act.cuh (0: none, SiLU)
+    int group_rows;                  // PARTIAL: every group_rows features (whole tiles) have T token rows of their own in x; 0: all the same
 };
 
 // ------------------------------------------------------------------------------- kernel
@@ -79,7 +80,7 @@ template <int BN, int MODE>
 __global__ void __launch_bounds__(TC_THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                void *__restrict__ out, int T, int N, int K, int kb_per_split, long long slice_stride,
-               long long ldo, int stages, int up_row_offset, int early_w, float act_limit) {
+               long long ldo, int stages, int up_row_offset, int early_w, float act_limit, int group_rows) {
     pdl_launch_dependents();
     constexpr int A_TILES = MODE == TC_PARTIAL ? 1 : 2;
     constexpr uint32_t A_BYTES = TC_BM * TC_BK * 2;
@@ -100,6 +101,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 
     int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     int n0 = blockIdx.x * TC_BM, t0 = blockIdx.y * BN;
+    const int x0 = t0 + (group_rows ? n0 / group_rows * T : 0);     // grouped: every group_rows features have token rows of their own
     int total_kb = (K + TC_BK - 1) / TC_BK;
     int kb0 = blockIdx.z * kb_per_split;
     int num_kb = min(kb_per_split, total_kb - kb0);
@@ -144,7 +146,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             }
             pdl_wait();                               // the activations are the predecessor's output
             for (int kb = 0; kb < pre; ++kb)
-                tma_load_2d(base + (uint32_t)kb * STAGE_BYTES + A_TILES * A_BYTES, &map_x, full_bar(kb), (kb0 + kb) * TC_BK, t0);
+                tma_load_2d(base + (uint32_t)kb * STAGE_BYTES + A_TILES * A_BYTES, &map_x, full_bar(kb), (kb0 + kb) * TC_BK, x0);
             int stage = pre == stages ? 0 : pre;
             uint32_t phase = pre == stages ? 1 : 0;
             for (int kb = pre; kb < num_kb; ++kb) {
@@ -154,7 +156,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                 int kc = (kb0 + kb) * TC_BK;
                 tma_load_2d(sa, &map_w, full_bar(stage), kc, n0);
                 if (A_TILES == 2) tma_load_2d(sa + A_BYTES, &map_w, full_bar(stage), kc, up_row_offset + n0);
-                tma_load_2d(sa + A_TILES * A_BYTES, &map_x, full_bar(stage), kc, t0);
+                tma_load_2d(sa + A_TILES * A_BYTES, &map_x, full_bar(stage), kc, x0);
                 if (++stage == stages) { stage = 0; phase ^= 1; }
             }
         }
@@ -526,6 +528,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                 const int split = tile / tiles_nt, tw = tile % tiles_nt;       // a tile of the output and its slice of K
                 int n0 = tile_n(tw) * 256 + (int)rank * TC_BM;
                 int t0 = tile_t(tw) * TCP_BN + (int)rank * (TCP_BN / 2);
+                if (MODE == TC_PARTIAL && prep.group_rows) t0 += tile_n(tw) * 256 / prep.group_rows * T;
                 if (MODE == TC_SWIGLU_T) n0 = tile_n(tw) * TC_BM + (rank ? up_row_offset : 0);     // this rank's half of the N operand: gate rows, or up rows
                 if (MODE == TC_QKV_PREP) n0 = (2 * tile_n(tw) + (int)rank) * TC_BM;                  // one head's rows from each rank
                 const int kb_end = min(num_kb, (split + 1) * kb_per_split);
@@ -899,6 +902,7 @@ static bool tc_wide(int T, int N) { return g_wide && T > g_wide_min && T <= 128 
 // fill, the last tile's epilogue); the slices' float32 planes cost their write and their read
 // by the consumer as far as they no longer fit L2 (measured at 3,072 tokens: the down product in
 // three slices 227 + 89 us with its norm, whole 251 + 47).
+static int tc_splits(int T, int N, int K, bool wide);
 static long long pair_cost(int T, int N, int K, int s, long long *waves_out = nullptr) {
     const long long tiles = (long long)((N + 255) / 256) * ((T + TCP_BN - 1) / TCP_BN);
     const int total_kb = (K + TC_BK - 1) / TC_BK;
@@ -912,7 +916,9 @@ static long long pair_cost(int T, int N, int K, int s, long long *waves_out = nu
     return waves * (g_pair_overhead_kb + per) + planes / 2100000;
 }
 
-KESTREL_API int kestrel_gemm_tc_splits(int T, int N, int K) {
+KESTREL_API int kestrel_gemm_tc_splits(int T, int N, int K) { return tc_splits(T, N, K, tc_wide(T, N)); }
+
+static int tc_splits(int T, int N, int K, bool wide) {
     if (T > g_pair_min_tokens) {
         // many tokens on CTA pairs: tiles of 256 x 256 over the pairs of SMs; K is cut only where
         // that fills idle pairs
@@ -927,7 +933,6 @@ KESTREL_API int kestrel_gemm_tc_splits(int T, int N, int K) {
         return best;
     }
     int bn = T <= 16 ? 16 : T <= 32 ? 32 : T <= 64 ? 64 : T <= 128 ? 128 : 256;
-    const bool wide = tc_wide(T, N);
     long long tiles = (long long)((N + TC_BM - 1) / TC_BM) * ((T + bn - 1) / bn) / (wide ? 2 : 1);
     int total_kb = (K + TC_BK - 1) / TC_BK;
     int slots = kestrel_sms() * (bn <= 64 && !wide ? g_ctas_per_sm : 1);          // wider token tiles take an SM's shared memory alone
@@ -957,7 +962,7 @@ KESTREL_API int kestrel_gemm_tc_plan(const void *x, const void *w, int T, int N,
 
 template <int BN, int MODE>
 static int launch_tc(const CUtensorMap &mw, const CUtensorMap &mx, void *out, int T, int N, int K, int splits,
-                     long long slice_stride, long long ldo, int up_off, int early_w, float act_limit, cudaStream_t stream) {
+                     long long slice_stride, long long ldo, int up_off, int early_w, float act_limit, cudaStream_t stream, int group_rows = 0) {
     constexpr int A_TILES = MODE == TC_PARTIAL ? 1 : 2;
     constexpr int STAGE_BYTES = A_TILES * TC_BM * TC_BK * 2 + BN * TC_BK * 2;
     int total_kb = (K + TC_BK - 1) / TC_BK;
@@ -977,7 +982,7 @@ static int launch_tc(const CUtensorMap &mw, const CUtensorMap &mx, void *out, in
     }
     dim3 grid((N + TC_BM - 1) / TC_BM, (T + BN - 1) / BN, splits);
     if (grid.y > 65535) return kestrel_fail(-2, "gemm_tc: T=%d needs more than 65535 token tiles", T);
-    kestrel_launch(gemm_tc_kernel<BN, MODE>, dim3(grid), dim3(TC_THREADS), smem, stream, mw, mx, out, T, N, K, per, slice_stride, ldo, stages, up_off, early_w, act_limit);
+    kestrel_launch(gemm_tc_kernel<BN, MODE>, dim3(grid), dim3(TC_THREADS), smem, stream, mw, mx, out, T, N, K, per, slice_stride, ldo, stages, up_off, early_w, act_limit, group_rows);
     return kestrel_check_launch("gemm_tc");
 }
 
@@ -1125,6 +1130,49 @@ KESTREL_API int kestrel_gemm_tc_w(const void *x, const void *w, float *out, int 
     KESTREL_REQUIRE(splits >= 1 && splits <= total_kb && ((total_kb + splits - 1) / splits) * (splits - 1) < total_kb,
                     "gemm_tc: %d slices over %d k-blocks would leave a slice empty", splits, total_kb);
     return dispatch_tc<TC_PARTIAL>(x, w, out, T, N, N, K, ldx, ldw, ldo, splits, slice_stride, 0, weights_static ? 1 : 0, stream);
+}
+
+// Several products in one launch: rows [g group_rows, (g + 1) group_rows) of w (the last group may have fewer) meet token rows
+// [g T, (g + 1) T) of x; out float32 [splits, T, N] as above, N all rows of w.  _plan: 0 if this form does not take the sizes (a group that is
+// no whole number of feature tiles), else the number of K slices.
+KESTREL_API int kestrel_gemm_tc_grouped_plan(const void *x, const void *w, int T, int N, int K, int group_rows, long long ldx, long long ldw) {
+    if (T <= 0 || N <= 0 || group_rows <= 0 || !kestrel_gemm_tc_supported(x, w, T, N, K, ldx, ldw)) return 0;
+    const bool many = T > g_pair_min_tokens;
+    if (group_rows % (many ? 256 : TC_BM) != 0 || (many && (!g_pairs || !g_persistent))) return 0;
+    return tc_splits(T, N, K, false);
+}
+
+KESTREL_API int kestrel_gemm_tc_grouped(const void *x, const void *w, float *out, int T, int N, int K, int group_rows, long long ldx, long long ldw,
+                                        long long ldo, int splits, long long slice_stride, int weights_static, cudaStream_t stream) {
+    if (T == 0) return 0;
+    KESTREL_REQUIRE(kestrel_gemm_tc_grouped_plan(x, w, T, N, K, group_rows, ldx, ldw) > 0, "gemm_tc_grouped: sizes T=%d N=%d K=%d in groups of %d", T, N, K, group_rows);
+    const int total_kb = (K + TC_BK - 1) / TC_BK, groups = (N + group_rows - 1) / group_rows;
+    KESTREL_REQUIRE(splits >= 1 && splits <= total_kb && ((total_kb + splits - 1) / splits) * (splits - 1) < total_kb,
+                    "gemm_tc_grouped: %d slices over %d k-blocks would leave a slice empty", splits, total_kb);
+    CUtensorMap mw, mx;
+    int rc = kestrel_tensor_map_bf16(&mw, w, N, K, ldw, TC_BM);
+    if (rc) return rc;
+    if (T > g_pair_min_tokens) {
+        rc = kestrel_tensor_map_bf16(&mx, x, groups * T, K, ldx, TCP_BN / 2);
+        if (rc) return rc;
+        QkvPrepParams prep = {};
+        prep.group_rows = group_rows;
+        rc = launch_tc_pair<TC_PARTIAL>(mw, mx, out, T, N, K, ldo, 0, 0, splits, slice_stride, stream, prep);
+        return rc > 0 ? kestrel_fail(-3, "gemm_tc_grouped: CTA pairs cannot be scheduled here") : rc;
+    }
+    const int bn = T <= 16 ? 16 : T <= 32 ? 32 : T <= 64 ? 64 : T <= 128 ? 128 : 256;
+    rc = kestrel_tensor_map_bf16(&mx, x, groups * T, K, ldx, bn);
+    if (rc) return rc;
+    const int early = weights_static ? 1 : 0;
+#define TG_CASE(B) return launch_tc<B, TC_PARTIAL>(mw, mx, out, T, N, K, splits, slice_stride, ldo, 0, early, 0.f, stream, group_rows)
+    switch (bn) {
+        case 16: TG_CASE(16);
+        case 32: TG_CASE(32);
+        case 64: TG_CASE(64);
+        case 128: TG_CASE(128);
+        default: TG_CASE(256);
+    }
+#undef TG_CASE
 }
 
 // The same for a w that the preceding kernel may have written.

@@ -2,6 +2,8 @@
 //
 //   residual[t] += y / sqrt(mean(y^2) + eps) * w,     copy[t] = residual[t] in the storage type (where a copy is given)
 //
+// or, with a second weight, copy[t] = the norm of the new residual[t]: the input of the sublayer that follows.
+//
 // with y either a product (float32 slices in ascending order, plus a bias) or the sum of a routed feed-forward that was never
 // written out (`MoeSource`): the chosen experts' weighted rows in the order of choice, the identity experts' weights times
 // the input row, and an expert that every token takes times its gate.  A block takes a row, its threads the row's float4s; the
@@ -53,7 +55,8 @@ __device__ __forceinline__ void pn_store(__nv_bfloat16 *p, const float4 v) {
 
 template <typename T, int NV, typename Source>
 __global__ void __launch_bounds__(PN_MAX_THREADS)
-post_norm_kernel(float *__restrict__ residual, const Source src, const float *__restrict__ w, float eps, T *__restrict__ copy, int d) {
+post_norm_kernel(float *__restrict__ residual, const Source src, const float *__restrict__ w, float eps, T *__restrict__ copy,
+                 const float *__restrict__ next_w, float next_eps, int d) {
     constexpr bool MOE = sizeof(Source) == sizeof(MoeSource);
     pdl_launch_dependents();
     __shared__ float red[PN_MAX_THREADS / 32];
@@ -147,16 +150,39 @@ post_norm_kernel(float *__restrict__ residual, const Source src, const float *__
         x[c].z += v[c].z * mul * g[c].z;
         x[c].w += v[c].w * mul * g[c].w;
         pn_store(residual + (size_t)t * d + i, x[c]);
-        if (copy) pn_store(copy + (size_t)t * d + i, x[c]);
+        if (copy && !next_w) pn_store(copy + (size_t)t * d + i, x[c]);
+    }
+    if (!next_w) return;
+    ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {
+        const int i = 4 * (tid + c * nt);
+        if (i >= d) continue;
+        g[c] = pn_load(next_w + i);
+        ss = fmaf(x[c].x, x[c].x, fmaf(x[c].y, x[c].y, fmaf(x[c].z, x[c].z, fmaf(x[c].w, x[c].w, ss))));
+    }
+    ss = warp_sum(ss);
+    __syncthreads();                                  // everyone has read the first sums
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    tot = 0.f;
+    for (int k = 0; k < nt / 32; ++k) tot += red[k];
+    const float mul2 = 1.0f / sqrtf(tot / (float)d + next_eps);
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {
+        const int i = 4 * (tid + c * nt);
+        if (i >= d) continue;
+        pn_store(copy + (size_t)t * d + i, make_float4(x[c].x * mul2 * g[c].x, x[c].y * mul2 * g[c].y, x[c].z * mul2 * g[c].z, x[c].w * mul2 * g[c].w));
     }
 }
 
 template <typename T, typename Source>
-static int pn_launch(float *residual, const Source &src, const float *w, float eps, T *copy, int n_tokens, int d, cudaStream_t stream) {
+static int pn_launch(float *residual, const Source &src, const float *w, float eps, T *copy, int n_tokens, int d, cudaStream_t stream,
+                     const float *next_w = nullptr, float next_eps = 0.f) {
     int nt = (d / 4 + 31) / 32 * 32;
     if (nt > PN_MAX_THREADS) nt = PN_MAX_THREADS;
     const int nv = (d / 4 + nt - 1) / nt;
-#define PN_CASE(N) kestrel_launch(post_norm_kernel<T, N, Source>, dim3(n_tokens), dim3(nt), 0, stream, residual, src, w, eps, copy, d)
+#define PN_CASE(N) kestrel_launch(post_norm_kernel<T, N, Source>, dim3(n_tokens), dim3(nt), 0, stream, residual, src, w, eps, copy, next_w, next_eps, d)
     if (nv <= 1) PN_CASE(1);
     else if (nv <= 2) PN_CASE(2);
     else if (nv <= 4) PN_CASE(4);
@@ -176,6 +202,17 @@ KESTREL_API int kestrel_post_norm_add(float *residual, const float *y, int S, lo
     if (dtype == KESTREL_F32) return pn_launch<float>(residual, src, w, eps, (float *)copy, T, d, stream);
     if (dtype == KESTREL_BF16) return pn_launch<__nv_bfloat16>(residual, src, w, eps, (__nv_bfloat16 *)copy, T, d, stream);
     return kestrel_fail(-2, "post_norm_add: unknown dtype %d", dtype);
+}
+
+// copy[t] = the norm of the new residual[t] with the weight next_w
+KESTREL_API int kestrel_post_norm_add_norm(float *residual, const float *y, int S, long long stride, const float *bias, const float *w, float eps,
+                                           const float *next_w, float next_eps, void *copy, int dtype, int T, int d, cudaStream_t stream) {
+    if (T == 0) return 0;
+    KESTREL_REQUIRE(T > 0 && S > 0 && kestrel_post_norm_takes(d) && stride % 4 == 0 && next_w && copy, "post_norm_add_norm: bad sizes T=%d d=%d", T, d);
+    const ProductSource src = {y, S, (size_t)stride, bias};
+    if (dtype == KESTREL_F32) return pn_launch<float>(residual, src, w, eps, (float *)copy, T, d, stream, next_w, next_eps);
+    if (dtype == KESTREL_BF16) return pn_launch<__nv_bfloat16>(residual, src, w, eps, (__nv_bfloat16 *)copy, T, d, stream, next_w, next_eps);
+    return kestrel_fail(-2, "post_norm_add_norm: unknown dtype %d", dtype);
 }
 
 KESTREL_API int kestrel_post_norm_add_moe(float *residual, const float *y, const int *pair_row, const int *ids, const float *weights, int top, int experts,

@@ -7,6 +7,7 @@
 //   scan          linear_recurrence.cu, the form that reads the old state with a bonus for the token's own write
 //   (output)      head_norm_act: per-head norm, weight, silu of the gate's product
 #include "common.cuh"
+#include "recurrence_step.cuh"
 #include <math.h>
 
 template <typename T> struct TmVec;
@@ -119,4 +120,95 @@ KESTREL_API int kestrel_time_mix_gates(const float *partial, int S, long long sl
     else return kestrel_fail(-2, "time_mix_gates: unknown dtype %d", dtype);
 #undef TG_GO
     return kestrel_check_launch("time_mix_gates");
+}
+
+// ---- a step of few tokens: state, read-out, norm, gate of a (request, head); and the request's last h into its slot ------------
+template <typename T, int VEC>
+__global__ void __launch_bounds__(RST_THREADS)
+time_mix_step_kernel(const float *__restrict__ p, int S, size_t slice_stride, int ld, const float *__restrict__ z, int Sz, size_t z_stride,
+                     const float *__restrict__ w0, const float *__restrict__ u, const float *__restrict__ norm_w, float eps, float scale,
+                     const T *__restrict__ hrow, int width, float *__restrict__ state, size_t state_stride, size_t state_off, size_t last_off,
+                     const int *__restrict__ cu_seqlens, const int *__restrict__ slots, T *__restrict__ out, long long ldo, int H, int d) {
+    __shared__ float r_s[256], k_s[256], v_s[256], g_s[256], w_s[256], ru_s[256], part_s[RST_THREADS * VEC], red[RST_THREADS / 32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, n = H * d;
+    const int t0 = cu_seqlens[seq], t1 = cu_seqlens[seq + 1];
+    if (t0 == t1) return;
+    float *slot = state + (size_t)slots[seq] * state_stride, *Sg = slot + state_off + (size_t)h * d * d;
+    const RstLayout l = rst_layout<VEC>(d);
+    for (int t = t0; t < t1; ++t) {
+        const size_t row = (size_t)t * ld + (size_t)h * d;
+        for (int i = tid; i < 4 * d; i += RST_THREADS) {
+            const int what = i / d, c = i % d;
+            const float x = sum_slices(p, S, slice_stride, row + (size_t)what * n + c);
+            (what == 0 ? r_s : what == 1 ? k_s : what == 2 ? v_s : g_s)[c] = x;
+        }
+        for (int c = tid; c < d; c += RST_THREADS)
+            w_s[c] = expf(-expf(sum_slices(z, Sz, z_stride, (size_t)t * n + (size_t)h * d + c) + w0[(size_t)h * d + c]));
+        __syncthreads();
+        float bonus = 0.f;                            // (r . (u k)) times v: the token's own write
+        for (int c = tid; c < d; c += RST_THREADS) bonus = fmaf(r_s[c] * u[(size_t)h * d + c], k_s[c], bonus);
+        bonus = rst_block_sum(bonus, red);
+        if (l.rg < l.groups) {
+            float acc[VEC], v[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) { acc[e] = 0.f; v[e] = v_s[l.c0 + e]; }
+            for (int i0 = l.rg; i0 < d; i0 += 8 * l.groups) {          // eight rows' loads in flight
+                float s[8][VEC];
+#pragma unroll
+                for (int r = 0; r < 8; ++r) {
+                    const int i = i0 + r * l.groups;
+                    if (i < d) rst_load<VEC>(s[r], Sg + (size_t)i * d + l.c0);
+                }
+#pragma unroll
+                for (int r = 0; r < 8; ++r) {
+                    const int i = i0 + r * l.groups;
+                    if (i >= d) continue;
+                    const float k = k_s[i], q = r_s[i], w = w_s[i];
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        acc[e] = fmaf(s[r][e], q, acc[e]);
+                        s[r][e] = fmaf(w, s[r][e], k * v[e]);
+                    }
+                    rst_store<VEC>(Sg + (size_t)i * d + l.c0, s[r]);
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) part_s[l.rg * d + l.c0 + e] = acc[e];
+        }
+        __syncthreads();
+        float o = 0.f;
+        if (tid < d) {                                // d <= RST_THREADS: a thread a value channel
+            for (int r = 0; r < l.groups; ++r) o += part_s[r * d + tid];
+            o = fmaf(bonus, v_s[tid], o);
+        }
+        const float tot = rst_block_sum(o * o, red);
+        if (tid < d) {
+            const float g = g_s[tid];
+            out[(size_t)t * ldo + (size_t)h * d + tid] =
+                from_f32<T>(o * (1.0f / sqrtf(tot / (float)d + eps)) * norm_w[(size_t)h * d + tid] * (g / (1.0f + expf(-g))) * scale);
+        }
+        __syncthreads();                              // the next token overwrites the shared rows
+    }
+    float *last = slot + last_off;                    // the heads share the row out
+    for (int i = h * RST_THREADS + tid; i < width; i += H * RST_THREADS) last[i] = to_f32<T>(hrow[(size_t)(t1 - 1) * width + i]);
+}
+
+KESTREL_API int kestrel_time_mix_step(const float *partial, int S, long long slice_stride, int ld, const float *z, int Sz, long long z_stride, const float *w0,
+                                      const float *u, const float *norm_w, float eps, float scale, const void *h, int width, float *state,
+                                      long long state_stride, long long state_off, long long last_off, const int *cu_seqlens, const int *slots, void *out,
+                                      long long ldo, int dtype, int nseq, int H, int d, cudaStream_t stream) {
+    if (nseq == 0) return 0;
+    KESTREL_REQUIRE(nseq > 0 && nseq <= 65535 && S > 0 && Sz > 0 && H > 0 && d > 0 && d <= 256 && ld >= 4 * H * d && width > 0 && state_off >= 0 &&
+                    last_off >= state_off + (long long)H * d * d, "time_mix_step: bad sizes H=%d d=%d", H, d);
+    const bool vec = d % 4 == 0 && state_stride % 4 == 0 && state_off % 4 == 0 && ((uintptr_t)state & 15) == 0;
+#define TS_GO(TT, V) kestrel_launch(time_mix_step_kernel<TT, V>, dim3(H, nseq), dim3(RST_THREADS), 0, stream, partial, S, (size_t)slice_stride, ld, z, Sz, \
+                                    (size_t)z_stride, w0, u, norm_w, eps, scale, (const TT *)h, width, state, (size_t)state_stride, (size_t)state_off, \
+                                    (size_t)last_off, cu_seqlens, slots, (TT *)out, ldo, H, d)
+    if (dtype == KESTREL_F32) { if (vec) TS_GO(float, 4); else TS_GO(float, 1); }
+    else if (dtype == KESTREL_BF16) { if (vec) TS_GO(__nv_bfloat16, 4); else TS_GO(__nv_bfloat16, 1); }
+    else return kestrel_fail(-2, "time_mix_step: unknown dtype %d", dtype);
+#undef TS_GO
+    return kestrel_check_launch("time_mix_step");
 }

@@ -161,6 +161,17 @@ class StreamCopy:
         self.data = data
 
 
+class NormedStream(StreamCopy):
+    """The residual stream after a norm, in the storage type, handed to the block that starts with that very norm (``norm``, the object):
+    nothing is left to add, and the norm is done."""
+
+    __slots__ = ("norm",)
+
+    def __init__(self, data: torch.Tensor, norm):
+        super().__init__(data)
+        self.norm = norm
+
+
 def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
     """out[t] = table[ids[t]] widened to float32, times ``scale``."""
     _need(table, "embed.table", dims=2)
@@ -487,29 +498,38 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None,
     return out
 
 
-def linear_groups(x: torch.Tensor, w: torch.Tensor, groups: int) -> Partials:
-    """``groups`` products of equal size over inputs of their own: columns [s n, (s + 1) n) of the result are x[s] times rows
-    [s n, (s + 1) n) of w, transposed; x [>= groups, T, K] contiguous, w [groups n, K].  The weights are a model's (`gemm_tc`)."""
+def linear_groups(x: torch.Tensor, w: torch.Tensor, group_rows: int) -> Partials:
+    """Products over inputs of their own, side by side: columns [s n, (s + 1) n) of the result, n = ``group_rows``, are x[s] times rows
+    [s n, (s + 1) n) of w, transposed; x [groups, T, K] contiguous, w [N, K], the last group may have fewer rows.  One launch where the
+    tensor-core product takes the groups, a launch a group otherwise.  The weights are a model's (`gemm_tc`)."""
     _need(x, "linear_groups.x", dims=3)
     _need(w, "linear_groups.w", x.dtype, 2)
-    T, K = x.shape[1:]
+    G, T, K = x.shape
     N = w.shape[0]
-    n = N // groups
-    if x.shape[0] < groups or w.shape[1] != K or N != groups * n:
-        raise KernelError(f"linear_groups: x {tuple(x.shape)}, w {tuple(w.shape)}, {groups} groups")
+    if w.shape[1] != K or not (G - 1) * group_rows < N <= G * group_rows:
+        raise KernelError(f"linear_groups: x {tuple(x.shape)}, w {tuple(w.shape)}, groups of {group_rows} rows")
     lib = library()
-    plan = lib.kestrel_gemm_tc_plan(x.data_ptr(), w.data_ptr(), T, n, K, K, w.stride(0)) if x.dtype == torch.bfloat16 else 0
-    if plan > 0 and (T * K * x.element_size()) % 16 == 0 and (n * w.stride(0) * w.element_size()) % 16 == 0:
-        out = torch.empty((plan, T, N), dtype=torch.float32, device=x.device)
-        for s in range(groups):
-            _check(lib.kestrel_gemm_tc_w(x[s].data_ptr(), w[s * n:].data_ptr(), out[0, 0, s * n:].data_ptr(), T, n, K, K, w.stride(0), N, plan, T * N, 1,
-                                         _stream()))
+    bf16 = x.dtype == torch.bfloat16
+    S = lib.kestrel_gemm_tc_grouped_plan(x.data_ptr(), w.data_ptr(), T, N, K, int(group_rows), K, w.stride(0)) if bf16 and linear_groups_fused else 0
+    if S > 0:
+        out = torch.empty((S, T, N), dtype=torch.float32, device=x.device)
+        _check(lib.kestrel_gemm_tc_grouped(x.data_ptr(), w.data_ptr(), out.data_ptr(), T, N, K, int(group_rows), K, w.stride(0), N, S, T * N, 1, _stream()))
         return Partials(out)
-    out = torch.empty((1, T, N), dtype=torch.float32, device=x.device)
-    for s in range(groups):
-        _check(lib.kestrel_gemm_plain(x[s].data_ptr(), w[s * n:].data_ptr(), out[0, 0, s * n:].data_ptr(), _code(x, "linear_groups.x"), T, n, K, K,
-                                      w.stride(0), N, _stream()))
+    parts = [(s, s * group_rows, min(group_rows, N - s * group_rows)) for s in range(G)]
+    # every group in the same number of slices, the one that suits the first
+    S = lib.kestrel_gemm_tc_plan(x.data_ptr(), w.data_ptr(), T, group_rows, K, K, w.stride(0)) if bf16 else 0
+    ok = S > 0 and all(lib.kestrel_gemm_tc_supported(x[s].data_ptr(), w[n0:].data_ptr(), T, n, K, K, w.stride(0)) for s, n0, n in parts)
+    out = torch.empty((S if ok else 1, T, N), dtype=torch.float32, device=x.device)
+    for s, n0, n in parts:
+        if ok:
+            _check(lib.kestrel_gemm_tc_w(x[s].data_ptr(), w[n0:].data_ptr(), out[0, 0, n0:].data_ptr(), T, n, K, K, w.stride(0), N, S, T * N, 1, _stream()))
+        else:
+            _check(lib.kestrel_gemm_plain(x[s].data_ptr(), w[n0:].data_ptr(), out[0, 0, n0:].data_ptr(), _code(x, "linear_groups.x"), T, n, K, K,
+                                          w.stride(0), N, _stream()))
     return Partials(out)
+
+
+linear_groups_fused = True       # tests switch the one-launch form off to hold both forms against each other
 
 
 def linear_add_into(x: torch.Tensor, w: torch.Tensor, residual: torch.Tensor) -> bool:
@@ -957,6 +977,25 @@ def post_norm_add(residual: torch.Tensor, y, weight: torch.Tensor, eps: float, c
         raise KernelError("post_norm_add: the bias does not fit the row")
     _check(lib.kestrel_post_norm_add(residual.data_ptr(), y.data.data_ptr(), y.slices, y.slice_stride, _p(y.bias), weight.data_ptr(), float(eps),
                                      _p(copy), _code(copy, "post_norm_add.copy") if copy is not None else F32, T, d, _stream()))
+
+
+def post_norm_add_norm(residual: torch.Tensor, y: Partials, weight: torch.Tensor, eps: float, next_weight: torch.Tensor, next_eps: float,
+                       out: torch.Tensor) -> None:
+    """residual += y / sqrt(mean(y^2) + eps) * weight over the row, then out = the norm of the new residual with ``next_weight``."""
+    _need(residual, "post_norm_add_norm.residual", torch.float32, 2)
+    _need(weight, "post_norm_add_norm.weight", torch.float32, 1)
+    _need(next_weight, "post_norm_add_norm.next_weight", torch.float32, 1)
+    _need(out, "post_norm_add_norm.out", dims=2)
+    T, d = residual.shape
+    lib = library()
+    if not lib.kestrel_post_norm_takes(d):
+        add_gated_normed(residual, y, None, weight, eps, next_weight, next_eps, out)
+        return
+    if y.tokens != T or y.width != d or weight.shape[0] != d or next_weight.shape[0] != d or out.shape != residual.shape or \
+            (y.bias is not None and y.bias.shape[0] != d):
+        raise KernelError("post_norm_add_norm: shapes differ")
+    _check(lib.kestrel_post_norm_add_norm(residual.data_ptr(), y.data.data_ptr(), y.slices, y.slice_stride, _p(y.bias), weight.data_ptr(), float(eps),
+                                          next_weight.data_ptr(), float(next_eps), out.data_ptr(), _code(out, "post_norm_add_norm.out"), T, d, _stream()))
 
 
 def embed_copy(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -1679,6 +1718,47 @@ def time_mix_gates(p: Partials, z: Partials, w0: torch.Tensor, n: int, h: torch.
     return r, w, k, v
 
 
+def time_mix_step(p: Partials, z: Partials, w0: torch.Tensor, u: torch.Tensor, norm_w: torch.Tensor, eps: float, scale: float, h: torch.Tensor,
+                  state: torch.Tensor, state_off: int, last_off: int, batch, out: torch.Tensor, H: int, d: int) -> None:
+    """Steps of few tokens: from the products [r | k | v | gate] and z to the normed, weighted and gated heads times ``scale`` in one kernel,
+    into a place inside a wider matrix."""
+    T = h.shape[0]
+    _need(h, "time_mix_step.h", dims=2)
+    _need(state, "time_mix_step.state", torch.float32, 2)
+    _need_rows(out, "time_mix_step.out", T, H * d)
+    if p.bias is not None or z.bias is not None or p.tokens != T or z.tokens != T or p.width < 4 * H * d or z.width != H * d or out.dtype != h.dtype or \
+            last_off + h.shape[1] > state.shape[1]:
+        raise KernelError("time_mix_step: shapes differ, or a bias is pending")
+    _check(library().kestrel_time_mix_step(p.data.data_ptr(), p.slices, p.slice_stride, p.width, z.data.data_ptr(), z.slices, z.slice_stride, w0.data_ptr(),
+                                           u.data_ptr(), norm_w.data_ptr(), float(eps), float(scale), h.data_ptr(), h.shape[1], state.data_ptr(),
+                                           state.stride(0), int(state_off), int(last_off), batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(),
+                                           out.data_ptr(), out.stride(0), _code(out, "time_mix_step.out"), batch.num_seqs, H, d, _stream()))
+
+
+def time_mix_chunks(p: Partials, z: Partials, w0: torch.Tensor, u: torch.Tensor, norm_w: torch.Tensor, eps: float, scale: float, h: torch.Tensor,
+                    state: torch.Tensor, state_off: int, last_off: int, batch, out: torch.Tensor, H: int, d: int) -> None:
+    """The same for prompt portions, in chunks on the tensor cores (bfloat16)."""
+    T, dev = h.shape[0], h.device
+    _need(h, "time_mix_chunks.h", torch.bfloat16, 2)
+    _need(state, "time_mix_chunks.state", torch.float32, 2)
+    _need_rows(out, "time_mix_chunks.out", T, H * d)
+    if p.bias is not None or z.bias is not None or p.tokens != T or z.tokens != T or p.width < 4 * H * d or z.width != H * d or \
+            out.dtype != torch.bfloat16 or last_off + h.shape[1] > state.shape[1]:
+        raise KernelError("time_mix_chunks: shapes differ, or a bias is pending")
+    tile_seq, tile_row0, first = chunk_tiles(batch, dev)
+    tiles = tile_seq.shape[0]
+    operands = torch.empty((3, T, H * d), dtype=torch.bfloat16, device=dev)
+    log_w = torch.empty((T, H * d), dtype=torch.float32, device=dev)
+    scratch = torch.empty((tiles * H * (2 * d * d + d),), dtype=torch.float32, device=dev)
+    _check(library().kestrel_time_mix_chunks(
+        p.data.data_ptr(), p.slices, p.slice_stride, p.width, z.data.data_ptr(), z.slices, z.slice_stride, w0.data_ptr(), u.data_ptr(), norm_w.data_ptr(),
+        float(eps), float(scale), h.data_ptr(), h.shape[1], state.data_ptr(), state.stride(0), int(state_off), int(last_off),
+        batch.seq_of_token.data_ptr(), batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), tile_seq.data_ptr(), tile_row0.data_ptr(), first.data_ptr(),
+        tiles, operands.data_ptr(), log_w.data_ptr(), scratch.data_ptr(), out.data_ptr(), out.stride(0), T, batch.num_seqs, H, d, _stream()))
+    global launches
+    launches += 3
+
+
 # ---- a state-space mixer with a scalar decay per head -----------------------------------------------
 
 def ssm_expand(act: torch.Tensor, fused: Partials, col_dt: int, dt_bias: torch.Tensor, A_log: torch.Tensor, H: int, G: int, N: int, P: int):
@@ -1710,6 +1790,127 @@ def ssm_out(o: torch.Tensor, act: torch.Tensor, D: torch.Tensor, fused: Partials
     _check(library().kestrel_ssm_out(o.data_ptr(), act.data_ptr(), D.data_ptr(), fused.data.data_ptr(), fused.slices, fused.slice_stride, fused.width,
                                      int(col_z), weight.data_ptr(), float(eps), out.data_ptr(), _code(out, "ssm_out.out"), T, H, G, N, P, int(parts),
                                      _stream()))
+
+
+def ssm_step(fused: Partials, col_z: int, col_x: int, col_dt: int, conv_w: torch.Tensor, conv_b: torch.Tensor, dt_bias: torch.Tensor,
+             A_log: torch.Tensor, D: torch.Tensor, state: torch.Tensor, tail_off: int, batch, H: int, G: int, N: int, P: int) -> torch.Tensor:
+    """Steps of few tokens: convolution, state, read-out, skip and gate in one kernel; returns the gated y float32 [T, H P], for `part_norm`."""
+    _need(state, "ssm_step.state", torch.float32, 2)
+    C, taps = conv_w.shape
+    if fused.bias is not None or C != H * P + 2 * G * N or max(col_z + H * P, col_x + C, col_dt + H) > fused.width or \
+            tail_off + (taps - 1) * C > state.shape[1]:
+        raise KernelError("ssm_step: shapes differ, or a bias is pending")
+    y = torch.empty((fused.tokens, H * P), dtype=torch.float32, device=state.device)
+    _check(library().kestrel_ssm_step(fused.data.data_ptr(), fused.slices, fused.slice_stride, fused.width, int(col_z), int(col_x), int(col_dt),
+                                      conv_w.data_ptr(), conv_b.data_ptr(), taps, dt_bias.data_ptr(), A_log.data_ptr(), D.data_ptr(), state.data_ptr(),
+                                      state.stride(0), int(tail_off), batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), y.data_ptr(),
+                                      batch.num_seqs, H, G, N, P, _stream()))
+    global launches
+    launches += 1 if taps > 1 else 0
+    return y
+
+
+def part_norm(y: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, parts: int) -> None:
+    """out = y / sqrt(mean(y^2) + eps) in ``parts`` equal parts of a row, times ``weight``."""
+    _need(y, "part_norm.y", torch.float32, 2)
+    _need(weight, "part_norm.weight", torch.float32, 1)
+    _need(out, "part_norm.out", dims=2)
+    T, inner = y.shape
+    if out.shape != y.shape or weight.shape[0] != inner or inner % parts:
+        raise KernelError("part_norm: shapes differ")
+    _check(library().kestrel_part_norm(y.data_ptr(), weight.data_ptr(), float(eps), out.data_ptr(), _code(out, "part_norm.out"), T, inner, int(parts),
+                                       _stream()))
+
+
+def chunk_tiles(batch, device):
+    """The step's tokens in chunks per request, as the chunked recurrences take them: (request of each chunk, its first token among the
+    request's, every request's first chunk), int32 on the device, made once a step."""
+    chunk = library().kestrel_decay_chunk_tokens()
+    tile_seq, tile_row0 = row_tiles(batch, 1, chunk)
+    kept = batch.__dict__.setdefault("_row_tiles", {})
+    if ("first", chunk) not in kept:
+        first = [0]
+        for n in batch.counts:
+            first.append(first[-1] + -(-n // chunk))
+        kept[("first", chunk)] = torch.tensor(first, dtype=torch.int32).to(device, non_blocking=True)
+    return tile_seq, tile_row0, kept[("first", chunk)]
+
+
+def ssm_chunks(act: torch.Tensor, fused: Partials, col_z: int, col_dt: int, dt_bias: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor,
+               state: torch.Tensor, batch, H: int, G: int, N: int, P: int) -> torch.Tensor:
+    """Prompt portions in chunks on the tensor cores: from act = [x | B | C] (bfloat16, after the convolution) and the product's gate and step
+    columns to the gated y float32 [T, H P], for `part_norm`."""
+    _need(act, "ssm_chunks.act", torch.bfloat16, 2)
+    _need(state, "ssm_chunks.state", torch.float32, 2)
+    T, dev = act.shape[0], act.device
+    if act.shape[1] != H * P + 2 * G * N or fused.tokens != T or fused.bias is not None or state.shape[1] < H * N * P:
+        raise KernelError("ssm_chunks: shapes differ, or a bias is pending")
+    lib = library()
+    step, log_decay = (torch.empty((T, H), dtype=torch.float32, device=dev) for _ in range(2))
+    _check(lib.kestrel_ssm_steps(fused.data.data_ptr(), fused.slices, fused.slice_stride, fused.width, int(col_dt), dt_bias.data_ptr(), A_log.data_ptr(),
+                                 step.data_ptr(), log_decay.data_ptr(), T, H, _stream()))
+    tile_seq, tile_row0, first = chunk_tiles(batch, dev)
+    tiles = tile_seq.shape[0]
+    scratch = torch.empty((tiles * H * (2 * N * P + 1),), dtype=torch.float32, device=dev)
+    y = torch.empty((T, H * P), dtype=torch.float32, device=dev)
+    _check(lib.kestrel_ssm_chunks(act.data_ptr(), act.shape[1], step.data_ptr(), log_decay.data_ptr(), D.data_ptr(), fused.data.data_ptr(), fused.slices,
+                                  fused.slice_stride, fused.width, int(col_z), state.data_ptr(), state.stride(0), 0, batch.cu_seqlens.data_ptr(),
+                                  batch.slots.data_ptr(), tile_seq.data_ptr(), tile_row0.data_ptr(), first.data_ptr(), tiles, scratch.data_ptr(),
+                                  y.data_ptr(), batch.num_seqs, H, G, N, P, _stream()))
+    global launches
+    launches += 2
+    return y
+
+
+def delta_head_step(fused: Partials, col_g: int, col_beta: int, col_a: int, conv_w: torch.Tensor, A_log: torch.Tensor, dt_bias: torch.Tensor,
+                    norm_w: torch.Tensor, eps: float, state: torch.Tensor, tail_off: int, batch, out: torch.Tensor, H: int, G: int, d: int, dv: int) -> bool:
+    """Steps of few tokens of a delta rule with one decay per head: everything between the fused product and the output product in one
+    kernel; False (nothing has run) for sizes it does not take."""
+    lib = library()
+    if not lib.kestrel_delta_head_step_takes(int(d), int(dv)):
+        return False
+    _need(state, "delta_head_step.state", torch.float32, 2)
+    _need(out, "delta_head_step.out", dims=2)
+    C, taps = conv_w.shape
+    if fused.bias is not None or C != 2 * G * d + H * dv or max(C, col_g + H * dv, col_beta + H, col_a + H) > fused.width or \
+            tail_off + (taps - 1) * C > state.shape[1] or out.shape != (fused.tokens, H * dv):
+        raise KernelError("delta_head_step: shapes differ, or a bias is pending")
+    _check(lib.kestrel_delta_head_step(fused.data.data_ptr(), fused.slices, fused.slice_stride, fused.width, int(col_g), int(col_beta), int(col_a),
+                                       conv_w.data_ptr(), taps, A_log.data_ptr(), dt_bias.data_ptr(), norm_w.data_ptr(), float(eps), state.data_ptr(),
+                                       state.stride(0), int(tail_off), batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), out.data_ptr(),
+                                       _code(out, "delta_head_step.out"), batch.num_seqs, H, G, d, dv, _stream()))
+    global launches
+    launches += 1 if taps > 1 else 0
+    return True
+
+
+def delta_chunks(act: torch.Tensor, fused: Partials, col_g: int, col_beta: int, col_a: int, A_log: torch.Tensor, dt_bias: torch.Tensor,
+                 norm_w: torch.Tensor, eps: float, state: torch.Tensor, batch, out: torch.Tensor, H: int, G: int, d: int, dv: int) -> None:
+    """Prompt portions of a delta rule with one decay per head, in chunks on the tensor cores: from act = [q | k | v] (bfloat16, after
+    convolution and silu) and the product's columns to the normed, weighted and gated heads."""
+    _need(act, "delta_chunks.act", torch.bfloat16, 2)
+    _need(out, "delta_chunks.out", torch.bfloat16, 2)
+    _need(state, "delta_chunks.state", torch.float32, 2)
+    T, dev = act.shape[0], act.device
+    if act.shape[1] != 2 * G * d + H * dv or fused.tokens != T or fused.bias is not None or state.shape[1] < H * d * dv or out.shape != (T, H * dv):
+        raise KernelError("delta_chunks: shapes differ, or a bias is pending")
+    lib = library()
+    f32 = dict(dtype=torch.float32, device=dev)
+    qs, ks, beta, la = torch.empty((T, G), **f32), torch.empty((T, G), **f32), torch.empty((T, H), **f32), torch.empty((T, H), **f32)
+    _check(lib.kestrel_delta_steps(act.data_ptr(), act.shape[1], fused.data.data_ptr(), fused.slices, fused.slice_stride, fused.width, int(col_beta),
+                                   int(col_a), A_log.data_ptr(), dt_bias.data_ptr(), qs.data_ptr(), ks.data_ptr(), beta.data_ptr(), la.data_ptr(), T, H, G,
+                                   d, _stream()))
+    tile_seq, tile_row0, first = chunk_tiles(batch, dev)
+    tiles = tile_seq.shape[0]
+    scratch = torch.empty((tiles * H * (64 * (d + dv) + 68 + d * dv),), **f32)
+    u = torch.empty((2, T, H * dv), dtype=torch.bfloat16, device=dev)
+    _check(lib.kestrel_delta_chunks(act.data_ptr(), act.shape[1], G, qs.data_ptr(), ks.data_ptr(), beta.data_ptr(), la.data_ptr(), norm_w.data_ptr(),
+                                    float(eps), fused.data.data_ptr(), fused.slices, fused.slice_stride, fused.width, int(col_g), state.data_ptr(),
+                                    state.stride(0), 0, batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), tile_seq.data_ptr(), tile_row0.data_ptr(),
+                                    first.data_ptr(), tiles, scratch.data_ptr(), u[0].data_ptr(), u[1].data_ptr(), out.data_ptr(), batch.num_seqs, H, d,
+                                    dv, _stream()))
+    global launches
+    launches += 2
 
 
 # ---- retention: linear attention with a fixed decay per head -----------------------------------------

@@ -280,11 +280,36 @@ KESTREL_API int kestrel_token_shift(const void *h, const float *mu, int n, const
 /* r, k, v = the product's columns 0, n, 2 n; w = exp(-exp(z + w0)), z a product [T, n]; every request's last h goes into its slot */
 KESTREL_API int kestrel_time_mix_gates(const float *partial, int S, long long slice_stride, int ld, const float *z, int Sz, long long z_stride, const float *w0, float *r_out, float *k_out, float *v_out, float *w_out, int n, const void *h, int dtype, int d, float *state, long long state_stride, long long state_off, const int *seq_of_token, const int *cu_seqlens, const int *slots, int T, kestrel_stream_t stream);
 
+/* steps of few tokens: state, read-out, norm per head, weight, silu gate (columns 3 n of the product), times scale, into rows of ldo numbers; h's last row into the slot at last_off */
+KESTREL_API int kestrel_time_mix_step(const float *partial, int S, long long slice_stride, int ld, const float *z, int Sz, long long z_stride, const float *w0, const float *u, const float *norm_w, float eps, float scale, const void *h, int width, float *state, long long state_stride, long long state_off, long long last_off, const int *cu_seqlens, const int *slots, void *out, long long ldo, int dtype, int nseq, int H, int d, kestrel_stream_t stream);
+/* prompt portions in chunks of kestrel_decay_chunk_tokens() tokens on the tensor cores (time_mix_chunks.cu; bfloat16, d a multiple of 8 up to 128), the same from the products to the gated heads: tiles list the chunks (request, first token among the request's), first_tile [nseq + 1] each request's first; operands 3 T H d bfloat16, log_w T H d floats, scratch tiles H (2 d d + d) floats */
+KESTREL_API int kestrel_time_mix_chunks(const float *partial, int S, long long slice_stride, int ld, const float *z, int Sz, long long z_stride, const float *w0, const float *u, const float *norm_w, float eps, float scale, const void *h, int width, float *state, long long state_stride, long long state_off, long long last_off, const int *seq_of_token, const int *cu_seqlens, const int *slots, const int *tile_seq, const int *tile_row0, const int *first_tile, int tiles, void *operands, float *log_w, float *scratch, void *out, long long ldo, int T, int nseq, int H, int d, kestrel_stream_t stream);
+
 /* ---- a state-space mixer with a scalar decay per head (ssm.cu); act [T, H P + 2 G N] = x | B | C ---- */
 /* dt = softplus(column col_dt + h of the product + dt_bias): r = C, k = B of the head's group, v = dt x, w = exp(-exp(A_log) dt), as the scan of linear_recurrence.cu takes them */
 KESTREL_API int kestrel_ssm_expand(const float *act, const float *partial, int S, long long slice_stride, int ld, int col_dt, const float *dt_bias, const float *A_log, float *r_out, float *w_out, float *k_out, float *v_out, int T, int H, int G, int N, int P, kestrel_stream_t stream);
 /* out = (o + D x) silu(z), normed (eps) in `parts` equal parts of the H P columns, times w; z the product's columns from col_z */
 KESTREL_API int kestrel_ssm_out(const float *o, const float *act, const float *D, const float *partial, int S, long long slice_stride, int ld, int col_z, const float *w, float eps, void *out, int dtype, int T, int H, int G, int N, int P, int parts, kestrel_stream_t stream);
+/* step sizes dt and logarithms of the decays, -exp(A_log) dt, float32 [T, H] */
+KESTREL_API int kestrel_ssm_steps(const float *partial, int S, long long slice_stride, int ld, int col_dt, const float *dt_bias, const float *A_log, float *step, float *log_decay, int T, int H, kestrel_stream_t stream);
+/* steps of few tokens: convolution (tail at tail_off behind the state), state, read-out, + D x, times silu(z): y [T, H P] float32 */
+KESTREL_API int kestrel_ssm_step(const float *partial, int S, long long slice_stride, int ld, int col_z, int col_x, int col_dt, const float *conv_w, const float *conv_b, int taps, const float *dt_bias, const float *A_log, const float *D, float *state, long long state_stride, long long tail_off, const int *cu_seqlens, const int *slots, float *y, int nseq, int H, int G, int N, int P, kestrel_stream_t stream);
+/* out = y / sqrt(mean(y^2) + eps) in `parts` equal parts of a row of `inner` numbers, times w [inner] */
+KESTREL_API int kestrel_part_norm(const float *y, const float *w, float eps, void *out, int dtype, int T, int inner, int parts, kestrel_stream_t stream);
+
+/* ---- scalar decays per head and token in chunks of 64 tokens on the tensor cores (decay_chunks.cu, delta_chunks.cu; bfloat16 rows, sizes multiples of 8); tiles list the chunks (request, first token among the request's), first_tile [nseq + 1] each request's first ---- */
+KESTREL_API int kestrel_decay_chunk_tokens(void);
+/* the state-space mixer from act [T, ld_act >= x: H P | B: G N | C: G N] to y as kestrel_ssm_step leaves it; scratch tiles H (2 N P + 1) floats */
+KESTREL_API int kestrel_ssm_chunks(const void *act, long long ld_act, const float *step, const float *log_decay, const float *D, const float *partial, int S, long long slice_stride, int ld, int col_z, float *state, long long state_stride, long long state_off, const int *cu_seqlens, const int *slots, const int *tile_seq, const int *tile_row0, const int *first_tile, int tiles, float *scratch, float *y, int nseq, int H, int G, int N, int P, kestrel_stream_t stream);
+/* the delta rule with one decay per head: act [T, ld_act >= q: G d | k: G d | v: H dv] after convolution and silu; q_scale, k_scale [T, G] what makes q (times d^-1/2) and k unit vectors; beta, log_decay [T, H] */
+KESTREL_API int kestrel_delta_steps(const void *act, long long ld_act, const float *partial, int S, long long slice_stride, int ld, int col_beta, int col_a, const float *A_log, const float *dt_bias, float *q_scale, float *k_scale, float *beta, float *log_decay, int T, int H, int G, int d, kestrel_stream_t stream);
+/* (d <= 128) to out [T, H dv] bfloat16 = norm per head(o) w silu(columns col_g of the product); scratch tiles H (64 (d + dv) + 68 + d dv) floats; u_hi, u_lo [T, H dv] bfloat16: room for what the tokens write */
+KESTREL_API int kestrel_delta_chunks(const void *act, long long ld_act, int G, const float *q_scale, const float *k_scale, const float *beta, const float *log_decay, const float *w, float eps, const float *partial, int S, long long slice_stride, int ld, int col_g, float *state, long long state_stride, long long state_off, const int *cu_seqlens, const int *slots, const int *tile_seq, const int *tile_row0, const int *first_tile, int tiles, float *scratch, void *u_hi, void *u_lo, void *out, int nseq, int H, int d, int dv, kestrel_stream_t stream);
+/* its last part: the outputs of all chunks from the states in front of them (before [tiles, H, 2, d, dv] bfloat16) and the tokens' writes */
+KESTREL_API int kestrel_delta_chunks_out(const void *act, long long ld_act, int G, const void *u_hi, const void *u_lo, const float *q_scale, const float *k_scale, const float *log_decay, const void *before, const float *w, float eps, const float *partial, int S, long long slice_stride, int ld, int col_g, const int *cu_seqlens, const int *tile_seq, const int *tile_row0, int tiles, void *out, int H, int d, int dv, kestrel_stream_t stream);
+/* steps of few tokens, one decay per head: everything between the fused product [q | k | v ... gate at col_g, beta at col_beta, decay logits at col_a] and the output product; sizes by _takes */
+KESTREL_API int kestrel_delta_head_step_takes(int d, int dv);
+KESTREL_API int kestrel_delta_head_step(const float *partial, int S, long long slice_stride, int ld, int col_g, int col_beta, int col_a, const float *conv_w, int taps, const float *A_log, const float *dt_bias, const float *norm_w, float eps, float *state, long long state_stride, long long tail_off, const int *cu_seqlens, const int *slots, void *out, int dtype, int nseq, int H, int G, int d, int dv, kestrel_stream_t stream);
 /* ---- retention: a fixed decay per head (retention.cu) ---- */
 /* product columns [q: H d | k: H d | v: H dv | ...]: q, k turned by position (first `rot` dimensions, rotate-half), k times d^-1/2; q_out, k_out [T, H d], v_out [T, H dv] in `dtype`; w_out (may be NULL) [T, H d] = the head's decay */
 KESTREL_API int kestrel_retention_prepare(const float *partial, int S, long long slice_stride, int ld, const int *positions, const float *inv_freq, int rot, const float *decay, void *q_out, void *k_out, void *v_out, float *w_out, int dtype, int T, int H, int d, int dv, kestrel_stream_t stream);
@@ -307,6 +332,8 @@ KESTREL_API int kestrel_attention_decode_maps(const void *q, const void *k_cache
 KESTREL_API int kestrel_post_norm_takes(int d);
 /* residual[t] += y / sqrt(mean(y^2) + eps) w, y the sum of the slices plus the bias (may be NULL); copy[t] = residual[t] in `dtype` (may be NULL) */
 KESTREL_API int kestrel_post_norm_add(float *residual, const float *y, int S, long long stride, const float *bias, const float *w, float eps, void *copy, int dtype, int T, int d, kestrel_stream_t stream);
+/* the same, but copy[t] = the new residual[t] / sqrt(mean(.^2) + next_eps) next_w: the norm that follows */
+KESTREL_API int kestrel_post_norm_add_norm(float *residual, const float *y, int S, long long stride, const float *bias, const float *w, float eps, const float *next_w, float next_eps, void *copy, int dtype, int T, int d, kestrel_stream_t stream);
 /* the same where y is a routed feed-forward's sum, as kestrel_moe_combine_with would write it; x in `dtype` too */
 KESTREL_API int kestrel_post_norm_add_moe(float *residual, const float *y, const int *pair_row, const int *ids, const float *weights, int top, int experts, const void *x, long long ldx, const float *shared, int Ss, long long shared_stride, const float *z, int Sz, long long z_stride, int z_ld, int sg_col, const float *w, float eps, void *copy, int dtype, int T, int d, kestrel_stream_t stream);
 /* x[t] = table[ids[t]] in float32, copy[t] = the bfloat16 row itself */
@@ -356,6 +383,9 @@ KESTREL_API int kestrel_gemm_tc_add(const void *x, const void *w, float *residua
 KESTREL_API int kestrel_gemm_tc_act(const void *x, const void *w, void *out, int act, int T, int N, int K, long long ldx, long long ldw, long long ldo, kestrel_stream_t stream);
 /* the same with a bias [N] (may be NULL) before the activation; act 6: xIELU with its two numbers in act_p (NULL for the others) */
 KESTREL_API int kestrel_gemm_tc_act_with(const void *x, const void *w, const float *bias, void *out, int act, const float *act_p, int T, int N, int K, long long ldx, long long ldw, long long ldo, kestrel_stream_t stream);
+/* several products in one launch: rows [g group_rows, (g + 1) group_rows) of w (the last group may have fewer) meet token rows [g T, (g + 1) T) of x, N all rows of w; _plan: 0 where this form does not take the sizes, else the number of K slices */
+KESTREL_API int kestrel_gemm_tc_grouped_plan(const void *x, const void *w, int T, int N, int K, int group_rows, long long ldx, long long ldw);
+KESTREL_API int kestrel_gemm_tc_grouped(const void *x, const void *w, float *out, int T, int N, int K, int group_rows, long long ldx, long long ldw, long long ldo, int splits, long long slice_stride, int weights_static, kestrel_stream_t stream);
 KESTREL_API int kestrel_gemm_tc_swiglu_w(const void *x, const void *w, void *out, int T, int ff, int K, long long ldx, long long ldw, long long ldo, int weights_static, kestrel_stream_t stream);
 /* the same with the bounded activation of kestrel_gated_act where limit > 0 */
 KESTREL_API int kestrel_gemm_tc_gated_w(const void *x, const void *w, void *out, int T, int ff, int K, long long ldx, long long ldw, long long ldo, float limit, int weights_static, kestrel_stream_t stream);

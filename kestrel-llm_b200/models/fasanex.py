@@ -62,6 +62,8 @@ def build_fasanex(config: FasanexConfig, dtype: torch.dtype, device) -> DecoderM
         else:
             optional += [p + "norm2", p + "norm2b"]         # a layer without feed-forward has no use for them
         blocks.append(SandwichBlock(norm(p + "norm1"), mixer, norm(p + "norm1b"), None, norm2, ffn, norm2b, None, dtype, p))
+    for block, after in zip(blocks, blocks[1:]):
+        block.following = after.norm1                       # the last add of a layer makes the norm of the next one
     order = [LayerCall(block=i, cache=i) for i in range(len(blocks))]
     return DecoderModel(c, dtype, device, TokenEmbedding(c.vocab_size, W, dtype, device, "embed", scale=c.embedding_scale), None, blocks, order,
                         norm("final.norm"), LMHead(c.vocab_size, W, dtype, device, "head"), optional_tensors=optional)

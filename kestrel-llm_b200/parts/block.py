@@ -95,7 +95,10 @@ class SandwichBlock(Block):
 
     (``gate1`` / ``gate2`` None: no gate on that sublayer; ``ffn`` None: the first line alone.)  A
     sublayer's gate, second norm and add are one kernel, which also makes the norm that follows
-    inside the block; the block adds into the stream itself and hands nothing on."""
+    inside the block; the block adds into the stream itself and hands nothing on - or, where ``following`` names the norm that the
+    next block starts with and the last sublayer has no gate, the stream after that norm."""
+
+    following: Optional[RMSNorm] = None
 
     def __init__(self, norm1: RMSNorm, mixer: Mixer, norm1b: RMSNorm, gate1: Optional[Linear], norm2: Optional[RMSNorm],
                  ffn: Optional[FeedForward], norm2b: Optional[RMSNorm], gate2: Optional[Linear], dtype: torch.dtype, prefix: str,
@@ -120,19 +123,36 @@ class SandwichBlock(Block):
                     slots.append(WeightSlot(self.prefix + name + ".b", gate.bias, "bias"))
         return slots
 
+    def _add(self, residual: torch.Tensor, y, gate, norm: RMSNorm, following: Optional[RMSNorm]):
+        """residual += norm(y, gated); the stream after ``following`` where one is given."""
+        if following is None:
+            if gate is None:
+                ops.post_norm_add(residual, y, norm.weight, norm.eps)
+            else:
+                ops.add_gated_normed(residual, y, gate, norm.weight, norm.eps)
+            return None
+        h = torch.empty(residual.shape, dtype=self.dtype, device=residual.device)
+        if gate is None:
+            ops.post_norm_add_norm(residual, y, norm.weight, norm.eps, following.weight, following.eps, h)
+        else:
+            ops.add_gated_normed(residual, y, gate, norm.weight, norm.eps, following.weight, following.eps, h)
+        return h
+
     def forward(self, residual: torch.Tensor, pending, batch, cache):
-        h = self.norm1.add_forward(residual, pending, self.dtype)
+        if isinstance(pending, ops.NormedStream) and pending.norm is self.norm1:
+            h = pending.data
+        else:
+            h = self.norm1.add_forward(residual, None if isinstance(pending, ops.StreamCopy) else pending, self.dtype)
         y = self.mixer.forward(h, batch, cache)
         g = self.gate1.forward(h) if self.gate1 is not None else None
         if self.ffn is None:
-            ops.add_gated_normed(residual, y, g, self.norm1b.weight, self.norm1b.eps)
-            return residual, None
-        h = torch.empty(residual.shape, dtype=self.dtype, device=residual.device)
-        ops.add_gated_normed(residual, y, g, self.norm1b.weight, self.norm1b.eps, self.norm2.weight, self.norm2.eps, h)
-        z = self.ffn.forward(h, batch)
-        g = self.gate2.forward(h) if self.gate2 is not None else None
-        ops.add_gated_normed(residual, z, g, self.norm2b.weight, self.norm2b.eps)
-        return residual, None
+            h = self._add(residual, y, g, self.norm1b, self.following)
+        else:
+            h = self._add(residual, y, g, self.norm1b, self.norm2)
+            z = self.ffn.forward(h, batch)
+            g = self.gate2.forward(h) if self.gate2 is not None else None
+            h = self._add(residual, z, g, self.norm2b, self.following)
+        return residual, ops.NormedStream(h, self.following) if h is not None else None
 
 
 class PostNormBlock(Block):

@@ -16,6 +16,8 @@ W_b, W_a1 and W_g1 are one fused product.
 
 `ChannelDeltaMixer` is the layer above; `HeadDeltaMixer` has one decay per value head, a = exp(-exp(A_log[n]) softplus(W_a h + dt_bias))
 for all of a head's key channels, and the gate silu(W_g h) without the step through a low rank; everything it reads h with is one product.
+Its steps of at most `STEP_TOKENS` tokens per request run one kernel between the products, in bfloat16 longer ones run in chunks on the
+tensor cores.
 """
 from __future__ import annotations
 
@@ -92,6 +94,9 @@ class ChannelDeltaMixer(Mixer):
 
 
 class HeadDeltaMixer(Mixer):
+    STEP_TOKENS = 4
+    chunked = True             # tests switch the chunked form and the one-kernel form off to hold the forms against each other
+    one_kernel = True
     graph_safe = True          # forward launches kernels over device tensors of the batch only
 
     def __init__(self, width: int, heads: int, kv_heads: int, key_dim: int, value_dim: int, taps: int, norm_eps: float, dtype: torch.dtype,
@@ -132,8 +137,18 @@ class HeadDeltaMixer(Mixer):
         H, G, d, dv = self.H, self.G, self.d, self.dv
         fused = self.in_proj.forward(x)
         y = torch.empty((T, H * dv), dtype=self.dtype, device=dev)
-        act = torch.empty((T, self.C), dtype=f32, device=dev)
+        cols = (self.col_g, self.col_beta, self.col_a)
+        if batch.max_count <= self.STEP_TOKENS and self.one_kernel and \
+                ops.delta_head_step(fused, *cols, self.conv_w, self.A_log, self.dt_bias, self.norm_w, self.eps, cache.state, self.tail_off, batch, y,
+                                    H, G, d, dv):
+            return self.out.forward(y)
+        chunks = self.dtype == torch.bfloat16 and not batch.captured and self.chunked and d % 8 == 0 and dv % 8 == 0 and d <= 128 and dv <= 256 and \
+            fused.width % 2 == 0
+        act = torch.empty((T, self.C), dtype=torch.bfloat16 if chunks else f32, device=dev)
         ops.short_conv(fused, self.conv_w, None, cache.state, self.tail_off, batch, act)
+        if chunks:
+            ops.delta_chunks(act, fused, *cols, self.A_log, self.dt_bias, self.norm_w, self.eps, cache.state, batch, y, H, G, d, dv)
+            return self.out.forward(y)
         qn, kn = (torch.empty((T, G * d), dtype=f32, device=dev) for _ in range(2))
         decay, beta = torch.empty((T, H * d), dtype=f32, device=dev), torch.empty((T, H), dtype=f32, device=dev)
         ops.delta_gates(act, fused, self.col_beta, fused, self.A_log, self.dt_bias, qn, kn, decay, beta, H, G, d, col_a=self.col_a, per_head=True)

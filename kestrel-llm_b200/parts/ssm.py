@@ -9,7 +9,8 @@ With h the mixer's input, H heads of P value channels, G groups of N state chann
     out = W_o ( norm(y * silu(z)) * w )                                    the norm over `norm_groups` equal parts of the inner channels
 
 The state S and the convolution's last taps - 1 inputs live in the request's state slot, float32; step sizes, decays, recurrence,
-gate and norm are float32.
+gate and norm are float32.  Steps of at most `STEP_TOKENS` tokens per request run one kernel between the input product and the norm; in
+bfloat16 longer ones run in chunks on the tensor cores; the rest runs on the sequential scan that the other recurrences share.
 """
 from __future__ import annotations
 
@@ -23,6 +24,9 @@ from .linear import Linear
 
 
 class StateSpaceMixer(Mixer):
+    STEP_TOKENS = 4
+    chunked = True             # tests switch the chunked form and the one-kernel form off to hold the forms against each other
+    one_kernel = True
     graph_safe = True          # forward launches kernels over device tensors of the batch only
 
     def __init__(self, width: int, heads: int, value_dim: int, state: int, groups: int, norm_groups: int, taps: int, norm_eps: float,
@@ -62,10 +66,20 @@ class StateSpaceMixer(Mixer):
         H, G, N, P = self.H, self.G, self.N, self.P
         T, dev = x.shape[0], x.device
         fused = self.in_proj.forward(x)
-        act = torch.empty((T, self.C), dtype=torch.float32, device=dev)
-        ops.short_conv(fused, self.conv_w, self.conv_b, cache.state, self.tail_off, batch, act, col0=self.inner)
-        r, w, k, v = ops.ssm_expand(act, fused, self.col_dt, self.dt_bias, self.A_log, H, G, N, P)
-        o = ops.recurrence_scan(r, w, k, v, None, None, cache.state, 0, batch, H, N, P)
         y = torch.empty((T, self.inner), dtype=self.dtype, device=dev)
-        ops.ssm_out(o, act, self.D, fused, 0, self.norm_w, self.eps, y, H, G, N, P, self.parts)
+        if batch.max_count <= self.STEP_TOKENS and P <= 256 and self.one_kernel:
+            o = ops.ssm_step(fused, 0, self.inner, self.col_dt, self.conv_w, self.conv_b, self.dt_bias, self.A_log, self.D, cache.state, self.tail_off,
+                             batch, H, G, N, P)
+            ops.part_norm(o, self.norm_w, self.eps, y, self.parts)
+            return self.out.forward(y)
+        chunks = self.dtype == torch.bfloat16 and not batch.captured and self.chunked and N % 8 == 0 and P % 8 == 0 and P <= 256 and fused.width % 2 == 0
+        act = torch.empty((T, self.C), dtype=torch.bfloat16 if chunks else torch.float32, device=dev)
+        ops.short_conv(fused, self.conv_w, self.conv_b, cache.state, self.tail_off, batch, act, col0=self.inner)
+        if chunks:
+            o = ops.ssm_chunks(act, fused, 0, self.col_dt, self.dt_bias, self.A_log, self.D, cache.state, batch, H, G, N, P)
+            ops.part_norm(o, self.norm_w, self.eps, y, self.parts)
+        else:
+            r, w, k, v = ops.ssm_expand(act, fused, self.col_dt, self.dt_bias, self.A_log, H, G, N, P)
+            o = ops.recurrence_scan(r, w, k, v, None, None, cache.state, 0, batch, H, N, P)
+            ops.ssm_out(o, act, self.D, fused, 0, self.norm_w, self.eps, y, H, G, N, P, self.parts)
         return self.out.forward(y)
