@@ -1,7 +1,7 @@
 // The step between a fused query/key product and attention, for mixers whose queries and keys pass a short causal convolution and
 // whose values ARE their keys:
 //
-//   u[t, c] = sum_j w[c, j] x[t - (taps - 1) + j, c]        per column of [q: nq hd | k: nkv hd]; inputs before a request's first
+//   u[t, c] = sum_j w[j, c] x[t - (taps - 1) + j, c]        per column of [q: nq hd | k: nkv hd]; inputs before a request's first
 //                                                           token of this step from its state slot (as in short_conv.cu)
 //   v = u_k as it is, into the V pages;   q, k = u / sqrt(mean(u^2) + eps) * weight [hd] per head, then the first `rot`
 //   dimensions turned by position in rotate-half pairs (times `rot_scale`); q to its rows, k into the K pages.
@@ -46,7 +46,7 @@ attn_prepare_conv_kernel(const float *__restrict__ p, int S, size_t slice_stride
             const int i = lane + 32 * c;
             w[c] = i < hd && nw ? nw[i] : 1.f;
 #pragma unroll
-            for (int j = 0; j < TP; ++j) f[j][c] = i < hd && j >= TP - taps ? conv_w[((size_t)r * hd + i) * taps + j - (TP - taps)] : 0.f;
+            for (int j = 0; j < TP; ++j) f[j][c] = i < hd && j >= TP - taps ? conv_w[(size_t)(j - (TP - taps)) * C + (size_t)r * hd + i] : 0.f;
         }
         auto load = [&](float (&v)[PER], int t) {
 #pragma unroll
@@ -134,11 +134,146 @@ attn_prepare_conv_kernel(const float *__restrict__ p, int S, size_t slice_stride
     }
 }
 
+// The same where a head's size is 32, 64 or 128 and all of it is turned, or none: HD / 8 lanes take a head row, a lane the numbers
+// 4 j .. 4 j + 3 and their partners HD / 2 + 4 j .., so that loads and stores are vectors and a pair is turned inside a lane; all inputs of
+// a run of tokens are in flight together.
+#define APF_THREADS 128
+template <int N> struct ApfCount { static constexpr int value = N; };
+__device__ __forceinline__ void apf_store4(float *dst, const float *x) { *reinterpret_cast<float4 *>(dst) = make_float4(x[0], x[1], x[2], x[3]); }
+__device__ __forceinline__ void apf_store4(__nv_bfloat16 *dst, const float *x) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(x[0], x[1]), hi = __floats2bfloat162_rn(x[2], x[3]);
+    *reinterpret_cast<uint2 *>(dst) = make_uint2(*reinterpret_cast<uint32_t *>(&lo), *reinterpret_cast<uint32_t *>(&hi));
+}
+
+template <typename T, int HD, int TP, int RUN>
+__global__ void __launch_bounds__(APF_THREADS)
+attn_prepare_conv_rows_kernel(const float *__restrict__ p, int S, size_t slice_stride, int ld, const float *__restrict__ conv_w, int taps,
+                              const float *__restrict__ q_w, const float *__restrict__ k_w, float eps, const float *__restrict__ inv_freq, int rot,
+                              float rot_scale, const float *__restrict__ state, size_t state_stride, size_t tail_off, const int *__restrict__ positions,
+                              const int *__restrict__ seq_of_token, const int *__restrict__ cu_seqlens, const int *__restrict__ slots,
+                              const int *__restrict__ block_table, int table_stride, int page_size, T *__restrict__ k_cache, T *__restrict__ v_cache,
+                              T *__restrict__ q_out, int n_tokens, int nq, int nkv) {
+    constexpr int LANES = HD / 8, ROWS = APF_THREADS / LANES, HALF = HD / 2;
+    __shared__ float cs_s[RUN][HALF], sn_s[RUN][HALF];
+    pdl_launch_dependents();
+    // the step's description and the weights are not the predecessor's output
+    const int tid = threadIdx.x, j = tid % LANES, r = blockIdx.y * ROWS + tid / LANES, t0 = blockIdx.x * RUN, t1 = min(t0 + RUN, n_tokens);
+    const int C = (nq + nkv) * HD;
+    if (rot) {
+        for (int i = tid; i < (t1 - t0) * HALF; i += APF_THREADS) {
+            float sn, cs;
+            sincosf((float)positions[t0 + i / HALF] * inv_freq[i % HALF], &sn, &cs);
+            cs_s[i / HALF][i % HALF] = cs * rot_scale;
+            sn_s[i / HALF][i % HALF] = sn * rot_scale;
+        }
+    }
+    const bool live = r < nq + nkv, is_k = r >= nq;
+    float f[TP][8], w[8];
+    const float *nw = is_k ? k_w : q_w;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+        const int i = (e >> 2) * HALF + 4 * j + (e & 3);
+        w[e] = live && nw ? nw[i] : 1.f;
+#pragma unroll
+        for (int x = 0; x < TP; ++x) f[x][e] = live && x >= TP - taps ? conv_w[(size_t)(x - (TP - taps)) * C + (size_t)r * HD + i] : 0.f;
+    }
+    __syncthreads();
+    pdl_wait();
+    auto go = [&](auto count, int t, int q) {
+        constexpr int N = decltype(count)::value;
+        const int first = cu_seqlens[q];
+        float x[TP - 1 + N][8];
+#pragma unroll
+        for (int a = 0; a < TP - 1 + N; ++a) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[a][e] = 0.f;
+        }
+        const int n0 = t - first - (TP - 1);                  // the first input, among this step's tokens of the request
+        auto add = [&](float (&v)[8], const float *src) {
+            const float4 lo = *reinterpret_cast<const float4 *>(src), hi = *reinterpret_cast<const float4 *>(src + HALF);
+            v[0] += lo.x; v[1] += lo.y; v[2] += lo.z; v[3] += lo.w;
+            v[4] += hi.x; v[5] += hi.y; v[6] += hi.z; v[7] += hi.w;
+        };
+        if (live) {
+            const float *src = p + (size_t)t * ld + (size_t)r * HD + 4 * j - (size_t)(TP - 1) * ld;
+            for (int s = 0; s < S; ++s, src += slice_stride) {
+#pragma unroll
+                for (int a = 0; a < TP - 1 + N; ++a)
+                    if (a >= TP - taps && n0 + a >= 0 && t + a - (TP - 1) < t1) add(x[a], src + (size_t)a * ld);
+            }
+            if (n0 < 0) {
+                const float *tail = state + (size_t)slots[q] * state_stride + tail_off + (size_t)r * HD + 4 * j;
+#pragma unroll
+                for (int a = 0; a < TP - 1; ++a)
+                    if (a >= TP - taps && n0 + a < 0) add(x[a], tail + (size_t)(taps - 1 + n0 + a) * C);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < N; ++k) {
+            float y[8], ss = 0.f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                y[e] = 0.f;
+#pragma unroll
+                for (int a = 0; a < TP; ++a) y[e] = fmaf(f[a][e], x[k + a][e], y[e]);
+                ss = fmaf(y[e], y[e], ss);
+            }
+#pragma unroll
+            for (int sh = 1; sh < LANES; sh <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, sh);
+            const int tt = t + k;
+            if (!live || tt >= t1) continue;
+            T *dst;
+            if (is_k) {
+                const int pos = positions[tt], page = block_table[(size_t)q * table_stride + pos / page_size];
+                const size_t slot = (((size_t)page * nkv + (r - nq)) * page_size + pos % page_size) * HD;
+                dst = k_cache + slot;
+                apf_store4(v_cache + slot + 4 * j, y);
+                apf_store4(v_cache + slot + HALF + 4 * j, y + 4);
+            } else {
+                dst = q_out + ((size_t)tt * nq + r) * HD;
+            }
+            const float mul = 1.0f / sqrtf(ss / (float)HD + eps);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) y[e] *= mul * w[e];
+            if (rot) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float cs = cs_s[tt - t0][4 * j + e], sn = sn_s[tt - t0][4 * j + e], a = y[e], b = y[4 + e];
+                    y[e] = a * cs - b * sn;
+                    y[4 + e] = b * cs + a * sn;
+                }
+            }
+            apf_store4(dst + 4 * j, y);
+            apf_store4(dst + HALF + 4 * j, y + 4);
+        }
+    };
+    const int q0 = seq_of_token[t0];
+    if (RUN > 1 && seq_of_token[t1 - 1] == q0) {
+        go(ApfCount<RUN>(), t0, q0);
+    } else {
+        for (int t = t0; t < t1; ++t) go(ApfCount<1>(), t, seq_of_token[t]);
+    }
+}
+
 template <typename T>
 static void apc_launch(dim3 grid, cudaStream_t stream, const float *p, int S, size_t ss, int ld, const float *conv_w, int taps, const float *q_w,
                        const float *k_w, float eps, const float *inv_freq, int rot, float rot_scale, const float *state, size_t st, size_t to,
                        const int *positions, const int *seq_of_token, const int *cu, const int *slots, const int *table, int table_stride, int page_size,
                        T *k_cache, T *v_cache, T *q_out, int n_tokens, int nq, int nkv, int hd, int run) {
+    if ((hd == 32 || hd == 64 || hd == 128) && (rot == hd || rot == 0) && taps <= 4 && ld % 4 == 0 && ss % 4 == 0 && st % 4 == 0 && to % 4 == 0 &&
+        (((uintptr_t)p | (uintptr_t)state) & 15) == 0) {
+        const int per = APF_THREADS / (hd / 8), by = (nq + nkv + per - 1) / per;
+#define APF_GO(HD, R) kestrel_launch(attn_prepare_conv_rows_kernel<T, HD, 4, R>, dim3((n_tokens + R - 1) / R, by), dim3(APF_THREADS), 0, stream, p, S, ss, ld, conv_w, taps, \
+                                     q_w, k_w, eps, inv_freq, rot, rot_scale, state, st, to, positions, seq_of_token, cu, slots, table, table_stride, page_size, \
+                                     k_cache, v_cache, q_out, n_tokens, nq, nkv)
+#define APF_HD(HD) { if (run > 1) APF_GO(HD, APC_RUN); else APF_GO(HD, 1); }
+        if (hd == 32) APF_HD(32)
+        else if (hd == 64) APF_HD(64)
+        else APF_HD(128)
+#undef APF_HD
+#undef APF_GO
+        return;
+    }
 #define APC_GO(PER, TP) kestrel_launch(attn_prepare_conv_kernel<T, PER, TP>, grid, dim3(APC_WARPS * 32), 0, stream, p, S, ss, ld, conv_w, taps, q_w, k_w, eps, \
                                        inv_freq, rot, rot_scale, state, st, to, positions, seq_of_token, cu, slots, table, table_stride, page_size, k_cache, \
                                        v_cache, q_out, n_tokens, nq, nkv, hd, run)

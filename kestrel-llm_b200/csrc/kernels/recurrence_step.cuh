@@ -39,14 +39,14 @@ __device__ __forceinline__ float rst_block_sum(float x, float *red) {
     return tot;
 }
 // A column's causal convolution at token t of a step (first: the request's first token of it): inputs before that from the request's
-// tail [taps - 1][C] at channel c, which is the product's column col.
+// tail [taps - 1][C] at channel c of the filter w [taps][C], which is the product's column col.
 __device__ __forceinline__ float rst_conv(const float *__restrict__ p, int S, size_t slice_stride, int ld, int col, const float *__restrict__ w, int taps,
                                           const float *__restrict__ tail, int C, int c, int first, int t) {
     float y = 0.f;
     for (int j = 0; j < taps; ++j) {
         const int n = t - first - (taps - 1) + j;
         const float x = n >= 0 ? sum_slices(p, S, slice_stride, (size_t)(first + n) * ld + col) : tail[(size_t)(taps - 1 + n) * C + c];
-        y = fmaf(w[(size_t)c * taps + j], x, y);
+        y = fmaf(w[(size_t)j * C + c], x, y);
     }
     return y;
 }

@@ -1,6 +1,6 @@
 // Short causal convolutions over time, one filter per channel, in front of recurrences and of attention:
 //
-//   y[t, c] = act( sum_j w[c, j] u[t - (taps - 1) + j, c] (+ b[c]) ),   act the identity or silu
+//   y[t, c] = act( sum_j w[j, c] u[t - (taps - 1) + j, c] (+ b[c]) ),   act the identity or silu; w [taps][C]
 //
 // u are columns of a product (float32 slices); inputs before a request's first token of this step come from its state slot, which
 // keeps the last taps - 1 of them (float32 [taps - 1][C], oldest first; zeros for a new request) and is brought up to date by a
@@ -10,17 +10,14 @@
 
 #define SC_MAX_TAPS 9
 #define SC_THREADS 128
+#define SC_RUN 8          // tokens of a thread in steps of many
 
-template <int VEC> __device__ __forceinline__ void sc_load(float (&x)[VEC], const float *__restrict__ p, int S, size_t slice_stride, size_t off) {
+template <int VEC> __device__ __forceinline__ void sc_add(float (&x)[VEC], const float *__restrict__ p) {
     if constexpr (VEC == 1) {
-        x[0] = sum_slices(p, S, slice_stride, off);
+        x[0] += p[0];
     } else {
-        x[0] = x[1] = x[2] = x[3] = 0.f;
-#pragma unroll 4
-        for (int s = 0; s < S; ++s) {
-            const float4 v = *reinterpret_cast<const float4 *>(p + (size_t)s * slice_stride + off);
-            x[0] += v.x; x[1] += v.y; x[2] += v.z; x[3] += v.w;
-        }
+        const float4 v = *reinterpret_cast<const float4 *>(p);
+        x[0] += v.x; x[1] += v.y; x[2] += v.z; x[3] += v.w;
     }
 }
 template <int VEC> __device__ __forceinline__ void sc_store(float *dst, const float (&y)[VEC]) {
@@ -36,13 +33,15 @@ template <int VEC> __device__ __forceinline__ void sc_store(__nv_bfloat16 *dst, 
     }
 }
 
-// A thread takes VEC neighbouring channels and `run` tokens one after the other, the filter's inputs in registers.  TP >= taps:
-// the filter is padded in front with zeros.
-template <typename T, int VEC, int TP>
+template <int N> struct ScCount { static constexpr int value = N; };
+
+// A thread takes VEC neighbouring channels and RUN tokens, their inputs in registers.  TP >= taps: the filter is padded in front with
+// zeros.
+template <typename T, int VEC, int TP, int RUN>
 __global__ void __launch_bounds__(SC_THREADS)
 short_conv_kernel(const float *__restrict__ p, int S, size_t slice_stride, int ld, int col0, const float *__restrict__ w, const float *__restrict__ b,
                   int taps, int silu, const float *__restrict__ state, size_t state_stride, size_t tail_off, const int *__restrict__ seq_of_token,
-                  const int *__restrict__ cu_seqlens, const int *__restrict__ slots, T *__restrict__ out, int n_tokens, int C, int run) {
+                  const int *__restrict__ cu_seqlens, const int *__restrict__ slots, T *__restrict__ out, int n_tokens, int C) {
     pdl_launch_dependents();
     const int c0 = (blockIdx.y * SC_THREADS + threadIdx.x) * VEC;
     if (c0 >= C) return;
@@ -51,47 +50,56 @@ short_conv_kernel(const float *__restrict__ p, int S, size_t slice_stride, int l
     for (int e = 0; e < VEC; ++e) {
         bias[e] = b ? b[c0 + e] : 0.f;
 #pragma unroll
-        for (int j = 0; j < TP; ++j) f[j][e] = j >= TP - taps ? w[(size_t)(c0 + e) * taps + j - (TP - taps)] : 0.f;
+        for (int j = 0; j < TP; ++j) f[j][e] = j >= TP - taps ? w[(size_t)(j - (TP - taps)) * C + c0 + e] : 0.f;
     }
     pdl_wait();
-    const int t0 = blockIdx.x * run, t1 = min(t0 + run, n_tokens);
-    float x[TP][VEC];                                        // the inputs, the current token's last
-    int seq = -1, first = 0;
-    for (int t = t0; t < t1; ++t) {
-        const int q = seq_of_token[t];
-        if (q != seq) {
-            seq = q;
-            first = cu_seqlens[q];
-            const float *tail = state + (size_t)slots[q] * state_stride + tail_off;
+    const int t0 = blockIdx.x * RUN, t1 = min(t0 + RUN, n_tokens);
+    // N tokens of one request from t on: all of their inputs and the filter's earlier ones in flight together
+    auto go = [&](auto count, int t, int q) {
+        constexpr int N = decltype(count)::value;
+        const int first = cu_seqlens[q];
+        const float *tail = state + (size_t)slots[q] * state_stride + tail_off;
+        float x[TP - 1 + N][VEC];
 #pragma unroll
-            for (int j = 0; j < TP - 1; ++j) {
-                const int n = t - first - (TP - 1) + j;       // among this step's tokens of the request
-                if (j < TP - taps) {
+        for (int j = 0; j < TP - 1 + N; ++j) {
 #pragma unroll
-                    for (int e = 0; e < VEC; ++e) x[j][e] = 0.f;
-                } else if (n >= 0) {
-                    sc_load<VEC>(x[j], p, S, slice_stride, (size_t)(first + n) * ld + col0 + c0);
-                } else {
+            for (int e = 0; e < VEC; ++e) x[j][e] = 0.f;
+        }
+        const int n0 = t - first - (TP - 1);                  // the first input, among this step's tokens of the request
+        const float *src = p + (size_t)t * ld + col0 + c0 - (size_t)(TP - 1) * ld;
+        for (int s = 0; s < S; ++s, src += slice_stride) {
 #pragma unroll
-                    for (int e = 0; e < VEC; ++e) x[j][e] = tail[(size_t)(taps - 1 + n) * C + c0 + e];
+            for (int j = 0; j < TP - 1 + N; ++j)
+                if (j >= TP - taps && n0 + j >= 0 && t + j - (TP - 1) < t1) sc_add<VEC>(x[j], src + (size_t)j * ld);
+        }
+        if (n0 < 0) {
+#pragma unroll
+            for (int j = 0; j < TP - 1; ++j)
+                if (j >= TP - taps && n0 + j < 0) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) x[j][e] = tail[(size_t)(taps - 1 + n0 + j) * C + c0 + e];
                 }
+        }
+#pragma unroll
+        for (int k = 0; k < N; ++k) {
+            if (t + k >= t1) break;
+            float y[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                float a = 0.f;
+#pragma unroll
+                for (int j = 0; j < TP; ++j) a = fmaf(f[j][e], x[k + j][e], a);
+                a += bias[e];
+                y[e] = silu ? a / (1.0f + expf(-a)) : a;
             }
+            sc_store<VEC>(out + (size_t)(t + k) * C + c0, y);
         }
-        sc_load<VEC>(x[TP - 1], p, S, slice_stride, (size_t)t * ld + col0 + c0);
-        float y[VEC];
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-            float a = 0.f;
-#pragma unroll
-            for (int j = 0; j < TP; ++j) a = fmaf(f[j][e], x[j][e], a);
-            a += bias[e];
-            y[e] = silu ? a / (1.0f + expf(-a)) : a;
-        }
-        sc_store<VEC>(out + (size_t)t * C + c0, y);
-#pragma unroll
-        for (int j = 0; j + 1 < TP; ++j)
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) x[j][e] = x[j + 1][e];
+    };
+    const int q0 = seq_of_token[t0];
+    if (RUN > 1 && seq_of_token[t1 - 1] == q0) {
+        go(ScCount<RUN>(), t0, q0);
+    } else {
+        for (int t = t0; t < t1; ++t) go(ScCount<1>(), t, seq_of_token[t]);
     }
 }
 
@@ -119,13 +127,15 @@ __global__ void short_conv_tail_kernel(const float *__restrict__ p, int S, size_
 template <typename T, int VEC>
 static void sc_launch(const float *p, int S, size_t ss, int ld, int col0, const float *w, const float *b, int taps, int silu, const float *state, size_t st,
                       size_t to, const int *seq_of_token, const int *cu, const int *slots, T *out, int n_tokens, int C, cudaStream_t stream) {
-    const int run = n_tokens >= 512 ? 8 : 1;
+    const int run = n_tokens >= 512 ? SC_RUN : 1;
     const dim3 grid((n_tokens + run - 1) / run, (C / VEC + SC_THREADS - 1) / SC_THREADS);
-#define SC_GO(TP) kestrel_launch(short_conv_kernel<T, VEC, TP>, grid, dim3(SC_THREADS), 0, stream, p, S, ss, ld, col0, w, b, taps, silu, state, st, to, \
-                                 seq_of_token, cu, slots, out, n_tokens, C, run)
-    if (taps <= 2) SC_GO(2);
-    else if (taps <= 4) SC_GO(4);
-    else SC_GO(SC_MAX_TAPS);
+#define SC_GO(TP) if (run > 1) SC_RUN_GO(TP, SC_RUN); else SC_RUN_GO(TP, 1)
+#define SC_RUN_GO(TP, R) kestrel_launch(short_conv_kernel<T, VEC, TP, R>, grid, dim3(SC_THREADS), 0, stream, p, S, ss, ld, col0, w, b, taps, silu, state, st, to, \
+                                 seq_of_token, cu, slots, out, n_tokens, C)
+    if (taps <= 2) { SC_GO(2); }
+    else if (taps <= 4) { SC_GO(4); }
+    else { SC_GO(SC_MAX_TAPS); }
+#undef SC_RUN_GO
 #undef SC_GO
 }
 

@@ -476,6 +476,43 @@ __global__ void gate_columns_mul_kernel(const T *x, const float *__restrict__ g,
     out[t * ldo + i] = from_f32<T>(to_f32<T>(x[idx]) * (1.0f / (1.0f + expf(-z))) * scale);
 }
 
+// four neighbours a thread, where everything lies on vectors' boundaries; the same bits
+__device__ __forceinline__ float4 gcm_load(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ float4 gcm_load(const __nv_bfloat16 *p) {
+    const uint2 u = *reinterpret_cast<const uint2 *>(p);
+    const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162 *>(&u.x), b = *reinterpret_cast<const __nv_bfloat162 *>(&u.y);
+    return make_float4(__bfloat162float(a.x), __bfloat162float(a.y), __bfloat162float(b.x), __bfloat162float(b.y));
+}
+__device__ __forceinline__ void gcm_store(float *p, const float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void gcm_store(__nv_bfloat16 *p, const float4 v) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<uint32_t *>(&a), *reinterpret_cast<uint32_t *>(&b));
+}
+template <typename T>
+__global__ void gate_columns_mul4_kernel(const T *x, const float *__restrict__ g, int S, size_t slice_stride, int ld, int col0,
+                                         const float *__restrict__ bias, float scale, T *out, long long ldo, int n, size_t total) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t idx = 4 * ((size_t)blockIdx.x * blockDim.x + threadIdx.x);
+    if (idx >= total) return;
+    const size_t t = idx / n;
+    const int i = (int)(idx % n);
+    float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float *src = g + t * ld + col0 + i;
+#pragma unroll 4
+    for (int s = 0; s < S; ++s) {
+        const float4 v = gcm_load(src + (size_t)s * slice_stride);
+        z.x += v.x; z.y += v.y; z.z += v.z; z.w += v.w;
+    }
+    if (bias) { z.x += bias[col0 + i]; z.y += bias[col0 + i + 1]; z.z += bias[col0 + i + 2]; z.w += bias[col0 + i + 3]; }
+    float4 v = gcm_load(x + idx);
+    v.x = v.x * (1.0f / (1.0f + expf(-z.x))) * scale;
+    v.y = v.y * (1.0f / (1.0f + expf(-z.y))) * scale;
+    v.z = v.z * (1.0f / (1.0f + expf(-z.z))) * scale;
+    v.w = v.w * (1.0f / (1.0f + expf(-z.w))) * scale;
+    gcm_store(out + t * ldo + i, v);
+}
+
 KESTREL_API int kestrel_gate_columns_mul(void *x, int dtype, const float *g, int S, long long slice_stride, int ld, int col0, const float *bias,
                                          int T, int n, cudaStream_t stream) {
     return kestrel_gate_columns_mul_to(x, dtype, g, S, slice_stride, ld, col0, bias, 1.0f, x, n, T, n, stream);
@@ -488,6 +525,17 @@ KESTREL_API int kestrel_gate_columns_mul_to(const void *x, int dtype, const floa
     KESTREL_REQUIRE(T > 0 && n > 0 && S > 0 && col0 >= 0 && col0 + n <= ld && ldo >= n, "gate_columns_mul: bad sizes");
     size_t total = (size_t)T * n;
     unsigned blocks = (unsigned)((total + 255) / 256);
+    if (n % 4 == 0 && ld % 4 == 0 && col0 % 4 == 0 && slice_stride % 4 == 0 && ldo % 4 == 0 && (((uintptr_t)x | (uintptr_t)g | (uintptr_t)out) & 15) == 0 &&
+        (dtype == KESTREL_F32 || dtype == KESTREL_BF16)) {
+        blocks = (unsigned)((total / 4 + 255) / 256);
+        if (dtype == KESTREL_F32)
+            kestrel_launch(gate_columns_mul4_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float *)x, g, S, (size_t)slice_stride, ld, col0, bias,
+                           scale, (float *)out, ldo, n, total);
+        else
+            kestrel_launch(gate_columns_mul4_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16 *)x, g, S, (size_t)slice_stride, ld,
+                           col0, bias, scale, (__nv_bfloat16 *)out, ldo, n, total);
+        return kestrel_check_launch("gate_columns_mul");
+    }
     if (dtype == KESTREL_F32)
         kestrel_launch(gate_columns_mul_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float *)x, g, S, (size_t)slice_stride, ld, col0, bias, scale,
                        (float *)out, ldo, n, total);

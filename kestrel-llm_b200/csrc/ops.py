@@ -1116,7 +1116,7 @@ def attn_prepare_conv(qk: Partials, conv_w: torch.Tensor, q_norm_w: Optional[tor
                       rotation, state: torch.Tensor, tail_off: int, batch, block_table: torch.Tensor, page_size: int, k_cache: torch.Tensor,
                       v_cache: torch.Tensor, q_out: torch.Tensor, nq: int, nkv: int, hd: int) -> None:
     """Columns [q | k | ...] of a product for a mixer whose values are its keys: q and k through a causal convolution over time
-    (``conv_w`` [(nq + nkv) hd, taps]; earlier inputs from, the last ones to, the slot at ``tail_off``), k as it then is into the V
+    (``conv_w`` [taps, (nq + nkv) hd]; earlier inputs from, the last ones to, the slot at ``tail_off``), k as it then is into the V
     pages; q and k divided by their root mean square per head, times weights [hd] where given, turned by position (rotate-half pairs);
     q to ``q_out``, k into the K pages."""
     _need(q_out, "attn_prepare_conv.q_out", dims=2)
@@ -1126,8 +1126,8 @@ def attn_prepare_conv(qk: Partials, conv_w: torch.Tensor, q_norm_w: Optional[tor
     _need(k_cache, "attn_prepare_conv.k_cache", q_out.dtype, 4)
     _need(v_cache, "attn_prepare_conv.v_cache", q_out.dtype, 4)
     T, C = q_out.shape[0], (nq + nkv) * hd
-    taps = conv_w.shape[1]
-    if qk.tokens != T or qk.width < C or qk.bias is not None or q_out.shape[1] != nq * hd or conv_w.shape[0] != C or \
+    taps = conv_w.shape[0]
+    if qk.tokens != T or qk.width < C or qk.bias is not None or q_out.shape[1] != nq * hd or conv_w.shape[1] != C or \
             tail_off + (taps - 1) * C > state.shape[1]:
         raise KernelError("attn_prepare_conv: shapes differ, or a bias is pending")
     for c in (k_cache, v_cache):
@@ -1526,13 +1526,13 @@ def head_gemm_set_plain(on: bool = True) -> None:
 
 def short_conv(x: Partials, conv_w: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, tail_off: int, batch, out: torch.Tensor,
                col0: int = 0, silu: bool = True) -> None:
-    """out[t, c] = act(causal convolution over time of x's columns col0 .. col0 + C, plus ``bias``), C = conv_w.shape[0], act silu or
+    """out[t, c] = act(causal convolution over time of x's columns col0 .. col0 + C, plus ``bias``), ``conv_w`` [taps, C], act silu or
     nothing; inputs before the step come from, and the last taps - 1 inputs go to, each request's state slot (``state`` float32
     [slots, size], the tail [taps - 1, C] at ``tail_off``)."""
     _need(conv_w, "short_conv.w", torch.float32, 2)
     _need(state, "short_conv.state", torch.float32, 2)
     _need(out, "short_conv.out", dims=2)
-    C, taps = conv_w.shape
+    taps, C = conv_w.shape
     T = out.shape[0]
     if x.tokens != T or x.width < col0 + C or out.shape[1] != C or x.bias is not None or tail_off + (taps - 1) * C > state.shape[1]:
         raise KernelError("short_conv: shapes differ")
@@ -1796,7 +1796,7 @@ def ssm_step(fused: Partials, col_z: int, col_x: int, col_dt: int, conv_w: torch
              A_log: torch.Tensor, D: torch.Tensor, state: torch.Tensor, tail_off: int, batch, H: int, G: int, N: int, P: int) -> torch.Tensor:
     """Steps of few tokens: convolution, state, read-out, skip and gate in one kernel; returns the gated y float32 [T, H P], for `part_norm`."""
     _need(state, "ssm_step.state", torch.float32, 2)
-    C, taps = conv_w.shape
+    taps, C = conv_w.shape
     if fused.bias is not None or C != H * P + 2 * G * N or max(col_z + H * P, col_x + C, col_dt + H) > fused.width or \
             tail_off + (taps - 1) * C > state.shape[1]:
         raise KernelError("ssm_step: shapes differ, or a bias is pending")
@@ -1871,7 +1871,7 @@ def delta_head_step(fused: Partials, col_g: int, col_beta: int, col_a: int, conv
         return False
     _need(state, "delta_head_step.state", torch.float32, 2)
     _need(out, "delta_head_step.out", dims=2)
-    C, taps = conv_w.shape
+    taps, C = conv_w.shape
     if fused.bias is not None or C != 2 * G * d + H * dv or max(C, col_g + H * dv, col_beta + H, col_a + H) > fused.width or \
             tail_off + (taps - 1) * C > state.shape[1] or out.shape != (fused.tokens, H * dv):
         raise KernelError("delta_head_step: shapes differ, or a bias is pending")

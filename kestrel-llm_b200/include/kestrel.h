@@ -267,7 +267,7 @@ KESTREL_API int kestrel_head_norm_act_to(const float *o, const float *w, int w_s
 /* o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t, then S_t = diag(w_t) S_(t-1) + k_t v_t^T; u [H, d] */
 KESTREL_API int kestrel_recurrence_scan_bonus(const float *r, const float *w, const float *k, const float *v, const float *u, float *state, long long state_stride, long long state_off, const int *cu_seqlens, const int *slots, float *out, int nseq, int H, int d, int dv, kestrel_stream_t stream);
 
-/* ---- short causal convolutions per channel (short_conv.cu): out[t, c] = act(sum_j w[c, j] u[t - (taps - 1) + j, c] + bias[c]), u the product's columns col0 .. col0 + C, act silu or none; inputs before the step from, and the last taps - 1 inputs to, the request's state slot (float32 [taps - 1, C] at tail_off) ---- */
+/* ---- short causal convolutions per channel (short_conv.cu): out[t, c] = act(sum_j w[j, c] u[t - (taps - 1) + j, c] + bias[c]), u the product's columns col0 .. col0 + C, act silu or none; inputs before the step from, and the last taps - 1 inputs to, the request's state slot (float32 [taps - 1, C] at tail_off) ---- */
 KESTREL_API int kestrel_short_conv(const float *partial, int S, long long slice_stride, int ld, int col0, const float *w, const float *bias, int taps, int silu, float *state, long long state_stride, long long tail_off, const int *seq_of_token, const int *cu_seqlens, const int *slots, void *out, int dtype, int T, int nseq, int C, kestrel_stream_t stream);
 /* the second half alone: the last taps - 1 inputs into the slot */
 KESTREL_API int kestrel_short_conv_tail(const float *partial, int S, long long slice_stride, int ld, int col0, int taps, float *state, long long state_stride, long long tail_off, const int *cu_seqlens, const int *slots, int nseq, int C, kestrel_stream_t stream);

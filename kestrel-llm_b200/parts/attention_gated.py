@@ -96,7 +96,7 @@ class GatedWindowAttention(Mixer):
         self.proj = Linear(width, self.q_cols + self.kv_cols + self.gate_cols, dtype, device, bias=bias)
         self.out_features = heads * v_head_dim
         self.out = Linear(heads * v_head_dim, width, dtype, device, bias=bias if out_bias is None else bool(out_bias)) if out_proj else None
-        self.conv_w = torch.empty((self.q_cols + self.kv_cols, conv_taps), dtype=torch.float32, device=device) if conv_taps else None
+        self.conv_w = torch.empty((conv_taps, self.q_cols + self.kv_cols), dtype=torch.float32, device=device) if conv_taps else None
         self.state_off = 0         # where the mixer's own state starts in the request's slot (a container of two mixers moves it)
         self.state_size = max(4, (conv_taps - 1) * (self.q_cols + self.kv_cols)) if conv_taps else 0
         self.rotation = position.rotary() if position is not None else None
@@ -162,7 +162,7 @@ class GatedWindowAttention(Mixer):
         if self.out is not None:
             slots.append(WeightSlot(p + no, self.out.weight))
         if self.conv_w is not None:
-            slots += [WeightSlot(p + nq + ".conv", self.conv_w[:self.q_cols], "bias"), WeightSlot(p + nk + ".conv", self.conv_w[self.q_cols:], "bias")]
+            slots += [WeightSlot(p + nq + ".conv", self.conv_w.t()[:self.q_cols], "bias"), WeightSlot(p + nk + ".conv", self.conv_w.t()[self.q_cols:], "bias")]
         x = self.extra_names
         if self.proj.bias is not None:
             b = self.proj.bias

@@ -52,7 +52,7 @@ class ChannelDeltaMixer(Mixer):
         self.a2 = Linear(decay_rank, heads * key_dim, dtype, device)
         self.g2 = Linear(gate_rank, vv, dtype, device)
         self.out = Linear(vv, width, dtype, device)
-        self.conv_w = torch.empty((self.C, taps), dtype=torch.float32, device=device)
+        self.conv_w = torch.empty((taps, self.C), dtype=torch.float32, device=device)    # a checkpoint stores [C, taps]
         self.A_log = torch.empty((heads,), dtype=torch.float32, device=device)
         self.dt_bias = torch.empty((heads * key_dim,), dtype=torch.float32, device=device)
         self.norm_w = torch.empty((value_dim,), dtype=torch.float32, device=device)
@@ -67,8 +67,8 @@ class ChannelDeltaMixer(Mixer):
         return [WeightSlot(p + "q", w[:qk]), WeightSlot(p + "k", w[qk:2 * qk]), WeightSlot(p + "v", w[2 * qk:self.C]),
                 WeightSlot(p + "b", w[self.col_beta:self.col_a1]), WeightSlot(p + "a1", w[self.col_a1:self.col_g1]),
                 WeightSlot(p + "g1", w[self.col_g1:]),
-                WeightSlot(p + "q.conv", self.conv_w[:qk]), WeightSlot(p + "k.conv", self.conv_w[qk:2 * qk]),
-                WeightSlot(p + "v.conv", self.conv_w[2 * qk:]),
+                WeightSlot(p + "q.conv", self.conv_w.t()[:qk]), WeightSlot(p + "k.conv", self.conv_w.t()[qk:2 * qk]),
+                WeightSlot(p + "v.conv", self.conv_w.t()[2 * qk:]),
                 WeightSlot(p + "a2", self.a2.weight), WeightSlot(p + "g2", self.g2.weight), WeightSlot(p + "o", self.out.weight),
                 WeightSlot(p + "A_log", self.A_log, "bias"), WeightSlot(p + "dt_bias", self.dt_bias, "bias"),
                 WeightSlot(p + "norm", self.norm_w, "norm")]
@@ -115,7 +115,7 @@ class HeadDeltaMixer(Mixer):
         self.in_proj = Linear(width, self.C + vv + 2 * heads, dtype, device)
         self.out = Linear(vv, width, dtype, device)
         f32 = dict(dtype=torch.float32, device=device)
-        self.conv_w = torch.empty((self.C, taps), **f32)
+        self.conv_w = torch.empty((taps, self.C), **f32)       # a checkpoint stores [C, taps]
         self.A_log, self.dt_bias = torch.empty((heads,), **f32), torch.empty((heads,), **f32)
         self.norm_w = torch.empty((value_dim,), **f32)
         self.tail_off = (heads * key_dim * value_dim + 3) // 4 * 4     # the slot: S [H, d, dv], then the convolutions' tail [taps - 1, C]
@@ -128,8 +128,8 @@ class HeadDeltaMixer(Mixer):
         p, w, qk = self.prefix, self.in_proj.weight, self.G * self.d
         return [WeightSlot(p + "q", w[:qk]), WeightSlot(p + "k", w[qk:2 * qk]), WeightSlot(p + "v", w[2 * qk:self.C]),
                 WeightSlot(p + "g", w[self.col_g:self.col_beta]), WeightSlot(p + "b", w[self.col_beta:self.col_a]), WeightSlot(p + "a", w[self.col_a:]),
-                WeightSlot(p + "q.conv", self.conv_w[:qk], "bias"), WeightSlot(p + "k.conv", self.conv_w[qk:2 * qk], "bias"),
-                WeightSlot(p + "v.conv", self.conv_w[2 * qk:], "bias"), WeightSlot(p + "o", self.out.weight),
+                WeightSlot(p + "q.conv", self.conv_w.t()[:qk], "bias"), WeightSlot(p + "k.conv", self.conv_w.t()[qk:2 * qk], "bias"),
+                WeightSlot(p + "v.conv", self.conv_w.t()[2 * qk:], "bias"), WeightSlot(p + "o", self.out.weight),
                 WeightSlot(p + "A_log", self.A_log, "bias"), WeightSlot(p + "dt_bias", self.dt_bias, "bias"), WeightSlot(p + "norm", self.norm_w, "norm")]
 
     def forward(self, x: torch.Tensor, batch, cache) -> ops.Partials:

@@ -47,7 +47,7 @@ class StateSpaceMixer(Mixer):
         self.in_proj = Linear(width, self.inner + self.C + heads, dtype, device)
         self.out = Linear(self.inner, width, dtype, device)
         f32 = dict(dtype=torch.float32, device=device)
-        self.conv_w, self.conv_b = torch.empty((self.C, taps), **f32), torch.empty((self.C,), **f32)
+        self.conv_w, self.conv_b = torch.empty((taps, self.C), **f32), torch.empty((self.C,), **f32)
         self.dt_bias, self.A_log, self.D = (torch.empty((heads,), **f32) for _ in range(3))
         self.norm_w = torch.empty((self.inner,), **f32)
         self.tail_off = (heads * state * value_dim + 3) // 4 * 4       # the slot: S [H, N, P], then the convolution's tail [taps - 1, C]
@@ -58,7 +58,7 @@ class StateSpaceMixer(Mixer):
 
     def weight_slots(self) -> List[WeightSlot]:
         p = self.prefix
-        return [WeightSlot(p + "in", self.in_proj.weight), WeightSlot(p + "conv", self.conv_w, "bias"), WeightSlot(p + "conv.b", self.conv_b, "bias"),
+        return [WeightSlot(p + "in", self.in_proj.weight), WeightSlot(p + "conv", self.conv_w.t(), "bias"), WeightSlot(p + "conv.b", self.conv_b, "bias"),
                 WeightSlot(p + "dt_bias", self.dt_bias, "bias"), WeightSlot(p + "A_log", self.A_log, "bias"), WeightSlot(p + "D", self.D, "norm"),
                 WeightSlot(p + "norm", self.norm_w, "norm"), WeightSlot(p + "o", self.out.weight)]
 
