@@ -88,8 +88,10 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     const int *table = p.block_table + (size_t)seq * p.table_stride;
     const int slice_len = attn_slice_len(p);
     const int first_tok = row0 / G, last_tok = (row0 + rows_here - 1) / G;
-    int k_hi = min(pos_begin + last_tok + 1, (slice + 1) * slice_len);          // exclusive
-    const int k_first = max(p.window > 0 ? max(0, pos_begin + first_tok - p.window + 1) : 0, slice * slice_len);
+    // a layer with a window may count its slices from the first tile that the window touches
+    const int seen = p.window > 0 ? max(0, pos_begin + first_tok - p.window + 1) : 0, slice0 = (p.slices_from_window ? seen / AD_BN * AD_BN : 0) + slice * slice_len;
+    int k_hi = min(pos_begin + last_tok + 1, slice0 + slice_len);          // exclusive
+    const int k_first = max(seen, slice0);
     const int k_lo = (k_first / AD_BN) * AD_BN;
     const int n_tiles = k_hi > k_lo ? (k_hi - k_lo + AD_BN - 1) / AD_BN : 0;
 
@@ -205,6 +207,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                 for (int e = 0; e < 4; ++e) {
                     int i = e >> 1;
                     float v = s[nt][e] * p.scale_log2;
+                    // cap * tanh(s / cap) in base-2 units, tanh(x) = 1 - 2 / (1 + e^2x) from one ex2 and one rcp
+                    if (p.cap_out > 0.f) v = fmaf(-2.0f * p.cap_out, HeadScore::score_rcp(1.0f + fast_exp2(v * p.cap_in)), p.cap_out);
                     if (!whole) {
                         int key = kbase + nt * 8 + 2 * (lane & 3) + (e & 1);
                         bool vis = key <= pos_r[i] && key >= lo_r[i] && key < k_hi && key >= k_first;
@@ -424,7 +428,20 @@ KESTREL_API int kestrel_attention_decode(const void *q, const void *k_cache, con
                                          int table_width, int table_stride, int page_size, int cache_pages, int T, int nq,
                                          int nkv, int hd, int window, int slices, int slice_len, const int *max_kv_ptr,
                                          float scale, cudaStream_t stream) {
+    return kestrel_attention_decode_capped(q, k_cache, v_cache, out, part_o, part_ml, tile_seq, tile_row0, tiles, cu_seqlens, kv_lens, block_table, table_width,
+                                           table_stride, page_size, cache_pages, T, nq, nkv, hd, window, slices, slice_len, max_kv_ptr, 0, scale, 0.f, stream);
+}
+
+// The same with scores bounded by softcap * tanh(s / softcap) (0: none); slices_from_window: slice s covers slice_len keys from the
+// first 64-key tile that the window of its rows touches plus s * slice_len, so slices * slice_len need reach the window only.
+KESTREL_API int kestrel_attention_decode_capped(const void *q, const void *k_cache, const void *v_cache, void *out,
+                                         float *part_o, float *part_ml, const int *tile_seq, const int *tile_row0,
+                                         int tiles, const int *cu_seqlens, const int *kv_lens, const int *block_table,
+                                         int table_width, int table_stride, int page_size, int cache_pages, int T, int nq,
+                                         int nkv, int hd, int window, int slices, int slice_len, const int *max_kv_ptr,
+                                         int slices_from_window, float scale, float softcap, cudaStream_t stream) {
     if (T == 0 || tiles == 0) return 0;
+    KESTREL_REQUIRE(softcap >= 0.f && (!slices_from_window || (window > 0 && !max_kv_ptr)), "attention_decode: slices from a window that is not there");
     KESTREL_REQUIRE(kestrel_attention_decode_supported(hd, page_size),
                     "attention_decode: head size %d with pages of %d keys; the head size must be 64 or 128 and the page size a multiple of 8 that divides 64 or is a multiple of it", hd, page_size);
     KESTREL_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0 && nq / nkv <= 16, "attention_decode: %d query heads over %d kv heads", nq, nkv);
@@ -444,8 +461,12 @@ KESTREL_API int kestrel_attention_decode(const void *q, const void *k_cache, con
     p.out = (__nv_bfloat16 *)out; p.part_o = part_o; p.part_ml = part_ml; p.tile_seq = tile_seq; p.tile_row0 = tile_row0;
     p.cu_seqlens = cu_seqlens; p.kv_lens = kv_lens; p.block_table = block_table; p.table_width = table_width;
     p.table_stride = table_stride; p.page_size = page_size; p.nq = nq; p.nkv = nkv; p.hd = hd; p.window = window;
-    p.slices = slices; p.slice_len = slice_len; p.max_kv_ptr = max_kv_ptr;
+    p.slices = slices; p.slice_len = slice_len; p.max_kv_ptr = max_kv_ptr; p.slices_from_window = slices_from_window;
     p.scale_log2 = scale * 1.4426950408889634f;
+    if (softcap > 0.f) {
+        p.cap_in = 2.0f / softcap;                    // on a score in base-2 units: 2^(v cap_in) = e^(2 s / cap)
+        p.cap_out = softcap * 1.4426950408889634f;
+    }
     // up to AD_MAX_CLUSTER slices are merged inside the kernel by a cluster; more go through scratch
     const bool cluster = slices > 1 && slices <= AD_MAX_CLUSTER;
     if (cluster) rc = hd == 64 ? launch_decode<64, true>(mk, mv, p, tiles, cache_pages, stream) : launch_decode<128, true>(mk, mv, p, tiles, cache_pages, stream);

@@ -26,6 +26,8 @@ struct AttnParams {
     ScoreOpts opts;
     int scored;
     int partial_only;               // attention_decode.cu: the unnormalised outputs go to part_o / part_ml even from one slice
+    float cap_in, cap_out;          // attention_decode.cu: a bound on the scores, in base-2 units (cap_out 0: none)
+    int slices_from_window;         // attention_decode.cu: slices count from the first key tile the window touches
     // two maps a head over the same values (differential attention); read by attention_tc.cu only
     DifferentialOpts maps;
 };

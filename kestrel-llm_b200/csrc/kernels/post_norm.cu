@@ -63,7 +63,13 @@ post_norm_kernel(float *__restrict__ residual, const Source src, const float *__
     __shared__ int row_s[PN_MAX_TOP];                 // MOE: the rows of the token's experts, -1 for an identity expert
     __shared__ float direct_s, gate_s;
     const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x, warp = tid >> 5, lane = tid & 31;
-    float4 v[NV];
+    float4 v[NV], g[NV], gn[NV];
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {                    // weights: before the wait
+        const int i = 4 * (tid + c * nt);
+        g[c] = i < d ? pn_load(w + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        gn[c] = next_w && i < d ? pn_load(next_w + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     if constexpr (MOE) {
         pdl_wait();
         if (tid < 32) {
@@ -124,15 +130,14 @@ post_norm_kernel(float *__restrict__ residual, const Source src, const float *__
 #pragma unroll
         for (int c = 0; c < NV; ++c) pn_add(v[c], b[c]);
     }
-    float4 x[NV], g[NV];
+    float4 x[NV];
     float ss = 0.f;
 #pragma unroll
     for (int c = 0; c < NV; ++c) {
         const int i = 4 * (tid + c * nt);
-        x[c] = g[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+        x[c] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (i >= d) continue;
         x[c] = pn_load(residual + (size_t)t * d + i);
-        g[c] = pn_load(w + i);
         ss = fmaf(v[c].x, v[c].x, fmaf(v[c].y, v[c].y, fmaf(v[c].z, v[c].z, fmaf(v[c].w, v[c].w, ss))));
     }
     ss = warp_sum(ss);
@@ -158,7 +163,6 @@ post_norm_kernel(float *__restrict__ residual, const Source src, const float *__
     for (int c = 0; c < NV; ++c) {
         const int i = 4 * (tid + c * nt);
         if (i >= d) continue;
-        g[c] = pn_load(next_w + i);
         ss = fmaf(x[c].x, x[c].x, fmaf(x[c].y, x[c].y, fmaf(x[c].z, x[c].z, fmaf(x[c].w, x[c].w, ss))));
     }
     ss = warp_sum(ss);
@@ -172,7 +176,7 @@ post_norm_kernel(float *__restrict__ residual, const Source src, const float *__
     for (int c = 0; c < NV; ++c) {
         const int i = 4 * (tid + c * nt);
         if (i >= d) continue;
-        pn_store(copy + (size_t)t * d + i, make_float4(x[c].x * mul2 * g[c].x, x[c].y * mul2 * g[c].y, x[c].z * mul2 * g[c].z, x[c].w * mul2 * g[c].w));
+        pn_store(copy + (size_t)t * d + i, make_float4(x[c].x * mul2 * gn[c].x, x[c].y * mul2 * gn[c].y, x[c].z * mul2 * gn[c].z, x[c].w * mul2 * gn[c].w));
     }
 }
 

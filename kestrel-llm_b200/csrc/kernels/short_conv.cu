@@ -90,7 +90,7 @@ short_conv_kernel(const float *__restrict__ p, int S, size_t slice_stride, int l
 #pragma unroll
                 for (int j = 0; j < TP; ++j) a = fmaf(f[j][e], x[k + j][e], a);
                 a += bias[e];
-                y[e] = silu ? a / (1.0f + expf(-a)) : a;
+                y[e] = !silu ? a : sizeof(T) == 2 ? __fdividef(a, 1.0f + __expf(-a)) : a / (1.0f + expf(-a));
             }
             sc_store<VEC>(out + (size_t)(t + k) * C + c0, y);
         }

@@ -1389,6 +1389,44 @@ def attention_decode_maps(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
     return True
 
 
+def attention_decode_capped(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch, block_table: torch.Tensor, page_size: int,
+                            out: torch.Tensor, nq: int, nkv: int, hd: int, window: int, scale: float, softcap: float = 0.0) -> bool:
+    """A step of one token per request on the TMA decode kernel (head size 64 or 128, at most 16 heads a group), scores bounded by
+    softcap * tanh(s / softcap) where given; keys - those of the window, or of the longest request - cut into slices that fill the device.
+    False if the step or the sizes are not taken; nothing has run then."""
+    lib = library()
+    if batch.max_count != 1 or nq // nkv > 16 or not lib.kestrel_attention_decode_supported(hd, int(page_size)):
+        return False
+    _need(q, "attention_decode_capped.q", torch.bfloat16, 2)
+    _need(out, "attention_decode_capped.out", torch.bfloat16, 2)
+    _need(k_cache, "attention_decode_capped.k_cache", torch.bfloat16, 4)
+    _need(v_cache, "attention_decode_capped.v_cache", torch.bfloat16, 4)
+    T = q.shape[0]
+    if q.shape[1] != nq * hd or out.shape != q.shape or tuple(k_cache.shape[1:]) != (nkv, page_size, hd) or v_cache.shape != k_cache.shape:
+        raise KernelError("attention_decode_capped: shapes differ")
+    n = int(batch.num_seqs)
+    tile_seq, tile_row0 = _single_token_tiles(n, q.device)
+    keys = min(window + 63, max(1, int(batch.max_kv_len))) if window and not batch.captured else window + 63 if window else max(1, int(batch.max_kv_len))
+    cand = max(1, min(lib.kestrel_attention_decode_slots(hd) // max(1, n * nkv), -(-keys // 128), 32))
+    in_cluster = lib.kestrel_attention_decode_cluster_slices()
+    if cand > in_cluster and keys <= 384 * in_cluster:
+        cand = in_cluster                      # few keys: what a slice saves is less than a second kernel that merges them costs
+    slice_len = (-(-keys // cand) + 63) // 64 * 64
+    slices = -(-keys // slice_len)
+    # a recorded step fixes the number of slices; without a window their length follows the longest request on the device
+    follow = batch.device_buffer.data_ptr() + 4 * int(batch.layout[_cdecl.constants()["KB_O_MAX_KV"]]) if batch.captured and not window else None
+    part = torch.empty((T * nq * slices * (hd + 2),), dtype=torch.float32, device=q.device) if slices > in_cluster else None
+    _check(lib.kestrel_attention_decode_capped(
+        q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), _p(part), part.data_ptr() + 4 * T * nq * slices * hd if part is not None else None,
+        tile_seq.data_ptr(), tile_row0.data_ptr(), n, batch.cu_seqlens.data_ptr(), batch.kv_lens.data_ptr(), block_table.data_ptr(), block_table.shape[1],
+        block_table.stride(0), int(page_size), int(k_cache.shape[0]), T, nq, nkv, hd, int(window), slices, slice_len, follow, 1 if window else 0,
+        float(scale), float(softcap), _stream()))
+    if part is not None:
+        global launches
+        launches += 1              # the merge kernel
+    return True
+
+
 def attention_window_maps(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch, block_table: torch.Tensor, page_size: int,
                           out: torch.Tensor, nq: int, nkv: int, dim: int, vd: int, scale: float, lambdas, diff: float, eps: float) -> bool:
     """Differential attention of a step of few tokens on the kernel of `attention_window`, whose merge of the keys' shares combines and

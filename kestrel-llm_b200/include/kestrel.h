@@ -419,6 +419,8 @@ KESTREL_API int kestrel_attention_tc_supported(int hd, int page_size);
 KESTREL_API int kestrel_attention_tc_slots(void);
 KESTREL_API int kestrel_attention_tc_error(void);
 KESTREL_API int kestrel_attention_decode(const void *q, const void *k_cache, const void *v_cache, void *out, float *part_o, float *part_ml, const int *tile_seq, const int *tile_row0, int tiles, const int *cu_seqlens, const int *kv_lens, const int *block_table, int table_width, int table_stride, int page_size, int cache_pages, int T, int nq, int nkv, int hd, int window, int slices, int slice_len, const int *max_kv_ptr, float scale, kestrel_stream_t stream);
+/* the same with scores bounded by softcap tanh(s / softcap) (0: none); slices_from_window 1: slices count from the first 64-key tile the window touches */
+KESTREL_API int kestrel_attention_decode_capped(const void *q, const void *k_cache, const void *v_cache, void *out, float *part_o, float *part_ml, const int *tile_seq, const int *tile_row0, int tiles, const int *cu_seqlens, const int *kv_lens, const int *block_table, int table_width, int table_stride, int page_size, int cache_pages, int T, int nq, int nkv, int hd, int window, int slices, int slice_len, const int *max_kv_ptr, int slices_from_window, float scale, float softcap, kestrel_stream_t stream);
 KESTREL_API int kestrel_attention_decode_supported(int hd, int page_size);
 KESTREL_API int kestrel_attention_decode_slots(int hd);
 KESTREL_API int kestrel_attention_decode_cluster_slices(void);

@@ -55,6 +55,7 @@ from .linear import Linear
 class GatedWindowAttention(Mixer):
     force_plain = False        # tests: bfloat16 through the plain kernel too, the twin of the tensor-core one
     tcgen05 = True             # tests: off, portions of head size 128 stay on the mma.sync kernel
+    decode = True              # tests: off, single tokens stay on the mma.sync kernel
     TC_SLICE = 512             # fewest keys a slice where a portion's key range is cut (softmax weights, no window)
     TC_SLICE_FILL = 148        # CTAs that the cut should reach: one an SM
     TC_MIN_ROWS = 64           # a step whose longest portion has more rows (tokens x heads of a group) takes the tcgen05 kernel
@@ -139,6 +140,7 @@ class GatedWindowAttention(Mixer):
         self.sink = torch.empty((heads,), **f32) if head_sink else None
         self.score = ops.ScoreOptions(softcap, self.r1, self.r2, self.pb, weighting, self.sink, self.rel, self.rel_bucket)
         self._scored = bool(softcap) or distance_bias or weighting != "softmax" or self.rel is not None
+        self._capped_only = not distance_bias and weighting == "softmax" and self.rel is None
         # checkpoint names of what the options add, after the projections' own names
         self.extra_names = dict(bias=".b", q_norm=names[0] + ".norm", k_norm=names[1] + ".norm", r1="r1", r2="r2", head_bias="pb",
                                 sink="sink", rel="rel")
@@ -245,6 +247,11 @@ class GatedWindowAttention(Mixer):
             ops.attention_tc(q, cache.k, cache.v, a, tile_seq, tile_row0, batch.cu_seqlens, batch.kv_lens, table, cache.page_size, self.heads,
                              self.kv_heads, 128, self.window, self.scale, slices=slices,
                              slice_len=slice_len, rows_per_tile=256, score=score)
+        elif self.dtype == torch.bfloat16 and not self.force_plain and self.decode and self._capped_only and gate is None and \
+                self.head_dim == self.v_head_dim and self.keep_first == 0 and \
+                ops.attention_decode_capped(q, cache.k, cache.v, batch, table, cache.page_size, a, self.heads, self.kv_heads, self.head_dim, self.window,
+                                            self.scale, self.score.softcap):
+            pass                                    # one token a request at head size 64 or 128
         elif self.dtype == torch.bfloat16 and not self.force_plain and \
                 ops.attention_window_supported(self.head_dim, self.v_head_dim, self.heads, self.kv_heads):
             ops.attention_window(q, cache.k, cache.v, batch, table, cache.page_size, a, self.heads, self.kv_heads, self.head_dim,

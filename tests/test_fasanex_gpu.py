@@ -288,6 +288,45 @@ def test_window_edges(dtype, decode, d, window):
         _close(got[i], want[i], dtype, f"window {window}, the row that asks", tol={"float32": 3e-4, "bfloat16": 5e-2}[dtype])
 
 
+@pytest.mark.parametrize("captured", [False, True])
+@pytest.mark.parametrize("d,G,H", [(128, 2, 4), (64, 1, 4), (128, 1, 16)])
+@pytest.mark.parametrize("window,cap", [(0, 5.0), (0, 0.0), (100, 5.0), (700, 8.0), (1500, 0.0), (4000, 6.0)])
+def test_single_tokens_on_the_decode_kernel(captured, window, cap, d, G, H):
+    """Capped scores over a window, or all keys, on the TMA decode kernel against the mma.sync kernel: requests of very unequal lengths in
+    one step, key ranges cut into slices inside a cluster and through scratch, with a recorded step's fixed number of slices."""
+    import torch
+    from types import SimpleNamespace
+    from kestrel_llm_b200.cache import CacheManager
+    from kestrel_llm_b200.csrc import ops
+    from kestrel_llm_b200.engine.batch import Entry, StepBatch
+    from kestrel_llm_b200.parts import PagedKVSpec
+    lengths = [1, 63, 64, 65, 700, 1499, 1500, 1501, 2900]
+    cache = CacheManager([PagedKVSpec(G, d)], torch.bfloat16, "cuda:0", 16, sum(-(-(n + 1) // 16) for n in lengths) + 4, 12, 1 << 12)
+    cache.shuffle_free(3)
+    gen = torch.Generator(device="cuda:0").manual_seed(d + window)
+    cache.k[0].normal_(0.0, 1.0, generator=gen)
+    cache.v[0].normal_(0.0, 1.0, generator=gen)
+    entries = []
+    for i, n in enumerate(lengths):
+        cache.admit(i)
+        cache.reserve(i, n)
+        cache.commit(i, n)
+        cache.reserve(i, 1)
+        entries.append(Entry(i, [0], []))
+    batch = StepBatch(entries, cache, "cuda:0")
+    if captured:
+        batch = SimpleNamespace(**{k: getattr(batch, k) for k in ("max_count", "num_seqs", "max_kv_len", "cu_seqlens", "kv_lens", "device_buffer", "layout",
+                                                                "positions", "seq_of_token", "num_tokens", "counts")}, captured=True)
+    q = torch.empty((len(lengths), H * d), dtype=torch.bfloat16, device="cuda:0").normal_(0.0, 1.0, generator=gen)
+    table = StepBatch.block_table(batch, 0) if not captured else StepBatch(entries, cache, "cuda:0").block_table(0)
+    out, want = torch.empty_like(q), torch.empty_like(q)
+    assert ops.attention_decode_capped(q, cache.k[0], cache.v[0], batch, table, 16, out, H, G, d, window, d ** -0.5, cap)
+    ops.raise_on_kernel_error()
+    ops.attention_plain_ex(q, cache.k[0], cache.v[0], batch.positions, batch.seq_of_token, table, 16, want, H, G, d, d, window, 0, None, d ** -0.5,
+                           ops.ScoreOptions(cap))
+    _close(out.float().cpu().numpy(), want.float().cpu().numpy(), "bfloat16", f"window {window}, cap {cap}", tol=1.5e-2)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_rotation_ramp_and_far_positions(dtype):
     """Positions into the thousands, a rotation over part of the head whose ramp starts and ends inside its pairs; the plain result with
