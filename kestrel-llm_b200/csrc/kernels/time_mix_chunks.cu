@@ -7,8 +7,8 @@
 //
 // The scores' exponents are sums of logarithms of decays, at most 0, but their two halves are not: e^{-L_j} alone overflows.  So a warp's
 // sixteen tokens take the state of the sums in front of THEM as the reference for all earlier sixteens - r_i e^{E_i - ref} and
-// k_j e^{ref - L_j} are both at most in size what r and k are, and their product is one on the tensor cores - and the pairs inside the
-// sixteen are summed channel by channel with their own exponent in float32.
+// k_j e^{ref - L_j} are both at most in size what r and k are, and their product is one on the tensor cores -, its last eight the same way
+// for its first eight, and the pairs inside an eight are summed channel by channel with their own exponent in float32.
 //
 // r, k, v are the bfloat16 operands the projections give; what the decays touch is float32 and enters a product as two bfloat16 terms.
 #include "decay_chunks.cuh"
@@ -222,33 +222,37 @@ time_mix_chunk_out_kernel(const TimeMixChunkParams p) {
     dc_load_rows<D>(Ks, p.k + t0 * ld + (size_t)h * d, ld, n, d, tid);
     dc_commit();
     load_slice(0);                                    // under the scores
-    for (int c = tid; c < D; c += 128) {
-        float s = 0.f;
-        const float *src = p.log_w + t0 * ld + (size_t)h * d + c;
-        us[c] = c < d ? p.u[(size_t)h * d + c] : 0.f;
-        Ls[c] = 0.f;
-        for (int j0 = 0; j0 < DC_C; j0 += 16) {
-            float lw[16];
+    // the running sums, in base-2 units: half a chunk's tokens of a channel a thread, all of its loads in flight; the second half
+    // then gets the first one's total
+    for (int idx = tid; idx < 2 * D; idx += 128) {
+        const int c = idx % D, j0 = idx / D * (DC_C / 2);
+        const float *src = p.log_w + (t0 + j0) * ld + (size_t)h * d + c;
+        float lw[DC_C / 2], s = 0.f;
 #pragma unroll
-            for (int j = 0; j < 16; ++j) lw[j] = j0 + j < n && c < d ? src[(size_t)(j0 + j) * ld] : 0.f;
+        for (int j = 0; j < DC_C / 2; ++j) lw[j] = j0 + j < n && c < d ? src[(size_t)j * ld] : 0.f;
 #pragma unroll
-            for (int j = 0; j < 16; ++j) {
-                s += lw[j];
-                Ls[(j0 + j + 1) * LDL + c] = s;
-            }
+        for (int j = 0; j < DC_C / 2; ++j) {
+            s += lw[j];
+            Ls[(j0 + j + 1) * LDL + c] = s * 1.4426950408889634f;
+        }
+        if (j0 == 0) {
+            us[c] = c < d ? p.u[(size_t)h * d + c] : 0.f;
+            Ls[c] = 0.f;
         }
     }
+    __syncthreads();
+    for (int idx = tid; idx < DC_C / 2 * D; idx += 128) Ls[(DC_C / 2 + 1 + idx / D) * LDL + idx % D] += Ls[DC_C / 2 * LDL + idx % D];
     dc_wait<1>();
     __syncthreads();
     const int g = lane >> 2, tq = lane & 3;
     const int v_row = (lane & 7) + ((lane >> 3) & 1) * 8, v_col = (lane >> 4) * 8;
     const int i0 = warp * 16 + g, i1 = i0 + 8;        // this lane's two rows
     auto pair = [](const __nv_bfloat16 *q) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(q)); };
-    // two neighbouring channels of a row of r, times e^{E_i - ref}, in two terms (ref null: nothing is subtracted)
+    // two neighbouring channels of a row of r, times 2^{E_i - ref}, in two terms (ref null: nothing is subtracted)
     auto r_terms = [&](int i, int c, const float *ref, uint32_t &hi, uint32_t &lo) {
         const float2 r = pair(Rs + i * (D + 8) + c), e = *reinterpret_cast<const float2 *>(Ls + i * LDL + c);
         const float2 m = ref ? *reinterpret_cast<const float2 *>(ref + c) : make_float2(0.f, 0.f);
-        dc_split2(r.x * __expf(e.x - m.x), r.y * __expf(e.y - m.y), hi, lo);
+        dc_split2(r.x * fast_exp2(e.x - m.x), r.y * fast_exp2(e.y - m.y), hi, lo);
     };
     uint32_t ph[DC_C / 16][4], pl[DC_C / 16][4];      // the scores as two terms, in the layout of an A operand
     {
@@ -257,7 +261,13 @@ time_mix_chunk_out_kernel(const TimeMixChunkParams p) {
         for (int j = 0; j < DC_C / 8; ++j)
 #pragma unroll
             for (int c = 0; c < 4; ++c) s[j][c] = 0.f;
-        const float *ref = Ls + warp * 16 * LDL;
+        // two neighbouring channels of a key, times 2^{ref - L_j}, in two terms
+        auto k_terms = [&](int j, int c, const float *ref, uint32_t &hi, uint32_t &lo) {
+            const float2 k = pair(Ks + j * (D + 8) + c), l = *reinterpret_cast<const float2 *>(Ls + (j + 1) * LDL + c),
+                         m = *reinterpret_cast<const float2 *>(ref + c);
+            dc_split2(k.x * fast_exp2(m.x - l.x), k.y * fast_exp2(m.y - l.y), hi, lo);
+        };
+        const float *ref = Ls + warp * 16 * LDL, *mid = ref + 8 * LDL;
         if (warp > 0) {                               // keys of the earlier sixteens (the branch is a warp's)
             for (int kk = 0; kk < k_steps; ++kk) {
                 uint32_t a[4], al[4];
@@ -269,55 +279,59 @@ time_mix_chunk_out_kernel(const TimeMixChunkParams p) {
                 for (int jt = 0; jt < 6; ++jt) {
                     if (jt >= 2 * warp) continue;
                     uint32_t b[2], bl[2];
-                    const int j = jt * 8 + g;
 #pragma unroll
-                    for (int x = 0; x < 2; ++x) {
-                        const int c = kk * 16 + 2 * tq + 8 * x;
-                        const float2 k = pair(Ks + j * (D + 8) + c), l = *reinterpret_cast<const float2 *>(Ls + (j + 1) * LDL + c),
-                                     m = *reinterpret_cast<const float2 *>(ref + c);
-                        dc_split2(k.x * __expf(m.x - l.x), k.y * __expf(m.y - l.y), b[x], bl[x]);
-                    }
+                    for (int x = 0; x < 2; ++x) k_terms(jt * 8 + g, kk * 16 + 2 * tq + 8 * x, ref, b[x], bl[x]);
                     mma_bf16(s[jt], a, b[0], b[1]);
                     mma_bf16(s[jt], a, bl[0], bl[1]);
                     mma_bf16(s[jt], al, b[0], b[1]);
                 }
             }
         }
-        // pairs inside the sixteen: this lane's rows i0, i1 and columns j = 16 warp + 8 jj + 2 tq + {0, 1}
-        float q[2][2][2];                             // [row][jj][column]
+        // inside the sixteen: the last eight tokens with the first eight once more as a product, the sums in front of the eighth as the
+        // reference (the rows of the first eight stay out of it)
+        float x8[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int kk = 0; kk < k_steps; ++kk) {
+            uint32_t a[4] = {0, 0, 0, 0}, al[4] = {0, 0, 0, 0}, b[2], bl[2];
+            r_terms(i1, kk * 16 + 2 * tq, mid, a[1], al[1]);
+            r_terms(i1, kk * 16 + 2 * tq + 8, mid, a[3], al[3]);
 #pragma unroll
-        for (int x = 0; x < 8; ++x) q[x >> 2][(x >> 1) & 1][x & 1] = 0.f;
+            for (int x = 0; x < 2; ++x) k_terms(warp * 16 + g, kk * 16 + 2 * tq + 8 * x, mid, b[x], bl[x]);
+            mma_bf16(x8, a, b[0], b[1]);
+            mma_bf16(x8, a, bl[0], bl[1]);
+            mma_bf16(x8, al, b[0], b[1]);
+        }
+        // and the pairs inside each eight: this lane's row i0 + 8 a with columns j = 16 warp + 8 a + 2 tq + {0, 1}
+        float q[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
         const int jb = warp * 16 + 2 * tq;
         for (int c = 0; c < d; c += 2) {
             const float2 uu = *reinterpret_cast<const float2 *>(us + c);
-            float2 r[2], e[2];
 #pragma unroll
             for (int a = 0; a < 2; ++a) {
-                r[a] = pair(Rs + (i0 + 8 * a) * (D + 8) + c);
-                e[a] = *reinterpret_cast<const float2 *>(Ls + (i0 + 8 * a) * LDL + c);
-            }
-#pragma unroll
-            for (int jj = 0; jj < 2; ++jj)
+                const int i = i0 + 8 * a;
+                const float2 r = pair(Rs + i * (D + 8) + c), e = *reinterpret_cast<const float2 *>(Ls + i * LDL + c);
 #pragma unroll
                 for (int b = 0; b < 2; ++b) {
-                    const int j = jb + 8 * jj + b;
+                    const int j = jb + 8 * a + b;
                     const float2 k = pair(Ks + j * (D + 8) + c), l = *reinterpret_cast<const float2 *>(Ls + (j + 1) * LDL + c);
-#pragma unroll
-                    for (int a = 0; a < 2; ++a) {
-                        const int i = i0 + 8 * a;
-                        const float fx = i == j ? uu.x : __expf(fminf(e[a].x - l.x, 0.f)), fy = i == j ? uu.y : __expf(fminf(e[a].y - l.y, 0.f));
-                        q[a][jj][b] = fmaf(r[a].x * k.x, fx, fmaf(r[a].y * k.y, fy, q[a][jj][b]));
-                    }
+                    const float fx = i == j ? uu.x : fast_exp2(fminf(e.x - l.x, 0.f)), fy = i == j ? uu.y : fast_exp2(fminf(e.y - l.y, 0.f));
+                    q[a][b] = fmaf(r.x * k.x, fx, fmaf(r.y * k.y, fy, q[a][b]));
                 }
+            }
         }
 #pragma unroll
         for (int jt = 0; jt < DC_C / 8; ++jt) {
-            const int jj = jt & 1;
             if ((jt >> 1) != warp) continue;
+            const int a = jt & 1;                     // the eight this column tile belongs to
 #pragma unroll
-            for (int a = 0; a < 2; ++a)
-#pragma unroll
-                for (int b = 0; b < 2; ++b) s[jt][2 * a + b] = i0 + 8 * a >= jb + 8 * jj + b ? q[a][jj][b] : 0.f;
+            for (int b = 0; b < 2; ++b) {
+                if (a == 0) {
+                    s[jt][b] = i0 >= jb + b ? q[0][b] : 0.f;
+                    s[jt][2 + b] = x8[2 + b];
+                } else {
+                    s[jt][b] = 0.f;
+                    s[jt][2 + b] = i1 >= jb + 8 + b ? q[1][b] : 0.f;
+                }
+            }
         }
 #pragma unroll
         for (int jp = 0; jp < DC_C / 16; ++jp)
