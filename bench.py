@@ -441,7 +441,7 @@ def run_zidivik(args) -> int:
                    "gate_columns_mul", "latent_rotate_queries", "add_row", "differential_combine", "retention_prepare", "retention_step", "retention_chunks",
                    "moe_route_scored", "attention_tc_maps", "attention_window_maps", "attention_decode_maps", "post_norm_add", "embed_copy",
                    "attn_prepare_conv", "token_shift", "linear_groups", "time_mix_gates", "recurrence_scan_bonus", "ssm_expand", "ssm_out", "ssm_step", "ssm_chunks", "part_norm", "delta_head_step",
-                   "delta_chunks", "time_mix_step", "time_mix_chunks", "post_norm_add_norm"]
+                   "delta_chunks", "time_mix_step", "time_mix_chunks", "post_norm_add_norm", "attention_decode_capped"]
 
     def measure(cfg, label):
         model = resolve_architecture(cfg.architecture).build(cfg, torch.bfloat16, dev)
