@@ -28,8 +28,8 @@ rows / 2, beyond that min(rows - 1, rows / 2 + floor(ln(n / (rows / 2)) / ln(far
 once on the host in float64 for the distances 0 .. far.  ``element_gate``: the gate is a number per ELEMENT of the
 concatenated heads (heads * v_head_dim logits of the mixer's input, further columns of the fused product) instead of
 one per head.  ``conv_taps`` > 0: q and k pass a causal convolution over time per channel, directly after their projection; its last
-conv_taps - 1 inputs are state of the request.  ``values_from_keys`` (with ``conv_taps``): there is no value projection, a key as it
-leaves the convolution - before norm and rotation - is its own value.
+conv_taps - 1 inputs are state of the request.  ``values_from_keys`` (with ``conv_taps``): there is no value projection; the
+convolved key is cached twice, once plain as the value and once normed and turned as the key that scores.
 
 `heads_into` runs everything in front of the output projection and leaves the gated heads, times a factor, in a place inside a
 wider matrix: for a container that projects the heads of two mixers by one product (``out_proj=False``: the mixer has no output
