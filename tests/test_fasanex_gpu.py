@@ -141,6 +141,15 @@ MIXERS = [
     ("delta 4/1 x 64/128", T.delta(4, 1, 64, 128, 4), None),
     ("joined 6/2 x 16 beside 2 x 24", T.parallel(6, 2, 16, 3, 0.3, 9.0, 13, T.rot(8, 100.0, SC), 2, 24, 8), None),
     ("joined 2/2 x 10 beside 3 x 12", T.parallel(2, 2, 10, 2, 0.5, 0.0, 40, T.rot(10, 1000.0), 3, 12, 5, (1.5, -0.4)), None),
+    ("attention 4/2 x 64, rotated whole", _left(4, 2, 64, conv=4, window=40), "left"),
+    ("attention 2/1 x 128, two taps, no rotation", _left(2, 1, 128, conv=2, rotary=None), "left"),
+    ("time mixing 1 x 96, rank 200", _right(1, 96, 200), "right"),
+    ("time mixing 2 x 128, rank 32", _right(2, 128, 32), "right"),
+    ("time mixing 3 x 40, rank 8", _right(3, 40, 8), "right"),
+    ("state space 2 x 136, state 48, 1 part", T.mamba2(2, 136, 48, 2, 1, 4), None),
+    ("state space 1 x 300, state 16", T.mamba2(1, 300, 16, 1, 1, 3), None),
+    ("delta 1/1 x 200/24", T.delta(1, 1, 200, 24, 2), None),
+    ("delta 6/3 x 40/8", T.delta(6, 3, 40, 8, 3), None),
 ]
 IDS = [m[0] for m in MIXERS]
 
@@ -395,7 +404,7 @@ def test_bounded_activation_in_the_products_epilogue(limit, T_, ff, K):
     _close(sliced.float().cpu().numpy(), want, "bfloat16", "on slices", scale=scale, tol=1e-2)
 
 
-@pytest.mark.parametrize("which", [7, 9, 12, 13, 14, 16, 18])
+@pytest.mark.parametrize("which", [7, 9, 12, 13, 14, 16, 18, 24, 25, 26, 29])
 def test_chunked_and_stepwise_forms_against_the_sequential_scan(which):
     """bfloat16: portions in chunks on the tensor cores and steps of few tokens in one kernel, against the same mixer on the sequential
     float32 scan: they round their operands alike, so they stand closer to each other than to the plain statement; decays from slow to
